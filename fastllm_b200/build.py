@@ -31,6 +31,8 @@ NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
     "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v",
 ]
+# translation units that state fp32 results exactly (32-bit angles, norms, matrix products) are compiled without fast-math
+PRECISE_UNITS = {"stream32", "full32"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fopenmp", "-march=x86-64-v3", "-Wall", "-Wno-unused-function"]
 
 
@@ -50,17 +52,23 @@ def _run(cmd: list[str], log: Path | None = None) -> None:
         raise RuntimeError("build step failed: " + " ".join(cmd))
 
 
-def build_kernels(force: bool = False) -> Path:
+# kernel files of models whose layers are latent attention and table-routed experts
+LATENT_UNITS = ("attn_mla", "attn_window", "elementwise", "full32", "gemm_bf16", "moe", "sampling", "stream32")
+
+
+def build_kernels(force: bool = False, units: tuple | None = None, out: Path | None = None) -> Path:
+    """``units``: compile and link these files only (into ``out``)."""
     OBJ.mkdir(exist_ok=True)
     LIB.mkdir(exist_ok=True)
     headers = sorted(CSRC.glob("*.cuh")) + sorted(CSRC.glob("*.h"))
-    sources = sorted(CSRC.glob("*.cu"))
-    out = LIB / "libfb_kernels.so"
+    sources = sorted(s for s in CSRC.glob("*.cu") if units is None or s.stem in units)
+    out = out or LIB / "libfb_kernels.so"
     jobs = []
     for src in sources:
         obj = OBJ / (src.stem + ".o")
         if force or _newer(src, headers, obj):
-            jobs.append((["nvcc", *NVCC_FLAGS, "-I", str(CSRC), "-c", str(src), "-o", str(obj)], OBJ / (src.stem + ".ptxas.log")))
+            flags = [f for f in NVCC_FLAGS if not (f == "--use_fast_math" and src.stem in PRECISE_UNITS)]
+            jobs.append((["nvcc", *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)], OBJ / (src.stem + ".ptxas.log")))
     if jobs:
         with ThreadPoolExecutor(max_workers=min(len(jobs), os.cpu_count() or 4)) as ex:
             list(ex.map(lambda j: _run(*j), jobs))
@@ -68,6 +76,22 @@ def build_kernels(force: bool = False) -> Path:
     if force or jobs or not out.exists():
         _run(["nvcc", "-shared", "-o", str(out), *map(str, objs), "-gencode", "arch=compute_100a,code=sm_100a"])
     return out
+
+
+def ensure_for(model_dir) -> None:
+    """Native libraries for serving the model in ``model_dir`` from a checkout without built files: the host runtime and the kernels
+    its layers launch.  A full kernel library that is there already is used as it is."""
+    from .models.config import load_config
+    from .ops import _lib
+
+    if not (LIB / "libfb_runtime.so").exists():
+        build_runtime()
+    if (LIB / "libfb_kernels.so").exists():
+        return
+    if load_config(model_dir).mixers is None:
+        build_kernels()
+        return
+    _lib.use_library(build_kernels(units=LATENT_UNITS, out=LIB / "libfb_kernels_latent.so"))
 
 
 def build_runtime(force: bool = False) -> Path:

@@ -1,0 +1,335 @@
+// Prefill attention with one key / value head per query head and an optional sliding window, for sm_100a (tcgen05 + TMEM).
+//
+// Keys and values are contiguous rows (the expanded latents of the keys a batch reads).  One CTA owns one head and up to 256
+// consecutive new tokens of one request as two blocks of 128 query rows; both blocks read the same 64-key K / V steps, loaded once,
+// and their softmax runs on two warp groups, so the tensor core alternates between the blocks:
+//     S_b[128 q x 64 k] = Q_b * K^T        O_b[128 q x V] += P_b * V          b = 0, 1
+// A block takes part only in the steps its rows see (the causal frontier at one end, the window at the other).  Head widths are
+// any multiple of 8: the operand maps are bounded per head, so the tail of a 64-column tile is zero.  The epilogue normalises and
+// applies the elementwise output gate o * sigmoid(g) where the layer has one.
+#include "ptx.cuh"
+#include "launch.h"
+#include "tmap.h"
+
+FB_DEFINE_ERROR_API(attn_window)
+
+namespace fb {
+
+constexpr int KID_ATTN_WINDOW = 16;
+constexpr int AW_KV = 64;                          // keys per step
+constexpr int AW_QT = 128 * 128;                   // bytes of a [128 rows x 64 cols] tile
+constexpr int AW_KT = AW_KV * 128;                 // bytes of a [64 rows x 64 cols] tile
+constexpr int AW_PT = 128 * AW_KV * 2;
+constexpr int AW_SMEM_MAX = 227 * 1024;
+
+struct AttnWindowParams {
+  // [n_blocks][6] = packed row of the first query, its position, query rows (<= 256), row of the request's first key, that key's
+  // position, (unused)
+  const int* blocks;
+  uint16_t* out; long long ld_out;
+  const uint16_t* gate; long long ld_gate;
+  int D, V, dt, vt;                               // head widths, their 64-column tiles
+  int stages, window;
+  float scale_log2;
+  uint32_t idesc_s, idesc_o;
+};
+
+template <bool BF16>
+__global__ void __launch_bounds__(320, 1)
+attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                   const AttnWindowParams p) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int dt = p.dt, vt = p.vt, stages = p.stages;
+  const int stage_bytes = (dt + vt) * AW_KT;
+  uint8_t* q_smem = smem;                                   // [2 blocks][dt] tiles of 16 KB
+  uint8_t* kv_smem = smem + 2 * dt * AW_QT;                 // [stages] x (K tiles, V tiles)
+  uint8_t* p_smem = kv_smem + stages * stage_bytes;         // [2 blocks] x 16 KB
+  uint64_t* bars = reinterpret_cast<uint64_t*>(p_smem + 2 * AW_PT);
+  uint64_t* full_k = bars;                                  // [4]
+  uint64_t* full_v = bars + 4;
+  uint64_t* empty = bars + 8;
+  uint64_t* q_full = bars + 12;
+  uint64_t* s_full = bars + 13;       // [2]
+  uint64_t* p_ready = bars + 15;      // [2]
+  uint64_t* o_full = bars + 17;       // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int head = blockIdx.x;
+  const int* blk = p.blocks + 6 * blockIdx.y;
+  const int q_row0 = blk[0], pos0 = blk[1], rows = blk[2], key_row0 = blk[3], key0 = blk[4];
+  // first key of the block's first row, one past the last key of its last row
+  int lo = key0;
+  if (p.window > 0 && pos0 - p.window + 1 > lo) lo = pos0 - p.window + 1;
+  const int hi = pos0 + rows;
+  const int n_steps = (hi - lo + AW_KV - 1) / AW_KV;
+  // steps [f, e) of query block b
+  int f[2], e[2];
+  f[0] = 0;
+  e[0] = (pos0 + (rows < 128 ? rows : 128) - lo + AW_KV - 1) / AW_KV;
+  if (rows > 128) {
+    int lo1 = lo;
+    if (p.window > 0 && pos0 + 128 - p.window + 1 > lo1) lo1 = pos0 + 128 - p.window + 1;
+    f[1] = (lo1 - lo) / AW_KV;
+    e[1] = n_steps;
+  } else {
+    f[1] = e[1] = n_steps;
+  }
+  bool dead = false;
+
+  if (threadIdx.x == 0) {
+    for (int s = 0; s < stages; ++s) { mbar_init(&full_k[s], 1); mbar_init(&full_v[s], 1); mbar_init(&empty[s], 1); }
+    mbar_init(q_full, 1);
+    for (int b = 0; b < 2; ++b) { mbar_init(&s_full[b], 1); mbar_init(&p_ready[b], 128); mbar_init(&o_full[b], 1); }
+    mbar_init_fence();
+    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem0 = *tmem_slot;
+  // columns: S_0 [0,64) S_1 [64,128) O_0 [128, 128 + 64 vt) O_1 behind it
+  const uint32_t o_cols = (uint32_t)(vt * 64);
+
+  if (warp == 0) {
+    if (elect_one()) {
+      const int nb = rows > 128 ? 2 : 1;
+      mbar_expect_tx(q_full, nb * dt * AW_QT);
+      for (int b = 0; b < nb; ++b)
+        for (int j = 0; j < dt; ++j) tma_load_3d(q_smem + (b * dt + j) * AW_QT, &tmQ, q_full, j * 64, head, q_row0 + b * 128);
+      for (int it = 0; it < n_steps; ++it) {
+        const int s = it % stages;
+        const uint32_t ph = (uint32_t)(it / stages) & 1u;
+        if (!mbar_wait(&empty[s], ph ^ 1u, dead, KID_ATTN_WINDOW, 1)) break;
+        const int row = key_row0 + (lo - key0) + it * AW_KV;
+        uint8_t* kb = kv_smem + s * stage_bytes;
+        uint8_t* vb = kb + dt * AW_KT;
+        mbar_expect_tx(&full_k[s], dt * AW_KT);
+        for (int j = 0; j < dt; ++j) tma_load_3d(kb + j * AW_KT, &tmK, &full_k[s], j * 64, head, row);
+        mbar_expect_tx(&full_v[s], vt * AW_KT);
+        for (int j = 0; j < vt; ++j) tma_load_3d(vb + j * AW_KT, &tmV, &full_v[s], j * 64, head, row);
+      }
+    }
+    __syncwarp();
+  } else if (warp == 1) {
+    if (elect_one()) {
+      const uint32_t qb = smem_u32(q_smem), pb = smem_u32(p_smem);
+      const int ks = (p.D + 15) / 16;              // 16-wide k steps of the S product
+      auto issue_s = [&](int b, uint32_t kb) {
+        for (int k = 0; k < ks; ++k) {
+          const uint64_t da = make_smem_desc(qb + (b * dt + (k >> 2)) * AW_QT + (k & 3) * 32, 16, 1024, SWZ_128B);
+          const uint64_t db = make_smem_desc(kb + (k >> 2) * AW_KT + (k & 3) * 32, 16, 1024, SWZ_128B);
+          umma_f16(tmem0 + (uint32_t)(b * 64), da, db, p.idesc_s, k != 0 ? 1u : 0u);
+        }
+        umma_commit(&s_full[b]);
+      };
+      bool ok = mbar_wait(q_full, 0, dead, KID_ATTN_WINDOW, 2);
+      if (ok) ok = mbar_wait(&full_k[0], 0, dead, KID_ATTN_WINDOW, 3);
+      if (ok) {
+        tc_fence_after_sync();
+        for (int b = 0; b < 2; ++b)
+          if (f[b] == 0 && e[b] > 0) issue_s(b, smem_u32(kv_smem));
+      }
+      for (int it = 0; ok && it < n_steps; ++it) {
+        const int s = it % stages, s1 = (it + 1) % stages;
+        const uint32_t ph = (uint32_t)(it / stages) & 1u, ph1 = (uint32_t)((it + 1) / stages) & 1u;
+        const uint32_t vb = smem_u32(kv_smem + s * stage_bytes + dt * AW_KT);
+        const uint32_t kb1 = smem_u32(kv_smem + s1 * stage_bytes);
+        bool have_v = false, have_k1 = false;
+        for (int b = 0; b < 2; ++b) {
+          if (it >= f[b] && it < e[b]) {
+            if (!mbar_wait(&p_ready[b], (uint32_t)(it - f[b]) & 1u, dead, KID_ATTN_WINDOW, 4)) { ok = false; break; }
+            if (!have_v && !mbar_wait(&full_v[s], ph, dead, KID_ATTN_WINDOW, 5)) { ok = false; break; }
+            have_v = true;
+            tc_fence_after_sync();
+            // O_b += P_b * V : A = P_b (K-major, 64 keys), B = V step MN-major (16 keys per MMA)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              const uint64_t da = make_smem_desc(pb + b * AW_PT + k * 32, 16, 1024, SWZ_128B);
+              const uint64_t db = make_smem_desc(vb + k * 2048, AW_KT, 1024, SWZ_128B);
+              umma_f16(tmem0 + 128u + (uint32_t)b * o_cols, da, db, p.idesc_o, (it != f[b] || k != 0) ? 1u : 0u);
+            }
+            umma_commit(&o_full[b]);
+          }
+          if (it + 1 >= f[b] && it + 1 < e[b]) {
+            if (!have_k1 && !mbar_wait(&full_k[s1], ph1, dead, KID_ATTN_WINDOW, 6)) { ok = false; break; }
+            have_k1 = true;
+            tc_fence_after_sync();
+            issue_s(b, kb1);
+          }
+        }
+        if (ok) {
+          // (a step no block used for V has its load outstanding: the slot may only be refilled once it has landed)
+          if (!have_v && !mbar_wait(&full_v[s], ph, dead, KID_ATTN_WINDOW, 7)) break;
+          umma_commit(&empty[s]);
+        }
+      }
+    }
+    __syncwarp();
+  } else {
+    const int b = (warp - 2) >> 2;               // query block of this warp group
+    const int q = warp & 3;                      // TMEM lane quarter: warps 2..5 -> 2,3,0,1 ; 6..9 -> 2,3,0,1
+    const int r = q * 32 + lane;
+    const int pos_b = pos0 + b * 128, pos = pos_b + r;
+    const int first = p.window > 0 ? pos - p.window + 1 : 0;
+    const uint32_t lane_off = (uint32_t)(q * 32) << 16;
+    const uint32_t tmem_s = tmem0 + (uint32_t)(b * 64), tmem_o = tmem0 + 128u + (uint32_t)b * o_cols;
+    uint8_t* prow = p_smem + b * AW_PT + r * 128;
+    const int it0 = f[b], it1 = e[b];
+    float m_run = -INFINITY, l_run = 0.f;
+    for (int it = it0; it < it1; ++it) {
+      const uint32_t iph = (uint32_t)(it - it0) & 1u;
+      mbar_wait(&s_full[b], iph, dead, KID_ATTN_WINDOW, 8);
+      tc_fence_after_sync();
+      const int kv0 = lo + it * AW_KV;
+      uint32_t sreg[64];
+      tmem_ld_32x32b_x32(tmem_s + lane_off, sreg);
+      tmem_ld_32x32b_x32(tmem_s + lane_off + 32, sreg + 32);
+      tmem_ld_wait();
+      // only steps on the causal diagonal or on the window's edge pay for the mask
+      const bool full_step = kv0 + AW_KV - 1 <= pos_b && (p.window <= 0 || kv0 > pos_b + 127 - p.window);
+      float m_new = m_run;
+      if (full_step) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) {
+          const float sv = __uint_as_float(sreg[j]) * p.scale_log2;
+          sreg[j] = __float_as_uint(sv);
+          m_new = fmaxf(m_new, sv);
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) {
+          const int kv = kv0 + j;
+          const float sv = (kv <= pos && kv >= first) ? __uint_as_float(sreg[j]) * p.scale_log2 : -INFINITY;
+          sreg[j] = __float_as_uint(sv);
+          m_new = fmaxf(m_new, sv);
+        }
+      }
+      const float m_use = m_new == -INFINITY ? 0.f : m_new;
+      const float alpha = exp2f(m_run - m_use);
+      if (it > it0) {
+        // the previous P * V of this block must be complete before P is overwritten or O is rescaled
+        mbar_wait(&o_full[b], iph ^ 1u, dead, KID_ATTN_WINDOW, 9);
+        tc_fence_after_sync();
+        if (__any_sync(0xffffffffu, alpha != 1.0f)) {
+#pragma unroll 1
+          for (int c0 = 0; c0 < (int)o_cols; c0 += 32) {
+            uint32_t oreg[32];
+            tmem_ld_32x32b_x32(tmem_o + lane_off + c0, oreg);
+            tmem_ld_wait();
+#pragma unroll
+            for (int j = 0; j < 32; ++j) oreg[j] = __float_as_uint(__uint_as_float(oreg[j]) * alpha);
+            tmem_st_32x32b_x32(tmem_o + lane_off + c0, oreg);
+          }
+          tmem_st_wait();
+        }
+      }
+      float l_add = 0.f;
+#pragma unroll
+      for (int g = 0; g < 8; ++g) {
+        uint32_t pk[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const float p0 = exp2f(__uint_as_float(sreg[8 * g + 2 * j]) - m_use);
+          const float p1 = exp2f(__uint_as_float(sreg[8 * g + 2 * j + 1]) - m_use);
+          pk[j] = pack_16<BF16>(p0, p1);
+          l_add += p0 + p1;
+        }
+        *reinterpret_cast<uint4*>(prow + ((g ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+      }
+      l_run = l_run * alpha + l_add;
+      m_run = m_new;
+      fence_proxy_async_smem();
+      tc_fence_before_sync();
+      mbar_arrive(&p_ready[b]);
+    }
+    if (it1 > it0) {
+      mbar_wait(&o_full[b], (uint32_t)(it1 - it0 - 1) & 1u, dead, KID_ATTN_WINDOW, 10);
+      tc_fence_after_sync();
+      const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      const bool live = b * 128 + r < rows;
+      const size_t row = (size_t)(q_row0 + b * 128 + r);
+      uint16_t* orow = p.out + row * p.ld_out + (size_t)head * p.V;
+      const uint16_t* grow = p.gate != nullptr ? p.gate + row * p.ld_gate + (size_t)head * p.V : nullptr;
+#pragma unroll 1
+      for (int c0 = 0; c0 < p.V; c0 += 32) {
+        uint32_t oreg[32];
+        __syncwarp();
+        tmem_ld_32x32b_x32(tmem_o + lane_off + c0, oreg);
+        tmem_ld_wait();
+        if (live) {
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            if (c0 + 8 * g >= p.V) break;
+            float v[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = __uint_as_float(oreg[8 * g + j]) * inv_l;
+            if (grow != nullptr) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(grow + c0 + 8 * g);
+              const float2 g0 = unpack_16<BF16>(gv.x), g1 = unpack_16<BF16>(gv.y), g2 = unpack_16<BF16>(gv.z), g3 = unpack_16<BF16>(gv.w);
+              const float gg[8] = {g0.x, g0.y, g1.x, g1.y, g2.x, g2.y, g3.x, g3.y};
+#pragma unroll
+              for (int j = 0; j < 8; ++j) v[j] *= 1.0f / (1.0f + __expf(-gg[j]));
+            }
+            *reinterpret_cast<uint4*>(orow + c0 + 8 * g) =
+                make_uint4(pack_16<BF16>(v[0], v[1]), pack_16<BF16>(v[2], v[3]), pack_16<BF16>(v[4], v[5]), pack_16<BF16>(v[6], v[7]));
+          }
+        }
+      }
+    }
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) tmem_dealloc(tmem0, 512);
+}
+
+// Ring depth that fits beside the queries and probabilities; 0: the head widths are outside the kernel.
+static int window_stages(int D, int V) {
+  const int dt = (D + 63) / 64, vt = (V + 63) / 64;
+  if (vt > 3) return 0;                                       // 2 accumulators of 64 vt columns beside S: 512 TMEM columns
+  const int fixed = 2 * dt * AW_QT + 2 * AW_PT + 256 + 1024;
+  const int n = (AW_SMEM_MAX - fixed) / ((dt + vt) * AW_KT);
+  return n < 2 ? 0 : n > 4 ? 4 : n;
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+extern "C" int fb_attn_window_supported(int D, int V) { return D > 0 && V > 0 && D % 8 == 0 && V % 8 == 0 && window_stages(D, V) > 0 ? 1 : 0; }
+
+// q: packed rows [T, >= H * D] (row stride ld_q), k: [n_keys, >= H * D], v: [n_keys, >= H * V], out [T, H * V], gate (optional) like out.
+extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* k, long long ld_k, const void* v, long long ld_v, int n_keys,
+                              void* out, long long ld_out, const void* gate, long long ld_gate, const int* blocks, int n_blocks, int H,
+                              int D, int V, int window, float scale, int dtype, void* stream_) {
+  if (n_blocks <= 0) return 0;
+  const int stages = window_stages(D, V);
+  if (stages == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || n_keys <= 0 || H <= 0 || n_blocks > 65535 || window < 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
+    return -1;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  CUtensorMap tmQ, tmK, tmV;
+  if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
+  if (!make_tmap_3d(&tmK, k, D, H, n_keys, D, ld_k, 64, AW_KV)) return -2;
+  if (!make_tmap_3d(&tmV, v, V, H, n_keys, V, ld_v, 64, AW_KV)) return -2;
+  AttnWindowParams p;
+  p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
+  p.D = D; p.V = V; p.dt = (D + 63) / 64; p.vt = (V + 63) / 64; p.stages = stages; p.window = window;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  const uint32_t fm = dtype == 1 ? 1u : 0u;
+  p.idesc_s = make_idesc(fm, fm, 0, 0, 128, AW_KV);
+  p.idesc_o = make_idesc(fm, fm, 0, 1, 128, p.vt * 64);
+  const int smem = 2 * p.dt * AW_QT + stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
+  const dim3 grid(H, n_blocks);
+  if (dtype == 1) {
+    static DeviceOnce cfg;
+    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);
+    attn_window_kernel<true><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);
+  } else {
+    static DeviceOnce cfg;
+    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);
+    attn_window_kernel<false><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);
+  }
+  return (int)cudaGetLastError();
+}

@@ -1,0 +1,193 @@
+// 32-bit and any-size forms of a model's matrix products and of latent attention (CUDA cores, fp32 FMAs).
+//
+// They serve models run in float32, where the tensor core has no full-precision mode, and 16-bit shapes outside the tensor-core
+// kernels' tiling.  Compiled without fast-math.
+#include "ptx.cuh"
+#include "launch.h"
+
+FB_DEFINE_ERROR_API(full32)
+
+namespace fb {
+
+template <int DT> struct F32In;
+template <> struct F32In<0> { typedef uint16_t T; static __device__ __forceinline__ float ld(uint16_t v) { return __half2float(__ushort_as_half(v)); }
+                              static __device__ __forceinline__ uint16_t st(float v) { return __half_as_ushort(__float2half_rn(v)); } };
+template <> struct F32In<1> { typedef uint16_t T; static __device__ __forceinline__ float ld(uint16_t v) { return __bfloat162float(__ushort_as_bfloat16(v)); }
+                              static __device__ __forceinline__ uint16_t st(float v) { return __bfloat16_as_ushort(__float2bfloat16_rn(v)); } };
+template <> struct F32In<2> { typedef float T; static __device__ __forceinline__ float ld(float v) { return v; } static __device__ __forceinline__ float st(float v) { return v; } };
+
+// out[m, n] = act(sum_k X[m, k] W[n, k]) (* sigmoid(gate[m, n])), or residual[m, n] + alpha * (...) in fp32.
+// blockIdx.z selects a batch (its own weight rows, column slices of X and out) or, with `counts`, an expert and its segment of rows.
+struct Full32Params {
+  const void* X; const void* W; void* out;
+  const float* residual; const void* gate; const void* bias;
+  int M, N, K;
+  long long ldx, ldw, ld_out, ld_res, ld_gate;
+  long long batch_w_rows, batch_x_cols, batch_out_cols;
+  const int* counts; const int* offsets;
+  float alpha;
+  int relu2, out_f32;
+};
+
+template <int DT>
+__global__ void __launch_bounds__(256) gemm_full32_kernel(const Full32Params p) {
+  typedef typename F32In<DT>::T T;
+  constexpr int BM = 64, BN = 64, BK = 16;
+  __shared__ float xs[BK][BM + 4], ws[BK][BN + 4];
+  const int z = blockIdx.z;
+  int M = p.M;
+  long long row0 = 0;
+  if (p.counts != nullptr) { M = p.counts[z]; row0 = p.offsets[z]; }
+  const int n0 = blockIdx.x * BN;
+  const T* X = reinterpret_cast<const T*>(p.X) + z * p.batch_x_cols;
+  const T* W = reinterpret_cast<const T*>(p.W) + z * p.batch_w_rows * p.ldw;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  for (int m0 = blockIdx.y * BM; m0 < M; m0 += gridDim.y * BM) {
+    float acc[4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+    for (int k0 = 0; k0 < p.K; k0 += BK) {
+      for (int i = threadIdx.x; i < BM * BK; i += 256) {
+        const int r = i / BK, k = i - r * BK;
+        const bool in_k = k0 + k < p.K;
+        xs[k][r] = (in_k && m0 + r < M) ? F32In<DT>::ld(X[(row0 + m0 + r) * p.ldx + k0 + k]) : 0.f;
+        ws[k][r] = (in_k && n0 + r < p.N) ? F32In<DT>::ld(W[(long long)(n0 + r) * p.ldw + k0 + k]) : 0.f;
+      }
+      __syncthreads();
+#pragma unroll
+      for (int k = 0; k < BK; ++k) {
+        float a[4], b[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { a[i] = xs[k][ty * 4 + i]; b[i] = ws[k][tx * 4 + i]; }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+      }
+      __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int m = m0 + ty * 4 + i;
+      if (m >= M) continue;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int n = n0 + tx * 4 + j;
+        if (n >= p.N) continue;
+        float v = acc[i][j];
+        const long long c = z * p.batch_out_cols + n;
+        if (p.bias != nullptr) v += F32In<DT>::ld(reinterpret_cast<const T*>(p.bias)[n]);
+        if (p.relu2) { v = fmaxf(v, 0.f); v *= v; }
+        if (p.gate != nullptr) v *= 1.0f / (1.0f + expf(-F32In<DT>::ld(reinterpret_cast<const T*>(p.gate)[(row0 + m) * p.ld_gate + c])));
+        if (p.residual != nullptr) v = p.residual[(row0 + m) * p.ld_res + c] + p.alpha * v;
+        if (p.out_f32) reinterpret_cast<float*>(p.out)[(row0 + m) * p.ld_out + c] = v;
+        else reinterpret_cast<T*>(p.out)[(row0 + m) * p.ld_out + c] = F32In<DT>::st(v);
+      }
+    }
+  }
+}
+
+// Latent attention of one (row, head) per CTA over the paged latent cache, any latent width:
+//   score[j] = scale * q[row, head] . c[j],  out = sum_j softmax(score)[j] c[j],  first <= j <= position
+// 128 threads: a warp scores one key at a time (lanes over the latent), then every thread accumulates its latent columns.
+constexpr int L32_KEYS = 64;
+template <int DT>
+__global__ void __launch_bounds__(128) latent_attn32_kernel(const typename F32In<DT>::T* __restrict__ q, const typename F32In<DT>::T* __restrict__ pool,
+                                                            typename F32In<DT>::T* __restrict__ out, const int* __restrict__ page_table,
+                                                            const int* __restrict__ kv_lens, int max_pages, int page_len, int H, int R,
+                                                            int ld, int window, float scale) {
+  extern __shared__ float sm[];
+  float* qs = sm;                       // [R]
+  float* os = sm + R;                   // [R] running output
+  __shared__ float sc[L32_KEYS];
+  __shared__ int rows[L32_KEYS];
+  const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int n = kv_lens[t];
+  const int first = (window > 0 && n > window) ? n - window : 0;
+  const typename F32In<DT>::T* qp = q + ((size_t)t * H + h) * ld;
+  for (int i = tid; i < R; i += 128) { qs[i] = F32In<DT>::ld(qp[i]); os[i] = 0.f; }
+  float m_run = -INFINITY, l_run = 0.f;
+  for (int j0 = first; j0 < n; j0 += L32_KEYS) {
+    const int cnt = n - j0 < L32_KEYS ? n - j0 : L32_KEYS;
+    __syncthreads();
+    if (tid < cnt) {
+      const int j = j0 + tid, pg = j / page_len;
+      rows[tid] = pg < max_pages ? page_table[(size_t)t * max_pages + pg] * page_len + (j - pg * page_len) : 0;
+    }
+    __syncthreads();
+    for (int j = warp; j < cnt; j += 4) {
+      const typename F32In<DT>::T* c = pool + (size_t)rows[j] * ld;
+      float s = 0.f;
+      for (int i = lane; i < R; i += 32) s = fmaf(qs[i], F32In<DT>::ld(c[i]), s);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      if (lane == 0) sc[j] = s * scale;
+    }
+    __syncthreads();
+    float mx = m_run;
+    for (int j = 0; j < cnt; ++j) mx = fmaxf(mx, sc[j]);
+    const float fac = m_run == -INFINITY ? 0.f : expf(m_run - mx);
+    __syncthreads();
+    if (tid < cnt) sc[tid] = expf(sc[tid] - mx);
+    __syncthreads();
+    float l = 0.f;
+    for (int j = 0; j < cnt; ++j) l += sc[j];
+    l_run = l_run * fac + l;
+    m_run = mx;
+    for (int i = tid; i < R; i += 128) {
+      float a = os[i] * fac;
+      for (int j = 0; j < cnt; ++j) a = fmaf(sc[j], F32In<DT>::ld(pool[(size_t)rows[j] * ld + i]), a);
+      os[i] = a;
+    }
+  }
+  const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  typename F32In<DT>::T* op = out + ((size_t)t * H + h) * ld;
+  for (int i = tid; i < ld; i += 128) op[i] = F32In<DT>::st(i < R ? os[i] * inv : 0.f);
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+// dt: 0 fp16, 1 bf16, 2 fp32 operands.  batch > 1: see Full32Params.  counts / offsets (optional): grouped rows, `batch` experts whose
+// weights are batch_w_rows rows apart; max_rows bounds an expert's rows.
+extern "C" int fb_gemm_full32(const void* X, const void* W, void* out, const void* bias, const float* residual, const void* gate, int M,
+                              int N, int K, int batch, long long ldx, long long ldw, long long ld_out, long long ld_res, long long ld_gate,
+                              long long batch_w_rows, long long batch_x_cols, long long batch_out_cols, const int* counts,
+                              const int* offsets, float alpha, int relu2, int out_f32, int dt, void* stream) {
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
+  if (K <= 0 || dt < 0 || dt > 2 || batch > 65535) return -1;
+  Full32Params p{X, W, out, residual, gate, bias, M, N, K, ldx, ldw, ld_out, ld_res, ld_gate, batch_w_rows, batch_x_cols, batch_out_cols,
+                 counts, offsets, alpha, relu2, out_f32};
+  int gy = (M + 63) / 64;
+  if (counts != nullptr && gy > 8) gy = 8;            // an expert rarely gets more; the kernel strides over the rest
+  if (gy > 65535) gy = 65535;
+  const dim3 grid((N + 63) / 64, gy, batch);
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (dt == 0) gemm_full32_kernel<0><<<grid, 256, 0, s>>>(p);
+  else if (dt == 1) gemm_full32_kernel<1><<<grid, 256, 0, s>>>(p);
+  else gemm_full32_kernel<2><<<grid, 256, 0, s>>>(p);
+  return (int)cudaGetLastError();
+}
+
+// q / out: [T, H, ld], pool: [num_slots, ld], latent width R <= ld.  page_table [T, max_pages] and kv_lens [T] belong to the rows: row t
+// sees keys [max(0, kv_lens[t] - window), kv_lens[t]).
+extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, const int* page_table, const int* kv_lens, int T, int H, int R,
+                                int ld, int max_pages, int page_len, int window, float scale, int dt, void* stream) {
+  if (T <= 0 || H <= 0) return 0;
+  if (R <= 0 || ld < R || R > 24576 || H > 65535 || max_pages <= 0 || page_len <= 0 || dt < 0 || dt > 2) return -1;
+  const size_t smem = (size_t)R * 8;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define GO(DT)                                                                                                                     \
+  {                                                                                                                                \
+    static DeviceOnce cfg;                                                                                                         \
+    if (cfg.need()) cudaFuncSetAttribute(latent_attn32_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 24576 * 8);         \
+    latent_attn32_kernel<DT><<<dim3(T, H), 128, smem, s>>>((const F32In<DT>::T*)q, (const F32In<DT>::T*)pool, (F32In<DT>::T*)out,  \
+                                                           page_table, kv_lens, max_pages, page_len, H, R, ld, window, scale);     \
+  }
+  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
+  return (int)cudaGetLastError();
+}

@@ -247,7 +247,7 @@ extern "C" int fb_gemm_pick_split(int M, int N, int K, int slots) {
   // Largest power-of-two split whose CTAs are all resident at once (slots = SMs x CTAs per SM) and that leaves
   // at least 8 k-blocks per rank.
   const int n_tiles = (N + 127) / 128;
-  const int kb = K / 64;
+  const int kb = (K + 63) / 64;
   int best = 1;
   for (int s = 2; s <= 8; s *= 2) {
     if (n_tiles * s > slots) break;
@@ -299,26 +299,19 @@ extern "C" int fb_gemm_route(const void* X, const void* W, int M, int E, int K, 
 #undef FB_RT
 }
 
-extern "C" int fb_gemm_16bit(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
-                             int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit, void* stream_) {
-  return fb_gemm_16bit_wait(X, W, out, bias, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype, flags, nsplit, nullptr, nullptr, stream_);
-}
-
-// Same, for activations that a fused collective broadcast without waiting for its peers (small-M path only): the kernel
-// itself waits until the arrival counter *wait_cnt has reached *wait_expect before it reads X.  Returns -3 when a wait
-// is requested for a shape that the small-M kernel does not cover.
-extern "C" int fb_gemm_16bit_wait(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
+static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
                                   int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit,
-                                  const void* wait_cnt, const void* wait_expect, void* stream_) {
+                                  const void* wait_cnt, const void* wait_expect, float alpha, void* stream_) {
   using namespace fb;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0) return 0;
-  if (K % 64 != 0 || N % 8 != 0 || (dtype != 0 && dtype != 1)) return -1;
+  if (K % 8 != 0 || N % 8 != 0 || (dtype != 0 && dtype != 1)) return -1;
   if ((flags & GEMM_SWIGLU) && (N % 128 != 0)) return -1;
   GemmParams p;
   p.out = out; p.bias = bias; p.residual = residual;
   p.M = M; p.N = N; p.K = K; p.ld_out = ld_out; p.ld_res = ld_res;
-  p.kb_total = K / 64;
+  p.kb_total = (K + 63) / 64;             // a last partial block: both operand maps end at column K, TMA fills the rest with zeros
+  p.alpha = alpha;
   p.flags = flags;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
@@ -384,6 +377,28 @@ extern "C" int fb_gemm_16bit_wait(const void* X, const void* W, void* out, const
   if (bn == 256)
     return (int)(bf16 ? launch_largem<256, true>(tmX, tmW, p, stream) : launch_largem<256, false>(tmX, tmW, p, stream));
   return (int)(bf16 ? launch_largem<128, true>(tmX, tmW, p, stream) : launch_largem<128, false>(tmX, tmW, p, stream));
+}
+
+// Same, for activations that a fused collective broadcast without waiting for its peers (small-M path only): the kernel
+// itself waits until the arrival counter *wait_cnt has reached *wait_expect before it reads X.  Returns -3 when a wait
+// is requested for a shape that the small-M kernel does not cover.
+extern "C" int fb_gemm_16bit_wait(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
+                                  int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit,
+                                  const void* wait_cnt, const void* wait_expect, void* stream_) {
+  return gemm_16bit_impl(X, W, out, bias, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype, flags, nsplit, wait_cnt, wait_expect, 1.f, stream_);
+}
+
+extern "C" int fb_gemm_16bit(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
+                             int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit, void* stream_) {
+  return gemm_16bit_impl(X, W, out, bias, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype, flags, nsplit, nullptr, nullptr, 1.f, stream_);
+}
+
+// Models with an fp32 residual stream: out_f32 = residual_f32 + alpha * (X W^T); `out` may be `residual`.
+extern "C" int fb_gemm_16bit_res32(const void* X, const void* W, float* out, const float* residual, int M, int N, int K, int ldx,
+                                   int ldw, int ld_out, int ld_res, float alpha, int dtype, void* stream_) {
+  using namespace fb;
+  return gemm_16bit_impl(X, W, out, nullptr, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype,
+                         GEMM_RESIDUAL | GEMM_RES_F32 | GEMM_OUT_F32, 0, nullptr, nullptr, alpha, stream_);
 }
 
 // QKV projection (head_dim 128, M <= 256, N = (Hq + 2 Hkv) * 128) with split / per-head RMSNorm / RoPE / paged-cache append in
@@ -456,18 +471,20 @@ extern "C" int fb_gemm_qkv_post(const void* X, const void* W, const void* bias, 
 // Batched small-M GEMM, one launch for `batch` independent products that share the token rows:
 //   out[m, z * out_cols + n] = sum_k X[m, z * x_cols + k] * W[z * N + n, k]      (z < batch, n < N, k < K)
 // X: [M, >= batch * x_cols] (row stride ldx), W: [batch * N, K] (row stride ldw), out row stride ld_out; 16-bit in and out.
-// Used for the absorbed multi-head-latent-attention projections (one small matrix per head).  M <= 256, K % 64 == 0,
-// N % 8 == 0, x_cols % 8 == 0, out_cols % 4 == 0.
-extern "C" int fb_gemm_16bit_batched(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw, int ld_out,
-                                     int x_cols, int out_cols, int dtype, void* stream_) {
+// Used for the absorbed multi-head-latent-attention projections (one small matrix per head).  M <= 256, K % 8 == 0
+// (a partial last k block of 64 reads the neighbouring slice of X against zero-filled weight columns), N % 4 == 0, x_cols % 8 == 0, out_cols % 4 == 0.
+// `gate` (optional, 16-bit, row stride ld_gate): out[m, c] is multiplied by sigmoid(gate[m, c]).
+extern "C" int fb_gemm_16bit_batched_gate(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw,
+                                          int ld_out, int x_cols, int out_cols, const void* gate, int ld_gate, int dtype, void* stream_) {
   using namespace fb;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
-  if (M > 256 || K % 64 != 0 || N % 8 != 0 || x_cols % 8 != 0 || out_cols % 4 != 0 || batch > 65535 || (dtype != 0 && dtype != 1)) return -1;
+  if (M > 256 || K % 8 != 0 || N % 4 != 0 || x_cols % 8 != 0 || out_cols % 4 != 0 || ld_gate % 4 != 0 || batch > 65535 || (dtype != 0 && dtype != 1)) return -1;
   GemmParams p;
   p.out = out; p.bias = nullptr; p.residual = nullptr;
   p.M = M; p.N = N; p.K = K; p.ld_out = ld_out; p.ld_res = 0;
-  p.kb_total = K / 64; p.kb_per_split = p.kb_total;
+  p.kb_total = (K + 63) / 64; p.kb_per_split = p.kb_total;
+  p.gate = gate; p.ld_gate = ld_gate;
   p.flags = 0;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
@@ -494,4 +511,9 @@ extern "C" int fb_gemm_16bit_batched(const void* X, const void* W, void* out, in
                         : launch_smallm<256, false, 1>(tmW, tmX, p, 1, n_tiles, stream, batch));
   }
 #undef FB_BT
+}
+
+extern "C" int fb_gemm_16bit_batched(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw, int ld_out,
+                                     int x_cols, int out_cols, int dtype, void* stream_) {
+  return fb_gemm_16bit_batched_gate(X, W, out, M, N, K, batch, ldx, ldw, ld_out, x_cols, out_cols, nullptr, 0, dtype, stream_);
 }

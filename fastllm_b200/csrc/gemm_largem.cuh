@@ -45,7 +45,19 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
             v[j] += b.x; v[j + 1] += b.y;
           }
         }
-        if (p.flags & GEMM_RESIDUAL) {
+        if (p.flags & GEMM_RELU2) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = relu2_f(v[j]);
+        }
+        if ((p.flags & GEMM_RESIDUAL) && (p.flags & GEMM_RES_F32)) {
+          const float4* rp = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.residual) + (size_t)m * p.ld_res + n0);
+#pragma unroll
+          for (int g = 0; g < 8; ++g) {
+            const float4 rv = rp[g];
+            v[g * 4 + 0] = rv.x + p.alpha * v[g * 4 + 0]; v[g * 4 + 1] = rv.y + p.alpha * v[g * 4 + 1];
+            v[g * 4 + 2] = rv.z + p.alpha * v[g * 4 + 2]; v[g * 4 + 3] = rv.w + p.alpha * v[g * 4 + 3];
+          }
+        } else if (p.flags & GEMM_RESIDUAL) {
           const uint4* rp = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.residual) + (size_t)m * p.ld_res + n0);
 #pragma unroll
           for (int g = 0; g < 4; ++g) {

@@ -44,6 +44,8 @@ enum GemmFlags : int {
   GEMM_RESIDUAL = 2,   // += residual[m, n]
   GEMM_SWIGLU = 4,     // out[m, i] = silu(gate) * up   (N_out = N / 2)
   GEMM_OUT_F32 = 8,    // write fp32 instead of the 16-bit input dtype
+  GEMM_RES_F32 = 16,   // with GEMM_RESIDUAL: the residual is fp32 and the product is scaled first, residual + alpha * acc
+  GEMM_RELU2 = 32,     // out = relu(acc)^2
   GEMM_FP4_F16W = 256, // fp4 weights, fp16 activations: the scale table lies within fp16's range (host-checked): half2 de-quantiser
 };
 
@@ -71,9 +73,14 @@ struct GemmParams {
   // z * batch_x_cols, the output at column z * batch_out_cols -- one launch for a GEMM per attention head (the absorbed
   // multi-head-latent-attention projections, where every head has its own small matrix and its own slice of the activations).
   int batch_w_rows = 0, batch_x_cols = 0, batch_out_cols = 0;
+  float alpha = 1.f;                         // GEMM_RES_F32
+  const void* gate = nullptr;                // 16-bit [M, >= N] (batched: + z * batch_out_cols): out = acc * sigmoid(gate)
+  int ld_gate = 0;
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float relu2_f(float x) { const float r = fmaxf(x, 0.f); return r * r; }
 
 // OCC = CTAs meant to be co-resident per SM: 1 -> deep ring (~200 KB), 2 -> two CTAs share the SM so that one
 // streams weights while the other is in its prologue / epilogue.
@@ -137,7 +144,17 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
           acc.x += b0.x; acc.y += b0.y; acc.z += b1.x; acc.w += b1.y;
         }
       }
-      if (p.flags & GEMM_RESIDUAL) {
+      if (p.flags & GEMM_RELU2) { acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y); acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w); }
+      if (p.gate != nullptr) {
+        const uint2 gv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p.gate) + (size_t)j * p.ld_gate +
+                                                         (size_t)blockIdx.z * (size_t)p.batch_out_cols + n_out);
+        const float2 g0 = unpack_16<BF16>(gv.x), g1 = unpack_16<BF16>(gv.y);
+        acc.x *= sigmoid_f(g0.x); acc.y *= sigmoid_f(g0.y); acc.z *= sigmoid_f(g1.x); acc.w *= sigmoid_f(g1.y);
+      }
+      if ((p.flags & GEMM_RESIDUAL) && (p.flags & GEMM_RES_F32)) {
+        const float4 rv = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.residual) + (size_t)j * p.ld_res + n_out);
+        acc.x = rv.x + p.alpha * acc.x; acc.y = rv.y + p.alpha * acc.y; acc.z = rv.z + p.alpha * acc.z; acc.w = rv.w + p.alpha * acc.w;
+      } else if (p.flags & GEMM_RESIDUAL) {
         const uint2 rv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p.residual) + (size_t)j * p.ld_res + n_out);
         float2 r0 = unpack_16<BF16>(rv.x), r1 = unpack_16<BF16>(rv.y);
         acc.x += r0.x; acc.y += r0.y; acc.z += r1.x; acc.w += r1.y;

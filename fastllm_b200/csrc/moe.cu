@@ -222,6 +222,58 @@ __global__ void moe_combine_kernel(const uint16_t* __restrict__ ys, const int* _
   }
 }
 
+// Plans of all table-routed layers of a model in one launch, one CTA per layer: the experts of a token are the entries of its
+// id's row of the layer's table, so the whole forward pass's routing is known once the token ids are.
+//   meta  [L][4] = (table address, top, experts, table rows);  counts / offsets [L][e_stride], total [L], pos [L][T * k_stride]
+// Rows inside an expert's segment come in no particular order (every row's product is computed by itself).
+__global__ void __launch_bounds__(1024)
+moe_plan_table_kernel(const long long* __restrict__ meta, const int* __restrict__ ids, int T, int* __restrict__ counts,
+                      int* __restrict__ offsets, int* __restrict__ pos, int* __restrict__ total_rows, int e_stride, int k_stride, int pad) {
+  __shared__ int s_cnt[1024];
+  __shared__ int s_off[1024];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int l = blockIdx.x;
+  const int* table = reinterpret_cast<const int*>(meta[4 * l]);
+  const int top = (int)meta[4 * l + 1], E = (int)meta[4 * l + 2], rows = (int)meta[4 * l + 3];
+  counts += (size_t)l * e_stride; offsets += (size_t)l * e_stride; pos += (size_t)l * T * k_stride;
+  const int pairs = T * top;
+  auto expert = [&](int i) {
+    int id = ids[i / top];
+    id = id < 0 ? 0 : (id >= rows ? rows - 1 : id);
+    const int e = table[(size_t)id * top + i % top];
+    return e < 0 || e >= E ? -1 : e;
+  };
+  for (int e = threadIdx.x; e < E; e += blockDim.x) s_cnt[e] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const int e = expert(i);
+    if (e >= 0) atomicAdd(&s_cnt[e], 1);
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    int carry = 0;
+    for (int base = 0; base < E; base += 32) {
+      const int e = base + threadIdx.x;
+      const int c = e < E ? (s_cnt[e] + pad - 1) / pad * pad : 0;
+      int incl = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, incl, o);
+        if ((int)threadIdx.x >= o) incl += v;
+      }
+      if (e < E) { counts[e] = s_cnt[e]; offsets[e] = s_off[e] = carry + incl - c; }
+      carry += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (threadIdx.x == 0) total_rows[l] = carry;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const int e = expert(i);
+    pos[i] = e < 0 ? -1 : atomicAdd(&s_off[e], 1);
+  }
+}
+
 // grouped dense GEMM: one (expert, chunk) per blockIdx.z
 template <int MPAD, bool BF16>
 __global__ void __launch_bounds__(192, 1)
@@ -293,6 +345,15 @@ extern "C" int fb_moe_plan(const int* idx, int T, int topk, int first, int n_loc
   return (int)cudaGetLastError();
 }
 
+extern "C" int fb_moe_plan_table(const long long* meta, int L, const int* ids, int T, int* counts, int* offsets, int* pos, int* total_rows,
+                                 int e_stride, int k_stride, int pad, void* stream) {
+  if (L <= 0 || T <= 0) return 0;
+  if (e_stride <= 0 || e_stride > 1024 || k_stride <= 0) return -1;
+  launch_k(moe_plan_table_kernel, dim3(L), dim3(1024), 0, reinterpret_cast<cudaStream_t>(stream), 0, meta, ids, T, counts, offsets, pos,
+           total_rows, e_stride, k_stride, pad);
+  return (int)cudaGetLastError();
+}
+
 extern "C" int fb_moe_gather(const void* x, const int* pos, void* xs, int T, int topk, int H, void* stream) {
   if (T <= 0) return 0;
   if (H % 8 != 0) return -1;
@@ -310,14 +371,16 @@ extern "C" int fb_moe_combine(const void* ys, const int* pos, const float* w, co
   return (int)cudaGetLastError();
 }
 
-// Grouped Y_e = X_e W_e^T over the sorted buffer.  Xs: [rows_cap, K] sorted rows; W: stacked [E_local * N, K]; out: [rows_cap, N or N/2].
+// Grouped Y_e = X_e W_e^T over the sorted buffer.  Xs: [rows_cap, K] sorted rows; W: stacked [E_local * N, K] with every
+// expert's rows padded to a multiple of 128; out: [rows_cap, N or N/2].
 // max_rows_per_expert bounds the chunk count (T for decode: every token could pick the same expert).
 extern "C" int fb_moe_grouped_gemm(const void* Xs, const void* W, void* out, const void* bias, const int* counts, const int* offsets,
                                    int rows_cap, int E_local, int N, int K, int ld_out, int max_rows_per_expert, int dtype, int flags,
                                    int total_rows, void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (E_local <= 0 || rows_cap <= 0) return 0;
-  if (K % 64 != 0 || N % 128 != 0 || (dtype != 0 && dtype != 1)) return -1;
+  if (K % 8 != 0 || N % 8 != 0 || ((flags & GEMM_SWIGLU) && N % 128 != 0) || (dtype != 0 && dtype != 1)) return -1;
+  const int n_rows_w = (N + 127) / 128 * 128;
   const bool bf16 = dtype == 1;
   // rows per chunk: low 16 bits of max_rows_per_expert = most rows an expert can get, high 16 bits = chunk size hint (0: auto)
   const int hint = max_rows_per_expert >> 16;
@@ -328,20 +391,20 @@ extern "C" int fb_moe_grouped_gemm(const void* Xs, const void* W, void* out, con
   GemmParams p;
   p.out = out; p.bias = bias; p.residual = nullptr;
   p.M = 0; p.N = N; p.K = K; p.ld_out = ld_out; p.ld_res = 0;
-  p.kb_total = K / 64; p.flags = flags;
+  p.kb_total = (K + 63) / 64; p.flags = flags;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
-  const int n_tiles = N / 128;
+  const int n_tiles = n_rows_w / 128;
   // k split: keep clusters small, experts already provide parallelism
   int nsplit = 1;
   while (nsplit < 4 && n_tiles * E_local * nsplit < 148 && (p.kb_total / (nsplit * 2)) >= 8) nsplit *= 2;
   p.kb_per_split = (p.kb_total + nsplit - 1) / nsplit;
   p.idesc = make_idesc(bf16 ? 1 : 0, bf16 ? 1 : 0, 0, 0, 128, mpad);
   MoeGroupInfo gi;
-  gi.counts = counts; gi.offsets = offsets; gi.rows_per_chunk = mpad; gi.chunks = chunks; gi.n_rows_w = N; gi.out_stride_e = 0;
+  gi.counts = counts; gi.offsets = offsets; gi.rows_per_chunk = mpad; gi.chunks = chunks; gi.n_rows_w = n_rows_w; gi.out_stride_e = 0;
   gi.ld_bias_e = N;
   CUtensorMap tmW, tmX;
-  if (!make_tmap_2d(&tmW, W, (uint64_t)E_local * N, K, K, 128, 64, 2, 3)) return -2;
+  if (!make_tmap_2d(&tmW, W, (uint64_t)E_local * n_rows_w, K, K, 128, 64, 2, 3)) return -2;
   if (!make_tmap_2d(&tmX, Xs, rows_cap, K, K, mpad, 64, 2, 3)) return -2;
   int nz = E_local * chunks;
   gi.n_local = E_local; gi.compact = 0;

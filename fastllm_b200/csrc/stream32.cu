@@ -1,0 +1,286 @@
+// Operators of models whose residual stream is fp32: token embedding plus sinusoidal positions, RMSNorm of an fp32 row into the
+// activation type, latent RMSNorm into the cache, and the mixture-of-experts combine that ends in residual and norm.
+//
+// One CTA owns a row; the row stays in shared memory between the reduction and the normalised write, so every operand is read
+// once.  Compiled without fast-math: angles, square roots and divisions are the correctly rounded fp32 ones.
+// Activation type codes: 0 fp16, 1 bf16, 2 fp32.
+#include "ptx.cuh"
+#include "launch.h"
+
+FB_DEFINE_ERROR_API(stream32)
+
+namespace fb {
+
+template <int DT>
+struct Act;
+template <>
+struct Act<0> {
+  typedef uint16_t T;
+  static __device__ __forceinline__ float ld(uint16_t v) { return __half2float(__ushort_as_half(v)); }
+  static __device__ __forceinline__ uint16_t st(float v) { return __half_as_ushort(__float2half_rn(v)); }
+};
+template <>
+struct Act<1> {
+  typedef uint16_t T;
+  static __device__ __forceinline__ float ld(uint16_t v) { return __bfloat162float(__ushort_as_bfloat16(v)); }
+  static __device__ __forceinline__ uint16_t st(float v) { return __bfloat16_as_ushort(__float2bfloat16_rn(v)); }
+};
+template <>
+struct Act<2> {
+  typedef float T;
+  static __device__ __forceinline__ float ld(float v) { return v; }
+  static __device__ __forceinline__ float st(float v) { return v; }
+};
+
+// four consecutive elements; the vector forms need 4-element alignment, which the launchers check
+template <int DT>
+__device__ __forceinline__ void ld4(const typename Act<DT>::T* p, float* v) {
+  if (DT == 2) {
+    const float4 t = *reinterpret_cast<const float4*>(p);
+    v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+  } else {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = unpack_16<DT == 1>(t.x), b = unpack_16<DT == 1>(t.y);
+    v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+  }
+}
+template <int DT>
+__device__ __forceinline__ void st4(typename Act<DT>::T* p, const float* v) {
+  if (DT == 2) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+  } else {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_16<DT == 1>(v[0], v[1]), pack_16<DT == 1>(v[2], v[3]));
+  }
+}
+
+__device__ __forceinline__ float block_sum32(float v, float* sh) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  if ((threadIdx.x & 31) == 0) sh[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) t += sh[w];
+  return t;
+}
+
+// y = row * inv * w from the shared-memory copy of the row
+template <int DT, int VEC>
+__device__ __forceinline__ void norm_write(const float* row, const typename Act<DT>::T* w, typename Act<DT>::T* y, int H, float inv) {
+  if (VEC == 4) {
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+      float wv[4], o[4];
+      ld4<DT>(w + i, wv);
+      const float4 r = *reinterpret_cast<const float4*>(row + i);
+      o[0] = r.x * inv * wv[0]; o[1] = r.y * inv * wv[1]; o[2] = r.z * inv * wv[2]; o[3] = r.w * inv * wv[3];
+      st4<DT>(y + i, o);
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) y[i] = Act<DT>::st(row[i] * inv * Act<DT>::ld(w[i]));
+  }
+}
+
+// y[row] = RMSNorm(x[row]) * w
+template <int DT, int VEC>
+__global__ void rmsnorm32_kernel(const float* __restrict__ x, const typename Act<DT>::T* __restrict__ w, typename Act<DT>::T* __restrict__ y,
+                                 int H, int ldx, int ldy, float eps) {
+  extern __shared__ float row[];
+  __shared__ float sh[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* xp = x + (size_t)blockIdx.x * ldx;
+  float ss = 0.f;
+  if (VEC == 4) {
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(xp + i);
+      *reinterpret_cast<float4*>(row + i) = v;
+      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+  } else {
+    for (int i = threadIdx.x; i < H; i += blockDim.x) { const float v = xp[i]; row[i] = v; ss += v * v; }
+  }
+  ss = block_sum32(ss, sh);
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  norm_write<DT, VEC>(row, w, y + (size_t)blockIdx.x * ldy, H, inv);
+}
+
+// h[t] = table[ids[t]] + sinusoid(positions[t]) in fp32, and its RMSNorm.  inv_freq[i] = 10000^(-2i / H) in double; the angle is
+// reduced to [-pi, pi] in double, so a far position costs no accuracy.
+template <int DT>
+__global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ positions, const typename Act<DT>::T* __restrict__ table,
+                                      const double* __restrict__ inv_freq, const typename Act<DT>::T* __restrict__ w, float* __restrict__ h,
+                                      typename Act<DT>::T* __restrict__ y, int H, int vocab, float eps) {
+  extern __shared__ float row[];
+  __shared__ float sh[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
+  const typename Act<DT>::T* e = table + (size_t)id * H;
+  float* hp = h + (size_t)t * H;
+  const double pos = (double)positions[t];
+  float ss = 0.f;
+  for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
+    float a = Act<DT>::ld(e[2 * i]);
+    if (inv_freq != nullptr) {
+      const double ang = pos * inv_freq[i];
+      const float red = (float)(ang - 6.283185307179586476925 * rint(ang * 0.15915494309189533577));
+      float s, c;
+      sincosf(red, &s, &c);
+      a += s;
+      if (2 * i + 1 < H) {
+        const float b = Act<DT>::ld(e[2 * i + 1]) + c;
+        hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b;
+      }
+    } else if (2 * i + 1 < H) {
+      const float b = Act<DT>::ld(e[2 * i + 1]);
+      hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b;
+    }
+    hp[2 * i] = a; row[2 * i] = a; ss += a * a;
+  }
+  ss = block_sum32(ss, sh);
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  norm_write<DT, 1>(row, w, y + (size_t)t * H, H, inv);
+}
+
+// pool[slot] = RMSNorm over the first `n` columns of x[t] (columns [n, ld) of the entry are zero); slots < 0 go to `spare`
+template <int DT>
+__global__ void latent_norm_kernel(const typename Act<DT>::T* __restrict__ x, int ldx, const typename Act<DT>::T* __restrict__ w,
+                                   const int* __restrict__ slots, typename Act<DT>::T* __restrict__ pool, int n, int ld, long long spare, float eps) {
+  extern __shared__ float row[];
+  __shared__ float sh[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  const typename Act<DT>::T* xp = x + (size_t)t * ldx;
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = Act<DT>::ld(xp[i]); row[i] = v; ss += v * v; }
+  ss = block_sum32(ss, sh);
+  const float inv = 1.0f / sqrtf(ss / (float)n + eps);
+  const int slot = slots[t];
+  typename Act<DT>::T* yp = pool + (size_t)(slot < 0 ? spare : (long long)slot) * ld;
+  for (int i = threadIdx.x; i < ld; i += blockDim.x) yp[i] = Act<DT>::st(i < n ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+}
+
+// h[t] += alpha * (sum_k wk * ys[pos[t, k]] + shared[t]), then y[t] = RMSNorm(h[t]) * w.  wts == nullptr: every weight is `wconst`.
+template <int DT, int VEC>
+__global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict__ ys, const int* __restrict__ pos, const float* __restrict__ wts,
+                                          float wconst, const typename Act<DT>::T* __restrict__ shared_y, float* __restrict__ h,
+                                          const typename Act<DT>::T* __restrict__ w, typename Act<DT>::T* __restrict__ y, int topk, int H,
+                                          float alpha, float eps) {
+  extern __shared__ float row[];
+  __shared__ float sh[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  float* hp = h + (size_t)t * H;
+  float ss = 0.f;
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+    float acc[VEC], v[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) acc[j] = 0.f;
+    for (int k = 0; k < topk; ++k) {
+      const int r = pos[(size_t)t * topk + k];
+      if (r < 0) continue;
+      const float wk = wts != nullptr ? wts[(size_t)t * topk + k] : wconst;
+      if (VEC == 4) ld4<DT>(ys + (size_t)r * H + i, v); else v[0] = Act<DT>::ld(ys[(size_t)r * H + i]);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc[j] += wk * v[j];
+    }
+    if (shared_y != nullptr) {
+      if (VEC == 4) ld4<DT>(shared_y + (size_t)t * H + i, v); else v[0] = Act<DT>::ld(shared_y[(size_t)t * H + i]);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc[j] += v[j];
+    }
+    if (VEC == 4) ld4<2>(hp + i, v); else v[0] = hp[i];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { v[j] += alpha * acc[j]; ss += v[j] * v[j]; row[i + j] = v[j]; }
+    if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
+  }
+  ss = block_sum32(ss, sh);
+  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+  norm_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
+}
+
+// dst[i] = src[idx[i]] for rows of `vecs` 16-byte units
+__global__ void gather_rows_kernel(const uint4* __restrict__ src, const long long* __restrict__ idx, uint4* __restrict__ dst, int rows, int vecs) {
+  const long long total = (long long)rows * vecs;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int r = (int)(i / vecs), c = (int)(i - (long long)r * vecs);
+    dst[i] = src[idx[r] * vecs + c];
+  }
+}
+
+constexpr int S32_MAX_ROW = 49152;           // floats of the shared-memory row buffer
+static int row_threads(int H, int vec) {
+  int n = (H / vec + 31) / 32 * 32;
+  return n < 64 ? 64 : n > 512 ? 512 : n;
+}
+
+}  // namespace fb
+
+using namespace fb;
+
+#define S32_LAUNCH(kern, grid, threads, H, stream, ...)                                                                            \
+  {                                                                                                                                \
+    static DeviceOnce cfg_;                                                                                                        \
+    if (cfg_.need()) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, S32_MAX_ROW * 4);                     \
+    launch_k(kern, dim3(grid), dim3(threads), (size_t)(H) * 4, reinterpret_cast<cudaStream_t>(stream), 0, __VA_ARGS__);             \
+  }
+
+extern "C" int fb_rmsnorm32(const float* x, const void* w, void* y, int M, int H, int ldx, int ldy, float eps, int dt, void* stream) {
+  if (M <= 0) return 0;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  const bool vec = H % 4 == 0 && ldx % 4 == 0 && ldy % 4 == 0;
+  const int th = row_threads(H, vec ? 4 : 1);
+#define GO(DT, V) S32_LAUNCH((rmsnorm32_kernel<DT, V>), M, th, H, stream, x, (const Act<DT>::T*)w, (Act<DT>::T*)y, H, ldx, ldy, eps)
+  if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
+  else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const void* table, const double* inv_freq, const void* w, float* h,
+                                 void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  const int th = row_threads(H, 2);
+#define GO(DT) S32_LAUNCH((embed_pos_norm_kernel<DT>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
+  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+extern "C" int fb_latent_norm(const void* x, int ldx, const void* w, const int* slots, void* pool, int T, int n, int ld, long long spare,
+                              float eps, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (n <= 0 || ld < n || n > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  const int th = row_threads(ld, 2);
+#define GO(DT) S32_LAUNCH((latent_norm_kernel<DT>), T, th, n, stream, (const Act<DT>::T*)x, ldx, (const Act<DT>::T*)w, slots, (Act<DT>::T*)pool, n, ld, spare, eps)
+  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+extern "C" int fb_moe_combine_norm32(const void* ys, const int* pos, const float* wts, float wconst, const void* shared_y, float* h,
+                                     const void* w, void* y, int T, int topk, int H, float alpha, float eps, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  const bool vec = H % 4 == 0;
+  const int th = row_threads(H, vec ? 4 : 1);
+#define GO(DT, V) S32_LAUNCH((moe_combine_norm32_kernel<DT, V>), T, th, H, stream, (const Act<DT>::T*)ys, pos, wts, wconst, (const Act<DT>::T*)shared_y, h, (const Act<DT>::T*)w, (Act<DT>::T*)y, topk, H, alpha, eps)
+  if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
+  else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+extern "C" int fb_gather_rows(const void* src, const long long* idx, void* dst, int rows, int row_bytes, void* stream) {
+  if (rows <= 0) return 0;
+  if (row_bytes <= 0 || row_bytes % 16 != 0) return -1;
+  const int vecs = row_bytes / 16;
+  long long blocks = ((long long)rows * vecs + 255) / 256;
+  if (blocks > 148 * 16) blocks = 148 * 16;
+  launch_k(gather_rows_kernel, dim3((unsigned)blocks), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), 0, (const uint4*)src, idx, (uint4*)dst, rows, vecs);
+  return (int)cudaGetLastError();
+}

@@ -79,4 +79,20 @@ inline bool make_tmap_2d(CUtensorMap* out, const void* ptr, uint64_t rows, uint6
   return true;
 }
 
+// 3-D map over 16-bit data: (inner, mid, rows) with strides of `mid` and `row` elements, one mid index per box, 128-byte swizzle.
+// The inner extent bounds every box on its own, so a head narrower than the 64-column box is padded with zeros instead of with
+// its neighbour.  Not cached: prefill calls build it from fresh buffers.
+inline bool make_tmap_3d(CUtensorMap* out, const void* ptr, uint64_t inner, uint64_t mid, uint64_t rows, uint64_t mid_stride,
+                         uint64_t row_stride, uint32_t box_inner, uint32_t box_rows) {
+  EncodeTiledFn fn = get_encode_fn();
+  if (!fn) return false;
+  if ((reinterpret_cast<uintptr_t>(ptr) & 15) || ((mid_stride * 2) & 15) || ((row_stride * 2) & 15)) return false;
+  cuuint64_t gdim[3] = {inner, mid, rows};
+  cuuint64_t gstride[2] = {mid_stride * 2, row_stride * 2};
+  cuuint32_t box[3] = {box_inner, 1, box_rows};
+  cuuint32_t estr[3] = {1, 1, 1};
+  return fn(out, CU_TENSOR_MAP_DATA_TYPE_UINT16, 3, const_cast<void*>(ptr), gdim, gstride, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
 }  // namespace fb

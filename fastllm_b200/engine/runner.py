@@ -64,7 +64,7 @@ class _DecodeSlot:
         m = runner.model
         G = max(1, max([m.num_heads_local] + [lw.attn.heads or 0 for lw in m.layers]) // m.num_kv_heads_local)
         self.ws = None
-        if dev.type == "cuda" and not m.cfg.use_mla:
+        if dev.type == "cuda" and not m.cfg.use_mla and m.cfg.mixers is None:
             windows = {int(lw.attn.window) for lw in m.layers if lw.attn.window}
             # one sliding-window length per model is planned alongside the full list (layers alternate local / global)
             self.ws = A.DecodeWorkspace(bsz, m.num_kv_heads_local, G, P, dev, m.cfg.head_dim, window=windows.pop() if len(windows) == 1 else 0)
@@ -93,7 +93,8 @@ class ModelRunner:
         self.steps = 0
         self.kernel_launches = 0
         self.launches_per_decode_step = 0
-        model.rope_tables()
+        if model.rope_mode != A.ROPE_NONE:
+            model.rope_tables()
 
     def _agree_on_pages(self, num_pages: int) -> int:
         """Page ids are chosen by the scheduler rank and used by every rank: all pools get the smallest planned size."""
@@ -121,6 +122,8 @@ class ModelRunner:
         c = self.model.cfg
         if getattr(self.model, "layer_devices", None) is not None:
             return False        # one graph cannot span the devices of a layer-split placement
+        if c.mixers is not None:       # every kernel of these layers is captured; experts must be on the grouped path
+            return all(lw.mlp.experts is None or lw.mlp.experts.stacked is not None for lw in self.model.layers)
         if c.use_mla and not (c.kv_lora_rank == 512 and c.qk_rope_head_dim == 64 and self.model.dtype in (torch.float16, torch.bfloat16)):
             return False        # latent shapes outside the MLA decode kernel run the PyTorch evaluation
         kvd = getattr(self.model, "kv_dtype", None)
@@ -143,7 +146,8 @@ class ModelRunner:
     # ---------------------------------------------------------------------------------------------
     def prefill(self, chunks, keep_hidden: bool = False, mtp_hidden=None):
         """chunks: list of (token_ids, start_pos, pages, want_logits). Returns fp32 logits ``[R, V_local]``
-        for the chunks that asked for them (last token of the chunk), in order.
+        for the chunks that asked for them, in order.  ``want_logits``: True for the last token of the chunk, an integer n > 1 for
+        its last n tokens, a list for the tokens at these places of the chunk.
 
         ``keep_hidden``: the final-normed rows of the whole packed batch stay in ``model.last_hidden`` (the draft head reads
         them).  ``mtp_hidden``: run the draft head instead of the decoder -- the chunks then hold, per position, the token that
@@ -185,7 +189,9 @@ class ModelRunner:
             cu.append(cu[-1] + n)
             kv_lens.append(start + n)
             pt[b, :len(pages)] = pages
-            if want:
+            if isinstance(want, (list, tuple)):
+                rows.extend(cu[-2] + int(w) for w in want)
+            elif want:
                 # True: the chunk's last row; an integer n > 1: its last n rows (speculative verification reads them all)
                 nrows = 1 if want is True else max(1, min(int(want), n))
                 rows.extend(range(cu[-1] - nrows, cu[-1]))
@@ -211,6 +217,7 @@ class ModelRunner:
             if ex_rows:
                 fb.expert_rows = torch.tensor(ex_rows, dtype=torch.long, device=dev)
         fb.kv_max_host = max(kv_lens) if kv_lens else 0
+        fb.kv_lens_host = kv_lens
         if mtp_hidden is not None:
             logits, x = self.model.mtp_forward(fb, mtp_hidden, self.kv.pools)
             return (logits if rows else None), x

@@ -80,6 +80,15 @@ def dequant_awq(qweight: torch.Tensor, qzeros: torch.Tensor, scales: torch.Tenso
 # name canonicalisation: every family is mapped onto the Llama naming that loader.shard understands
 # ---------------------------------------------------------------------------------------------------
 _RENAMES = [
+    # Patesun
+    (r"^embed$", "model.embed_tokens.weight"), (r"^final\.norm$", "model.norm.weight"), (r"^head$", "lm_head.weight"),
+    (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"), (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
+    (r"^l(\d+)\.mix\.dkv\.norm$", r"model.layers.\1.self_attn.kv_a_layernorm.weight"), (r"^l(\d+)\.mix\.dkv$", r"model.layers.\1.self_attn.kv_a_proj.weight"),
+    (r"^l(\d+)\.mix\.uk$", r"model.layers.\1.self_attn.k_b_proj.weight"), (r"^l(\d+)\.mix\.uv$", r"model.layers.\1.self_attn.v_b_proj.weight"),
+    (r"^l(\d+)\.mix\.([qgo])$", r"model.layers.\1.self_attn.\2_proj.weight"), (r"^l(\d+)\.mlp\.(up|down)$", r"model.layers.\1.mlp.\2_proj.weight"),
+    (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
+    (r"^l(\d+)\.mlp\.shared\.(gate|up|down)$", r"model.layers.\1.mlp.shared_experts.\2_proj.weight"),
+    (r"^l(\d+)\.mlp\.table$", r"model.layers.\1.mlp.token_table"),
     (r"\.mlp\.moe_statics\.e_score_correction_bias", ".mlp.gate.e_score_correction_bias"),          # Ernie-4.5-MoE
     (r"\.block_sparse_moe\.e_score_correction_bias", ".mlp.gate.e_score_correction_bias"),          # MiniMax-M2
     (r"\.mlp\.e_score_correction_bias", ".mlp.gate.e_score_correction_bias"),
@@ -306,6 +315,8 @@ def load_model(path: str | Path, device="cuda", dtype=None, wdtype: str = "auto"
         if tp is not None and tp.size > 1:
             raise NotImplementedError("cogvlm runs on one rank")
         m = CogVLMModel(cfg, device, dtype, tp, ep)
+    elif cfg.mixers is not None and tp is not None and tp.size > 1:
+        raise NotImplementedError(f"{cfg.model_type} runs on one rank")
     else:
         m = DecoderModel(cfg, device, dtype, tp, ep)
     m.moe_disk = moe_device == "disk"

@@ -104,6 +104,12 @@ def build_layer(m, i: int, t: dict, wdtype="dense", moe_wdtype=None):
         f.ln = _to(g("post_attention_layernorm.weight"), m)
         a.post_ln = _to(g("post_self_attn_layernorm.weight"), m)     # GLM-4
         f.post_ln = _to(g("post_mlp_layernorm.weight"), m)
+    if cfg.mixers is not None:
+        _build_listed_layer(m, i, lw, g, wdtype, moe_wdtype or wdtype)
+        while len(m.layers) <= i:
+            m.layers.append(None)
+        m.layers[i] = lw
+        return
     if cfg.layer_windows is not None and i < len(cfg.layer_windows):
         a.window = int(cfg.layer_windows[i])
     elif cfg.sliding_window and cfg.sliding_window < cfg.max_position:
@@ -301,6 +307,50 @@ def build_layer(m, i: int, t: dict, wdtype="dense", moe_wdtype=None):
     m.layers[i] = lw
 
 
+def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
+    """Mixer and feed-forward of a model that lists its layers (``cfg.mixers`` / ``cfg.ffs``).  Widths are padded with zero rows and
+    columns to what the kernels tile (the padding stays zero through every product)."""
+    from ..ops import latent as LA
+
+    cfg = m.cfg
+    spec, ff = cfg.mixers[i], cfg.ffs[i]
+    t = lambda k: _to(g("self_attn." + k + ".weight"), m)
+    exact = m.dtype == torch.float32
+
+    def lin(w, kind=wdtype, interleaved=False):
+        l = LinearWeight.from_dense(w, kind, None, interleaved, act_dtype=m.dtype)
+        l.exact32 = exact
+        return l
+
+    def gate_up(gw, uw, kind):
+        if m.on_cuda:
+            return lin(B.interleave_gate_up(LA.pad_rows(_to(gw, m), 64), LA.pad_rows(_to(uw, m), 64)), kind, True)
+        return lin(torch.cat([_to(gw, m), _to(uw, m)], dim=0), kind)
+
+    def down(w, kind, mult):
+        return lin(LA.pad_cols(_to(w, m), mult if m.on_cuda else 1).contiguous(), kind)
+
+    la, in_w = LA.build(spec, t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"))
+    la.in_proj = lin(in_w)
+    lw.latent = la
+    lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
+    f = lw.mlp
+    if ff.kind == "none":
+        f.absent = True
+    elif ff.kind == "dense":
+        f.act = ff.act
+        f.up = lin(LA.pad_rows(_to(g("mlp.up_proj.weight"), m), 8 if m.on_cuda else 1))
+        f.down = down(g("mlp.down_proj.weight"), wdtype, 8)
+    else:
+        f.route_table = g("mlp.token_table").to(m.device, torch.int32).contiguous()
+        names = [f"mlp.experts.{e}." for e in range(ff.experts)]
+        f.experts = MOE.ExpertWeights(ff.experts, 0, [gate_up(g(n + "gate_proj.weight"), g(n + "up_proj.weight"), moe_wdtype) for n in names],
+                                      [down(g(n + "down_proj.weight"), moe_wdtype, 64) for n in names])
+        if ff.shared_ff:
+            f.shared_gate_up = gate_up(g("mlp.shared_experts.gate_proj.weight"), g("mlp.shared_experts.up_proj.weight"), wdtype)
+            f.shared_down = down(g("mlp.shared_experts.down_proj.weight"), wdtype, 64)
+
+
 def build_linear_attn(m, g, ln, W, layer_idx: int = 0):
     """Gated-DeltaNet weights of one layer for this rank.  Accepts the grouped layout of Qwen3-Next (``in_proj_qkvz`` /
     ``in_proj_ba``, rows grouped per key head) and the plain layout of Qwen3.5 (``in_proj_qkv``, ``in_proj_z``, ``in_proj_b``,
@@ -406,7 +456,13 @@ def build_top(m, t: dict, wdtype="dense"):
         if head is t["model.embed_tokens.weight"] and m.embed is not None and hb is None:
             m.lm_head = LinearWeight("dense", m.embed, dtype=m.dtype)
         else:
+            if cfg.mixers is not None and m.on_cuda and head.shape[0] % 8:
+                from ..ops.latent import pad_rows
+
+                m.vocab_pad_from = head.shape[0]                  # the head's GEMM wants a multiple of 8 rows
+                head = pad_rows(head, 8)
             m.lm_head = _lin(m, head, "dense", hb)
+            m.lm_head.exact32 = cfg.mixers is not None and m.dtype == torch.float32
 
 
 def finalize_model(m, top_fn, layer_fn, wdtype="dense", moe_wdtype=None):
@@ -419,7 +475,12 @@ def finalize_model(m, top_fn, layer_fn, wdtype="dense", moe_wdtype=None):
     for i in range(m.cfg.num_layers):
         if staged is not None:
             m.device = staged[i]           # the builders place tensors on m.device
-        build_layer(m, i, layer_fn(i), wdtype, moe_wdtype)
+        src = m.cfg.layer_runs[i] if m.cfg.layer_runs is not None else i
+        if m.cfg.layer_runs is not None and src in m.cfg.layer_runs[:i]:
+            m.layers.append(m.layers[m.cfg.layer_runs.index(src)])       # another pass over the same weights
+            continue
+        build_layer(m, i, layer_fn(src) if src == i else {k.replace(f"model.layers.{src}.", f"model.layers.{i}.", 1): v for k, v in layer_fn(src).items()},
+                    wdtype, moe_wdtype)
         progress.emit("load_weights", i + 1, m.cfg.num_layers)
     m.device = home
     if staged is not None:                 # the head runs where the last layer left the activations

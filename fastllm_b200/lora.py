@@ -59,7 +59,7 @@ def _block(pairs, rows):
 def load_adapter(model, name: str, adapter_dir) -> int:
     """Attach the adapter in ``adapter_dir`` to ``model`` under ``name``; returns the number of adapted projections."""
     cfg = model.cfg
-    if model.tp.size != 1 or cfg.use_mla:
+    if model.tp.size != 1 or cfg.use_mla or cfg.mixers is not None:
         raise NotImplementedError("run-time adapters cover dense-attention models on one tensor-parallel rank; "
                                   "use llm.model(path, lora=adapter_dir) to merge the adapter at load")
     lo = _read(adapter_dir)

@@ -12,6 +12,31 @@ from pathlib import Path
 
 
 @dataclass
+class LatentSpec:
+    """Latent attention of one layer: per-head keys and values are projections of one cached, RMS-normalised latent row; no
+    positions enter the scores."""
+    heads: int
+    dim: int                # query / key dimensions per head
+    vdim: int
+    kv_rank: int
+    scale: float
+    window: int = 0         # keys a query sees, itself included (0: all before it)
+
+
+@dataclass
+class FFSpec:
+    """Feed-forward of one layer where the layers of a model differ: "dense" (up -> act -> down), "moe" (routed SwiGLU experts plus
+    an optional shared one) or "none"."""
+    kind: str = "none"
+    ff: int = 0
+    act: str = "relu2"
+    experts: int = 0
+    top: int = 0
+    expert_ff: int = 0
+    shared_ff: int = 0      # 0: no shared expert
+
+
+@dataclass
 class ModelConfig:
     model_type: str = "llama"
     architectures: list = field(default_factory=list)
@@ -94,6 +119,14 @@ class ModelConfig:
     lin_conv_kernel: int = 4
     lin_kind: str = "gdn"                  # "gdn" Gated DeltaNet | "lightning" decayed linear attention (MiniMax-Text-01 / M1)
     lin_block: int = 256                   # lightning attention: block length of the chunked evaluation
+    # models whose layers are listed one by one (Patesun): the mixer and feed-forward of every layer, and which layer's weights each
+    # run of the stack uses (looped layers appear once per pass; num_layers counts the runs, every run has its own cache)
+    mixers: list | None = None             # LatentSpec per run
+    ffs: list | None = None                # FFSpec per run
+    layer_runs: list | None = None
+    residual_f32: bool = False             # the residual stream is fp32; sub-layer outputs join it times residual_mult
+    residual_mult: float = 1.0
+    pos_embed_base: float = 0.0            # > 0: sinusoidal positions with this base are added to the token embedding
     # DeepNorm-style residual (MiniMax-Text-01 / M1): the block input is normalised first and the NORMALISED rows are the
     # residual: y = alpha * norm(x) + beta * f(norm(x)).  (alpha, beta) for full-attention layers, linear layers, MLPs.
     postnorm_residual: bool = False
@@ -154,6 +187,8 @@ def from_hf_dict(d: dict) -> ModelConfig:
             if k in d and k not in inner:
                 inner[k] = d[k]
         d = inner
+    if d.get("architecture") == "Patesun":
+        return _patesun(d)
     mt = d.get("model_type", "llama")
     if "CogVLMForCausalLM" in (d.get("architectures") or []) or mt == "CogVLMForCausalLM":
         mt = "cogvlm"                                   # the checkpoint's config names no model_type
@@ -521,6 +556,55 @@ def _step_family(c: ModelConfig, g, mt: str) -> None:
     c.first_k_dense = 0
 
 
+def _patesun(d: dict) -> ModelConfig:
+    """Patesun: a list of layers (latent attention with a sliding window and an output gate; ReLU^2 MLP or experts picked by token
+    id), a span of layers that runs several times, fp32 residuals with a multiplier, sinusoidal positions."""
+    L = d["layers"]
+    mixers, ffs = [], []
+    for i, spec in enumerate(L):
+        if spec.get("type") != "latent_attention":
+            raise NotImplementedError(f"Patesun: layer {i} has mixer '{spec.get('type')}'")
+        m = spec["mixer"]
+        mixers.append(LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]),
+                                 int((m.get("mask") or {}).get("size") or 0)))
+        f = spec.get("mlp")
+        if f is None:
+            ffs.append(FFSpec())
+        elif f.get("kind") == "dense":
+            ffs.append(FFSpec("dense", ff=int(f["ff"])))
+        elif f.get("kind") == "moe":
+            ffs.append(FFSpec("moe", act="silu", experts=int(f["router"]["experts"]), top=int(f["router"]["top"]),
+                              expert_ff=int(f["expert"]["ff"]), shared_ff=int((f.get("shared") or {}).get("ff") or 0)))
+        else:
+            raise NotImplementedError(f"Patesun: layer {i} has feed-forward '{f.get('kind')}'")
+    runs = list(range(len(L)))
+    loop = d.get("loop")
+    if loop:
+        a, b = int(loop["start"]), int(loop["stop"])
+        runs = runs[:a] + runs[a:b] * int(loop["times"]) + runs[b:]
+    c = ModelConfig(model_type="patesun", raw=d, architectures=["Patesun"])
+    c.vocab_size, c.hidden_size = int(d["vocab"]), int(d["width"])
+    c.layer_runs = runs
+    c.num_layers = len(runs)
+    c.mixers, c.ffs = [mixers[i] for i in runs], [ffs[i] for i in runs]
+    c.num_heads = c.num_kv_heads = max((m.heads for m in mixers), default=1)
+    c.head_dim = max((m.dim for m in mixers), default=1)
+    c.intermediate_size = max((f.ff for f in ffs), default=0)
+    c.num_experts = max((f.experts for f in ffs), default=0)
+    c.num_experts_per_tok = max((f.top for f in ffs), default=0)
+    c.moe_intermediate_size = max((f.expert_ff for f in ffs), default=0)
+    c.rms_eps = float(d["norm"]["eps"])
+    c.residual_f32 = True
+    c.residual_mult = float(d.get("residual_mult", 1.0))
+    c.pos_embed_base = 10000.0
+    c.rope_mode = "none"
+    c.max_position = int(d.get("max_position_embeddings", 1 << 20))
+    c.eos_token_ids = _eos_list(d.get("eos_token_id"))
+    c.bos_token_id = d.get("bos_token_id")
+    c.torch_dtype = str(d.get("torch_dtype", d.get("dtype", "bfloat16"))).replace("torch.", "")
+    return c
+
+
 def load_config(path: str | Path) -> ModelConfig:
     p = Path(path)
     if p.is_dir():
@@ -650,6 +734,21 @@ def preset(name: str) -> ModelConfig:
                                  scoring_func="sigmoid", topk_method="noaux_tc", norm_topk_prob=True, q_lora_rank=128,
                                  kv_lora_rank=64, qk_nope_head_dim=32, qk_rope_head_dim=16, v_head_dim=32,
                                  rms_norm_eps=1e-6, rope_theta=10000.0, max_position_embeddings=2048))
+    if name == "tiny-patesun":           # two windows and head shapes, a looped layer, dense / table-routed / no feed-forward
+        mx = lambda h, d, v, r, w: {"heads": h, "dim": d, "vdim": v, "kv_rank": r, "scale": d ** -0.5, "mask": {"size": w}}
+        moe = {"kind": "moe", "expert": {"ff": 64}, "router": {"experts": 6, "top": 3}, "shared": {"ff": 128}}
+        return from_hf_dict(dict(architecture="Patesun", vocab=512, width=192, norm={"eps": 1e-5}, residual_mult=0.5,
+                                 loop={"start": 1, "stop": 2, "times": 2},
+                                 layers=[{"type": "latent_attention", "mixer": mx(4, 48, 32, 72, 24), "mlp": {"kind": "dense", "ff": 320}},
+                                         {"type": "latent_attention", "mixer": mx(6, 32, 40, 128, 33), "mlp": moe},
+                                         {"type": "latent_attention", "mixer": mx(2, 64, 64, 64, 150), "mlp": None}]))
+    if name == "patesun-9b":             # layers of a served model's size: 2048-token windows, 64 experts of 1024
+        mx = {"heads": 32, "dim": 128, "vdim": 128, "kv_rank": 512, "scale": 128 ** -0.5, "mask": {"size": 2048}}
+        moe = {"kind": "moe", "expert": {"ff": 1024}, "router": {"experts": 64, "top": 6}, "shared": {"ff": 2048}}
+        return from_hf_dict(dict(architecture="Patesun", vocab=128256, width=4096, norm={"eps": 1e-6}, residual_mult=0.4,
+                                 loop={"start": 1, "stop": 5, "times": 2},
+                                 layers=[{"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": 14336}}]
+                                 + [{"type": "latent_attention", "mixer": mx, "mlp": moe} for _ in range(7)]))
     if name == "tiny-deepseek-v32":      # latent attention with the sparse-attention indexer (selection size 32)
         return from_hf_dict(dict(model_type="deepseek_v32", vocab_size=512, hidden_size=256, num_hidden_layers=2,
                                  num_attention_heads=4, num_key_value_heads=4, intermediate_size=512,

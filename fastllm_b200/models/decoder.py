@@ -22,7 +22,9 @@ import torch.nn.functional as F
 
 from ..ops import attention as A
 from ..ops import basic as B
+from ..ops import latent as LA
 from ..ops import moe as MOE
+from ..ops import stream32 as S
 from ..ops.quant import LinearWeight
 from .config import ModelConfig
 
@@ -49,6 +51,7 @@ class ForwardBatch:
     rope_pos3: torch.Tensor | None = None
     expert_rows: torch.Tensor | None = None      # rows evaluated with a model's visual-expert weights (models/cogvlm.py)
     keep_hidden: bool = False                    # leave the final-normed rows of the whole batch in ``model.last_hidden``
+    kv_lens_host: list | None = None             # kv_lens as known on the host (prefill batches)
     kv_max_host: int = 0                         # longest context of the batch, known on the host (sparse-attention switch)
 
 
@@ -123,6 +126,9 @@ class MLPWeights:
         self.up: LinearWeight | None = None      # two-matrix MLPs (no gate): up -> activation -> down
         self.down: LinearWeight | None = None
         self.post_ln = None      # sandwich norm on the MLP output
+        self.act = ""            # activation of a two-matrix MLP where it is the layer's own (default: the model's hidden_act)
+        self.absent = False      # the layer has no feed-forward
+        self.route_table = None  # int32 [vocab, top]: experts of every token id (no router), equal weights
         self.act_limit = 0.0     # clamp inside the dense / shared-expert SwiGLU (Step-3.5); 0: none
         # MoE
         self.router = None          # fp32 [E, H]
@@ -140,6 +146,7 @@ class LayerWeights:
     def __init__(self):
         self.attn = AttentionWeights()
         self.mlp = MLPWeights()
+        self.latent: LA.LatentWeights | None = None    # latent attention without positions (``attn`` keeps its norm and output projection)
         self.lin: LinearAttnWeights | None = None      # set instead of ``attn`` projections on linear-attention layers
 
 
@@ -178,6 +185,7 @@ class DecoderModel:
         self.num_kv_heads_local = max(1, cfg.num_kv_heads // self.tp.size)
         self.kv_replicas = max(1, self.tp.size // cfg.num_kv_heads)
         self._rope = None
+        self.vocab_pad_from = 1 << 62     # logit columns from here on are padding of the output head
         self._fused_active = False
         self._beta = 1.0                  # scale of the running sub-layer's contribution (DeepNorm-style residual models)
         self.layer_devices = None          # per-layer devices for the layer-split placement (None: everything on self.device)
@@ -247,6 +255,8 @@ class DecoderModel:
     def kv_cache_shape(self, num_pages: int):
         """Per-layer page-pool shapes of this rank: (K shape, V shape or None for MLA)."""
         c = self.cfg
+        if c.mixers is not None:
+            return self.kv_cache_shape_layer(0, num_pages)
         if c.use_mla:
             # one spare page at the end: rows that must not be cached (padded decode rows) are written there
             idx = (num_pages + 1, A.PAGE_LEN, 1, c.index_head_dim) if (c.index_topk and getattr(self, "has_indexer", False)) else None
@@ -254,7 +264,17 @@ class DecoderModel:
         s = (num_pages, A.PAGE_LEN, self.num_kv_heads_local, c.head_dim)
         return s, s
 
+    def kv_cache_shape_layer(self, i: int, num_pages: int):
+        """Pool shapes of layer ``i``: the model-wide ones, or a latent row per token where layers are listed one by one (plus a
+        spare page for rows that must not be cached)."""
+        if self.cfg.mixers is None:
+            return self.kv_cache_shape(num_pages)
+        return (num_pages + 1, A.PAGE_LEN, 1, (self.cfg.mixers[i].kv_rank + 7) // 8 * 8), None
+
     def kv_bytes_per_page(self) -> int:
+        if self.cfg.mixers is not None:
+            n = sum(math.prod(self.kv_cache_shape_layer(i, 1)[0][1:]) for i in range(self.cfg.num_layers))
+            return n * torch.finfo(self.dtype).bits // 8
         ks, vs = self.kv_cache_shape(1)
         n = math.prod(ks) + (math.prod(vs) if vs else 0)
         paged_layers = sum(1 for i in range(self.cfg.num_layers) if not self.cfg.layer_is_linear(i)) + (1 if self.mtp is not None else 0)
@@ -291,7 +311,7 @@ class DecoderModel:
         dt = table[name]
         if dt == self.dtype:
             return
-        if self.cfg.use_mla:
+        if self.cfg.use_mla or self.cfg.mixers is not None:
             raise NotImplementedError("the MLA latent cache is kept in the activation dtype")
         self.kv_dtype = dt
         self.general_attn = True              # prefill (and everything the decode kernel does not cover) evaluates attention in PyTorch
@@ -466,6 +486,8 @@ class DecoderModel:
         return self.tp.comm.row_linear(w, x, residual)
 
     def _norm(self, h, ln_w):
+        if self.cfg.residual_f32:
+            return S.rmsnorm32(h, ln_w, self.cfg.rms_eps)
         if self.cfg.norm_kind == "layernorm":
             return F.layer_norm(h.float(), (h.shape[-1],), ln_w.float(), self.ln_bias[id(ln_w)].float() if id(ln_w) in self.ln_bias else None,
                                 self.cfg.rms_eps).to(h.dtype)
@@ -506,6 +528,9 @@ class DecoderModel:
         all-gather to land: that wait moves into the consumer's GEMM, behind its weight prefetch.
         """
         c = self.cfg
+        if c.residual_f32:               # fp32 stream: the scaled sub-layer output is added in the GEMM's epilogue
+            h = w.add_to(x, h, c.residual_mult)
+            return h, S.rmsnorm32(h, next_ln, c.rms_eps)
         if next_ln is None:              # parallel block: the attention output joins the residual, the MLP's call normalises
             return self._row_parallel(w, x, h), None
         if self._beta != 1.0:            # DeepNorm-style residual: the sub-layer's contribution is scaled (linear in x)
@@ -586,6 +611,15 @@ class DecoderModel:
         B.linear_batched(o_lat.reshape(T, H * lora), lw.w_uv_c, H, lora, o, vd)
         return self._row_parallel_norm(lw.o, o, residual, next_ln, consumer=consumer)
 
+    def _latent_attention(self, lw: LayerWeights, x, fb: ForwardBatch, kv, residual, next_ln):
+        """Latent attention: merged [queries | gate | latent] projection, the normalised latent row into its cache slot, windowed
+        attention with the output gate in its epilogue, output projection onto the residual."""
+        la = lw.latent
+        proj = la.in_proj(x)
+        S.latent_norm(proj[:, la.latent_col:], la.kv_norm, fb.slots, kv[0], la.rank, self.cfg.rms_eps)
+        a = LA.attention(la, proj, kv[0], fb)
+        return self._row_parallel_norm(lw.attn.o, a, residual, next_ln)
+
     @staticmethod
     def _glu(gu, act: str, interleaved: bool):
         """``act(gate) * up`` for gated MLPs whose activation is not SiLU (GeGLU of the Gemma family, ...): one kernel."""
@@ -601,8 +635,35 @@ class DecoderModel:
             return B.linear(x, lw.router_16, out_f32=True)
         return torch.matmul(x.float(), lw.router.t())
 
-    def _mlp(self, lw: MLPWeights, x, residual, layer_idx, next_ln, consumer=None):
+    def _table_moe(self, lw: MLPWeights, x, h, fb: ForwardBatch, next_ln):
+        """Experts picked by the token id's table row, each with weight 1 / top, plus the shared expert; combine, residual add and
+        the next norm are one launch."""
         c = self.cfg
+        top = lw.route_table.shape[1]
+        shared = lw.shared_down(lw.shared_gate_up(x, swiglu=True)) if lw.shared_gate_up is not None else None
+        parts = None
+        if lw.experts.stacked is not None and x.is_cuda:
+            from ..ops import moe_grouped
+
+            plans = fb.__dict__.get("_table_plans")
+            if plans is None:
+                if self.__dict__.get("_table_router") is None:
+                    self._table_router = MOE.TableRouter([l.mlp for l in self.layers if l.mlp.route_table is not None], x.device)
+                plans = fb._table_plans = self._table_router.plan(fb.ids)
+            parts = moe_grouped.forward(x, None, None, lw.experts, combine=False, plan=plans[id(lw)])
+        if parts is not None:
+            return h, S.moe_combine_norm(parts[0], parts[1], None, 1.0 / top, shared, h, next_ln, c.residual_mult, c.rms_eps)
+        idx = lw.route_table[fb.ids.long()]
+        y = MOE.moe_forward(x, idx, torch.full(idx.shape, 1.0 / top, device=x.device), lw.experts)
+        rows = self._row_ids(x.shape[0], x.device).view(-1, 1)
+        return h, S.moe_combine_norm(y, rows, None, 1.0, shared, h, next_ln, c.residual_mult, c.rms_eps)
+
+    def _mlp(self, lw: MLPWeights, x, residual, layer_idx, next_ln, consumer=None, fb=None):
+        c = self.cfg
+        if lw.route_table is not None:
+            return self._table_moe(lw, x, residual, fb, next_ln)
+        if lw.act == "relu2":
+            return self._row_parallel_norm(lw.down, lw.up.relu2(x), residual, next_ln, lw.post_ln, consumer)
         if lw.experts is None and lw.up is not None:         # two-matrix MLP: up -> activation -> down
             u = lw.up(x).float()
             code = B.GLU_ACTS.get(c.hidden_act, 1)
@@ -681,7 +742,12 @@ class DecoderModel:
             fb.decode_planned = True
         if self.layer_devices is not None:
             return self._forward_staged(fb, kv_caches)
-        h = self.embed_tokens(fb.ids)
+        if c.residual_f32:
+            if self.__dict__.get("_pos_freq") is None:
+                self._pos_freq = S.sinusoid_inv_freq(c.hidden_size, c.pos_embed_base, self.device) if c.pos_embed_base else None
+            h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps)
+        else:
+            h, x = self.embed_tokens(fb.ids), None
         if fb.embed_rows is not None:
             h[fb.embed_rows] = fb.embed_vals.to(h.dtype)
         self._rope_override = None
@@ -694,8 +760,8 @@ class DecoderModel:
         if self._fused_active:
             h = fused.load_h(h)
         n_layers = len(self.layers)
-        l0 = self.layers[0]
-        x = self._norm(h, l0.lin.ln if l0.lin is not None else l0.attn.ln)
+        if x is None:
+            x = self._norm(h, self._entry_norm(0))
         for i, lw in enumerate(self.layers):
             # the projection that reads each fused collective's output first (it can take over the all-gather wait)
             mlp_first = lw.mlp.gate_up if lw.mlp.experts is None else None
@@ -706,6 +772,8 @@ class DecoderModel:
                 h = x * alpha if alpha != 1.0 else x
             if c.parallel_block:
                 h, _ = self._attention(lw.attn, x, fb, kv_caches[i], h, None, None)       # h + attention(x); the MLP reads x too
+            elif lw.latent is not None:
+                h, x = self._latent_attention(lw, x, fb, kv_caches[i], h, self._entry_norm(i + 1) if lw.mlp.absent else lw.mlp.ln)
             elif lw.lin is not None:
                 h, x = self._linear_attention(lw.lin, x, fb, kv_caches[i], h, lw.mlp.ln, mlp_first)
             else:
@@ -713,15 +781,16 @@ class DecoderModel:
             if c.postnorm_residual:
                 self._beta = mbeta
                 h = x * ma if ma != 1.0 else x
+            if lw.mlp.absent:
+                continue
+            next_ln = self._entry_norm(i + 1)
             if i + 1 < n_layers:
                 nl = self.layers[i + 1]
-                next_ln = nl.lin.ln if nl.lin is not None else nl.attn.ln
                 na = nl.attn
-                nxt = nl.lin.in_proj if nl.lin is not None else ((na.q_a if na.q_a is not None else na.q_b) if c.use_mla else na.qkv)
+                nxt = nl.latent.in_proj if nl.latent is not None else nl.lin.in_proj if nl.lin is not None else ((na.q_a if na.q_a is not None else na.q_b) if c.use_mla else na.qkv)
             else:
-                next_ln = self.final_norm
                 nxt = self.lm_head if fb.logit_rows is None else None
-            h, x = self._mlp(lw.mlp, x, h, i, next_ln, nxt)
+            h, x = self._mlp(lw.mlp, x, h, i, next_ln, nxt, fb)
         self._beta = 1.0
         self._rope_override = None
         # x is RMSNorm(h) with the final norm weight (row-wise, so selecting rows afterwards is equivalent)
@@ -732,12 +801,21 @@ class DecoderModel:
             B.flush_pending_wait()
             x = x.index_select(0, fb.logit_rows)
         logits = self.lm_head(x, out_f32=True)
+        if logits.shape[1] > self.vocab_pad_from:
+            logits = logits[:, :self.vocab_pad_from]
         B.flush_pending_wait()          # no-op unless the head ran outside the GEMM that waits itself
         if c.logit_scale != 1.0:
             logits = logits * c.logit_scale
         if c.final_softcap:
             logits = torch.tanh(logits / c.final_softcap) * c.final_softcap
         return logits
+
+    def _entry_norm(self, i: int):
+        """Weight of the norm that opens layer ``i`` (the final norm behind the last one)."""
+        if i >= len(self.layers):
+            return self.final_norm
+        lw = self.layers[i]
+        return lw.lin.ln if lw.lin is not None else lw.attn.ln
 
     def mtp_forward(self, fb: ForwardBatch, hidden: torch.Tensor, kv_caches):
         """Draft head over the packed rows of ``fb``: ``fb.ids`` are the tokens FOLLOWING each row's position, ``hidden`` the
@@ -889,6 +967,29 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
             mk(p + "input_layernorm.bias", (H,))
         if not cfg.parallel_block:
             ones(p + "post_attention_layernorm.weight", H)
+        if cfg.mixers is not None:
+            if cfg.ffs[i].kind == "none":
+                raw.pop(p + "post_attention_layernorm.weight")
+            sp, ff = cfg.mixers[i], cfg.ffs[i]
+            ap = p + "self_attn."
+            mk(ap + "q_proj.weight", (sp.heads * sp.dim, H))
+            mk(ap + "g_proj.weight", (sp.heads * sp.vdim, H))
+            mk(ap + "kv_a_proj.weight", (sp.kv_rank, H))
+            ones(ap + "kv_a_layernorm.weight", sp.kv_rank)
+            mk(ap + "k_b_proj.weight", (sp.heads * sp.dim, sp.kv_rank))
+            mk(ap + "v_b_proj.weight", (sp.heads * sp.vdim, sp.kv_rank))
+            mk(ap + "o_proj.weight", (H, sp.heads * sp.vdim))
+            if ff.kind == "dense":
+                mk(p + "mlp.up_proj.weight", (ff.ff, H))
+                mk(p + "mlp.down_proj.weight", (H, ff.ff))
+            elif ff.kind == "moe":
+                for nm, inter in [(f"mlp.experts.{e}.", ff.expert_ff) for e in range(ff.experts)] + ([("mlp.shared_experts.", ff.shared_ff)] if ff.shared_ff else []):
+                    mk(p + nm + "gate_proj.weight", (inter, H))
+                    mk(p + nm + "up_proj.weight", (inter, H))
+                    mk(p + nm + "down_proj.weight", (H, inter))
+                gen.manual_seed(_name_seed(seed, p + "mlp.token_table"))
+                raw[p + "mlp.token_table"] = torch.rand((cfg.vocab_size, ff.experts), device=dev, generator=gen).topk(ff.top, dim=1).indices.to(torch.int32)
+            return raw
         if cfg.layer_is_linear(i) and cfg.lin_kind == "lightning":
             HD = cfg.num_heads * cfg.head_dim
             mk(p + "self_attn.qkv_proj.weight", (3 * HD, H))

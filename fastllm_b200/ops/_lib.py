@@ -16,6 +16,7 @@ _LIB_DIR = Path(__file__).resolve().parent.parent / "lib"
 _lock = threading.Lock()
 _kernels = None
 _runtime = None
+_kernel_path = _LIB_DIR / "libfb_kernels.so"
 
 P = c_void_p
 I = c_int
@@ -28,6 +29,9 @@ _KERNEL_SIGS = {
     "fb_gemm_qkv_post": [P, P, P, I, I, I, I, I, I, P, P, P, I, P, P, P, P, P, P, P, P, I, I, I, I, F, F, P],
     "fb_gemm_route": [P, P, I, I, I, I, I, I, P, P, P, I, I, I, F, P],
     "fb_gemm_16bit_batched": [P, P, P, I, I, I, I, I, I, I, I, I, I, P],
+    "fb_gemm_16bit_batched_gate": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P],
+    "fb_gemm_16bit_res32": [P, P, P, P, I, I, I, I, I, I, I, F, I, P],
+    "fb_gemm_full32": [P, P, P, P, P, P, I, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, P, P, F, I, I, I, P],
     "fb_mla_post": [P, I, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, LL, F, I, P],
     "fb_gemm_pick_split": [I, I, I, I],
     "fb_rmsnorm": [P, P, P, P, I, I, I, I, F, F, I, P],
@@ -156,6 +160,12 @@ class _KernelProxy:
         return hasattr(self._lib, name)
 
 
+def use_library(path) -> None:
+    """Load the kernels from ``path`` (a library with the files some model needs) instead of the full one."""
+    global _kernel_path
+    _kernel_path = Path(path)
+
+
 def kernels():
     global _kernels
     if _kernels is not None:
@@ -163,7 +173,7 @@ def kernels():
     with _lock:
         if _kernels is not None:
             return _kernels
-        path = _LIB_DIR / "libfb_kernels.so"
+        path = _kernel_path
         if not path.exists():
             raise KernelLibraryMissing(
                 f"{path} not found: run `python -m fastllm_b200.build` (sm_100a kernels are required on GPU)")

@@ -15,7 +15,7 @@ import torch.nn.functional as F
 
 from . import _lib, cpu
 
-GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32 = 1, 2, 4, 8
+GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32, GEMM_RELU2 = 1, 2, 4, 8, 32
 
 
 def _ptr(t):
@@ -145,12 +145,64 @@ def _f32_split(w: torch.Tensor):
     return p
 
 
+_FULL32_CODE = {torch.float16: 0, torch.bfloat16: 1, torch.float32: 2}
+
+
+def linear_full32(x, w, bias=None, residual=None, alpha: float = 1.0, relu2: bool = False, gate=None, out=None, out_f32: bool = False,
+                  batch: int = 1, x_cols: int = 0, out_cols: int = 0, counts=None, offsets=None, n: int | None = None):
+    """``x @ w.T`` in fp32 arithmetic on the CUDA cores for any size (float32 models, 16-bit shapes outside the tensor-core tiling),
+    with optional ReLU^2, gate ``* sigmoid(gate)`` and fp32 ``residual + alpha * ...``.  ``batch`` > 1: the slices of
+    ``linear_batched``; with ``counts`` / ``offsets`` the rows of ``batch`` experts whose weights are stacked in ``w``
+    (``n`` rows each are used, the stack's own stride is its row count over ``batch``)."""
+    flush_pending_wait()
+    M, K = x.shape[0], w.shape[-1]
+    w2 = w.reshape(-1, K)
+    rows_w = w2.shape[0] // batch
+    N = n or rows_w
+    if out is None:
+        out = torch.empty((M, N), device=x.device, dtype=torch.float32 if (out_f32 or residual is not None) else x.dtype)
+    rc = _lib.kernels().fb_gemm_full32(_ptr(x), _ptr(w2), _ptr(out), _ptr(bias), _ptr(residual), _ptr(gate), M, N, K, batch, x.stride(0),
+                                       w2.stride(0), out.stride(0), residual.stride(0) if residual is not None else 0,
+                                       gate.stride(0) if gate is not None else 0, rows_w, x_cols, out_cols, _ptr(counts), _ptr(offsets),
+                                       float(alpha), 1 if relu2 else 0, 1 if out.dtype == torch.float32 else 0, _FULL32_CODE[x.dtype], _stream())
+    _lib.check(rc, "fb_gemm_full32")
+    return out
+
+
+def tc_operands_ok(x, w) -> bool:
+    """The 16-bit tensor-core GEMMs read ``x`` [M, K] and ``w`` [N, K] through TMA: 16-byte aligned rows of both."""
+    return bool(x.dtype in (torch.float16, torch.bfloat16) and w.dtype == x.dtype and w.shape[1] % 8 == 0 and w.shape[0] % 8 == 0
+                and x.stride(-1) == 1 and not (x.data_ptr() & 15) and (x.stride(0) * 2) % 16 == 0 and w.is_contiguous())
+
+
+def linear_res32(x, w, h, alpha: float):
+    """fp32 residual stream: ``h += alpha * (x @ w.T)`` in place, in the GEMM's epilogue."""
+    if not x.is_cuda:
+        flush_pending_wait()
+        h += alpha * (x.float() @ w.float().t())
+        return h
+    M, N, K = x.shape[0], w.shape[0], w.shape[1]
+    if not tc_operands_ok(x, w):
+        return linear_full32(x, w, residual=h, alpha=alpha, out=h)
+    flush_pending_wait()
+    step = M if (M <= 256 or N % 32 == 0) else 256
+    for m0 in range(0, M, step):
+        m1 = min(M, m0 + step)
+        rc = _lib.kernels().fb_gemm_16bit_res32(_ptr(x[m0:m1]), _ptr(w), _ptr(h[m0:m1]), _ptr(h[m0:m1]), m1 - m0, N, K, x.stride(0), w.stride(0),
+                                                h.stride(0), h.stride(0), float(alpha), dtype_code(x.dtype), _stream())
+        _lib.check(rc, "fb_gemm_16bit_res32")
+    return h
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: bool = False, interleaved: bool = True,
-           out_f32: bool = False, out: torch.Tensor | None = None, nsplit: int = 0) -> torch.Tensor:
-    """``y = x @ w.T`` with optional fused bias, SwiGLU (``w`` = gate/up stacked) and residual add.
+           out_f32: bool = False, out: torch.Tensor | None = None, nsplit: int = 0, relu2: bool = False) -> torch.Tensor:
+    """``y = x @ w.T`` with optional fused bias, SwiGLU (``w`` = gate/up stacked) or ReLU^2, and residual add.
 
     x: ``[M, K]`` (row stride may exceed K), w: ``[N, K]``.  16-bit CUDA tensors run the tcgen05 GEMM.
     """
+    if relu2 and (not x.is_cuda or x.dtype == torch.float32 or not tc_operands_ok(x, w)):
+        y = linear(x, w, bias, out_f32=out_f32)
+        return torch.relu(y).square()
     if not x.is_cuda:
         flush_pending_wait()
         # native kernels for decode-sized batches and for 16-bit weights (used in place); large fp32 GEMMs go to the BLAS
@@ -184,9 +236,11 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: b
         if residual is not None:
             y += residual.reshape(-1, residual.shape[-1]).float()
         return y.reshape(*lead, y.shape[-1])
-    if K % 64 != 0 or N % 8 != 0 or x.dtype not in (torch.float16, torch.bfloat16) or (x2.data_ptr() & 15) or (x2.stride(0) * 2) % 16:
+    if K % 8 != 0 or N % 8 != 0 or x.dtype not in (torch.float16, torch.bfloat16) or (x2.data_ptr() & 15) or (x2.stride(0) * 2) % 16:
         # shapes outside the tensor-core kernels' tiling (rare: odd projection widths): plain PyTorch definition
         flush_pending_wait()
+        if not swiglu and residual is None and x.dtype == w.dtype and x.dtype in _FULL32_CODE and w.is_contiguous() and out is None and bias is None:
+            return linear_full32(x2, w, out_f32=out_f32).reshape(*lead, N)
         return linear_ref(x, w, bias, residual, swiglu, interleaved, torch.float32 if out_f32 else None)
     if swiglu and not interleaved:
         raise ValueError("CUDA SwiGLU epilogue needs tile-interleaved gate/up weights (interleave_gate_up)")
@@ -194,7 +248,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: b
     if out is None:
         out = torch.empty((M, n_out), device=x.device, dtype=torch.float32 if out_f32 else x.dtype)
     flags = (GEMM_BIAS if bias is not None else 0) | (GEMM_RESIDUAL if residual is not None else 0) | \
-            (GEMM_SWIGLU if swiglu else 0) | (GEMM_OUT_F32 if out_f32 else 0)
+            (GEMM_SWIGLU if swiglu else 0) | (GEMM_OUT_F32 if out_f32 else 0) | (GEMM_RELU2 if relu2 else 0)
     res2 = residual.reshape(-1, residual.shape[-1]) if residual is not None else None
     lib = _lib.kernels()
     dt = dtype_code(x.dtype)
@@ -224,27 +278,33 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: b
     return out.reshape(*lead, n_out)
 
 
-def linear_batched(x: torch.Tensor, w: torch.Tensor, batch: int, x_cols: int, out: torch.Tensor, out_cols: int) -> torch.Tensor:
+def linear_batched(x: torch.Tensor, w: torch.Tensor, batch: int, x_cols: int, out: torch.Tensor, out_cols: int, gate=None) -> torch.Tensor:
     """``out[m, z * out_cols + n] = sum_k x[m, z * x_cols + k] * w[z, n, k]`` for ``z < batch``: one small GEMM per attention head
     in one launch (the absorbed multi-head-latent-attention projections).  x ``[M, >= batch * x_cols]``, w ``[batch, N, K]``
-    contiguous, out ``[M, >= batch * out_cols]`` (written in place and returned)."""
+    contiguous, out ``[M, >= batch * out_cols]`` (written in place and returned).  ``gate`` (like out): ``* sigmoid(gate)``."""
     M = x.shape[0]
     _, N, K = w.shape
-    ok = (x.is_cuda and x.dtype in (torch.float16, torch.bfloat16) and w.dtype == x.dtype and out.dtype == x.dtype and K % 64 == 0
+    ok = (x.is_cuda and x.dtype in (torch.float16, torch.bfloat16) and w.dtype == x.dtype and out.dtype == x.dtype and K % 8 == 0
           and N % 8 == 0 and x_cols % 8 == 0 and out_cols % 4 == 0 and x.stride(-1) == 1 and out.stride(-1) == 1
           and not (x.data_ptr() & 15) and not ((x.stride(0) * 2) & 15) and w.is_contiguous())
     if not ok:
         flush_pending_wait()
+        if x.is_cuda and w.dtype == x.dtype and out.dtype == x.dtype and w.is_contiguous() and x.dtype in _FULL32_CODE:
+            return linear_full32(x, w, gate=gate, out=out, batch=batch, x_cols=x_cols, out_cols=out_cols)
         xs = x.as_strided((M, batch, K), (x.stride(0), x_cols, 1))
         ov = out.as_strided((M, batch, N), (out.stride(0), out_cols, 1))
-        ov.copy_(torch.einsum("mzk,znk->mzn", xs.float(), w.float()).to(out.dtype))
+        y = torch.einsum("mzk,znk->mzn", xs.float(), w.float())
+        if gate is not None:
+            y = y * torch.sigmoid(gate.float()).as_strided((M, batch, N), (gate.shape[1], out_cols, 1))
+        ov.copy_(y.to(out.dtype))
         return out
     flush_pending_wait()
     lib = _lib.kernels()
     for m0 in range(0, M, 256):
         m1 = min(M, m0 + 256)
-        rc = lib.fb_gemm_16bit_batched(_ptr(x[m0:m1]), _ptr(w), _ptr(out[m0:m1]), m1 - m0, N, K, batch, x.stride(0), K, out.stride(0),
-                                       x_cols, out_cols, dtype_code(x.dtype), _stream())
+        rc = lib.fb_gemm_16bit_batched_gate(_ptr(x[m0:m1]), _ptr(w), _ptr(out[m0:m1]), m1 - m0, N, K, batch, x.stride(0), K, out.stride(0),
+                                            x_cols, out_cols, _ptr(gate[m0:m1] if gate is not None else None),
+                                            gate.stride(0) if gate is not None else 0, dtype_code(x.dtype), _stream())
         _lib.check(rc, "fb_gemm_16bit_batched")
     return out
 

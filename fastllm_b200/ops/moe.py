@@ -88,6 +88,36 @@ def route_fused(x, router_16, bias, topk, score_mode, renorm, route_scale=1.0):
     return idx, w
 
 
+class TableRouter:
+    """Routing by token id: every such layer has a table ``[vocab, top]`` of experts.  The plans of all layers depend on the ids
+    alone, so one launch at the start of a forward pass makes them (one CTA per layer; a layer that runs several times is planned once)."""
+
+    def __init__(self, layers, device):
+        self.layers = list({id(l): l for l in layers if l.experts is not None and l.experts.stacked is not None}.values())
+        self.e_stride = max(l.experts.count for l in self.layers)
+        self.k_stride = max(l.route_table.shape[1] for l in self.layers)
+        self.meta = torch.tensor([[l.route_table.data_ptr(), l.route_table.shape[1], l.experts.count, l.route_table.shape[0]] for l in self.layers],
+                                 dtype=torch.int64).to(device)
+
+    def plan(self, ids):
+        """id(layer) -> (counts, offsets, pos [T, top], total) as ``fb_moe_plan`` gives them."""
+        from .moe_grouped import PAD
+
+        L, T, dev = len(self.layers), ids.shape[0], ids.device
+        ctr = torch.empty((2 * L * self.e_stride + L,), device=dev, dtype=torch.int32)
+        counts, offsets, total = ctr[:L * self.e_stride], ctr[L * self.e_stride:2 * L * self.e_stride], ctr[2 * L * self.e_stride:]
+        pos = torch.empty((L, T * self.k_stride), device=dev, dtype=torch.int32)
+        rc = _lib.kernels().fb_moe_plan_table(_ptr(self.meta), L, _ptr(ids), T, _ptr(counts), _ptr(offsets), _ptr(pos), _ptr(total), self.e_stride,
+                                              self.k_stride, PAD, _stream())
+        _lib.check(rc, "fb_moe_plan_table")
+        out = {}
+        for i, l in enumerate(self.layers):
+            top, E = l.route_table.shape[1], l.experts.count
+            out[id(l)] = (counts[i * self.e_stride:i * self.e_stride + E], offsets[i * self.e_stride:i * self.e_stride + E],
+                          pos[i, :T * top].view(T, top), total[i:i + 1])
+        return out
+
+
 def route_group_top1(logits, groups: int, expert_scale=None):
     """Mixture of grouped experts (Pangu Pro MoE): the experts form ``groups`` equal, contiguous groups and the best-scoring
     expert of every group is taken; weight = softmax score (over all experts) x the expert's learned scale, not renormalised.
@@ -301,7 +331,7 @@ def mla_paged_attention(q_full, lat_pool, fb, scale, lora, select=None):
             and lat_pool.dtype == q_full.dtype and lat_pool.shape[1] == 128):
         from .attention import mla_decode
 
-        return mla_decode(q_full, lat_pool, fb.page_table, fb.kv_lens, scale)
+        return mla_decode(q_full, lat_pool, fb.page_table, fb.kv_lens, scale, lora=lora)
     out = torch.zeros((T, H, lora), device=q_full.device, dtype=q_full.dtype)
     page_len = lat_pool.shape[1]
     cu = fb.cu_q_host if fb.cu_q_host is not None else fb.cu_q.tolist()

@@ -13,12 +13,14 @@ import ctypes
 import torch
 
 from . import _lib
+from . import basic as B
 from . import quant_gemm as QG
 from .basic import GEMM_SWIGLU, _ptr, _stream, dtype_code
 
 P, I = ctypes.c_void_p, ctypes.c_int
 _lib.register_sigs({
     "fb_moe_plan": [P, I, I, I, I, P, P, P, P, I, P],
+    "fb_moe_plan_table": [P, I, P, I, P, P, P, P, I, I, I, P],
     "fb_moe_gather": [P, P, P, I, I, I, P],
     "fb_moe_combine": [P, P, P, P, P, I, I, I, I, P],
     "fb_moe_grouped_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
@@ -80,12 +82,17 @@ def stack_experts(experts) -> StackedExperts | None:
     if any(w.kind != kind or not w.interleaved or w.bias is not None for w in gu) or any(w.kind != kind or w.bias is not None for w in dn):
         return None
     two_i, hidden = gu[0].n, gu[0].k
-    if two_i % 128 != 0 or hidden % 128 != 0 or (two_i // 2) % 64 != 0:
+    if two_i % 128 != 0 or hidden % (8 if kind == "dense" else 128) != 0 or (two_i // 2) % 64 != 0:
         return None
     g = torch.cat([w.w for w in gu], dim=0).contiguous()
-    d = torch.cat([w.w for w in dn], dim=0).contiguous()
     if kind == "dense":
-        return StackedExperts(kind, g, d, len(gu), two_i // 2, hidden)
+        # a weight tile is 128 output rows of one expert: the down matrices are stacked a multiple of 128 rows apart
+        hp = (hidden + 127) // 128 * 128
+        d = torch.zeros((len(dn), hp, two_i // 2), dtype=dn[0].w.dtype, device=dn[0].w.device)
+        for e, w in enumerate(dn):
+            d[e, :hidden] = w.w
+        return StackedExperts(kind, g, d.view(len(dn) * hp, two_i // 2), len(gu), two_i // 2, hidden)
+    d = torch.cat([w.w for w in dn], dim=0).contiguous()
     if kind == "int4g" and (gu[0].group % 64 != 0 or hidden % gu[0].group != 0 or (two_i // 2) % gu[0].group != 0):
         return None
     if kind == "fp8" and (two_i // 2) % 128 != 0:
@@ -104,7 +111,7 @@ def prepare_model(m) -> None:
     """Stack the experts of every MoE layer; the per-expert tensors are replaced by views of the stacked matrices."""
     for lw in m.layers:
         ex = lw.mlp.experts
-        if ex is None or ex.count == 0 or ex.host or ex.act != "swiglu" or any(l.bias is not None for l in ex.gate_up + ex.down):
+        if ex is None or ex.stacked is not None or ex.count == 0 or ex.host or ex.act != "swiglu" or any(l.bias is not None for l in ex.gate_up + ex.down):
             continue
         st = stack_experts(ex)
         if st is None:
@@ -114,19 +121,36 @@ def prepare_model(m) -> None:
         two_i, H = 2 * st.inter, st.hidden
         for e in range(ex.count):       # drop the duplicate storage: per-expert weights become views of the stacked matrices
             ex.gate_up[e].w = st.gate_up[e * two_i:(e + 1) * two_i]
-            ex.down[e].w = st.down[e * H:(e + 1) * H]
+            hp = st.down.shape[0] // ex.count
+            ex.down[e].w = st.down[e * hp:e * hp + H]
         if QG.INT_A8 and st.kind in ("int8", "int4g") and st.gate_up.is_cuda and (st.kind == "int8" or st.group == 128) \
                 and H % 128 == 0 and st.inter % 128 == 0:
             _prepare_a8(st, ex)                    # scale tables of the integer path, before any CUDA graph is captured
 
 
-def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add: torch.Tensor | None = None, combine: bool = True):
-    """``combine=False`` stops before the weighted sum and returns ``(ys, pos, wts)`` for a fused cross-rank combine."""
+def _forward32(x, st, plan):
+    """The same steps on fp32 operands (CUDA-core products): sorted expert outputs and their positions."""
+    counts, offsets, pos, _ = plan
+    T, H = x.shape
+    topk = pos.shape[1]
+    rows_cap = T * topk + st.n_local * PAD + 128
+    xs = torch.empty((rows_cap, H), device=x.device, dtype=x.dtype)
+    _lib.check(_lib.kernels().fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, 2 * H, _stream()), "fb_moe_gather")
+    act = B.glu_act_ref(B.linear_full32(xs, st.gate_up, batch=st.n_local, counts=counts, offsets=offsets), "silu", True)
+    return B.linear_full32(act, st.down, batch=st.n_local, counts=counts, offsets=offsets, n=H), pos
+
+
+def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add: torch.Tensor | None = None, combine: bool = True, plan=None):
+    """``combine=False`` stops before the weighted sum and returns ``(ys, pos, wts)`` for a fused combine.  ``plan``: the routing
+    plan (counts, offsets, pos, total) where it is known already (``ops.moe.TableRouter``)."""
     st = experts.stacked
+    if st is not None and plan is not None and not combine and x.dtype == torch.float32 and st.kind == "dense" and st.gate_up.dtype == x.dtype:
+        ys, pos = _forward32(x, st, plan)
+        return ys, pos, wts
     if st is None or x.dtype not in (torch.float16, torch.bfloat16):
         return None
     T, H = x.shape
-    topk = idx.shape[1]
+    topk = (plan[2] if plan is not None else idx).shape[1]
     E = st.n_local
     dev = x.device
     lib = _lib.kernels()
@@ -138,14 +162,18 @@ def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add:
     if st.kind == "int4g" and QG.INT_A8 and mean <= 12:
         hint = 16          # the 16-row integer kernel has dedicated unpack warps; a second chunk re-reads its weights from L2
     max_rows = min(T, 0xFFFF) | (hint << 16)
-    counts = torch.empty(E, device=dev, dtype=torch.int32)
-    offsets = torch.empty(E, device=dev, dtype=torch.int32)
-    pos = torch.empty((T, topk), device=dev, dtype=torch.int32)
-    total = torch.empty(1, device=dev, dtype=torch.int32)
-    idx = idx.contiguous()
-    wts = wts.float().contiguous()
     s = _stream()
-    _lib.check(lib.fb_moe_plan(_ptr(idx), T, topk, experts.first, E, _ptr(counts), _ptr(offsets), _ptr(pos), _ptr(total), PAD, s), "fb_moe_plan")
+    if plan is not None:
+        counts, offsets, pos, total = plan
+    else:
+        counts = torch.empty(E, device=dev, dtype=torch.int32)
+        offsets = torch.empty(E, device=dev, dtype=torch.int32)
+        pos = torch.empty((T, topk), device=dev, dtype=torch.int32)
+        total = torch.empty(1, device=dev, dtype=torch.int32)
+        idx = idx.contiguous()
+        _lib.check(lib.fb_moe_plan(_ptr(idx), T, topk, experts.first, E, _ptr(counts), _ptr(offsets), _ptr(pos), _ptr(total), PAD, s), "fb_moe_plan")
+    if wts is not None:
+        wts = wts.float().contiguous()
     dt = dtype_code(x.dtype)
     fp8_native = st.kind == "fp8" and QG.FP8_NATIVE and H % 128 == 0 and st.inter % 128 == 0
     int_a8 = QG.INT_A8 and (st.kind == "int8" or (st.kind == "int4g" and st.group == 128)) and H % 128 == 0 and st.inter % 128 == 0

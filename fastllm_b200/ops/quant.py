@@ -199,7 +199,7 @@ def normalize_wdtype(name: str | None) -> tuple[str, int]:
 class LinearWeight:
     """Weight (+ optional bias) of one linear layer in one of the storage formats above."""
 
-    __slots__ = ("kind", "w", "scale", "zero", "bias", "group", "n", "k", "interleaved", "dtype", "_dq", "signed", "_a8", "adapters")
+    __slots__ = ("kind", "w", "scale", "zero", "bias", "group", "n", "k", "interleaved", "dtype", "_dq", "signed", "_a8", "adapters", "exact32")
     active_adapter: str | None = None       # name of the run-time low-rank adapter applied by every weight that carries it
 
     def __init__(self, kind, w, scale=None, zero=None, bias=None, group=0, dtype=torch.bfloat16, interleaved=False):
@@ -211,6 +211,7 @@ class LinearWeight:
         self._dq = None
         self._a8 = None
         self.adapters = None                # name -> (A [r, K], B [N, r]) run-time low-rank deltas (fastllm_b200/lora.py)
+        self.exact32 = False                # float32 operands on CUDA: fp32 FMAs instead of the split tensor-core product
         self.signed = False                 # int8 only: bytes hold q - 128 (the integer tensor-core path's operand form)
 
     @staticmethod
@@ -298,7 +299,33 @@ class LinearWeight:
             return y.float() if out_f32 else y
         return self._base(x, residual, swiglu, out_f32)
 
+    def _exact(self, x) -> bool:
+        return bool(self.exact32 and self.kind == "dense" and x.is_cuda and x.dtype == torch.float32 and self.w.dtype == torch.float32)
+
+    def _plain(self, x) -> bool:
+        """A dense product without a run-time adapter: the epilogues below can be fused into it."""
+        return self.kind == "dense" and self.w.dtype == x.dtype and not (LinearWeight.active_adapter is not None and self.adapters)
+
+    def add_to(self, x, h, alpha: float):
+        """fp32 residual stream: ``h += alpha * (W x)`` in place."""
+        if self._plain(x) and self.bias is None:
+            if self._exact(x):
+                return B.linear_full32(x, self.w, residual=h, alpha=alpha, out=h)
+            return B.linear_res32(x, self.w, h, alpha)
+        h.add_(self(x, out_f32=True), alpha=alpha)
+        return h
+
+    def relu2(self, x):
+        """``relu(W x)^2``"""
+        if self._plain(x) and self.bias is None:
+            return B.linear_full32(x, self.w, relu2=True) if self._exact(x) else B.linear(x, self.w, relu2=True)
+        return torch.relu(self(x)).square()
+
     def _base(self, x, residual=None, swiglu=False, out_f32=False):
+        if self._exact(x) and residual is None:
+            y = B.linear_full32(x.reshape(-1, x.shape[-1]), self.w, self.bias)
+            y = B.glu_act_ref(y, "silu", self.interleaved) if swiglu else y
+            return y.reshape(*x.shape[:-1], y.shape[-1])
         if self.kind == "dense":
             w = self.w
             if w.dtype != x.dtype:
