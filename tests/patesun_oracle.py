@@ -38,24 +38,22 @@ def latent(h, w, prefix, eps):
     return rms_norm(linear(w[prefix + "dkv"], h), w[prefix + "dkv.norm"], eps)
 
 
-def latent_scores(h, c, w, prefix, mixer):
-    """[heads, queries, keys] scaled scores before the mask."""
-    H, D = mixer["heads"], mixer["dim"]
-    q = linear(w[prefix + "q"], h).reshape(-1, H, D)
-    k = linear(w[prefix + "uk"], c).reshape(-1, H, D)
-    return torch.einsum("ihd,jhd->hij", q, k) * mixer["scale"]
+def latent_core(q, c, uk, uv, gate, mixer):
+    """Attention of the rows ``q`` [n, heads * dim], which are the last n of the len(c) tokens, over the latents ``c`` [L, rank];
+    ``gate`` [n, heads * vdim] is the projection before its sigmoid."""
+    n, L, H, D, V = q.shape[0], c.shape[0], mixer["heads"], mixer["dim"], mixer["vdim"]
+    k = linear(uk, c).reshape(L, H, D)
+    v = linear(uv, c).reshape(L, H, V)
+    s = torch.einsum("ihd,jhd->hij", q.reshape(n, H, D), k) * mixer["scale"]
+    s = s.masked_fill(~visible(L, (mixer.get("mask") or {}).get("size"))[L - n:], float("-inf"))
+    o = torch.einsum("hij,jhv->ihv", torch.softmax(s, dim=-1), v).reshape(n, H * V)
+    return o * torch.sigmoid(gate)
 
 
 def latent_attention(h, w, prefix, mixer, eps):
     """``h`` [n, width] is one whole sequence."""
-    n, H, V = h.shape[0], mixer["heads"], mixer["vdim"]
     c = latent(h, w, prefix, eps)
-    s = latent_scores(h, c, w, prefix, mixer)
-    s = s.masked_fill(~visible(n, (mixer.get("mask") or {}).get("size")), float("-inf"))
-    p = torch.softmax(s, dim=-1)
-    v = linear(w[prefix + "uv"], c).reshape(-1, H, V)
-    o = torch.einsum("hij,jhv->ihv", p, v).reshape(n, H * V)
-    o = o * torch.sigmoid(linear(w[prefix + "g"], h))
+    o = latent_core(linear(w[prefix + "q"], h), c, w[prefix + "uk"], w[prefix + "uv"], linear(w[prefix + "g"], h), mixer)
     return linear(w[prefix + "o"], o)
 
 
