@@ -41,6 +41,10 @@ def parse_args():
     ap.add_argument("--output-len", type=int, default=256)
     ap.add_argument("--dtype", default="auto", help="weight dtype: auto(bf16) | int8 | int4g128 | fp8 | nvfp4 | mxfp4")
     ap.add_argument("--comm", default="auto", choices=["auto", "fused", "nccl"])
+    ap.add_argument("--layers", default="", choices=["", "patesun"],
+                    help="instead of the headline: throughput and kernel times of this design's layers beside the closest other family")
+    ap.add_argument("--layer-sizes", default="2k,4k,7k")
+    ap.add_argument("--layer-parts", default="kernels,steps")
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--device", default="cuda", choices=["cuda", "cpu"],
                     help="cpu: the CPU configuration (fp32, C++ backend); use with --model qwen3-0.6b --batch 1 --prompt-len 128 --output-len 128")
@@ -312,6 +316,11 @@ def run_cpu(args):
 
 def main():
     args = parse_args()
+    if args.layers:
+        from fastllm_b200.utils import layer_bench
+
+        layer_bench.run(args.layer_sizes.split(","), "steps" in args.layer_parts, "kernels" in args.layer_parts)
+        return
     if args.device == "cpu" and args.impl == "ours":
         run_cpu(args)
         return

@@ -214,9 +214,8 @@ def _absorbed(lw, q, gate, pool, page_table, kv_lens, out):
     B.linear_batched(o_lat.view(n, H * lw.ld), lw.w_uv, H, lw.ld, out, lw.vdim, gate=gate)
 
 
-def _expanded(lw, grp, q, gate, pool, out):
-    keys = S.gather_rows(pool.view(-1, lw.ld), grp.key_idx)
-    kv = B.linear(keys, lw.w_ukv)
+def window_attention(lw, grp, q, gate, kv, out):
+    """Prefill kernel over one group's expanded keys and values ``kv`` [n_keys, >= heads * (dim + vdim)]."""
     H = lw.heads
     k, v = kv[:, :H * lw.dim], kv[:, H * lw.dim:]
     rc = _lib.kernels().fb_attn_window(_ptr(q), q.stride(0), q.shape[0], _ptr(k), kv.stride(0), _ptr(v), kv.stride(0), kv.shape[0], _ptr(out),
@@ -243,7 +242,7 @@ def attention(lw, proj, pool, fb):
                   pl.kv_lens, part)
         out.index_copy_(0, pl.rows, part)
     for grp in pl.groups:
-        _expanded(lw, grp, q, gate, pool, out)
+        window_attention(lw, grp, q, gate, B.linear(S.gather_rows(pool.view(-1, lw.ld), grp.key_idx), lw.w_ukv), out)
     return out
 
 
