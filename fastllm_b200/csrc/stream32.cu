@@ -105,7 +105,7 @@ __global__ void rmsnorm32_kernel(const float* __restrict__ x, const typename Act
 
 // h[t] = table[ids[t]] + sinusoid(positions[t]) in fp32, and its RMSNorm.  inv_freq[i] = 10000^(-2i / H) in double; the angle is
 // reduced to [-pi, pi] in double, so a far position costs no accuracy.
-template <int DT>
+template <int DT, int VEC>
 __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ positions, const typename Act<DT>::T* __restrict__ table,
                                       const double* __restrict__ inv_freq, const typename Act<DT>::T* __restrict__ w, float* __restrict__ h,
                                       typename Act<DT>::T* __restrict__ y, int H, int vocab, float eps) {
@@ -120,27 +120,34 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
   float* hp = h + (size_t)t * H;
   const double pos = (double)positions[t];
   float ss = 0.f;
-  for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
-    float a = Act<DT>::ld(e[2 * i]);
-    if (inv_freq != nullptr) {
-      const double ang = pos * inv_freq[i];
-      const float red = (float)(ang - 6.283185307179586476925 * rint(ang * 0.15915494309189533577));
-      float s, c;
-      sincosf(red, &s, &c);
-      a += s;
-      if (2 * i + 1 < H) {
-        const float b = Act<DT>::ld(e[2 * i + 1]) + c;
-        hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b;
-      }
-    } else if (2 * i + 1 < H) {
-      const float b = Act<DT>::ld(e[2 * i + 1]);
-      hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b;
+  auto add_pos = [&](int i, float& a, float& b) {
+    const double ang = pos * inv_freq[i];
+    const float red = (float)(ang - 6.283185307179586476925 * rint(ang * 0.15915494309189533577));
+    float s, c;
+    sincosf(red, &s, &c);
+    a += s; b += c;
+  };
+  if (VEC == 4) {
+    for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
+      float v[4];
+      ld4<DT>(e + i, v);
+      if (inv_freq != nullptr) { add_pos(i / 2, v[0], v[1]); add_pos(i / 2 + 1, v[2], v[3]); }
+      st4<2>(hp + i, v);
+      st4<2>(row + i, v);
+      ss += v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
     }
-    hp[2 * i] = a; row[2 * i] = a; ss += a * a;
+  } else {
+    for (int i = threadIdx.x; 2 * i < H; i += blockDim.x) {
+      const bool two = 2 * i + 1 < H;
+      float a = Act<DT>::ld(e[2 * i]), b = two ? Act<DT>::ld(e[2 * i + 1]) : 0.f;
+      if (inv_freq != nullptr) add_pos(i, a, b);
+      hp[2 * i] = a; row[2 * i] = a; ss += a * a;
+      if (two) { hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b; }
+    }
   }
   ss = block_sum32(ss, sh);
   const float inv = 1.0f / sqrtf(ss / (float)H + eps);
-  norm_write<DT, 1>(row, w, y + (size_t)t * H, H, inv);
+  norm_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
 }
 
 // pool[slot] = RMSNorm over the first `n` columns of x[t] (columns [n, ld) of the entry are zero); slots < 0 go to `spare`
@@ -244,9 +251,11 @@ extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const voi
                                  void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
-  const int th = row_threads(H, 2);
-#define GO(DT) S32_LAUNCH((embed_pos_norm_kernel<DT>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
-  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+  const bool vec = H % 4 == 0;
+  const int th = row_threads(H, vec ? 4 : 2);
+#define GO(DT, V) S32_LAUNCH((embed_pos_norm_kernel<DT, V>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
+  if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
+  else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
   return (int)cudaGetLastError();
 }
