@@ -968,9 +968,10 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
         if not cfg.parallel_block:
             ones(p + "post_attention_layernorm.weight", H)
         if cfg.mixers is not None:
-            if cfg.ffs[i].kind == "none":
+            run = cfg.layer_runs.index(i)                 # i names a layer's weights; its specs are listed per run
+            sp, ff = cfg.mixers[run], cfg.ffs[run]
+            if ff.kind == "none":
                 raw.pop(p + "post_attention_layernorm.weight")
-            sp, ff = cfg.mixers[i], cfg.ffs[i]
             ap = p + "self_attn."
             mk(ap + "q_proj.weight", (sp.heads * sp.dim, H))
             mk(ap + "g_proj.weight", (sp.heads * sp.vdim, H))
