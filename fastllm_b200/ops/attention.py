@@ -551,9 +551,9 @@ class MlaWorkspace:
 
 def mla_decode(q_full, lat_pool, page_table, seq_lens, scale, ws: MlaWorkspace | None = None, lora: int | None = None, window: int = 0):
     """q_full ``[B, H, dq]`` (absorbed q_nope | rotated q_pe), lat_pool ``[pages, 128, 1, dq]`` -> ``[B, H, lora]``; the values are
-    the first ``lora`` of the ``dq`` columns (default: all).  ``window`` > 0: the last ``window`` tokens only."""
+    the first ``lora`` of the ``dq`` columns (default: up to 512 of them).  ``window`` > 0: the last ``window`` tokens only."""
     B, H, dq = q_full.shape
-    lora = lora or dq
+    lora = lora or min(dq, 512)
     if ws is None:
         cap = 1 << max(4, (B - 1).bit_length())
         key = (q_full.device, cap, H, lora)

@@ -37,6 +37,7 @@ class StackedExperts:
     def __init__(self, kind, gate_up, down, n_local, inter, hidden, group=0, gu_scale=None, gu_zero=None, dn_scale=None, dn_zero=None):
         self.kind, self.gate_up, self.down, self.n_local, self.inter, self.hidden, self.group = kind, gate_up, down, n_local, inter, hidden, group
         self.gu_scale, self.gu_zero, self.dn_scale, self.dn_zero = gu_scale, gu_zero, dn_scale, dn_zero
+        self.part_signed = None        # the same per matrix (gate_up, down) where only one's shape is taken by that path
         self.signed = False            # int8: the stacked bytes hold q - 128 (operand form of the integer tensor-core path)
         self.a8 = None                 # (gate_up scale, zero / min, down scale, zero / min) in the integer kernel's layout
 
@@ -118,6 +119,7 @@ def prepare_model(m) -> None:
             continue
         ex.stacked = st
         st.signed = st.kind == "int8" and all(w.signed for w in ex.gate_up + ex.down)
+        st.part_signed = tuple(st.kind == "int8" and all(w.signed for w in ws) for ws in (ex.gate_up, ex.down))
         two_i, H = 2 * st.inter, st.hidden
         for e in range(ex.count):       # drop the duplicate storage: per-expert weights become views of the stacked matrices
             ex.gate_up[e].w = st.gate_up[e * two_i:(e + 1) * two_i]
@@ -228,13 +230,14 @@ def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add:
                    "fb_gemm_i8(down)")
     else:
         qm = {"int8": 1, "int4g": 2, "fp8": 3, "fp4": 4}[st.kind]
-        grp = -1 if st.signed else (st.group or 0)           # -1: int8 bytes hold q - 128
+        gu_signed, dn_signed = (True, True) if st.signed else (st.part_signed or (False, False))
+        g_gu, g_dn = (-1 if sg else (st.group or 0) for sg in (gu_signed, dn_signed))           # -1: int8 bytes hold q - 128
         f16w = QG.GEMM_FP4_F16W if (st.kind == "fp4" and getattr(st, "fp4_f16w", False)) else 0
         _lib.check(lib.fb_moe_grouped_gemm_quant(_ptr(xs), _ptr(st.gate_up), _ptr(st.gu_scale), _ptr(st.gu_zero), _ptr(act), _ptr(counts),
-                                                 _ptr(offsets), rows_cap, E, 2 * st.inter, H, st.inter, max_rows, dt, qm, grp,
+                                                 _ptr(offsets), rows_cap, E, 2 * st.inter, H, st.inter, max_rows, dt, qm, g_gu,
                                                  GEMM_SWIGLU | f16w, T * topk, s), "fb_moe_grouped_gemm_quant(gate_up)")
         _lib.check(lib.fb_moe_grouped_gemm_quant(_ptr(act), _ptr(st.down), _ptr(st.dn_scale), _ptr(st.dn_zero), _ptr(ys), _ptr(counts),
-                                                 _ptr(offsets), rows_cap, E, H, st.inter, H, max_rows, dt, qm, grp, f16w, T * topk, s),
+                                                 _ptr(offsets), rows_cap, E, H, st.inter, H, max_rows, dt, qm, g_dn, f16w, T * topk, s),
                    "fb_moe_grouped_gemm_quant(down)")
     if not combine:
         return ys, pos, wts
