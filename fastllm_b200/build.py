@@ -32,7 +32,7 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v",
 ]
 # translation units that state fp32 results exactly (32-bit angles, norms, matrix products) are compiled without fast-math
-PRECISE_UNITS = {"stream32", "full32"}
+PRECISE_UNITS = {"stream32", "full32", "gla"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fopenmp", "-march=x86-64-v3", "-Wall", "-Wno-unused-function"]
 
 
@@ -52,8 +52,9 @@ def _run(cmd: list[str], log: Path | None = None) -> None:
         raise RuntimeError("build step failed: " + " ".join(cmd))
 
 
-# kernel files of models whose layers are latent attention and table-routed experts
-LATENT_UNITS = ("attn_mla", "attn_window", "elementwise", "full32", "gemm_bf16", "moe", "sampling", "stream32")
+# kernel files of models whose layers are listed one by one: what all of them launch, and what each kind of mixer adds
+LISTED_UNITS = ("elementwise", "full32", "gemm_bf16", "moe", "sampling", "stream32")
+MIXER_UNITS = {"LatentSpec": ("attn_mla", "attn_window"), "AttnSpec": ("attn_grouped", "attn_window"), "GLASpec": ("gla",)}
 
 
 def build_kernels(force: bool = False, units: tuple | None = None, out: Path | None = None) -> Path:
@@ -88,10 +89,12 @@ def ensure_for(model_dir) -> None:
         build_runtime()
     if (LIB / "libfb_kernels.so").exists():
         return
-    if load_config(model_dir).mixers is None:
+    mixers = load_config(model_dir).mixers
+    if mixers is None:
         build_kernels()
         return
-    _lib.use_library(build_kernels(units=LATENT_UNITS, out=LIB / "libfb_kernels_latent.so"))
+    extra = sorted({u for m in mixers for u in MIXER_UNITS[type(m).__name__]})
+    _lib.use_library(build_kernels(units=(*LISTED_UNITS, *extra), out=LIB / ("libfb_kernels_" + "_".join(extra) + ".so")))
 
 
 def build_runtime(force: bool = False) -> Path:

@@ -1,6 +1,7 @@
-// Prefill attention with one key / value head per query head and an optional sliding window, for sm_100a (tcgen05 + TMEM).
+// Prefill attention with an optional sliding window or chunk mask, for sm_100a (tcgen05 + TMEM).
 //
-// Keys and values are contiguous rows (the expanded latents of the keys a batch reads).  One CTA owns one head and up to 256
+// Keys and values are contiguous rows (the expanded latents of the keys a batch reads, one head per query head) or the cache pages
+// themselves (grouped-query attention: a step of 64 keys lies inside one 128-token page).  One CTA owns one head and up to 256
 // consecutive new tokens of one request as two blocks of 128 query rows; both blocks read the same 64-key K / V steps, loaded once,
 // and their softmax runs on two warp groups, so the tensor core alternates between the blocks:
 //     S_b[128 q x 64 k] = Q_b * K^T        O_b[128 q x V] += P_b * V          b = 0, 1
@@ -24,15 +25,24 @@ constexpr int AW_SMEM_MAX = 227 * 1024;
 
 struct AttnWindowParams {
   // [n_blocks][6] = packed row of the first query, its position, query rows (<= 256), row of the request's first key, that key's
-  // position, (unused)
+  // position, request (row of the page table)
   const int* blocks;
   uint16_t* out; long long ld_out;
   const uint16_t* gate; long long ld_gate;
   int D, V, dt, vt;                               // head widths, their 64-column tiles
   int stages, window;
+  int chunk;                                      // > 0 (instead of a window): a query sees the keys of its own chunk of positions
+  int group;                                      // query heads per key / value head
+  const int* page_table; int max_pages, num_pages;     // null: contiguous keys
   float scale_log2;
   uint32_t idesc_s, idesc_o;
 };
+
+// first position a query at `pos` sees
+__device__ __forceinline__ int aw_first(const AttnWindowParams& p, int pos) {
+  if (p.chunk > 0) return pos - pos % p.chunk;
+  return p.window > 0 ? pos - p.window + 1 : 0;
+}
 
 template <bool BF16>
 __global__ void __launch_bounds__(320, 1)
@@ -56,12 +66,12 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head = blockIdx.x;
+  const int head = blockIdx.x, kv_head = head / p.group;
   const int* blk = p.blocks + 6 * blockIdx.y;
   const int q_row0 = blk[0], pos0 = blk[1], rows = blk[2], key_row0 = blk[3], key0 = blk[4];
   // first key of the block's first row, one past the last key of its last row
-  int lo = key0;
-  if (p.window > 0 && pos0 - p.window + 1 > lo) lo = pos0 - p.window + 1;
+  int lo = max(key0, aw_first(p, pos0));
+  if (p.page_table != nullptr) lo &= ~(AW_KV - 1);          // a step never straddles two pages; the mask drops what lies before
   const int hi = pos0 + rows;
   const int n_steps = (hi - lo + AW_KV - 1) / AW_KV;
   // steps [f, e) of query block b
@@ -69,9 +79,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   f[0] = 0;
   e[0] = (pos0 + (rows < 128 ? rows : 128) - lo + AW_KV - 1) / AW_KV;
   if (rows > 128) {
-    int lo1 = lo;
-    if (p.window > 0 && pos0 + 128 - p.window + 1 > lo1) lo1 = pos0 + 128 - p.window + 1;
-    f[1] = (lo1 - lo) / AW_KV;
+    f[1] = (max(lo, aw_first(p, pos0 + 128)) - lo) / AW_KV;
     e[1] = n_steps;
   } else {
     f[1] = e[1] = n_steps;
@@ -103,13 +111,19 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const int s = it % stages;
         const uint32_t ph = (uint32_t)(it / stages) & 1u;
         if (!mbar_wait(&empty[s], ph ^ 1u, dead, KID_ATTN_WINDOW, 1)) break;
-        const int row = key_row0 + (lo - key0) + it * AW_KV;
+        int row = key_row0 + (lo - key0) + it * AW_KV;
+        if (p.page_table != nullptr) {
+          const int key = lo + it * AW_KV;
+          int page = (key >> 7) < p.max_pages ? p.page_table[(size_t)blk[5] * p.max_pages + (key >> 7)] : 0;
+          if ((unsigned)page >= (unsigned)p.num_pages) { report_error(ERR_BAD_ARG, KID_ATTN_WINDOW, 20); page = 0; }
+          row = page * 128 + (key & 127);
+        }
         uint8_t* kb = kv_smem + s * stage_bytes;
         uint8_t* vb = kb + dt * AW_KT;
         mbar_expect_tx(&full_k[s], dt * AW_KT);
-        for (int j = 0; j < dt; ++j) tma_load_3d(kb + j * AW_KT, &tmK, &full_k[s], j * 64, head, row);
+        for (int j = 0; j < dt; ++j) tma_load_3d(kb + j * AW_KT, &tmK, &full_k[s], j * 64, kv_head, row);
         mbar_expect_tx(&full_v[s], vt * AW_KT);
-        for (int j = 0; j < vt; ++j) tma_load_3d(vb + j * AW_KT, &tmV, &full_v[s], j * 64, head, row);
+        for (int j = 0; j < vt; ++j) tma_load_3d(vb + j * AW_KT, &tmV, &full_v[s], j * 64, kv_head, row);
       }
     }
     __syncwarp();
@@ -173,7 +187,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const int q = warp & 3;                      // TMEM lane quarter: warps 2..5 -> 2,3,0,1 ; 6..9 -> 2,3,0,1
     const int r = q * 32 + lane;
     const int pos_b = pos0 + b * 128, pos = pos_b + r;
-    const int first = p.window > 0 ? pos - p.window + 1 : 0;
+    const int first = aw_first(p, pos), first_all = aw_first(p, pos_b + 127);      // of this row; no earlier than any row of the block's
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const uint32_t tmem_s = tmem0 + (uint32_t)(b * 64), tmem_o = tmem0 + 128u + (uint32_t)b * o_cols;
     uint8_t* prow = p_smem + b * AW_PT + r * 128;
@@ -189,7 +203,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       tmem_ld_32x32b_x32(tmem_s + lane_off + 32, sreg + 32);
       tmem_ld_wait();
       // only steps on the causal diagonal or on the window's edge pay for the mask
-      const bool full_step = kv0 + AW_KV - 1 <= pos_b && (p.window <= 0 || kv0 > pos_b + 127 - p.window);
+      const bool full_step = kv0 + AW_KV - 1 <= pos_b && kv0 >= first_all;
       float m_new = m_run;
       if (full_step) {
 #pragma unroll
@@ -300,27 +314,14 @@ using namespace fb;
 
 extern "C" int fb_attn_window_supported(int D, int V) { return D > 0 && V > 0 && D % 8 == 0 && V % 8 == 0 && window_stages(D, V) > 0 ? 1 : 0; }
 
-// q: packed rows [T, >= H * D] (row stride ld_q), k: [n_keys, >= H * D], v: [n_keys, >= H * V], out [T, H * V], gate (optional) like out.
-extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* k, long long ld_k, const void* v, long long ld_v, int n_keys,
-                              void* out, long long ld_out, const void* gate, long long ld_gate, const int* blocks, int n_blocks, int H,
-                              int D, int V, int window, float scale, int dtype, void* stream_) {
-  if (n_blocks <= 0) return 0;
-  const int stages = window_stages(D, V);
-  if (stages == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || n_keys <= 0 || H <= 0 || n_blocks > 65535 || window < 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
-    return -1;
-  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
-  CUtensorMap tmQ, tmK, tmV;
-  if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
-  if (!make_tmap_3d(&tmK, k, D, H, n_keys, D, ld_k, 64, AW_KV)) return -2;
-  if (!make_tmap_3d(&tmV, v, V, H, n_keys, V, ld_v, 64, AW_KV)) return -2;
-  AttnWindowParams p;
-  p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
-  p.D = D; p.V = V; p.dt = (D + 63) / 64; p.vt = (V + 63) / 64; p.stages = stages; p.window = window;
+static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, AttnWindowParams p, int n_blocks, int H, float scale,
+                         int dtype, cudaStream_t stream) {
+  p.dt = (p.D + 63) / 64; p.vt = (p.V + 63) / 64; p.stages = window_stages(p.D, p.V);
   p.scale_log2 = scale * 1.4426950408889634f;
   const uint32_t fm = dtype == 1 ? 1u : 0u;
   p.idesc_s = make_idesc(fm, fm, 0, 0, 128, AW_KV);
   p.idesc_o = make_idesc(fm, fm, 0, 1, 128, p.vt * 64);
-  const int smem = 2 * p.dt * AW_QT + stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
+  const int smem = 2 * p.dt * AW_QT + p.stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
   const dim3 grid(H, n_blocks);
   if (dtype == 1) {
     static DeviceOnce cfg;
@@ -332,4 +333,43 @@ extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* 
     attn_window_kernel<false><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);
   }
   return (int)cudaGetLastError();
+}
+
+// q: packed rows [T, >= H * D] (row stride ld_q), k: [n_keys, >= H * D], v: [n_keys, >= H * V], out [T, H * V], gate (optional) like out.
+extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* k, long long ld_k, const void* v, long long ld_v, int n_keys,
+                              void* out, long long ld_out, const void* gate, long long ld_gate, const int* blocks, int n_blocks, int H,
+                              int D, int V, int window, float scale, int dtype, void* stream_) {
+  if (n_blocks <= 0) return 0;
+  if (window_stages(D, V) == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || n_keys <= 0 || H <= 0 || n_blocks > 65535 || window < 0 || ld_out % 8 != 0 ||
+      ld_gate % 8 != 0)
+    return -1;
+  CUtensorMap tmQ, tmK, tmV;
+  if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
+  if (!make_tmap_3d(&tmK, k, D, H, n_keys, D, ld_k, 64, AW_KV)) return -2;
+  if (!make_tmap_3d(&tmV, v, V, H, n_keys, V, ld_v, 64, AW_KV)) return -2;
+  AttnWindowParams p = {};
+  p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
+  p.D = D; p.V = V; p.window = window; p.group = 1;
+  return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
+}
+
+// Grouped-query form over the cache pages: k_pool [num_slots, G, D], v_pool [num_slots, G, V], 128 slots a page; query head h uses
+// key / value head h / (H / G).  page_table: [requests, max_pages], a block's request is blocks[.][5].
+extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const void* k_pool, const void* v_pool, long long num_slots,
+                                    const int* page_table, int max_pages, void* out, long long ld_out, const void* gate, long long ld_gate,
+                                    const int* blocks, int n_blocks, int H, int G, int D, int V, int window, int chunk, float scale, int dtype,
+                                    void* stream_) {
+  if (n_blocks <= 0) return 0;
+  if (window_stages(D, V) == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || num_slots < 128 || H <= 0 || G <= 0 || H % G != 0 || n_blocks > 65535 ||
+      window < 0 || chunk < 0 || max_pages <= 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
+    return -1;
+  CUtensorMap tmQ, tmK, tmV;
+  if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
+  if (!make_tmap_3d(&tmK, k_pool, D, G, num_slots, D, (long long)G * D, 64, AW_KV)) return -2;
+  if (!make_tmap_3d(&tmV, v_pool, V, G, num_slots, V, (long long)G * V, 64, AW_KV)) return -2;
+  AttnWindowParams p = {};
+  p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
+  p.D = D; p.V = V; p.window = window; p.chunk = chunk; p.group = H / G;
+  p.page_table = page_table; p.max_pages = max_pages; p.num_pages = (int)(num_slots / 128);
+  return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }

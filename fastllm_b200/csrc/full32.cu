@@ -1,4 +1,4 @@
-// 32-bit and any-size forms of a model's matrix products and of latent attention (CUDA cores, fp32 FMAs).
+// 32-bit and any-size forms of a model's matrix products, of latent attention and of grouped-query attention (CUDA cores, fp32 FMAs).
 //
 // They serve models run in float32, where the tensor core has no full-precision mode, and 16-bit shapes outside the tensor-core
 // kernels' tiling.  Compiled without fast-math.
@@ -147,6 +147,83 @@ __global__ void __launch_bounds__(128) latent_attn32_kernel(const typename F32In
   for (int i = tid; i < ld; i += 128) op[i] = F32In<DT>::st(i < R ? os[i] * inv : 0.f);
 }
 
+// Grouped-query attention of one (row, query head) per CTA over paged keys and values, any widths, fp32 arithmetic:
+//   out = (sum_j softmax(scale q . k_j) v_j) * sigmoid(gate),  first(position) <= j <= position
+// Row t sees the keys of its own page-table row; its position is kv_lens[t] - 1.  chunk: first = position - position % chunk; window:
+// first = position - window + 1; neither: 0.
+struct Grouped32Params {
+  const void* q; const void* k_pool; const void* v_pool; void* out; const void* gate;
+  long long ld_q, ld_out, ld_gate;
+  const int* page_table; const int* kv_lens;
+  int H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk;
+  float scale;
+};
+
+template <int DT>
+__global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Params p) {
+  typedef typename F32In<DT>::T T;
+  extern __shared__ float sm[];
+  float* qs = sm;                       // [Dp]
+  float* os = sm + p.Dp;                // [Vp] running output
+  __shared__ float sc[L32_KEYS];
+  __shared__ int rows[L32_KEYS];
+  const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = h / (p.H / p.G);
+  const int n = p.kv_lens[t], pos = n - 1;
+  int first = 0;
+  if (p.chunk > 0) first = n > 0 ? pos - pos % p.chunk : 0;
+  else if (p.window > 0 && n > p.window) first = n - p.window;
+  const T* qp = reinterpret_cast<const T*>(p.q) + (size_t)t * p.ld_q + (size_t)h * p.Dp;
+  const T* kp = reinterpret_cast<const T*>(p.k_pool);
+  const T* vp = reinterpret_cast<const T*>(p.v_pool);
+  for (int i = tid; i < p.Dp; i += 128) qs[i] = F32In<DT>::ld(qp[i]);
+  for (int i = tid; i < p.Vp; i += 128) os[i] = 0.f;
+  float m_run = -INFINITY, l_run = 0.f;
+  for (int j0 = first; j0 < n; j0 += L32_KEYS) {
+    const int cnt = n - j0 < L32_KEYS ? n - j0 : L32_KEYS;
+    __syncthreads();
+    if (tid < cnt) {
+      const int j = j0 + tid, pg = j / p.page_len;
+      int page = pg < p.max_pages ? p.page_table[(size_t)t * p.max_pages + pg] : 0;
+      if ((unsigned)page >= (unsigned)p.num_pages) page = 0;
+      rows[tid] = page * p.page_len + (j - pg * p.page_len);
+    }
+    __syncthreads();
+    for (int j = warp; j < cnt; j += 4) {
+      const T* c = kp + ((size_t)rows[j] * p.G + g) * p.Dp;
+      float s = 0.f;
+      for (int i = lane; i < p.D; i += 32) s = fmaf(qs[i], F32In<DT>::ld(c[i]), s);
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      if (lane == 0) sc[j] = s * p.scale;
+    }
+    __syncthreads();
+    float mx = m_run;
+    for (int j = 0; j < cnt; ++j) mx = fmaxf(mx, sc[j]);
+    const float fac = m_run == -INFINITY ? 0.f : expf(m_run - mx);
+    __syncthreads();
+    if (tid < cnt) sc[tid] = expf(sc[tid] - mx);
+    __syncthreads();
+    float l = 0.f;
+    for (int j = 0; j < cnt; ++j) l += sc[j];
+    l_run = l_run * fac + l;
+    m_run = mx;
+    for (int i = tid; i < p.Vp; i += 128) {
+      float a = os[i] * fac;
+      for (int j = 0; j < cnt; ++j) a = fmaf(sc[j], F32In<DT>::ld(vp[((size_t)rows[j] * p.G + g) * p.Vp + i]), a);
+      os[i] = a;
+    }
+  }
+  const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  T* op = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.Vp;
+  const T* gp = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + (size_t)h * p.Vp : nullptr;
+  for (int i = tid; i < p.Vp; i += 128) {
+    float v = os[i] * inv;
+    if (gp != nullptr) v *= 1.0f / (1.0f + expf(-F32In<DT>::ld(gp[i])));
+    op[i] = F32In<DT>::st(v);
+  }
+}
+
 }  // namespace fb
 
 using namespace fb;
@@ -186,6 +263,29 @@ extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, cons
     if (cfg.need()) cudaFuncSetAttribute(latent_attn32_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 24576 * 8);         \
     latent_attn32_kernel<DT><<<dim3(T, H), 128, smem, s>>>((const F32In<DT>::T*)q, (const F32In<DT>::T*)pool, (F32In<DT>::T*)out,  \
                                                            page_table, kv_lens, max_pages, page_len, H, R, ld, window, scale);     \
+  }
+  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// See Grouped32Params; q / out / gate: T rows, pools [num_pages * page_len, G, Dp / Vp].
+extern "C" int fb_grouped_attn32(const void* q, long long ld_q, const void* k_pool, const void* v_pool, void* out, long long ld_out,
+                                 const void* gate, long long ld_gate, const int* page_table, const int* kv_lens, int T, int H, int G, int D,
+                                 int Dp, int Vp, int max_pages, int num_pages, int page_len, int window, int chunk, float scale, int dt,
+                                 void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G <= 0 || H % G != 0 || H > 65535 || D <= 0 || Dp < D || Vp <= 0 || Dp + Vp > 49152 || max_pages <= 0 || num_pages <= 0 ||
+      page_len <= 0 || window < 0 || chunk < 0 || dt < 0 || dt > 2)
+    return -1;
+  Grouped32Params p{q, k_pool, v_pool, out, gate, ld_q, ld_out, ld_gate, page_table, kv_lens, H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, scale};
+  const size_t smem = (size_t)(Dp + Vp) * 4;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+#define GO(DT)                                                                                                          \
+  {                                                                                                                     \
+    static DeviceOnce cfg;                                                                                              \
+    if (cfg.need()) cudaFuncSetAttribute(grouped_attn32_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 49152 * 4); \
+    grouped_attn32_kernel<DT><<<dim3(T, H), 128, smem, s>>>(p);                                                         \
   }
   if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
 #undef GO

@@ -46,6 +46,7 @@ enum GemmFlags : int {
   GEMM_OUT_F32 = 8,    // write fp32 instead of the 16-bit input dtype
   GEMM_RES_F32 = 16,   // with GEMM_RESIDUAL: the residual is fp32 and the product is scaled first, residual + alpha * acc
   GEMM_RELU2 = 32,     // out = relu(acc)^2
+  GEMM_GLU_CLAMP = 64, // with GEMM_SWIGLU: g = min(gate, act_limit), u = clamp(up, +-act_limit), out = g * sigmoid(act_alpha * g) * (u + 1)
   GEMM_FP4_F16W = 256, // fp4 weights, fp16 activations: the scale table lies within fp16's range (host-checked): half2 de-quantiser
 };
 
@@ -76,10 +77,16 @@ struct GemmParams {
   float alpha = 1.f;                         // GEMM_RES_F32
   const void* gate = nullptr;                // 16-bit [M, >= N] (batched: + z * batch_out_cols): out = acc * sigmoid(gate)
   int ld_gate = 0;
+  float act_limit = 0.f, act_alpha = 1.f;    // GEMM_GLU_CLAMP
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + __expf(-x)); }
+__device__ __forceinline__ float glu_clamp_f(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return g * sigmoid_f(alpha * g) * (u + 1.0f);
+}
 __device__ __forceinline__ float relu2_f(float x) { const float r = fmaxf(x, 0.f); return r * r; }
 
 // OCC = CTAs meant to be co-resident per SM: 1 -> deep ring (~200 KB), 2 -> two CTAs share the SM so that one
@@ -132,8 +139,13 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
           acc.x += b0.x; acc.y += b0.y; acc.z += b1.x; acc.w += b1.y;
           acc2.x += u0.x; acc2.y += u0.y; acc2.z += u1.x; acc2.w += u1.y;
         }
-        acc.x = silu_f(acc.x) * acc2.x; acc.y = silu_f(acc.y) * acc2.y;
-        acc.z = silu_f(acc.z) * acc2.z; acc.w = silu_f(acc.w) * acc2.w;
+        if (p.flags & GEMM_GLU_CLAMP) {
+          acc.x = glu_clamp_f(acc.x, acc2.x, p.act_limit, p.act_alpha); acc.y = glu_clamp_f(acc.y, acc2.y, p.act_limit, p.act_alpha);
+          acc.z = glu_clamp_f(acc.z, acc2.z, p.act_limit, p.act_alpha); acc.w = glu_clamp_f(acc.w, acc2.w, p.act_limit, p.act_alpha);
+        } else {
+          acc.x = silu_f(acc.x) * acc2.x; acc.y = silu_f(acc.y) * acc2.y;
+          acc.z = silu_f(acc.z) * acc2.z; acc.w = silu_f(acc.w) * acc2.w;
+        }
         if (n_out >= (p.N >> 1)) continue;
       } else {
         n_out = n_tile * 128 + c;

@@ -1,8 +1,8 @@
 // Mixture-of-experts execution for sm_100a: routing plan, token gather, grouped expert GEMMs, weighted combine.
 //
 //   moe_plan     one CTA: per-local-expert token counts, segment offsets padded to 16 rows, and for every (token, k)
-//                pair its row in the expert-sorted buffer (-1 if the expert lives on another rank).  Deterministic:
-//                rows inside a segment follow (token, k) order.
+//                pair its row in the expert-sorted buffer (-1 if the expert lives on another rank).  Up to 4096 pairs
+//                the rows inside a segment follow (token, k) order.
 //   moe_gather   copies each routed token row into its sorted position
 //   grouped GEMM the swap-AB tcgen05 decode GEMM run once per (expert, 128/256-token chunk) through blockIdx.z; the
 //                weight tile coordinate is offset into the stacked expert matrix, the activation tile into the sorted
@@ -33,42 +33,7 @@ struct MoeGroupInfo {
   int n_local, compact;    // compact: grid.z enumerates existing (expert, chunk) pairs (moe_find_item)
 };
 
-// counts/offsets/pos for the experts in [first, first + n_local)
-__global__ void moe_plan_kernel(const int* __restrict__ idx, int T, int topk, int first, int n_local, int* __restrict__ counts,
-                                int* __restrict__ offsets, int* __restrict__ pos, int* __restrict__ total_rows, int pad) {
-  __shared__ int s_cnt[1024];
-  __shared__ int s_off[1025];
-  const int e = threadIdx.x;
-  pdl_launch_dependents();
-  pdl_wait();
-  const int pairs = T * topk;
-  int c = 0;
-  if (e < n_local) {
-    for (int i = 0; i < pairs; ++i) c += (idx[i] == first + e);
-  }
-  s_cnt[e] = e < n_local ? c : 0;
-  __syncthreads();
-  if (e == 0) {
-    int acc = 0;
-    for (int i = 0; i < n_local; ++i) { s_off[i] = acc; acc += (s_cnt[i] + pad - 1) / pad * pad; }
-    s_off[n_local] = acc;
-    *total_rows = acc;
-  }
-  __syncthreads();
-  if (e < n_local) {
-    counts[e] = s_cnt[e];
-    offsets[e] = s_off[e];
-    int r = s_off[e];
-    for (int i = 0; i < pairs; ++i)
-      if (idx[i] == first + e) pos[i] = r++;
-  }
-  // pairs whose expert is not local
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int x = idx[i];
-    if (x < first || x >= first + n_local) pos[i] = -1;
-  }
-}
-
+// counts / offsets / pos of the experts in [first, first + n_local).
 // Small problems (pairs <= 4096): one thread per (token, k) pair; rank inside the expert segment = number of earlier pairs
 // routed to the same expert, so the order is deterministic without any sorting pass.
 __global__ void moe_plan_small_kernel(const int* __restrict__ idx, int pairs, int first, int n_local, int* __restrict__ counts,
@@ -177,6 +142,45 @@ moe_plan_warp_kernel(const int* __restrict__ idx, int pairs, int first, int n_lo
     const int e = i < pairs ? s_idx[i] : -1;
     const uint32_t same = __match_any_sync(0xffffffffu, e);
     if (i < pairs) pos[i] = e < 0 ? -1 : s_off[e] + (int)s_w[c * n_local + e] + __popc(same & lt_mask);
+  }
+}
+
+// Large problems: counts by shared-memory atomics, then rows handed out by atomics (rows inside an expert's segment come in no
+// particular order: every row's product stands alone).
+__global__ void __launch_bounds__(1024)
+moe_plan_large_kernel(const int* __restrict__ idx, int pairs, int first, int n_local, int* __restrict__ counts, int* __restrict__ offsets,
+                      int* __restrict__ pos, int* __restrict__ total_rows, int pad) {
+  __shared__ int s_cnt[1024];
+  __shared__ int s_off[1024];
+  pdl_launch_dependents();
+  pdl_wait();
+  for (int e = threadIdx.x; e < n_local; e += blockDim.x) s_cnt[e] = 0;
+  __syncthreads();
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const int e = idx[i] - first;
+    if (e >= 0 && e < n_local) atomicAdd(&s_cnt[e], 1);
+  }
+  __syncthreads();
+  if (threadIdx.x < 32) {
+    int carry = 0;
+    for (int base = 0; base < n_local; base += 32) {
+      const int e = base + threadIdx.x;
+      const int c = e < n_local ? (s_cnt[e] + pad - 1) / pad * pad : 0;
+      int incl = c;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, incl, o);
+        if ((int)threadIdx.x >= o) incl += v;
+      }
+      if (e < n_local) { counts[e] = s_cnt[e]; offsets[e] = s_off[e] = carry + incl - c; }
+      carry += __shfl_sync(0xffffffffu, incl, 31);
+    }
+    if (threadIdx.x == 0) *total_rows = carry;
+  }
+  __syncthreads();
+  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
+    const int e = idx[i] - first;
+    pos[i] = e >= 0 && e < n_local ? atomicAdd(&s_off[e], 1) : -1;
   }
 }
 
@@ -338,10 +342,7 @@ extern "C" int fb_moe_plan(const int* idx, int T, int topk, int first, int n_loc
     launch_k(moe_plan_small_kernel, dim3(1), dim3(1024), 0, reinterpret_cast<cudaStream_t>(stream), 0, idx, T * topk, first, n_local, counts, offsets, pos, total_rows, pad);
     return (int)cudaGetLastError();
   }
-  int threads = 32;
-  while (threads < n_local) threads <<= 1;
-  if (threads < 256) threads = 256;
-  launch_k(moe_plan_kernel, dim3(1), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), 0, idx, T, topk, first, n_local, counts, offsets, pos, total_rows, pad);
+  launch_k(moe_plan_large_kernel, dim3(1), dim3(1024), 0, reinterpret_cast<cudaStream_t>(stream), 0, idx, T * topk, first, n_local, counts, offsets, pos, total_rows, pad);
   return (int)cudaGetLastError();
 }
 
@@ -371,12 +372,24 @@ extern "C" int fb_moe_combine(const void* ys, const int* pos, const float* w, co
   return (int)cudaGetLastError();
 }
 
+extern "C" int fb_moe_grouped_gemm_act(const void* Xs, const void* W, void* out, const void* bias, const int* counts, const int* offsets,
+                                       int rows_cap, int E_local, int N, int K, int ld_out, int max_rows_per_expert, int dtype, int flags,
+                                       int total_rows, float act_limit, float act_alpha, void* stream_);
+
 // Grouped Y_e = X_e W_e^T over the sorted buffer.  Xs: [rows_cap, K] sorted rows; W: stacked [E_local * N, K] with every
 // expert's rows padded to a multiple of 128; out: [rows_cap, N or N/2].
 // max_rows_per_expert bounds the chunk count (T for decode: every token could pick the same expert).
 extern "C" int fb_moe_grouped_gemm(const void* Xs, const void* W, void* out, const void* bias, const int* counts, const int* offsets,
                                    int rows_cap, int E_local, int N, int K, int ld_out, int max_rows_per_expert, int dtype, int flags,
                                    int total_rows, void* stream_) {
+  return fb_moe_grouped_gemm_act(Xs, W, out, bias, counts, offsets, rows_cap, E_local, N, K, ld_out, max_rows_per_expert, dtype, flags, total_rows, 0.f,
+                                 1.f, stream_);
+}
+
+// act_limit / act_alpha: constants of the GEMM_GLU_CLAMP activation.
+extern "C" int fb_moe_grouped_gemm_act(const void* Xs, const void* W, void* out, const void* bias, const int* counts, const int* offsets,
+                                       int rows_cap, int E_local, int N, int K, int ld_out, int max_rows_per_expert, int dtype, int flags,
+                                       int total_rows, float act_limit, float act_alpha, void* stream_) {
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (E_local <= 0 || rows_cap <= 0) return 0;
   if (K % 8 != 0 || N % 8 != 0 || ((flags & GEMM_SWIGLU) && N % 128 != 0) || (dtype != 0 && dtype != 1)) return -1;
@@ -392,6 +405,7 @@ extern "C" int fb_moe_grouped_gemm(const void* Xs, const void* W, void* out, con
   p.out = out; p.bias = bias; p.residual = nullptr;
   p.M = 0; p.N = N; p.K = K; p.ld_out = ld_out; p.ld_res = 0;
   p.kb_total = (K + 63) / 64; p.flags = flags;
+  p.act_limit = act_limit; p.act_alpha = act_alpha;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
   const int n_tiles = n_rows_w / 128;

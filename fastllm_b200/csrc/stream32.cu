@@ -1,5 +1,6 @@
-// Operators of models whose residual stream is fp32: token embedding plus sinusoidal positions, RMSNorm of an fp32 row into the
-// activation type, latent RMSNorm into the cache, and the mixture-of-experts combine that ends in residual and norm.
+// Operators of models whose residual stream is fp32: token embedding plus sinusoidal or learned positions, RMSNorm of an fp32 row
+// into the activation type, latent RMSNorm into the cache, per-head norm + rotary + cache append, and the end of a sub-layer (output
+// norm, residual, next norm) for a plain output or a mixture-of-experts combine.
 //
 // One CTA owns a row; the row stays in shared memory between the reduction and the normalised write, so every operand is read
 // once.  Compiled without fast-math: angles, square roots and divisions are the correctly rounded fp32 ones.
@@ -79,6 +80,15 @@ __device__ __forceinline__ void norm_write(const float* row, const typename Act<
   }
 }
 
+// the same, or the row itself where there is no weight
+template <int DT, int VEC>
+__device__ __forceinline__ void row_write(const float* row, const typename Act<DT>::T* w, typename Act<DT>::T* y, int H, float inv) {
+  if (w != nullptr) { norm_write<DT, VEC>(row, w, y, H, inv); return; }
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+    if (VEC == 4) st4<DT>(y + i, row + i); else y[i] = Act<DT>::st(row[i]);
+  }
+}
+
 // y[row] = RMSNorm(x[row]) * w
 template <int DT, int VEC>
 __global__ void rmsnorm32_kernel(const float* __restrict__ x, const typename Act<DT>::T* __restrict__ w, typename Act<DT>::T* __restrict__ y,
@@ -103,12 +113,14 @@ __global__ void rmsnorm32_kernel(const float* __restrict__ x, const typename Act
   norm_write<DT, VEC>(row, w, y + (size_t)blockIdx.x * ldy, H, inv);
 }
 
-// h[t] = table[ids[t]] + sinusoid(positions[t]) in fp32, and its RMSNorm.  inv_freq[i] = 10000^(-2i / H) in double; the angle is
-// reduced to [-pi, pi] in double, so a far position costs no accuracy.
+// h[t] = table[ids[t]] + position in fp32, and its RMSNorm (w == nullptr: the row itself; y == nullptr: h only).  inv_freq: the position
+// is sines and cosines, inv_freq[i] = 10000^(-2i / H) in double; the angle is reduced to [-pi, pi] in double, so a far position costs
+// no accuracy.  pos_table: it is row positions[t] of a learned table.
 template <int DT, int VEC>
 __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ positions, const typename Act<DT>::T* __restrict__ table,
-                                      const double* __restrict__ inv_freq, const typename Act<DT>::T* __restrict__ w, float* __restrict__ h,
-                                      typename Act<DT>::T* __restrict__ y, int H, int vocab, float eps) {
+                                      const double* __restrict__ inv_freq, const typename Act<DT>::T* __restrict__ pos_table, int pos_rows,
+                                      const typename Act<DT>::T* __restrict__ w, float* __restrict__ h, typename Act<DT>::T* __restrict__ y, int H,
+                                      int vocab, float eps) {
   extern __shared__ float row[];
   __shared__ float sh[32];
   pdl_launch_dependents();
@@ -118,7 +130,10 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
   id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
   const typename Act<DT>::T* e = table + (size_t)id * H;
   float* hp = h + (size_t)t * H;
-  const double pos = (double)positions[t];
+  int row_p = positions[t];
+  const double pos = (double)row_p;
+  row_p = row_p < 0 ? 0 : (row_p >= pos_rows ? pos_rows - 1 : row_p);
+  const typename Act<DT>::T* pe = pos_table != nullptr ? pos_table + (size_t)row_p * H : nullptr;
   float ss = 0.f;
   auto add_pos = [&](int i, float& a, float& b) {
     const double ang = pos * inv_freq[i];
@@ -132,6 +147,11 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
       float v[4];
       ld4<DT>(e + i, v);
       if (inv_freq != nullptr) { add_pos(i / 2, v[0], v[1]); add_pos(i / 2 + 1, v[2], v[3]); }
+      if (pe != nullptr) {
+        float u[4];
+        ld4<DT>(pe + i, u);
+        v[0] += u[0]; v[1] += u[1]; v[2] += u[2]; v[3] += u[3];
+      }
       st4<2>(hp + i, v);
       st4<2>(row + i, v);
       ss += v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
@@ -141,13 +161,15 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
       const bool two = 2 * i + 1 < H;
       float a = Act<DT>::ld(e[2 * i]), b = two ? Act<DT>::ld(e[2 * i + 1]) : 0.f;
       if (inv_freq != nullptr) add_pos(i, a, b);
+      if (pe != nullptr) { a += Act<DT>::ld(pe[2 * i]); if (two) b += Act<DT>::ld(pe[2 * i + 1]); }
       hp[2 * i] = a; row[2 * i] = a; ss += a * a;
       if (two) { hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b; }
     }
   }
+  if (y == nullptr) return;
   ss = block_sum32(ss, sh);
   const float inv = 1.0f / sqrtf(ss / (float)H + eps);
-  norm_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
+  row_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
 }
 
 // pool[slot] = RMSNorm over the first `n` columns of x[t] (columns [n, ld) of the entry are zero); slots < 0 go to `spare`
@@ -169,14 +191,15 @@ __global__ void latent_norm_kernel(const typename Act<DT>::T* __restrict__ x, in
   for (int i = threadIdx.x; i < ld; i += blockDim.x) yp[i] = Act<DT>::st(i < n ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
 }
 
-// h[t] += alpha * (sum_k wk * ys[pos[t, k]] + shared[t]), then y[t] = RMSNorm(h[t]) * w.  wts == nullptr: every weight is `wconst`.
+// z[t] = sum_k wk * ys[pos[t, k]] + shared[t]; with an output norm z = RMSNorm(z) * post; h[t] += alpha * z; then y[t] = RMSNorm(h[t]) * w.
+// wts == nullptr: every weight is `wconst`.  pos == nullptr: z[t] = ys[t].  w == nullptr: y[t] = h[t].  y == nullptr: h only.
 template <int DT, int VEC>
 __global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict__ ys, const int* __restrict__ pos, const float* __restrict__ wts,
                                           float wconst, const typename Act<DT>::T* __restrict__ shared_y, float* __restrict__ h,
-                                          const typename Act<DT>::T* __restrict__ w, typename Act<DT>::T* __restrict__ y, int topk, int H,
-                                          float alpha, float eps) {
+                                          const typename Act<DT>::T* __restrict__ post, const typename Act<DT>::T* __restrict__ w,
+                                          typename Act<DT>::T* __restrict__ y, int topk, int H, float alpha, float eps) {
   extern __shared__ float row[];
-  __shared__ float sh[32];
+  __shared__ float sh[2][32];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
@@ -186,27 +209,137 @@ __global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict_
     float acc[VEC], v[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) acc[j] = 0.f;
-    for (int k = 0; k < topk; ++k) {
-      const int r = pos[(size_t)t * topk + k];
-      if (r < 0) continue;
-      const float wk = wts != nullptr ? wts[(size_t)t * topk + k] : wconst;
-      if (VEC == 4) ld4<DT>(ys + (size_t)r * H + i, v); else v[0] = Act<DT>::ld(ys[(size_t)r * H + i]);
+    if (pos == nullptr) {
+      if (VEC == 4) ld4<DT>(ys + (size_t)t * H + i, acc); else acc[0] = Act<DT>::ld(ys[(size_t)t * H + i]);
+    } else {
+      for (int k = 0; k < topk; ++k) {
+        const int r = pos[(size_t)t * topk + k];
+        if (r < 0) continue;
+        const float wk = wts != nullptr ? wts[(size_t)t * topk + k] : wconst;
+        if (VEC == 4) ld4<DT>(ys + (size_t)r * H + i, v); else v[0] = Act<DT>::ld(ys[(size_t)r * H + i]);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) acc[j] += wk * v[j];
+        for (int j = 0; j < VEC; ++j) acc[j] += wk * v[j];
+      }
     }
     if (shared_y != nullptr) {
       if (VEC == 4) ld4<DT>(shared_y + (size_t)t * H + i, v); else v[0] = Act<DT>::ld(shared_y[(size_t)t * H + i]);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) acc[j] += v[j];
     }
+    if (post != nullptr) {                     // the thread's own columns wait in shared memory for the output norm
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) { ss += acc[j] * acc[j]; row[i + j] = acc[j]; }
+      continue;
+    }
     if (VEC == 4) ld4<2>(hp + i, v); else v[0] = hp[i];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) { v[j] += alpha * acc[j]; ss += v[j] * v[j]; row[i + j] = v[j]; }
     if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
   }
-  ss = block_sum32(ss, sh);
-  const float inv = 1.0f / sqrtf(ss / (float)H + eps);
-  norm_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
+  if (post != nullptr) {
+    ss = block_sum32(ss, sh[0]);
+    const float inv = 1.0f / sqrtf(ss / (float)H + eps);
+    ss = 0.f;
+    for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+      float pv[VEC], v[VEC];
+      if (VEC == 4) { ld4<DT>(post + i, pv); ld4<2>(hp + i, v); } else { pv[0] = Act<DT>::ld(post[i]); v[0] = hp[i]; }
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) { v[j] += alpha * (row[i + j] * inv * pv[j]); ss += v[j] * v[j]; row[i + j] = v[j]; }
+      if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
+    }
+  }
+  if (y == nullptr) return;
+  float inv = 1.f;
+  if (w != nullptr) {
+    ss = block_sum32(ss, sh[1]);
+    inv = 1.0f / sqrtf(ss / (float)H + eps);
+  }
+  row_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);       // (without a weight every thread writes the columns it owns)
+}
+
+// xs[pos[t, k]] = wts[t, k] * x[t] for fp32 rows: one CTA per row, all its experts' copies
+template <int DT, int VEC>
+__global__ void moe_gather_scaled_kernel(const float* __restrict__ x, const int* __restrict__ pos, const float* __restrict__ wts,
+                                         typename Act<DT>::T* __restrict__ xs, int topk, int H) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int t = blockIdx.x;
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+    float v[VEC], o[VEC];
+    if (VEC == 4) ld4<2>(x + (size_t)t * H + i, v); else v[0] = x[(size_t)t * H + i];
+    for (int k = 0; k < topk; ++k) {
+      const int r = pos[(size_t)t * topk + k];
+      if (r < 0) continue;
+      const float wk = wts[(size_t)t * topk + k];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = wk * v[j];
+      if (VEC == 4) st4<DT>(xs + (size_t)r * H + i, o); else xs[(size_t)r * H + i] = Act<DT>::st(o[0]);
+    }
+  }
+}
+
+// Per-head RMS norm, interleaved rotary positions and cache append of a merged projection [queries | gate | keys | values], one warp
+// per (token, head), fp32 arithmetic.  Heads are D wide, stored Dp (values Vp); queries are rewritten in place, keys and values go to
+// their cache slots (slot < 0: nowhere).  rot: leading dimensions that turn; cos / sin tables [tab_rows, rot / 2].
+struct HeadPostParams {
+  void* proj; long long ld;
+  const int* positions; const int* slots;
+  int T, H, G, D, Dp, Vp, k_col, v_col, rot;
+  const void* q_norm; const void* k_norm;
+  const float* cos_tab; const float* sin_tab;
+  int tab_rows, num_slots;
+  void* k_pool; void* v_pool;
+  float eps;
+};
+
+template <int DT>
+__global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParams p) {
+  typedef typename Act<DT>::T T;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int units = p.H + 2 * p.G;
+  const long long u = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (u >= (long long)p.T * units) return;
+  const int lane = threadIdx.x & 31;
+  const int t = (int)(u / units), k = (int)(u - (long long)t * units);
+  T* row = reinterpret_cast<T*>(p.proj) + (size_t)t * p.ld;
+  const int slot = p.slots[t];
+  const bool cached = slot >= 0 && slot < p.num_slots;
+  if (k >= p.H + p.G) {                                    // values
+    if (!cached) return;
+    const int g = k - p.H - p.G;
+    const T* src = row + p.v_col + g * p.Vp;
+    T* dst = reinterpret_cast<T*>(p.v_pool) + ((size_t)slot * p.G + g) * p.Vp;
+    for (int i = lane; i < p.Vp; i += 32) dst[i] = src[i];
+    return;
+  }
+  const bool is_k = k >= p.H;
+  if (is_k && !cached) return;
+  T* src = is_k ? row + p.k_col + (k - p.H) * p.Dp : row + (size_t)k * p.Dp;
+  T* dst = is_k ? reinterpret_cast<T*>(p.k_pool) + ((size_t)slot * p.G + (k - p.H)) * p.Dp : src;
+  const T* nw = reinterpret_cast<const T*>(is_k ? p.k_norm : p.q_norm);
+  float ss = 0.f;
+  for (int i = lane; i < p.D; i += 32) { const float v = Act<DT>::ld(src[i]); ss += v * v; }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  const float inv = 1.0f / sqrtf(ss / (float)p.D + p.eps);
+  int pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.tab_rows ? p.tab_rows - 1 : pos);
+  const int half = p.rot >> 1;
+  const float* ct = p.cos_tab + (size_t)pos * half;
+  const float* st = p.sin_tab + (size_t)pos * half;
+  for (int j = lane; 2 * j < p.Dp; j += 32) {              // pairs (Dp is even; beyond D the row is zero and stays zero)
+    const int i0 = 2 * j, i1 = 2 * j + 1;
+    float a = i0 < p.D ? Act<DT>::ld(src[i0]) * inv * Act<DT>::ld(nw[i0]) : 0.f;
+    float b = i1 < p.D ? Act<DT>::ld(src[i1]) * inv * Act<DT>::ld(nw[i1]) : 0.f;
+    if (j < half) {
+      const float c = ct[j], s = st[j], u0 = a;
+      a = u0 * c - b * s;
+      b = b * c + u0 * s;
+    }
+    dst[i0] = Act<DT>::st(a);
+    dst[i1] = Act<DT>::st(b);
+  }
 }
 
 // dst[i] = src[idx[i]] for rows of `vecs` 16-byte units
@@ -247,13 +380,13 @@ extern "C" int fb_rmsnorm32(const float* x, const void* w, void* y, int M, int H
   return (int)cudaGetLastError();
 }
 
-extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const void* table, const double* inv_freq, const void* w, float* h,
-                                 void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
+extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const void* table, const double* inv_freq, const void* pos_table,
+                                 int pos_rows, const void* w, float* h, void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
   if (T <= 0) return 0;
-  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2 || (pos_table != nullptr && pos_rows <= 0)) return -1;
   const bool vec = H % 4 == 0;
   const int th = row_threads(H, vec ? 4 : 2);
-#define GO(DT, V) S32_LAUNCH((embed_pos_norm_kernel<DT, V>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
+#define GO(DT, V) S32_LAUNCH((embed_pos_norm_kernel<DT, V>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)pos_table, pos_rows, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
   if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
   else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
@@ -272,12 +405,12 @@ extern "C" int fb_latent_norm(const void* x, int ldx, const void* w, const int* 
 }
 
 extern "C" int fb_moe_combine_norm32(const void* ys, const int* pos, const float* wts, float wconst, const void* shared_y, float* h,
-                                     const void* w, void* y, int T, int topk, int H, float alpha, float eps, int dt, void* stream) {
+                                     const void* post, const void* w, void* y, int T, int topk, int H, float alpha, float eps, int dt, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
   const bool vec = H % 4 == 0;
   const int th = row_threads(H, vec ? 4 : 1);
-#define GO(DT, V) S32_LAUNCH((moe_combine_norm32_kernel<DT, V>), T, th, H, stream, (const Act<DT>::T*)ys, pos, wts, wconst, (const Act<DT>::T*)shared_y, h, (const Act<DT>::T*)w, (Act<DT>::T*)y, topk, H, alpha, eps)
+#define GO(DT, V) S32_LAUNCH((moe_combine_norm32_kernel<DT, V>), T, th, H, stream, (const Act<DT>::T*)ys, pos, wts, wconst, (const Act<DT>::T*)shared_y, h, (const Act<DT>::T*)post, (const Act<DT>::T*)w, (Act<DT>::T*)y, topk, H, alpha, eps)
   if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
   else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
@@ -291,5 +424,37 @@ extern "C" int fb_gather_rows(const void* src, const long long* idx, void* dst, 
   long long blocks = ((long long)rows * vecs + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   launch_k(gather_rows_kernel, dim3((unsigned)blocks), dim3(256), 0, reinterpret_cast<cudaStream_t>(stream), 0, (const uint4*)src, idx, (uint4*)dst, rows, vecs);
+  return (int)cudaGetLastError();
+}
+
+// x: fp32 [T, H]; xs: sorted rows of type dt.
+extern "C" int fb_moe_gather_scaled(const float* x, const int* pos, const float* wts, void* xs, int T, int topk, int H, int dt, void* stream_) {
+  if (T <= 0) return 0;
+  if (H <= 0 || topk <= 0 || dt < 0 || dt > 2) return -1;
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  const bool vec = H % 4 == 0;
+  const int th = row_threads(H, vec ? 4 : 1);
+#define GO(DT, V) launch_k(moe_gather_scaled_kernel<DT, V>, dim3(T), dim3(th), 0, stream, 0, x, pos, wts, (Act<DT>::T*)xs, topk, H)
+  if (vec) { if (dt == 0) GO(0, 4); else if (dt == 1) GO(1, 4); else GO(2, 4); }
+  else { if (dt == 0) GO(0, 1); else if (dt == 1) GO(1, 1); else GO(2, 1); }
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// See HeadPostParams.  G = 0: queries only (the layer reads another layer's cache).
+extern "C" int fb_head_norm_rope(void* proj, long long ld, const int* positions, const int* slots, int T, int H, int G, int D, int Dp, int Vp,
+                                 int k_col, int v_col, int rot, const void* q_norm, const void* k_norm, const float* cos_tab,
+                                 const float* sin_tab, int tab_rows, int num_slots, void* k_pool, void* v_pool, float eps, int dt, void* stream_) {
+  if (T <= 0) return 0;
+  if (H <= 0 || G < 0 || D <= 0 || Dp < D || (Dp & 1) || Vp <= 0 || rot < 0 || (rot & 1) || rot > D || dt < 0 || dt > 2 || q_norm == nullptr) return -1;
+  if (rot > 0 && (cos_tab == nullptr || sin_tab == nullptr || tab_rows <= 0)) return -1;
+  if (G > 0 && (k_norm == nullptr || k_pool == nullptr || v_pool == nullptr)) return -1;
+  HeadPostParams p{proj, ld, positions, slots, T, H, G, D, Dp, Vp, k_col, v_col, rot, q_norm, k_norm, cos_tab, sin_tab, tab_rows, num_slots, k_pool, v_pool, eps};
+  const long long units = (long long)T * (H + 2 * G);
+  const dim3 grid((unsigned)((units + 7) / 8));
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  if (dt == 0) launch_k(head_norm_rope_kernel<0>, grid, dim3(256), 0, stream, 0, p);
+  else if (dt == 1) launch_k(head_norm_rope_kernel<1>, grid, dim3(256), 0, stream, 0, p);
+  else launch_k(head_norm_rope_kernel<2>, grid, dim3(256), 0, stream, 0, p);
   return (int)cudaGetLastError();
 }

@@ -81,7 +81,7 @@ class LLMEngine:
 
             if control is not None or model.tp.size > 1:
                 raise NotImplementedError("a separate draft model runs on one rank")
-            if self.runner.state_slots or any(lw.lin is not None for lw in draft_model.layers):
+            if self.runner.state_slots or draft_model.cfg.has_linear_attn:
                 raise NotImplementedError("draft-model speculation needs attention-only target and draft models")
             if draft_model.cfg.vocab_size != model.cfg.vocab_size:
                 raise ValueError("the draft model's vocabulary differs from the target's")

@@ -105,7 +105,7 @@ class KVCache:
             if model.cfg.layer_is_linear(i):
                 # no pages: a convolution window and a delta-rule state per request slot; the last slot is scratch for
                 # padded decode rows
-                cs, rs = model.linear_state_shapes(state_slots + 1)
+                cs, rs = model.linear_state_shapes(state_slots + 1, i)
                 self.pools.append((torch.zeros(cs, device=dev, dtype=model.dtype), torch.zeros(rs, device=dev, dtype=torch.float32)))
                 continue
             lks, lvs = ks, vs

@@ -80,7 +80,10 @@ def dequant_awq(qweight: torch.Tensor, qzeros: torch.Tensor, scales: torch.Tenso
 # name canonicalisation: every family is mapped onto the Llama naming that loader.shard understands
 # ---------------------------------------------------------------------------------------------------
 _RENAMES = [
-    # Patesun
+    # Patesun, Vilulorn
+    (r"^pos$", "model.embed_positions.weight"), (r"^l(\d+)\.mix\.([qk])\.norm$", r"model.layers.\1.self_attn.\2_norm.weight"),
+    (r"^l(\d+)\.mix\.norm$", r"model.layers.\1.self_attn.o_norm.weight"), (r"^l(\d+)\.mix\.a2\.b$", r"model.layers.\1.self_attn.a2_proj.bias"),
+    (r"^l(\d+)\.mix\.(a1|a2|k|v)$", r"model.layers.\1.self_attn.\2_proj.weight"), (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight"),
     (r"^embed$", "model.embed_tokens.weight"), (r"^final\.norm$", "model.norm.weight"), (r"^head$", "lm_head.weight"),
     (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"), (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
     (r"^l(\d+)\.mix\.dkv\.norm$", r"model.layers.\1.self_attn.kv_a_layernorm.weight"), (r"^l(\d+)\.mix\.dkv$", r"model.layers.\1.self_attn.kv_a_proj.weight"),
@@ -328,7 +331,7 @@ def load_model(path: str | Path, device="cuda", dtype=None, wdtype: str = "auto"
 
     def top_fn():
         t = {}
-        for k in ("model.embed_tokens.weight", "model.norm.weight", "model.norm.bias", "lm_head.weight", "lm_head.bias"):
+        for k in ("model.embed_tokens.weight", "model.embed_positions.weight", "model.norm.weight", "model.norm.bias", "lm_head.weight", "lm_head.bias"):
             if ck.has(k):
                 t[k] = ck.raw(k)
         return t

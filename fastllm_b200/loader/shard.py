@@ -310,6 +310,9 @@ def build_layer(m, i: int, t: dict, wdtype="dense", moe_wdtype=None):
 def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
     """Mixer and feed-forward of a model that lists its layers (``cfg.mixers`` / ``cfg.ffs``).  Widths are padded with zero rows and
     columns to what the kernels tile (the padding stays zero through every product)."""
+    from ..models.config import AttnSpec, GLASpec
+    from ..ops import gla as GLA
+    from ..ops import grouped as GR
     from ..ops import latent as LA
 
     cfg = m.cfg
@@ -330,11 +333,25 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
     def down(w, kind, mult):
         return lin(LA.pad_cols(_to(w, m), mult if m.on_cuda else 1).contiguous(), kind)
 
-    la, in_w = LA.build(spec, t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"))
-    la.in_proj = lin(in_w)
-    lw.latent = la
-    lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
     f = lw.mlp
+    if cfg.output_norms:                    # the layer's two norms belong to its sub-layers' outputs
+        lw.attn.post_ln, f.post_ln, lw.attn.ln, f.ln = lw.attn.ln, f.ln, None, None
+    if isinstance(spec, GLASpec):
+        lw.gla, in_w = GLA.build(spec, *(t(k + "_proj") for k in ("q", "k", "v", "g", "a1", "a2")), _to(g("self_attn.a2_proj.bias"), m), t("o_norm"))
+        lw.gla.in_proj = lin(in_w)
+        lw.attn.o = lin(t("o_proj"))
+    elif isinstance(spec, AttnSpec):
+        own = spec.kv_from is None
+        lw.grouped, in_w = GR.build(spec, t("q_proj"), t("k_proj") if own else None, t("v_proj") if own else None, t("g_proj"), t("q_norm"),
+                                    t("k_norm") if own else None)
+        lw.grouped.in_proj = lin(in_w)
+        lw.attn.heads, lw.attn.rope = spec.heads, spec.rope
+        lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
+    else:
+        la, in_w = LA.build(spec, t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"))
+        la.in_proj = lin(in_w)
+        lw.latent = la
+        lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
     if ff.kind == "none":
         f.absent = True
     elif ff.kind == "dense":
@@ -342,10 +359,16 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
         f.up = lin(LA.pad_rows(_to(g("mlp.up_proj.weight"), m), 8 if m.on_cuda else 1))
         f.down = down(g("mlp.down_proj.weight"), wdtype, 8)
     else:
-        f.route_table = g("mlp.token_table").to(m.device, torch.int32).contiguous()
         names = [f"mlp.experts.{e}." for e in range(ff.experts)]
         f.experts = MOE.ExpertWeights(ff.experts, 0, [gate_up(g(n + "gate_proj.weight"), g(n + "up_proj.weight"), moe_wdtype) for n in names],
                                       [down(g(n + "down_proj.weight"), moe_wdtype, 64) for n in names])
+        if ff.act == "gptoss":
+            f.experts.act, f.experts.limit = "gptoss", ff.limit
+        if ff.router == "table":
+            f.route_table = g("mlp.token_table").to(m.device, torch.int32).contiguous()
+        else:
+            f.experts.scale_input = True
+            MOE.set_router(f, _to(g("mlp.gate.weight"), m), ff.top, m.on_cuda)
         if ff.shared_ff:
             f.shared_gate_up = gate_up(g("mlp.shared_experts.gate_proj.weight"), g("mlp.shared_experts.up_proj.weight"), wdtype)
             f.shared_down = down(g("mlp.shared_experts.down_proj.weight"), wdtype, 64)
@@ -432,6 +455,8 @@ def build_top(m, t: dict, wdtype="dense"):
     cfg, tp = m.cfg, m.tp
     m.embed = _to(t["model.embed_tokens.weight"], m)
     m.final_norm = _to(t["model.norm.weight"], m)
+    if cfg.pos_table:
+        m.pos_table = _to(t["model.embed_positions.weight"], m)
     if t.get("model.norm.bias") is not None:
         m.ln_bias[id(m.final_norm)] = _to(t["model.norm.bias"], m)
     head = t.get("lm_head.weight")

@@ -24,16 +24,42 @@ class LatentSpec:
 
 
 @dataclass
+class AttnSpec:
+    """Softmax attention of one layer with its own head counts and widths, per-head query / key norms, rotary positions and an
+    elementwise sigmoid gate on the heads."""
+    heads: int
+    kv_heads: int
+    dim: int                # query / key dimensions per head
+    vdim: int
+    scale: float
+    chunk: int = 0          # > 0: the sequence is cut into chunks of this many positions, a query sees the keys of its own chunk
+    rope: dict | None = None     # {"theta", "rot_dim", "scaling"}: interleaved pairs on the first rot_dim dimensions
+    kv_from: int | None = None   # the layer whose cached keys and values this one reads (it has no projections of them)
+
+
+@dataclass
+class GLASpec:
+    """Gated linear attention of one layer: a [dim, vdim] state per head whose key channels decay by sigmoid(z)^(1 / tau)."""
+    heads: int
+    dim: int
+    vdim: int
+    tau: float
+    rank: int = 16          # inner width of the decay projection (random init; a checkpoint's tensor says its own)
+
+
+@dataclass
 class FFSpec:
-    """Feed-forward of one layer where the layers of a model differ: "dense" (up -> act -> down), "moe" (routed SwiGLU experts plus
+    """Feed-forward of one layer where the layers of a model differ: "dense" (up -> act -> down), "moe" (routed gated experts plus
     an optional shared one) or "none"."""
     kind: str = "none"
     ff: int = 0
-    act: str = "relu2"
+    act: str = "relu2"      # experts: "silu" | "gptoss" (both branches clamped at `limit`)
     experts: int = 0
     top: int = 0
     expert_ff: int = 0
     shared_ff: int = 0      # 0: no shared expert
+    router: str = "table"   # "table": experts by token id | "sigmoid": the best scores of a projection, which scale the expert's input
+    limit: float = 0.0
 
 
 @dataclass
@@ -119,14 +145,16 @@ class ModelConfig:
     lin_conv_kernel: int = 4
     lin_kind: str = "gdn"                  # "gdn" Gated DeltaNet | "lightning" decayed linear attention (MiniMax-Text-01 / M1)
     lin_block: int = 256                   # lightning attention: block length of the chunked evaluation
-    # models whose layers are listed one by one (Patesun): the mixer and feed-forward of every layer, and which layer's weights each
-    # run of the stack uses (looped layers appear once per pass; num_layers counts the runs, every run has its own cache)
-    mixers: list | None = None             # LatentSpec per run
+    # models whose layers are listed one by one (Patesun, Vilulorn): the mixer and feed-forward of every layer, and which layer's
+    # weights each run of the stack uses (looped layers appear once per pass; num_layers counts the runs, every run has its own cache)
+    mixers: list | None = None             # LatentSpec / AttnSpec / GLASpec per run
     ffs: list | None = None                # FFSpec per run
     layer_runs: list | None = None
     residual_f32: bool = False             # the residual stream is fp32; sub-layer outputs join it times residual_mult
     residual_mult: float = 1.0
     pos_embed_base: float = 0.0            # > 0: sinusoidal positions with this base are added to the token embedding
+    pos_table: int = 0                     # > 0: rows of a learned position table that is added to the token embedding
+    output_norms: bool = False             # fp32 residual: norms sit on the sub-layers' outputs only, sub-layers read the residual itself
     # DeepNorm-style residual (MiniMax-Text-01 / M1): the block input is normalised first and the NORMALISED rows are the
     # residual: y = alpha * norm(x) + beta * f(norm(x)).  (alpha, beta) for full-attention layers, linear layers, MLPs.
     postnorm_residual: bool = False
@@ -187,8 +215,8 @@ def from_hf_dict(d: dict) -> ModelConfig:
             if k in d and k not in inner:
                 inner[k] = d[k]
         d = inner
-    if d.get("architecture") == "Patesun":
-        return _patesun(d)
+    if d.get("architecture") in LISTED:
+        return LISTED[d["architecture"]](d)
     mt = d.get("model_type", "llama")
     if "CogVLMForCausalLM" in (d.get("architectures") or []) or mt == "CogVLMForCausalLM":
         mt = "cogvlm"                                   # the checkpoint's config names no model_type
@@ -582,7 +610,16 @@ def _patesun(d: dict) -> ModelConfig:
     if loop:
         a, b = int(loop["start"]), int(loop["stop"])
         runs = runs[:a] + runs[a:b] * int(loop["times"]) + runs[b:]
-    c = ModelConfig(model_type="patesun", raw=d, architectures=["Patesun"])
+    c = _listed("Patesun", d, mixers, ffs, runs)
+    c.residual_mult = float(d.get("residual_mult", 1.0))
+    c.pos_embed_base = 10000.0
+    c.max_position = int(d.get("max_position_embeddings", 1 << 20))
+    return c
+
+
+def _listed(name: str, d: dict, mixers: list, ffs: list, runs: list) -> ModelConfig:
+    """What models with listed layers and an fp32 residual share."""
+    c = ModelConfig(model_type=name.lower(), raw=d, architectures=[name])
     c.vocab_size, c.hidden_size = int(d["vocab"]), int(d["width"])
     c.layer_runs = runs
     c.num_layers = len(runs)
@@ -595,14 +632,56 @@ def _patesun(d: dict) -> ModelConfig:
     c.moe_intermediate_size = max((f.expert_ff for f in ffs), default=0)
     c.rms_eps = float(d["norm"]["eps"])
     c.residual_f32 = True
-    c.residual_mult = float(d.get("residual_mult", 1.0))
-    c.pos_embed_base = 10000.0
-    c.rope_mode = "none"
-    c.max_position = int(d.get("max_position_embeddings", 1 << 20))
+    c.rope_mode = "none"                    # model-wide tables: none (a layer's mixer has its own)
+    if any(isinstance(m, GLASpec) for m in c.mixers):
+        c.layer_types = ["linear_attention" if isinstance(m, GLASpec) else "full_attention" for m in c.mixers]
     c.eos_token_ids = _eos_list(d.get("eos_token_id"))
     c.bos_token_id = d.get("bos_token_id")
     c.torch_dtype = str(d.get("torch_dtype", d.get("dtype", "bfloat16"))).replace("torch.", "")
     return c
+
+
+def _vilulorn(d: dict) -> ModelConfig:
+    """Vilulorn: gated linear attention layers and chunked grouped-query attention layers (which may read an earlier layer's keys and
+    values), experts picked by sigmoid scores that scale their inputs, norms on the sub-layers' outputs only, learned positions."""
+    L = d["layers"]
+    mixers, ffs = [], []
+    for i, spec in enumerate(L):
+        m, kind = spec["mixer"], spec.get("type")
+        if kind == "gla":
+            mixers.append(GLASpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["tau"])))
+        elif kind == "attention":
+            rot = m.get("rot")
+            rope = None
+            if rot and int(rot["dims"]):
+                sc = rot.get("scaling")
+                rope = {"theta": float(rot["base"]), "rot_dim": int(rot["dims"]),
+                        "scaling": {"rope_type": "llama3", "factor": float(sc["factor"]), "low_freq_factor": float(sc["low"]),
+                                    "high_freq_factor": float(sc["high"]), "original_max_position_embeddings": float(sc["original"])} if sc else None}
+            src = m.get("kv_from")
+            if src is not None and not (0 <= int(src) < i and isinstance(mixers[int(src)], AttnSpec) and mixers[int(src)].kv_from is None):
+                raise ValueError(f"Vilulorn: layer {i} cannot read the keys and values of layer {src}")
+            mixers.append(AttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                   int((m.get("mask") or {}).get("size") or 0), rope, int(src) if src is not None else None))
+        else:
+            raise NotImplementedError(f"Vilulorn: layer {i} has mixer '{kind}'")
+        f = spec.get("mlp")
+        if f is None:
+            ffs.append(FFSpec())
+        elif f.get("kind") == "moe":
+            ffs.append(FFSpec("moe", act="gptoss", experts=int(f["router"]["experts"]), top=int(f["router"]["top"]),
+                              expert_ff=int(f["expert"]["ff"]), router="sigmoid", limit=float(f["expert"]["limit"])))
+        else:
+            raise NotImplementedError(f"Vilulorn: layer {i} has feed-forward '{f.get('kind')}'")
+    c = _listed("Vilulorn", d, mixers, ffs, list(range(len(L))))
+    c.num_kv_heads = max((m.kv_heads for m in mixers if isinstance(m, AttnSpec)), default=1)
+    c.output_norms = True
+    c.pos_table = c.max_position = int(d["max_positions"])
+    return c
+
+
+# config.json "architecture" of designs whose layers are listed one by one
+LISTED = {"Patesun": _patesun, "Vilulorn": _vilulorn}
 
 
 def load_config(path: str | Path) -> ModelConfig:
@@ -749,6 +828,19 @@ def preset(name: str) -> ModelConfig:
                                  loop={"start": 1, "stop": 5, "times": 2},
                                  layers=[{"type": "latent_attention", "mixer": mx, "mlp": {"kind": "dense", "ff": 14336}}]
                                  + [{"type": "latent_attention", "mixer": mx, "mlp": moe} for _ in range(7)]))
+    if name in ("tiny-vilulorn", "vilulorn-7b"):
+        tiny = name.startswith("tiny")
+        rot = {"base": 1e4 if tiny else 5e5, "dims": 16 if tiny else 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 64 if tiny else 8192}}
+        at = ({"heads": 6, "kv_heads": 3, "dim": 40, "vdim": 24, "scale": 0.2, "mask": {"size": 50}, "rot": rot} if tiny else
+              {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 8192}, "rot": rot})
+        gl = {"heads": 3, "dim": 24, "vdim": 32, "tau": 8.0} if tiny else {"heads": 32, "dim": 128, "vdim": 128, "tau": 16.0}
+        moe = {"kind": "moe", "expert": {"ff": 48 if tiny else 1024, "limit": 4.0}, "router": {"experts": 5 if tiny else 64, "top": 2 if tiny else 6}}
+        layer = lambda t, m, f=moe: {"type": t, "mixer": m, "mlp": f}
+        block = [layer("attention", at), layer("gla", gl, None if tiny else moe), layer("attention", dict(at, kv_from=0)), layer("gla", gl)]
+        if not tiny:
+            block += [layer("gla", gl), layer("attention", at), layer("gla", gl), layer("attention", dict(at, kv_from=5))]
+        return from_hf_dict(dict(architecture="Vilulorn", vocab=512 if tiny else 128256, width=128 if tiny else 4096, norm={"eps": 1e-5},
+                                 max_positions=640 if tiny else 32768, layers=block))
     if name == "tiny-deepseek-v32":      # latent attention with the sparse-attention indexer (selection size 32)
         return from_hf_dict(dict(model_type="deepseek_v32", vocab_size=512, hidden_size=256, num_hidden_layers=2,
                                  num_attention_heads=4, num_key_value_heads=4, intermediate_size=512,

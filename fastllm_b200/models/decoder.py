@@ -22,11 +22,13 @@ import torch.nn.functional as F
 
 from ..ops import attention as A
 from ..ops import basic as B
+from ..ops import gla as GLA
+from ..ops import grouped as GR
 from ..ops import latent as LA
 from ..ops import moe as MOE
 from ..ops import stream32 as S
 from ..ops.quant import LinearWeight
-from .config import ModelConfig
+from .config import AttnSpec, GLASpec, ModelConfig
 
 
 @dataclass
@@ -129,6 +131,7 @@ class MLPWeights:
         self.act = ""            # activation of a two-matrix MLP where it is the layer's own (default: the model's hidden_act)
         self.absent = False      # the layer has no feed-forward
         self.route_table = None  # int32 [vocab, top]: experts of every token id (no router), equal weights
+        self.top = 0             # experts per token where it is the layer's own (listed layers with a scored router)
         self.act_limit = 0.0     # clamp inside the dense / shared-expert SwiGLU (Step-3.5); 0: none
         # MoE
         self.router = None          # fp32 [E, H]
@@ -146,7 +149,10 @@ class LayerWeights:
     def __init__(self):
         self.attn = AttentionWeights()
         self.mlp = MLPWeights()
-        self.latent: LA.LatentWeights | None = None    # latent attention without positions (``attn`` keeps its norm and output projection)
+        # mixers of listed layers (``attn`` keeps their norms and output projection)
+        self.latent: LA.LatentWeights | None = None    # latent attention without positions
+        self.grouped: GR.GroupedWeights | None = None  # grouped-query attention with its own widths, mask and rotary tables
+        self.gla: GLA.GLAWeights | None = None         # gated linear attention
         self.lin: LinearAttnWeights | None = None      # set instead of ``attn`` projections on linear-attention layers
 
 
@@ -176,6 +182,7 @@ class DecoderModel:
         self.tp = tp or TPInfo()
         self.ep = ep                       # parallel.ep.EPInfo or None
         self.embed = None                  # [vocab(/tp), H]
+        self.pos_table = None              # [positions, H] learned positions added to the embedding
         self.layers: list[LayerWeights] = []
         self.final_norm = None
         self.lm_head: LinearWeight | None = None
@@ -256,7 +263,8 @@ class DecoderModel:
         """Per-layer page-pool shapes of this rank: (K shape, V shape or None for MLA)."""
         c = self.cfg
         if c.mixers is not None:
-            return self.kv_cache_shape_layer(0, num_pages)
+            paged = [i for i in range(c.num_layers) if not c.layer_is_linear(i)]
+            return self.kv_cache_shape_layer(paged[0], num_pages) if paged else ((0,), None)
         if c.use_mla:
             # one spare page at the end: rows that must not be cached (padded decode rows) are written there
             idx = (num_pages + 1, A.PAGE_LEN, 1, c.index_head_dim) if (c.index_topk and getattr(self, "has_indexer", False)) else None
@@ -265,24 +273,39 @@ class DecoderModel:
         return s, s
 
     def kv_cache_shape_layer(self, i: int, num_pages: int):
-        """Pool shapes of layer ``i``: the model-wide ones, or a latent row per token where layers are listed one by one (plus a
-        spare page for rows that must not be cached)."""
+        """Pool shapes of layer ``i``: the model-wide ones, or those of its own mixer where layers are listed one by one (plus a spare
+        page for rows that must not be cached).  None: the layer reads the pools of layer ``kv_donor(i)``."""
         if self.cfg.mixers is None:
             return self.kv_cache_shape(num_pages)
-        return (num_pages + 1, A.PAGE_LEN, 1, (self.cfg.mixers[i].kv_rank + 7) // 8 * 8), None
+        sp = self.cfg.mixers[i]
+        if isinstance(sp, AttnSpec):
+            if sp.kv_from is not None:
+                return None
+            lead = (num_pages, A.PAGE_LEN, sp.kv_heads)
+            return (*lead, (sp.dim + 7) // 8 * 8), (*lead, (sp.vdim + 7) // 8 * 8)
+        return (num_pages + 1, A.PAGE_LEN, 1, (sp.kv_rank + 7) // 8 * 8), None
+
+    def kv_donor(self, i: int) -> int:
+        """The layer whose pools layer ``i`` reads."""
+        src = getattr(self.cfg.mixers[i], "kv_from", None) if self.cfg.mixers is not None else None
+        return i if src is None else src
 
     def kv_bytes_per_page(self) -> int:
         if self.cfg.mixers is not None:
-            n = sum(math.prod(self.kv_cache_shape_layer(i, 1)[0][1:]) for i in range(self.cfg.num_layers))
-            return n * torch.finfo(self.dtype).bits // 8
+            shapes = [self.kv_cache_shape_layer(i, 1) for i in range(self.cfg.num_layers) if not self.cfg.layer_is_linear(i)]
+            n = sum(math.prod(s[1:]) for pair in shapes if pair is not None for s in pair if s is not None)
+            return max(1, n * torch.finfo(self.dtype).bits // 8)
         ks, vs = self.kv_cache_shape(1)
         n = math.prod(ks) + (math.prod(vs) if vs else 0)
         paged_layers = sum(1 for i in range(self.cfg.num_layers) if not self.cfg.layer_is_linear(i)) + (1 if self.mtp is not None else 0)
         return n * max(1, paged_layers) * torch.finfo(getattr(self, "kv_dtype", None) or self.dtype).bits // 8
 
-    def linear_state_shapes(self, n_slots: int):
-        """Per linear-attention layer: (convolution window pool, delta-rule state pool) shapes for ``n_slots`` requests."""
+    def linear_state_shapes(self, n_slots: int, layer: int | None = None):
+        """Per linear-attention layer: (convolution window pool, recurrent state pool) shapes for ``n_slots`` requests."""
         c = self.cfg
+        if c.mixers is not None:               # every listed layer has its own state
+            sp = c.mixers[layer]
+            return (n_slots, 0, 0), (n_slots, sp.heads, sp.dim, sp.vdim)
         Hk, Hv = c.lin_num_k_heads // self.tp.size, c.lin_num_v_heads // self.tp.size
         if c.lin_kind == "lightning":          # no convolution window; one [D, D] state per head
             return (n_slots, 0, 0), (n_slots, Hv, c.lin_k_dim, c.lin_v_dim)
@@ -290,11 +313,12 @@ class DecoderModel:
         return (n_slots, C, c.lin_conv_kernel - 1), (n_slots, Hv, c.lin_k_dim, c.lin_v_dim)
 
     def linear_state_bytes_per_slot(self) -> int:
-        if not self.cfg.has_linear_attn:
-            return 0
-        cs, rs = self.linear_state_shapes(1)
-        n_lin = sum(1 for i in range(self.cfg.num_layers) if self.cfg.layer_is_linear(i))
-        return n_lin * (math.prod(cs) * torch.finfo(self.dtype).bits // 8 + math.prod(rs) * 4)
+        n = 0
+        for i in range(self.cfg.num_layers):
+            if self.cfg.layer_is_linear(i):
+                cs, rs = self.linear_state_shapes(1, i)
+                n += math.prod(cs) * torch.finfo(self.dtype).bits // 8 + math.prod(rs) * 4
+        return n
 
     def set_kv_cache_dtype(self, name: str | None) -> None:
         """``fp8_e4m3``: keys and values are stored as unscaled e4m3 (half the cache bytes); attention then runs on the
@@ -487,7 +511,7 @@ class DecoderModel:
 
     def _norm(self, h, ln_w):
         if self.cfg.residual_f32:
-            return S.rmsnorm32(h, ln_w, self.cfg.rms_eps)
+            return S.rmsnorm32(h, ln_w, self.cfg.rms_eps) if ln_w is not None else h.to(self.dtype)
         if self.cfg.norm_kind == "layernorm":
             return F.layer_norm(h.float(), (h.shape[-1],), ln_w.float(), self.ln_bias[id(ln_w)].float() if id(ln_w) in self.ln_bias else None,
                                 self.cfg.rms_eps).to(h.dtype)
@@ -528,6 +552,8 @@ class DecoderModel:
         all-gather to land: that wait moves into the consumer's GEMM, behind its weight prefetch.
         """
         c = self.cfg
+        if c.output_norms:               # fp32 stream, the sub-layer's output is normalised before it is added
+            return h, S.add_norm(h, w(x), post_ln, next_ln, c.rms_eps, c.residual_mult)
         if c.residual_f32:               # fp32 stream: the scaled sub-layer output is added in the GEMM's epilogue
             h = w.add_to(x, h, c.residual_mult)
             return h, S.rmsnorm32(h, next_ln, c.rms_eps)
@@ -620,6 +646,22 @@ class DecoderModel:
         a = LA.attention(la, proj, kv[0], fb)
         return self._row_parallel_norm(lw.attn.o, a, residual, next_ln)
 
+    def _grouped_attention(self, lw: LayerWeights, x, fb: ForwardBatch, kv, residual, next_ln):
+        """Grouped-query attention of a listed layer: merged [queries | gate | keys | values] projection, per-head norms + rotary + cache
+        append in one launch, chunked attention with the output gate in its epilogue, output projection onto the residual."""
+        gw = lw.grouped
+        proj = gw.in_proj(x)
+        _, cos, sin, _ = self._layer_geom(lw.attn, x.device) if lw.attn.rope is not None else (0, None, None, 0)
+        GR.post(gw, proj, fb, kv, cos, sin, self.cfg.rms_eps)
+        a = GR.attention(gw, proj, kv, fb)
+        return self._row_parallel_norm(lw.attn.o, a, residual, next_ln, lw.attn.post_ln)
+
+    def _gla(self, lw: LayerWeights, x, fb: ForwardBatch, state, residual, next_ln):
+        """Gated linear attention: merged [q | k | v | gate | decay rank] projection, the recurrence over the request's state with the
+        head norm and the gate, output projection onto the residual."""
+        a = GLA.mix(lw.gla, lw.gla.in_proj(x), fb, state[1], self.cfg.rms_eps)
+        return self._row_parallel_norm(lw.attn.o, a, residual, next_ln, lw.attn.post_ln)
+
     @staticmethod
     def _glu(gu, act: str, interleaved: bool):
         """``act(gate) * up`` for gated MLPs whose activation is not SiLU (GeGLU of the Gemma family, ...): one kernel."""
@@ -658,10 +700,31 @@ class DecoderModel:
         rows = self._row_ids(x.shape[0], x.device).view(-1, 1)
         return h, S.moe_combine_norm(y, rows, None, 1.0, shared, h, next_ln, c.residual_mult, c.rms_eps)
 
+    def _scored_moe(self, lw: MLPWeights, x, h, next_ln):
+        """Experts picked by sigmoid scores of a router; where the scores scale the experts' inputs the rows are scaled as they are
+        gathered (from the fp32 residual).  Combine, output norm, residual add and the next norm are one launch."""
+        c = self.cfg
+        idx, wts = MOE.route_scored(lw, x)
+        ex = lw.experts
+        parts = None
+        if ex.stacked is not None and x.is_cuda:
+            from ..ops import moe_grouped
+
+            parts = moe_grouped.forward(x, idx, wts, ex, combine=False, rows32=h if ex.scale_input else None)
+        if parts is not None:
+            return h, S.moe_combine_norm(parts[0], parts[1], None if ex.scale_input else wts, 1.0, None, h, next_ln, c.residual_mult, c.rms_eps,
+                                         post_w=lw.post_ln, dtype=self.dtype)
+        y = MOE.moe_forward(x, idx, wts, ex)
+        if lw.post_ln is not None:
+            return h, S.add_norm(h, y, lw.post_ln, next_ln, c.rms_eps, c.residual_mult)
+        return h, S.moe_combine_norm(y, self._row_ids(x.shape[0], x.device).view(-1, 1), None, 1.0, None, h, next_ln, c.residual_mult, c.rms_eps)
+
     def _mlp(self, lw: MLPWeights, x, residual, layer_idx, next_ln, consumer=None, fb=None):
         c = self.cfg
         if lw.route_table is not None:
             return self._table_moe(lw, x, residual, fb, next_ln)
+        if lw.top:
+            return self._scored_moe(lw, x, residual, next_ln)
         if lw.act == "relu2":
             return self._row_parallel_norm(lw.down, lw.up.relu2(x), residual, next_ln, lw.post_ln, consumer)
         if lw.experts is None and lw.up is not None:         # two-matrix MLP: up -> activation -> down
@@ -745,7 +808,7 @@ class DecoderModel:
         if c.residual_f32:
             if self.__dict__.get("_pos_freq") is None:
                 self._pos_freq = S.sinusoid_inv_freq(c.hidden_size, c.pos_embed_base, self.device) if c.pos_embed_base else None
-            h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps)
+            h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps, pos_table=self.pos_table)
         else:
             h, x = self.embed_tokens(fb.ids), None
         if fb.embed_rows is not None:
@@ -772,8 +835,9 @@ class DecoderModel:
                 h = x * alpha if alpha != 1.0 else x
             if c.parallel_block:
                 h, _ = self._attention(lw.attn, x, fb, kv_caches[i], h, None, None)       # h + attention(x); the MLP reads x too
-            elif lw.latent is not None:
-                h, x = self._latent_attention(lw, x, fb, kv_caches[i], h, self._entry_norm(i + 1) if lw.mlp.absent else lw.mlp.ln)
+            elif c.mixers is not None:
+                mixer = self._latent_attention if lw.latent is not None else self._gla if lw.gla is not None else self._grouped_attention
+                h, x = mixer(lw, x, fb, kv_caches[i], h, self._entry_norm(i + 1) if lw.mlp.absent else lw.mlp.ln)
             elif lw.lin is not None:
                 h, x = self._linear_attention(lw.lin, x, fb, kv_caches[i], h, lw.mlp.ln, mlp_first)
             else:
@@ -787,7 +851,8 @@ class DecoderModel:
             if i + 1 < n_layers:
                 nl = self.layers[i + 1]
                 na = nl.attn
-                nxt = nl.latent.in_proj if nl.latent is not None else nl.lin.in_proj if nl.lin is not None else ((na.q_a if na.q_a is not None else na.q_b) if c.use_mla else na.qkv)
+                mx = nl.latent or nl.grouped or nl.gla
+                nxt = mx.in_proj if mx is not None else nl.lin.in_proj if nl.lin is not None else ((na.q_a if na.q_a is not None else na.q_b) if c.use_mla else na.qkv)
             else:
                 nxt = self.lm_head if fb.logit_rows is None else None
             h, x = self._mlp(lw.mlp, x, h, i, next_ln, nxt, fb)
@@ -811,7 +876,7 @@ class DecoderModel:
         return logits
 
     def _entry_norm(self, i: int):
-        """Weight of the norm that opens layer ``i`` (the final norm behind the last one)."""
+        """Weight of the norm that opens layer ``i`` (the final norm behind the last one; None: the layer reads the residual itself)."""
         if i >= len(self.layers):
             return self.final_norm
         lw = self.layers[i]
@@ -975,11 +1040,25 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
             ap = p + "self_attn."
             mk(ap + "q_proj.weight", (sp.heads * sp.dim, H))
             mk(ap + "g_proj.weight", (sp.heads * sp.vdim, H))
-            mk(ap + "kv_a_proj.weight", (sp.kv_rank, H))
-            ones(ap + "kv_a_layernorm.weight", sp.kv_rank)
-            mk(ap + "k_b_proj.weight", (sp.heads * sp.dim, sp.kv_rank))
-            mk(ap + "v_b_proj.weight", (sp.heads * sp.vdim, sp.kv_rank))
             mk(ap + "o_proj.weight", (H, sp.heads * sp.vdim))
+            if isinstance(sp, GLASpec):
+                mk(ap + "k_proj.weight", (sp.heads * sp.dim, H))
+                mk(ap + "v_proj.weight", (sp.heads * sp.vdim, H))
+                mk(ap + "a1_proj.weight", (sp.rank, H))
+                mk(ap + "a2_proj.weight", (sp.heads * sp.dim, sp.rank))
+                ones(ap + "a2_proj.bias", sp.heads * sp.dim)
+                ones(ap + "o_norm.weight", sp.vdim)
+            elif isinstance(sp, AttnSpec):
+                ones(ap + "q_norm.weight", sp.dim)
+                if sp.kv_from is None:
+                    mk(ap + "k_proj.weight", (sp.kv_heads * sp.dim, H))
+                    mk(ap + "v_proj.weight", (sp.kv_heads * sp.vdim, H))
+                    ones(ap + "k_norm.weight", sp.dim)
+            else:
+                mk(ap + "kv_a_proj.weight", (sp.kv_rank, H))
+                ones(ap + "kv_a_layernorm.weight", sp.kv_rank)
+                mk(ap + "k_b_proj.weight", (sp.heads * sp.dim, sp.kv_rank))
+                mk(ap + "v_b_proj.weight", (sp.heads * sp.vdim, sp.kv_rank))
             if ff.kind == "dense":
                 mk(p + "mlp.up_proj.weight", (ff.ff, H))
                 mk(p + "mlp.down_proj.weight", (H, ff.ff))
@@ -988,6 +1067,9 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
                     mk(p + nm + "gate_proj.weight", (inter, H))
                     mk(p + nm + "up_proj.weight", (inter, H))
                     mk(p + nm + "down_proj.weight", (H, inter))
+                if ff.router != "table":
+                    mk(p + "mlp.gate.weight", (ff.experts, H))
+                    return raw
                 gen.manual_seed(_name_seed(seed, p + "mlp.token_table"))
                 raw[p + "mlp.token_table"] = torch.rand((cfg.vocab_size, ff.experts), device=dev, generator=gen).topk(ff.top, dim=1).indices.to(torch.int32)
             return raw
@@ -1081,6 +1163,8 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
     def top_tensors():
         raw.clear()
         mk("model.embed_tokens.weight", (cfg.vocab_size, H))
+        if cfg.pos_table:
+            mk("model.embed_positions.weight", (cfg.pos_table, H))
         ones("model.norm.weight", H)
         if cfg.norm_kind == "layernorm":
             mk("model.norm.bias", (H,))

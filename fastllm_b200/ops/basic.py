@@ -15,7 +15,7 @@ import torch.nn.functional as F
 
 from . import _lib, cpu
 
-GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32, GEMM_RELU2 = 1, 2, 4, 8, 32
+GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32, GEMM_RELU2, GEMM_GLU_CLAMP = 1, 2, 4, 8, 32, 64
 
 
 def _ptr(t):

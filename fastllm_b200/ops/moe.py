@@ -88,6 +88,30 @@ def route_fused(x, router_16, bias, topk, score_mode, renorm, route_scale=1.0):
     return idx, w
 
 
+def set_router(mlp, w, top: int, on_cuda: bool) -> None:
+    """Sigmoid router of a listed layer (``MLPWeights``): its projection ``w`` [E, H] in fp32 and, for the tensor-core GEMM, with rows
+    padded to the large-batch kernel's tiling (a -inf bias keeps the padding from being chosen)."""
+    mlp.router, mlp.top = w.float(), top
+    if on_cuda and w.dtype in (torch.float16, torch.bfloat16):
+        E = w.shape[0]
+        pad = -E % 32
+        mlp.router_16 = torch.cat([w, w.new_zeros((pad, w.shape[1]))]).contiguous()
+        if pad:
+            mlp.router_bias = torch.cat([torch.zeros(E), torch.full((pad,), float("-inf"))]).to(w.device)
+
+
+def route_scored(mlp, x):
+    """(experts int32 [T, top], their sigmoid scores fp32, not renormalised) of a router made by ``set_router``."""
+    if not x.is_cuda:
+        logits = torch.matmul(x.float(), mlp.router.t())
+    elif mlp.router_16 is not None and mlp.router_16.dtype == x.dtype:
+        logits = B.linear(x, mlp.router_16, out_f32=True)
+    else:
+        logits = B.linear_full32(x.float(), mlp.router)
+    bias = mlp.router_bias if mlp.router_bias is not None and mlp.router_bias.shape[0] == logits.shape[1] else None
+    return route_topk(logits, bias, mlp.top, 1, False)
+
+
 class TableRouter:
     """Routing by token id: every such layer has a table ``[vocab, top]`` of experts.  The plans of all layers depend on the ids
     alone, so one launch at the start of a forward pass makes them (one CTA per layer; a layer that runs several times is planned once)."""
@@ -144,7 +168,8 @@ class ExpertWeights:
         self.down = down
         self.stacked = None     # filled by ops.moe_grouped when a grouped kernel can take the whole set
         self.act = "swiglu"     # "gptoss": clamped gate/up, gate * sigmoid(1.702 gate) * (up + 1); "swiglu_clamp": see limit
-        self.limit = 0.0        # "swiglu_clamp" (Step-3.5): min(silu(gate), limit) * clamp(up, -limit, limit)
+        self.limit = 0.0        # "swiglu_clamp" (Step-3.5): min(silu(gate), limit) * clamp(up, -limit, limit); "gptoss": its clamp (0: 7)
+        self.scale_input = False    # the router's weight multiplies the expert's input, not its output
         self.host = False       # expert weights live in CPU memory and run on the native CPU backend (hybrid placement)
         self._host_arrays = None
 
@@ -192,14 +217,15 @@ def output_is_complete(ep) -> bool:
 
 
 def moe_forward(x, idx, wts, experts: ExpertWeights, ep=None):
-    """``y[t] = sum_k wts[t,k] * down_e(silu(gate_e x) * up_e x)`` over the experts this rank owns.
+    """``y[t] = sum_k wts[t,k] * down_e(silu(gate_e x) * up_e x)`` over the experts this rank owns (``scale_input``: the weight
+    multiplies x instead).
 
     Tokens are grouped by expert; each non-empty local expert runs the two GEMMs on its token group.
     With expert parallelism the result is this rank's partial sum (the caller all-reduces it).
     """
     if experts.host and experts.act == "swiglu":
         return _moe_forward_host(x, idx, wts, experts)
-    if experts.stacked is not None and x.is_cuda and experts.act == "swiglu":
+    if experts.stacked is not None and x.is_cuda and experts.act == "swiglu" and not experts.scale_input:
         from . import moe_grouped
 
         y = moe_grouped.forward(x, idx, wts, experts)
@@ -223,13 +249,15 @@ def moe_forward(x, idx, wts, experts: ExpertWeights, ep=None):
         rows = t_sorted[start:start + n]
         xe = x.index_select(0, rows)
         le = e - experts.first
+        if experts.scale_input:
+            xe = (xe.float() * w_sorted[start:start + n, None]).to(x.dtype)
         if experts.act == "gptoss":
-            he = experts.down[le](glu_gptoss(experts.gate_up[le](xe), experts.gate_up[le].interleaved))
+            he = experts.down[le](glu_gptoss(experts.gate_up[le](xe), experts.gate_up[le].interleaved, experts.limit or 7.0))
         elif experts.act == "swiglu_clamp":
             he = experts.down[le](glu_clamped(experts.gate_up[le](xe), experts.gate_up[le].interleaved, experts.limit))
         else:
             he = experts.down[le](experts.gate_up[le](xe, swiglu=True))
-        y.index_add_(0, rows, he.float() * w_sorted[start:start + n, None])
+        y.index_add_(0, rows, he.float() if experts.scale_input else he.float() * w_sorted[start:start + n, None])
         start += n
     return y.to(x.dtype)
 

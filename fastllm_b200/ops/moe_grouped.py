@@ -15,7 +15,8 @@ import torch
 from . import _lib
 from . import basic as B
 from . import quant_gemm as QG
-from .basic import GEMM_SWIGLU, _ptr, _stream, dtype_code
+from .basic import GEMM_GLU_CLAMP, GEMM_SWIGLU, _ptr, _stream, dtype_code
+from .stream32 import moe_gather_scaled
 
 P, I = ctypes.c_void_p, ctypes.c_int
 _lib.register_sigs({
@@ -24,11 +25,13 @@ _lib.register_sigs({
     "fb_moe_gather": [P, P, P, I, I, I, P],
     "fb_moe_combine": [P, P, P, P, P, I, I, I, I, P],
     "fb_moe_grouped_gemm": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, P],
+    "fb_moe_grouped_gemm_act": [P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, ctypes.c_float, ctypes.c_float, P],
     "fb_moe_grouped_gemm_quant": [P, P, P, P, P, P, P, I, I, I, I, I, I, I, I, I, I, I, P],
 }, ["moe"])
 
 GRAPH_SAFE = True
 PAD = 16
+GPTOSS_ALPHA = 1.702             # g * sigmoid(alpha g) * (u + 1)
 
 
 class StackedExperts:
@@ -112,7 +115,9 @@ def prepare_model(m) -> None:
     """Stack the experts of every MoE layer; the per-expert tensors are replaced by views of the stacked matrices."""
     for lw in m.layers:
         ex = lw.mlp.experts
-        if ex is None or ex.stacked is not None or ex.count == 0 or ex.host or ex.act != "swiglu" or any(l.bias is not None for l in ex.gate_up + ex.down):
+        if ex is None or ex.stacked is not None or ex.count == 0 or ex.host or any(l.bias is not None for l in ex.gate_up + ex.down):
+            continue
+        if ex.act != "swiglu" and not (ex.act == "gptoss" and ex.gate_up[0].kind == "dense"):
             continue
         st = stack_experts(ex)
         if st is None:
@@ -130,24 +135,42 @@ def prepare_model(m) -> None:
             _prepare_a8(st, ex)                    # scale tables of the integer path, before any CUDA graph is captured
 
 
-def _forward32(x, st, plan):
+def _make_plan(idx, experts):
+    """(counts, offsets, pos, total) of the pairs ``idx`` [T, top] (``fb_moe_plan``)."""
+    T, topk = idx.shape
+    dev, E = idx.device, experts.stacked.n_local
+    counts, offsets = torch.empty(E, device=dev, dtype=torch.int32), torch.empty(E, device=dev, dtype=torch.int32)
+    pos, total = torch.empty((T, topk), device=dev, dtype=torch.int32), torch.empty(1, device=dev, dtype=torch.int32)
+    idx = idx.contiguous()
+    _lib.check(_lib.kernels().fb_moe_plan(_ptr(idx), T, topk, experts.first, E, _ptr(counts), _ptr(offsets), _ptr(pos), _ptr(total), PAD, _stream()), "fb_moe_plan")
+    return counts, offsets, pos, total
+
+
+def _forward32(x, st, plan, experts, wts, rows32):
     """The same steps on fp32 operands (CUDA-core products): sorted expert outputs and their positions."""
+    from .moe import glu_gptoss
+
     counts, offsets, pos, _ = plan
     T, H = x.shape
     topk = pos.shape[1]
-    rows_cap = T * topk + st.n_local * PAD + 128
-    xs = torch.empty((rows_cap, H), device=x.device, dtype=x.dtype)
-    _lib.check(_lib.kernels().fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, 2 * H, _stream()), "fb_moe_gather")
-    act = B.glu_act_ref(B.linear_full32(xs, st.gate_up, batch=st.n_local, counts=counts, offsets=offsets), "silu", True)
+    xs = torch.empty((T * topk + st.n_local * PAD + 128, H), device=x.device, dtype=x.dtype)
+    if rows32 is not None:
+        moe_gather_scaled(rows32, pos, wts, xs)
+    else:
+        _lib.check(_lib.kernels().fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, 2 * H, _stream()), "fb_moe_gather")
+    gu = B.linear_full32(xs, st.gate_up, batch=st.n_local, counts=counts, offsets=offsets)
+    act = glu_gptoss(gu, True, experts.limit or 7.0) if experts.act == "gptoss" else B.glu_act_ref(gu, "silu", True)
     return B.linear_full32(act, st.down, batch=st.n_local, counts=counts, offsets=offsets, n=H), pos
 
 
-def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add: torch.Tensor | None = None, combine: bool = True, plan=None):
+def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add: torch.Tensor | None = None, combine: bool = True, plan=None,
+            rows32: torch.Tensor | None = None):
     """``combine=False`` stops before the weighted sum and returns ``(ys, pos, wts)`` for a fused combine.  ``plan``: the routing
-    plan (counts, offsets, pos, total) where it is known already (``ops.moe.TableRouter``)."""
+    plan (counts, offsets, pos, total) where it is known already (``ops.moe.TableRouter``).  ``rows32``: the experts' inputs are these
+    fp32 rows times the pair's weight, in place of ``x``."""
     st = experts.stacked
-    if st is not None and plan is not None and not combine and x.dtype == torch.float32 and st.kind == "dense" and st.gate_up.dtype == x.dtype:
-        ys, pos = _forward32(x, st, plan)
+    if st is not None and not combine and x.dtype == torch.float32 and st.kind == "dense" and st.gate_up.dtype == x.dtype:
+        ys, pos = _forward32(x, st, plan if plan is not None else _make_plan(idx, experts), experts, wts, rows32)
         return ys, pos, wts
     if st is None or x.dtype not in (torch.float16, torch.bfloat16):
         return None
@@ -165,15 +188,7 @@ def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add:
         hint = 16          # the 16-row integer kernel has dedicated unpack warps; a second chunk re-reads its weights from L2
     max_rows = min(T, 0xFFFF) | (hint << 16)
     s = _stream()
-    if plan is not None:
-        counts, offsets, pos, total = plan
-    else:
-        counts = torch.empty(E, device=dev, dtype=torch.int32)
-        offsets = torch.empty(E, device=dev, dtype=torch.int32)
-        pos = torch.empty((T, topk), device=dev, dtype=torch.int32)
-        total = torch.empty(1, device=dev, dtype=torch.int32)
-        idx = idx.contiguous()
-        _lib.check(lib.fb_moe_plan(_ptr(idx), T, topk, experts.first, E, _ptr(counts), _ptr(offsets), _ptr(pos), _ptr(total), PAD, s), "fb_moe_plan")
+    counts, offsets, pos, total = plan if plan is not None else _make_plan(idx, experts)
     if wts is not None:
         wts = wts.float().contiguous()
     dt = dtype_code(x.dtype)
@@ -193,12 +208,17 @@ def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add:
     elif int_a8:
         # gather fused with the int8 quantisation of the rows
         xq, sa, sx, ld_a = QG.quant_act_i8(x.contiguous(), pos=pos, topk=topk, rows_cap=rows_cap)
+    elif rows32 is not None:
+        xs = torch.empty((rows_cap, H), device=dev, dtype=x.dtype)
+        moe_gather_scaled(rows32, pos, wts, xs)
     else:
         xs = torch.empty((rows_cap, H), device=dev, dtype=x.dtype)
         _lib.check(lib.fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, H, s), "fb_moe_gather")
     if st.kind == "dense":
-        _lib.check(lib.fb_moe_grouped_gemm(_ptr(xs), _ptr(st.gate_up), _ptr(act), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E,
-                                           2 * st.inter, H, st.inter, max_rows, dt, GEMM_SWIGLU, T * topk, s), "fb_moe_grouped_gemm(gate_up)")
+        clamp = experts.act == "gptoss"
+        _lib.check(lib.fb_moe_grouped_gemm_act(_ptr(xs), _ptr(st.gate_up), _ptr(act), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E, 2 * st.inter, H,
+                                               st.inter, max_rows, dt, GEMM_SWIGLU | (GEMM_GLU_CLAMP if clamp else 0), T * topk,
+                                               (experts.limit or 7.0) if clamp else 0.0, GPTOSS_ALPHA, s), "fb_moe_grouped_gemm(gate_up)")
         _lib.check(lib.fb_moe_grouped_gemm(_ptr(act), _ptr(st.down), _ptr(ys), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E,
                                            H, st.inter, H, max_rows, dt, 0, T * topk, s), "fb_moe_grouped_gemm(down)")
     elif fp8_native:
