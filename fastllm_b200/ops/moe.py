@@ -47,7 +47,7 @@ def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group
 
 def route_topk(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0):
     """logits fp32 ``[M, E]`` -> (expert index int32 ``[M, topk]``, weight fp32 ``[M, topk]``)."""
-    if not logits.is_cuda or logits.shape[1] > 512:
+    if not logits.is_cuda or logits.shape[1] > 512 or topk > 32:        # beyond the kernel's registers: tensor ops
         return route_topk_ref(logits, bias, topk, score_mode, renorm, n_group, topk_group, route_scale)
     lg = logits.float().contiguous()
     M, E = lg.shape

@@ -1,8 +1,9 @@
-"""Throughput and kernel times of latent-attention models whose layers are listed one by one, beside the closest other family
-(multi-head latent attention with routed experts, DeepSeek-V3 layout) at equal sizes; random weights.
+"""Throughput and kernel times of models whose layers are listed one by one, beside the closest other family at equal sizes; random
+weights.
 
-``python bench.py --layers patesun`` prints one JSON line per measurement:
-  * ``step``   -- prefill and decode tokens/s of a short stack (one dense layer, three expert layers) through the engine's runner;
+``python bench.py --layers patesun`` (beside multi-head latent attention with routed experts, DeepSeek-V3 layout) and ``--layers
+vilulorn`` (beside Gated DeltaNet + gated attention with routed experts, Qwen3-Next layout) print one JSON line per measurement:
+  * ``step``   -- prefill and decode tokens/s of a stack of four layers through the engine's runner;
   * ``kernel`` -- one operator alone: microseconds, its bytes / FLOPs and the fraction of the measured copy bandwidth or GEMM peak.
 Operators are timed with CUDA events behind an L2 flush that also hides the host's launch time; the median of the repeats is kept.
 """
@@ -21,6 +22,12 @@ SIZES = {
     "7k": dict(width=7168, heads=128, rank=512, window=4096, ff=18432, experts=64, top=8, eff=2048, shared=2048),
 }
 HEAD, VOCAB, LAYERS = 128, 32768, 4
+HYBRID_SIZES = {
+    # width, query heads, key / value heads, linear heads, chunk, experts, top, expert ff
+    "2k": dict(width=2048, heads=16, kv=4, lin=16, chunk=4096, experts=64, top=6, eff=1024),
+    "4k": dict(width=4096, heads=32, kv=8, lin=32, chunk=4096, experts=64, top=6, eff=1024),
+    "7k": dict(width=7168, heads=64, kv=8, lin=56, chunk=8192, experts=64, top=8, eff=2048),
+}
 
 
 def patesun_config(z):
@@ -42,6 +49,27 @@ def mla_config(z):
                              n_shared_experts=z["shared"] // z["eff"], first_k_dense_replace=1, n_group=1, topk_group=1,
                              scoring_func="sigmoid", topk_method="noaux_tc", norm_topk_prob=True, kv_lora_rank=z["rank"],
                              qk_nope_head_dim=HEAD, qk_rope_head_dim=64, v_head_dim=HEAD, rms_norm_eps=1e-6, max_position_embeddings=65536))
+
+
+def vilulorn_config(z):
+    from ..models.config import from_hf_dict
+
+    at = {"heads": z["heads"], "kv_heads": z["kv"], "dim": HEAD, "vdim": HEAD, "scale": HEAD ** -0.5, "mask": {"size": z["chunk"]},
+          "rot": {"base": 5e5, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    gl = {"heads": z["lin"], "dim": HEAD, "vdim": HEAD, "tau": 16.0}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
+    return from_hf_dict(dict(architecture="Vilulorn", vocab=VOCAB, width=z["width"], norm={"eps": 1e-6}, max_positions=1 << 16,
+                             layers=[{"type": t, "mixer": m, "mlp": moe} for t, m in (("gla", gl), ("attention", at), ("gla", gl), ("attention", dict(at, kv_from=1)))]))
+
+
+def deltanet_config(z):
+    from ..models.config import from_hf_dict
+
+    return from_hf_dict(dict(model_type="qwen3_next", vocab_size=VOCAB, hidden_size=z["width"], num_hidden_layers=LAYERS, num_attention_heads=z["heads"],
+                             num_key_value_heads=z["kv"], head_dim=HEAD, intermediate_size=z["eff"], num_experts=z["experts"],
+                             num_experts_per_tok=z["top"], moe_intermediate_size=z["eff"], linear_num_key_heads=z["lin"], linear_num_value_heads=z["lin"],
+                             linear_key_head_dim=HEAD, linear_value_head_dim=HEAD, full_attention_interval=2, partial_rotary_factor=0.5, rms_norm_eps=1e-6,
+                             max_position_embeddings=65536))
 
 
 class Timer:
@@ -90,13 +118,14 @@ def bench_steps(family: str, cfg, size: str, cases, emit) -> None:
         pages = (ctx + 64) // 128 + 1
         runner = ModelRunner(model, EngineConfig(max_batch=batch, max_context=pages * 128, prefix_cache=False, graph_batch_sizes=[batch]), num_pages=batch * pages + 1)
         owned = [list(range(b * pages, (b + 1) * pages)) for b in range(batch)]
+        states = list(range(batch)) if runner.state_slots else None
         toks = torch.randint(0, VOCAB, (ctx,), generator=gen).tolist()
         per = max(1, 8192 // ctx)                       # requests of a prefill step of about 8192 tokens
         n_pre = min(per, batch)
 
         def prefill(first, count):
             for s in range(0, ctx, 8192):
-                runner.prefill([(toks[s:s + 8192], s, owned[b], s + 8192 >= ctx) for b in range(first, first + count)])
+                runner.prefill([(toks[s:s + 8192], s, owned[b], s + 8192 >= ctx, b if states else None) for b in range(first, first + count)])
 
         for _ in range(2):
             prefill(0, n_pre)
@@ -116,7 +145,7 @@ def bench_steps(family: str, cfg, size: str, cases, emit) -> None:
         ids = torch.randint(0, VOCAB, (batch,), generator=gen).tolist()
         pos = [ctx] * batch
         for _ in range(4):
-            runner.decode(ids, pos, owned)
+            runner.decode(ids, pos, owned, state_slots=states)
         slot = runner.slots[batch]
         torch.cuda.synchronize()
         ms = []
@@ -255,13 +284,153 @@ def bench_kernels(z, size: str, emit) -> None:
         torch.cuda.empty_cache()
 
 
-def run(sizes, steps: bool = True, kernels: bool = True, emit=None) -> None:
+def bench_hybrid_kernels(z, size: str, emit) -> None:
+    """Operators of the chunked-attention / gated-linear-attention stack, each before the like one of the Gated-DeltaNet stack."""
+    from ..models.config import AttnSpec, GLASpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import attention as A
+    from ..ops import basic as B
+    from ..ops import gla as GLA
+    from ..ops import grouped as GR
+    from ..ops import linear_attn as L
+    from ..ops import moe as MOE
+    from ..ops import moe_grouped as MG
+    from ..ops import stream32 as S
+    from ..ops._lib import kernels
+
+    tm = Timer()
+    hbm, tf, src = peaks()
+    dev, dt = "cuda", torch.bfloat16
+    W, H, G, N, C, E, top, eff = (z[k] for k in ("width", "heads", "kv", "lin", "chunk", "experts", "top", "eff"))
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=dt) * 0.05
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    rope = {"theta": 5e5, "rot_dim": 64, "scaling": None}
+    cos, sin = A.build_rope_tables(64, 65536, 5e5, None, dev)
+
+    def put(name, role, fn, nbytes, flops, **info):
+        us = tm.us(fn)
+        t_mem, t_mm = nbytes / hbm / 1e3, flops / tf / 1e6
+        emit(dict(kind="kernel", size=size, name=name, role=role, us=round(us, 2), gbytes=nbytes / 1e9, gflop=flops / 1e9,
+                  bound="memory" if t_mem > t_mm else "tensor", roofline_frac=round(max(t_mem, t_mm) / us, 4), peak=src, **info))
+
+    # recurrent step of 64 requests: state read and written once
+    Bn, D = 64, HEAD
+    gw, _ = GLA.build(GLASpec(N, D, D, 16.0), *(rnd(N * D, 16) for _ in range(4)), rnd(16, 16), rnd(N * D, 16), rnd(N * D), rnd(D))
+    st, slots = torch.zeros((Bn + 1, N, D, D), device=dev), i32(list(range(Bn)))
+    proj = rnd(Bn, gw.cols[-1] + 32)
+    fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=None, kv_lens=None, cu_q=None, is_decode=True, state_slots=slots)
+    nb = Bn * N * (2 * D * D * 4 + 5 * D * 2)
+    put("gla step", "new", lambda: GLA.mix(gw, proj, fb, st, 1e-6), nb, 0, batch=Bn)
+    mixed, ab, zz, par = rnd(Bn, 3 * N * D), rnd(Bn, N), rnd(Bn, N * D), torch.zeros(N, device=dev)
+    put("delta-rule step", "like", lambda: L.gated_delta_decode(mixed, ab, ab, zz, par, par, gw.norm, 1e-6, st, slots, N, N, D, D), nb, 0, batch=Bn)
+    # prompts: chunked forms
+    T = 8192
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        cu = [n * b for b in range(n_req + 1)]
+        proj, sl = rnd(T, gw.cols[-1] + 32), list(range(n_req))
+        fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=i32([[0]]), kv_lens=None, cu_q=i32(cu), cu_q_host=cu, state_slots=i32(sl), state_slots_host=sl)
+        nb, fl = T * N * D * 2 * 5, T * N * (4.0 * D * D + 2.0 * 64 * D)
+        put("gla prompt", "new", lambda: GLA.mix(gw, proj, fb, st, 1e-6), nb, fl, requests=n_req, tokens=n)
+        q, k, v, a = rnd(T, N, D), rnd(T, N, D), rnd(T, N, D), rnd(T, N)
+
+        def like():
+            o = L.gated_delta_rule(q, k, v, a, a, par, par, st, cu, sl, 1)
+            return L.rmsnorm_gated(o, v, gw.norm, 1e-6)
+        put("delta-rule prompt", "like", like, nb, fl, requests=n_req, tokens=n)
+        del q, k, v, a, proj
+    del st
+    # attention: decoded rows, prompts, post-processing
+    spec = AttnSpec(H, G, HEAD, HEAD, HEAD ** -0.5, C, rope)
+    at, _ = GR.build(spec, rnd(H * HEAD, 16), rnd(G * HEAD, 16), rnd(G * HEAD, 16), rnd(H * HEAD, 16), rnd(HEAD), rnd(HEAD))
+    ctxs = (C, 2 * C)
+    for ctx in ctxs:
+        pages = ctx // 128
+        pool = (rnd(Bn * pages, 128, G, HEAD), rnd(Bn * pages, 128, G, HEAD))
+        pt, lens = torch.randperm(Bn * pages, device=dev).to(torch.int32).view(Bn, pages), i32([ctx] * Bn)
+        fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=pt, kv_lens=lens, cu_q=None, is_decode=True)
+        proj = rnd(Bn, (at.v_col + G * HEAD + 31) // 32 * 32)
+        GR.attention(at, proj, pool, fb)
+        put("grouped decode", "new", lambda: GR.attention(at, proj, pool, fb), Bn * (C * G * HEAD * 4 + H * HEAD * 6), 4.0 * Bn * H * C * HEAD, batch=Bn, context=ctx, keys=C)
+        ws = A.DecodeWorkspace(Bn, G, H // G, pages, torch.device(dev), HEAD)
+        ws.plan(lens)
+        q = rnd(Bn, H * HEAD)
+        put("decode attention", "like", lambda: A.attn_decode(q, *pool, pt, lens, 0.1, H, G, HEAD, ws=ws, planned=True), Bn * (ctx * G * HEAD * 4 + H * HEAD * 4),
+            4.0 * Bn * H * ctx * HEAD, batch=Bn, context=ctx, keys=ctx)
+        del pool, ws
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        pages, cu = n // 128, [n * b for b in range(n_req + 1)]
+        pool = (rnd(n_req * pages, 128, G, HEAD), rnd(n_req * pages, 128, G, HEAD))
+        pt, lens = torch.arange(n_req * pages, device=dev, dtype=torch.int32).view(n_req, pages), i32([n] * n_req)
+        pos = torch.arange(T, device=dev, dtype=torch.int32)
+        fb = ForwardBatch(ids=pos, positions=pos % n, slots=pos, page_table=pt, kv_lens=lens, cu_q=i32(cu), cu_q_host=cu, kv_lens_host=[n] * n_req)
+        proj = rnd(T, (at.v_col + G * HEAD + 31) // 32 * 32)
+        causal = lambda m: m * (m + 1) // 2
+        seen = (n // C * causal(C) + causal(n % C)) * n_req
+        GR.attention(at, proj, pool, fb)
+        put("grouped prompt attention", "new", lambda: GR.attention(at, proj, pool, fb), T * (H * HEAD * 6 + G * HEAD * 4), 4.0 * seen * H * HEAD, requests=n_req, tokens=n)
+        q = rnd(T, H * HEAD)
+        put("prompt attention", "like", lambda: A.attn_prefill(q, *pool, pt, lens, fb.cu_q, 0.1, H, G, HEAD, cu_q_host=cu), T * (H * HEAD * 4 + G * HEAD * 4),
+            4.0 * causal(n) * n_req * H * HEAD, requests=n_req, tokens=n)
+    nb = T * (2 * H + 4 * G) * HEAD * 2
+    put("head norm + rotary + append", "new", lambda: GR.post(at, proj, fb, pool, cos, sin, 1e-6), nb, 0, rows=T)
+    qkv, nw = rnd(T, (H + 2 * G) * HEAD), rnd(HEAD)
+    put("qkv post", "like", lambda: A.qkv_post(qkv, fb.positions, fb.slots, *pool, H, G, HEAD, cos, sin, A.ROPE_INTERLEAVED, 64, nw, nw), nb, 0, rows=T)
+    del pool, proj, qkv
+    # row operators
+    h, y, nw = torch.randn(T, W, device=dev), rnd(T, W), torch.ones(W, device=dev, dtype=dt)
+    res = rnd(T, W)
+    put("output norm + residual", "new", lambda: S.add_norm(h, y, nw, None, 1e-6), T * W * 12, 0)
+    put("residual + norm", "like", lambda: B.rmsnorm(y, nw, 1e-6, residual=res), T * W * 8, 0)
+    ids, pos, table, ptab = torch.randint(0, VOCAB, (T,), device=dev, dtype=torch.int32), torch.arange(T, device=dev, dtype=torch.int32), rnd(VOCAB, W), rnd(T, W)
+    put("embedding + learned positions", "new", lambda: S.embed_pos_norm(ids, pos, table, None, None, 1e-6, pos_table=ptab), T * W * 10, 0)
+    put("embedding + norm", "like", lambda: B.rmsnorm(B.embedding(ids, table), nw, 1e-6), T * W * 8, 0)
+    # experts: routing, plan, gather, the two grouped products, combine
+    ex = MOE.ExpertWeights(E, 0, [], [])
+    ex.count, ex.act, ex.limit, ex.scale_input = E, "gptoss", 7.0, True
+    ex.stacked = MG.StackedExperts("dense", rnd(E * 2 * eff, W), rnd(E * W, eff), E, eff, W)
+    ey = MOE.ExpertWeights(E, 0, [], [])
+    ey.count, ey.stacked = E, ex.stacked
+
+    class _M:
+        router_bias = None
+    MOE.set_router(_M, rnd(E, W), top, True)
+    for M in (64, T):
+        x, h, res = rnd(M, W), torch.randn(M, W, device=dev), rnd(M, W)
+        logits, bias = torch.randn(M, E, device=dev), torch.zeros(E, device=dev)
+        put("router + top-k", "new", lambda: MOE.route_scored(_M, x), M * W * 2 + E * W * 2, 2.0 * M * E * W, rows=M)
+        put("router + top-k", "like", lambda: MOE.route_topk(B.linear(x, _M.router_16, out_f32=True), None, top, 0, True), M * W * 2 + E * W * 2, 2.0 * M * E * W, rows=M)
+        idx, wts = MOE.route_topk(logits, bias, top, 1, False)
+        fl, nb = 6.0 * M * top * W * eff, 3 * E * W * eff * 2 + M * top * (4 * W + 2 * eff) * 2
+
+        def new():
+            ys, p_, _ = MG.forward(x, idx, wts, ex, combine=False, rows32=h)
+            return S.moe_combine_norm(ys, p_, None, 1.0, None, h, None, 1.0, 1e-6, post_w=nw, dtype=dt)
+        put("experts, scaled inputs, output norm", "new", new, nb, fl, rows=M)
+        put("experts, residual, norm", "like", lambda: B.rmsnorm(MG.forward(x, idx, wts, ey), nw, 1e-6, residual=res), nb, fl, rows=M)
+        plan = MG._make_plan(idx, ex)
+        xs, rows = torch.empty((M * top + E * 16 + 128, W), device=dev, dtype=dt), M * top
+        put("scaled gather", "new", lambda: S.moe_gather_scaled(h, plan[2], wts, xs), M * W * 4 + rows * W * 2, 0, rows=M)
+        put("gather", "like", lambda: kernels().fb_moe_gather(B._ptr(x), B._ptr(plan[2]), B._ptr(xs), M, top, W, B._stream()), M * W * 2 + rows * W * 2, 0, rows=M)
+        put("combine, output norm, residual", "new", lambda: S.moe_combine_norm(xs, plan[2], None, 1.0, None, h, None, 1.0, 1e-6, post_w=nw, dtype=dt),
+            rows * W * 2 + M * W * 10, 0, rows=M)
+
+        def comb():
+            out = torch.empty((M, W), device=dev, dtype=dt)
+            kernels().fb_moe_combine(B._ptr(xs), B._ptr(plan[2]), B._ptr(wts), B._ptr(None), B._ptr(out), M, top, W, 1, B._stream())
+            return B.rmsnorm(out, nw, 1e-6, residual=res)
+        put("combine, residual, norm", "like", comb, rows * W * 2 + M * W * 8, 0, rows=M)
+    torch.cuda.empty_cache()
+
+
+def run(family: str, sizes, steps: bool = True, kernels: bool = True, emit=None) -> None:
     emit = emit or (lambda d: print(json.dumps(d), flush=True))
+    hybrid = family == "vilulorn"
     for size in sizes:
-        z = SIZES[size]
+        z = (HYBRID_SIZES if hybrid else SIZES)[size]
         if kernels:
-            bench_kernels(z, size, emit)
+            (bench_hybrid_kernels if hybrid else bench_kernels)(z, size, emit)
         torch.cuda.empty_cache()
         if steps:
-            for family, cfg in (("patesun", patesun_config(z)), ("mla", mla_config(z))):
-                bench_steps(family, cfg, size, ((1, z["window"]), (64, z["window"] // 2), (64, z["window"])), emit)
+            span = z["chunk" if hybrid else "window"]
+            for fam, cfg in ((("vilulorn", vilulorn_config(z)), ("deltanet", deltanet_config(z))) if hybrid else (("patesun", patesun_config(z)), ("mla", mla_config(z)))):
+                bench_steps(fam, cfg, size, ((1, span), (64, span // 2), (64, span)), emit)

@@ -8,17 +8,17 @@ import json
 import pytest
 import torch
 
+from . import listed_common as LC
 from . import patesun_oracle as O
+from .listed_common import DEVICES, PAGE, assert_close, few_threads, portions, save  # noqa: F401
 from fastllm_b200.engine import EngineConfig, GenerationConfig, LLMEngine
 from fastllm_b200.engine.replay import Replay, open_engine
-from fastllm_b200.loader import safetensors as st
 from fastllm_b200.loader.hf import load_model
 from fastllm_b200.models.decoder import ForwardBatch
 from fastllm_b200.ops import latent as LA
 from fastllm_b200.ops import stream32 as S
 
 gpu = pytest.mark.gpu
-PAGE = 128
 
 
 def mixer(heads, dim, vdim, rank, window, scale=None):
@@ -51,8 +51,6 @@ CONFIGS = {
     # one head, one expert, a window of one token, no loop, and full causal attention
     "ones": config([(mixer(1, 8, 8, 8, 1), moe(1, 1, 8, 8)), (mixer(1, 16, 8, 16, 0), {"kind": "dense", "ff": 8})], width=64, vocab=64, mult=0.7),
 }
-DEVICES = [pytest.param(("cpu", torch.float32), id="cpu"), pytest.param(("cuda", torch.float32), id="gpu32", marks=gpu),
-           pytest.param(("cuda", torch.bfloat16), id="gpu16", marks=gpu)]
 _CACHE: dict = {}
 
 
@@ -60,22 +58,6 @@ def weights(name):
     if name not in _CACHE:
         _CACHE[name] = O.random_weights(CONFIGS[name], seed=len(name))
     return _CACHE[name]
-
-
-def save(path, cfg, w):
-    path.mkdir(exist_ok=True)
-    (path / "config.json").write_text(json.dumps(cfg))
-    st.save_file(w, path / "model.safetensors")
-    return path
-
-
-@pytest.fixture(autouse=True, scope="module")
-def _few_threads():
-    """The matrices are tiny: more threads than a few only wait for one another."""
-    n = torch.get_num_threads()
-    torch.set_num_threads(min(n, 4))
-    yield
-    torch.set_num_threads(n)
 
 
 @pytest.fixture(scope="module")
@@ -102,42 +84,8 @@ def prompt(name, n, seed=0):
     return torch.randint(0, CONFIGS[name]["vocab"], (n,), generator=g).tolist()
 
 
-def assert_close(got, want, dtype, tol16=0.03):
-    """Root mean square of the difference relative to the logits' own, per row."""
-    err = ((got.double() - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()).max().item()
-    limit = 3e-5 if dtype == torch.float32 else tol16
-    assert err < limit, f"relative error {err:.3g}"
-
-
 def replay(models, name, where, reqs, schedule, max_tokens):
-    """Run a schedule of (request, count) steps; compares every position's logits with the whole-sequence oracle."""
-    device, dtype = where
-    eng = open_engine(models(name)[2], dtype, max_tokens, device)
-    rp, at, got = Replay(eng), {}, {r: [] for r in reqs}
-    free = eng.pm.num_free()
-    for step in schedule:
-        entries = []
-        for r, n in step:
-            lo = at.get(r, 0)
-            entries.append((r, reqs[r][lo:lo + n], list(range(n))))
-            at[r] = lo + n
-        out = rp.step(entries, [r for r, _ in step if at[r] == len(reqs[r])])
-        row = 0
-        for r, n in step:
-            got[r].append(out[row:row + n])
-            row += n
-    assert eng.pm.num_free() == free, "pages were not given back"
-    for r, toks in reqs.items():
-        assert at[r] == len(toks)
-        assert_close(torch.cat(got[r]), oracle(name, toks), dtype)
-
-
-def portions(n, sizes):
-    out, i = [], 0
-    while sum(out) < n:
-        out.append(min(sizes[i % len(sizes)], n - sum(out)))
-        i += 1
-    return out
+    LC.replay(models(name)[2], where, reqs, schedule, max_tokens, lambda toks: oracle(name, toks))
 
 
 # ---------------------------------------------------------------------------------------------------

@@ -147,8 +147,8 @@ def forward(cfg, w, tokens, dtype=torch.float64, layers_out=None):
     return linear(w["head"], rms_norm(x, w["final.norm"], eps))
 
 
-def random_weights(cfg, seed=0, scale=1.0):
-    """bfloat16 weights of the right names and shapes (norm weights around one)."""
+def random_weights(cfg, seed=0, scale=1.0, rank=16):
+    """bfloat16 weights of the right names and shapes (norm weights around one); ``rank``: inner width of the decay projections."""
     g = torch.Generator().manual_seed(seed)
     E, V = cfg["width"], cfg["vocab"]
     w = {}
@@ -169,12 +169,11 @@ def random_weights(cfg, seed=0, scale=1.0):
         mat(p + "mix.g", H * Vd, E)
         mat(p + "mix.o", E, H * Vd)
         if spec["type"] == "gla":
-            R = mx.get("_rank", 16)
             mat(p + "mix.k", H * D, E)
             mat(p + "mix.v", H * Vd, E)
             norm(p + "mix.norm", Vd)
-            mat(p + "mix.a1", R, E)
-            mat(p + "mix.a2", H * D, R, 2.0)
+            mat(p + "mix.a1", rank, E)
+            mat(p + "mix.a2", H * D, rank, 2.0)
             norm(p + "mix.a2.b", H * D, 0.5)
         else:
             norm(p + "mix.q.norm", D, 1.5)
