@@ -25,7 +25,7 @@ from .basic import _ptr, _stream
 P, I, FLT, LL = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _lib.register_sigs({
     "fb_gla_recurrent": [P, LL, P, P, P, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, FLT, FLT, FLT, I, P],
-    "fb_gla_chunked": [P, LL, P, P, P, P, P, I, P, I, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, FLT, FLT, FLT, I, P],
+    "fb_gla_chunked": [P, LL, P, P, P, P, P, I, P, I, P, P, P, P, LL, I, I, I, I, I, I, I, I, I, I, FLT, FLT, FLT, I, P],
 }, ["gla"])
 
 CHUNK = 64
@@ -90,13 +90,13 @@ def mix(w: GLAWeights, proj, fb, state, eps: float):
     pl = fb.__dict__.get("_gla_plan")
     if pl is None:
         pl = fb._gla_plan = _ChunkPlan(fb)
-    per_head = pl.n_chunks * w.dim * (w.vdim + 1)
+    sizes = [pl.n_chunks * w.dim * CHUNK, pl.n_chunks * w.dim * w.vdim, pl.n_chunks * w.dim]      # log-decays, increments, chunk decays
+    per_head = sum(sizes)
     step = max(1, min(w.heads, SCRATCH_BYTES // (4 * per_head)))
-    scratch = torch.empty((per_head * step,), device=proj.device, dtype=torch.float32)
-    dec = scratch[pl.n_chunks * step * w.dim * w.vdim:]
+    lg, inc, dec = torch.empty((per_head * step,), device=proj.device, dtype=torch.float32).split([x * step for x in sizes])
     for h0 in range(0, w.heads, step):
         rc = _lib.kernels().fb_gla_chunked(_ptr(proj), proj.stride(0), _ptr(w.a2), _ptr(w.a2_b), _ptr(w.norm), _ptr(state), _ptr(pl.chunks), pl.n_chunks,
-                                           _ptr(pl.reqs), pl.n_reqs, _ptr(scratch), _ptr(dec), _ptr(out), out.stride(0), w.heads, h0,
+                                           _ptr(pl.reqs), pl.n_reqs, _ptr(inc), _ptr(dec), _ptr(lg), _ptr(out), out.stride(0), w.heads, h0,
                                            min(step, w.heads - h0), w.dim, w.vdim, w.rank, kc, vc, gc, ac, w.dim ** -0.5, 1.0 / w.tau, float(eps),
                                            S.act_code(proj.dtype), _stream())
         _lib.check(rc, "fb_gla_chunked")

@@ -258,7 +258,29 @@ def model_kernel_table(model="qwen3-30b-a3b", wdtype="fp8", batch=128, prompt=51
     print(_lib.stop_profile().format())
 
 
+def gla(tokens=8192, heads=16, batch=64, step=False, iters=4):
+    """Gated linear attention: one prompt in chunks, or one decoded token of every request."""
+    from ..models.config import GLASpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import gla as GLA
+
+    dev, D = "cuda", 128
+    rnd = lambda *s: (torch.randn(*s, device=dev) * 0.1).bfloat16()
+    w, _ = GLA.build(GLASpec(heads, D, D, 16.0), *(rnd(heads * D, 16) for _ in range(4)), rnd(16, 16), rnd(heads * D, 16), rnd(heads * D), rnd(D))
+    T = batch if step else tokens
+    proj, state = rnd(T, w.cols[-1] + 32), torch.zeros((batch + 1, heads, D, D), device=dev)
+    slots, cu = list(range(batch if step else 1)), list(range(batch + 1)) if step else [0, tokens]
+    fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=torch.zeros((1, 1), device=dev, dtype=torch.int32), kv_lens=None,
+                      cu_q=torch.tensor(cu, device=dev, dtype=torch.int32), cu_q_host=cu, is_decode=step,
+                      state_slots=torch.tensor(slots, device=dev, dtype=torch.int32), state_slots_host=slots)
+    for _ in range(iters):
+        GLA.mix(w, proj, fb, state, 1e-6)
+    torch.cuda.synchronize()
+
+
 CASES = {
+    "gla_prompt": gla,
+    "gla_step": lambda: gla(heads=32, step=True),
     "model_kernel_table_qwen3_moe_fp8": model_kernel_table,
     "gemm_qkv_post": gemm_qkv_post,
     "attn_decode_kv8": attn_decode_kv8,
