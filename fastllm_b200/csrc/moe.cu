@@ -1,8 +1,8 @@
 // Mixture-of-experts execution for sm_100a: routing plan, token gather, grouped expert GEMMs, weighted combine.
 //
 //   moe_plan     one CTA: per-local-expert token counts, segment offsets padded to 16 rows, and for every (token, k)
-//                pair its row in the expert-sorted buffer (-1 if the expert lives on another rank).  Up to 4096 pairs
-//                the rows inside a segment follow (token, k) order.
+//                pair its row in the expert-sorted buffer (-1 if the expert lives on another rank).  Deterministic:
+//                rows inside a segment follow (token, k) order.
 //   moe_gather   copies each routed token row into its sorted position
 //   grouped GEMM the swap-AB tcgen05 decode GEMM run once per (expert, 128/256-token chunk) through blockIdx.z; the
 //                weight tile coordinate is offset into the stacked expert matrix, the activation tile into the sorted
@@ -145,42 +145,63 @@ moe_plan_warp_kernel(const int* __restrict__ idx, int pairs, int first, int n_lo
   }
 }
 
-// Large problems: counts by shared-memory atomics, then rows handed out by atomics (rows inside an expert's segment come in no
-// particular order: every row's product stands alone).
+// Large problems, the same order: every warp owns a contiguous run of pairs.  It counts its experts chunk by chunk (`match.any`, the first
+// lane of an expert adds), a scan over the warps turns the counts into first rows, and a second walk hands the rows out.
+// Shared memory: [32 warps][n_local] counters.
 __global__ void __launch_bounds__(1024)
 moe_plan_large_kernel(const int* __restrict__ idx, int pairs, int first, int n_local, int* __restrict__ counts, int* __restrict__ offsets,
                       int* __restrict__ pos, int* __restrict__ total_rows, int pad) {
+  extern __shared__ int s_run[];
   __shared__ int s_cnt[1024];
-  __shared__ int s_off[1024];
   pdl_launch_dependents();
   pdl_wait();
-  for (int e = threadIdx.x; e < n_local; e += blockDim.x) s_cnt[e] = 0;
-  __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int e = idx[i] - first;
-    if (e >= 0 && e < n_local) atomicAdd(&s_cnt[e], 1);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const uint32_t lt_mask = (1u << lane) - 1u;
+  int* run = s_run + warp * n_local;
+  for (int e = lane; e < n_local; e += 32) run[e] = 0;
+  __syncwarp();
+  const int per = ((pairs + 1023) / 1024) * 32;                // pairs of a warp, whole chunks
+  const int i0 = warp * per, i1 = min(pairs, i0 + per);
+  auto expert = [&](int i) {
+    const int e = i < i1 ? idx[i] - first : -1;
+    return e >= 0 && e < n_local ? e : -1;
+  };
+  for (int c = i0; c < i1; c += 32) {
+    const int e = expert(c + lane);
+    const uint32_t same = __match_any_sync(0xffffffffu, e);
+    if (e >= 0 && (same & lt_mask) == 0) run[e] += __popc(same);
+    __syncwarp();
   }
   __syncthreads();
-  if (threadIdx.x < 32) {
+  for (int e = threadIdx.x; e < n_local; e += blockDim.x) {
+    int n = 0;
+    for (int w = 0; w < 32; ++w) { const int v = s_run[w * n_local + e]; s_run[w * n_local + e] = n; n += v; }
+    s_cnt[e] = n;
+  }
+  __syncthreads();
+  if (warp == 0) {
     int carry = 0;
     for (int base = 0; base < n_local; base += 32) {
-      const int e = base + threadIdx.x;
-      const int c = e < n_local ? (s_cnt[e] + pad - 1) / pad * pad : 0;
+      const int e = base + lane, n = e < n_local ? s_cnt[e] : 0, c = (n + pad - 1) / pad * pad;
       int incl = c;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const int v = __shfl_up_sync(0xffffffffu, incl, o);
-        if ((int)threadIdx.x >= o) incl += v;
+        if (lane >= o) incl += v;
       }
-      if (e < n_local) { counts[e] = s_cnt[e]; offsets[e] = s_off[e] = carry + incl - c; }
+      if (e < n_local) { counts[e] = n; offsets[e] = s_cnt[e] = carry + incl - c; }
       carry += __shfl_sync(0xffffffffu, incl, 31);
     }
-    if (threadIdx.x == 0) *total_rows = carry;
+    if (lane == 0) *total_rows = carry;
   }
   __syncthreads();
-  for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
-    const int e = idx[i] - first;
-    pos[i] = e >= 0 && e < n_local ? atomicAdd(&s_off[e], 1) : -1;
+  for (int c = i0; c < i1; c += 32) {
+    const int e = expert(c + lane);
+    const uint32_t same = __match_any_sync(0xffffffffu, e);
+    if (c + lane < i1) pos[c + lane] = e < 0 ? -1 : s_cnt[e] + run[e] + __popc(same & lt_mask);
+    __syncwarp();
+    if (e >= 0 && (same & lt_mask) == 0) run[e] += __popc(same);
+    __syncwarp();
   }
 }
 
@@ -342,7 +363,10 @@ extern "C" int fb_moe_plan(const int* idx, int T, int topk, int first, int n_loc
     launch_k(moe_plan_small_kernel, dim3(1), dim3(1024), 0, reinterpret_cast<cudaStream_t>(stream), 0, idx, T * topk, first, n_local, counts, offsets, pos, total_rows, pad);
     return (int)cudaGetLastError();
   }
-  launch_k(moe_plan_large_kernel, dim3(1), dim3(1024), 0, reinterpret_cast<cudaStream_t>(stream), 0, idx, T * topk, first, n_local, counts, offsets, pos, total_rows, pad);
+  const size_t smem = (size_t)32 * n_local * 4;
+  static DeviceOnce cfg;
+  if (cfg.need()) cudaFuncSetAttribute(moe_plan_large_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 32 * 1024 * 4);
+  launch_k(moe_plan_large_kernel, dim3(1), dim3(1024), smem, reinterpret_cast<cudaStream_t>(stream), 0, idx, T * topk, first, n_local, counts, offsets, pos, total_rows, pad);
   return (int)cudaGetLastError();
 }
 

@@ -318,8 +318,8 @@ def load_model(path: str | Path, device="cuda", dtype=None, wdtype: str = "auto"
         if tp is not None and tp.size > 1:
             raise NotImplementedError("cogvlm runs on one rank")
         m = CogVLMModel(cfg, device, dtype, tp, ep)
-    elif cfg.mixers is not None and tp is not None and tp.size > 1:
-        raise NotImplementedError(f"{cfg.model_type} runs on one rank")
+    elif cfg.mixers is not None and ((tp is not None and tp.size > 1) or (device_map and len(set(map(str, staged))) > 1)):
+        raise NotImplementedError(f"{cfg.model_type} runs on one rank and one device")
     else:
         m = DecoderModel(cfg, device, dtype, tp, ep)
     m.moe_disk = moe_device == "disk"

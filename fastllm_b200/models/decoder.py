@@ -294,7 +294,7 @@ class DecoderModel:
         if self.cfg.mixers is not None:
             shapes = [self.kv_cache_shape_layer(i, 1) for i in range(self.cfg.num_layers) if not self.cfg.layer_is_linear(i)]
             n = sum(math.prod(s[1:]) for pair in shapes if pair is not None for s in pair if s is not None)
-            return max(1, n * torch.finfo(self.dtype).bits // 8)
+            return n * torch.finfo(self.dtype).bits // 8 or 1 << 20      # (no paged layer at all: a nominal size)
         ks, vs = self.kv_cache_shape(1)
         n = math.prod(ks) + (math.prod(vs) if vs else 0)
         paged_layers = sum(1 for i in range(self.cfg.num_layers) if not self.cfg.layer_is_linear(i)) + (1 if self.mtp is not None else 0)

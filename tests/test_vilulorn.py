@@ -561,6 +561,29 @@ def test_greedy_generation(models, where):
     assert again == outs or dtype != torch.float32
 
 
+def test_speculative_generation_matches_greedy(models):
+    """Drafts by prompt lookup: rejected drafts leave the recurrent state as if they had never been read."""
+    path = models("mixed")[2]
+    m = load_model(path, device="cpu", dtype=torch.float32)
+    prompts, outs = [prompt("mixed", 9, 5) * 4, [7, 8, 9] * 10], []
+    for spec in ("", "ngram"):
+        eng = LLMEngine(m, EngineConfig(max_batch=2, max_context=256, speculative=spec), num_pages=8)
+        outs.append(eng.generate(prompts, GenerationConfig(max_new_tokens=12, ignore_eos=True)))
+    assert outs[0] == outs[1]
+
+
+def test_layers_without_pages(tmp_path):
+    """A stack of recurrent layers only: no page pools, the scheduler runs on state slots."""
+    cfg = config([(gla(2, 16, 16, 4.0), moe(2, 1, 16, 1.0)), (gla(1, 24, 8, 2.0), None)], width=64, vocab=64)
+    w = O.random_weights(cfg, seed=1)
+    m = load_model(save(tmp_path / "m", cfg, w), device="cpu", dtype=torch.float32)
+    eng = LLMEngine(m, EngineConfig(max_batch=2, max_context=256, max_tokens=512))
+    toks = list(range(20))
+    out = eng.generate([toks, toks[:3]], GenerationConfig(max_new_tokens=3, ignore_eos=True))
+    logits = O.forward(cfg, w, toks + out[0][:-1])[19:]
+    assert [x.argmax().item() for x in logits] == out[0]
+
+
 def test_context_ends_with_the_position_table(models):
     path = models("ones")[2]
     eng = LLMEngine(load_model(path, device="cpu", dtype=torch.float32), EngineConfig(max_batch=2, max_context=4096), num_pages=16)
