@@ -353,8 +353,8 @@ extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* 
   return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }
 
-// Grouped-query form over the cache pages: k_pool [num_slots, G, D], v_pool [num_slots, G, V], 128 slots a page; query head h uses
-// key / value head h / (H / G).  page_table: [requests, max_pages], a block's request is blocks[.][5].
+// Grouped-query form over the cache pages: k_pool [num_slots, G, D], v_pool [num_slots, G, V], 128 slots a page; H / G
+// consecutive query heads share a key / value head.  page_table: [requests, max_pages], a block's request is blocks[.][5].
 extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const void* k_pool, const void* v_pool, long long num_slots,
                                     const int* page_table, int max_pages, void* out, long long ld_out, const void* gate, long long ld_gate,
                                     const int* blocks, int n_blocks, int H, int G, int D, int V, int window, int chunk, float scale, int dtype,

@@ -1,6 +1,7 @@
-// Gated linear attention for sm_100a: per head a [D, V] fp32 state whose key channels decay at their own data-dependent rate,
-//     S_t = diag(alpha_t) S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t,   alpha_t = sigmoid(W_a2 a_t + b)^(1 / tau),
-// then RMS norm of every head's output and * silu(gate).  q, k, v, gate and a_t are columns of one merged projection row.
+// Gated linear attention for sm_100a: per head a [D, V] fp32 state S whose key channels d forget at their own data-dependent rate.  A token
+// with query q, key k, value v and decay logits z does
+//     S[d, :] <- f[d] S[d, :] + k[d] v,   f[d] = sigmoid(z[d])^(1 / tau),   out = sum_d q[d] S[d, :],
+// then comes the RMS norm of every head's output and * silu(gate).  z = W_a2 a + b comes from a low-rank row a.  q, k, v, gate and a_t are columns of one merged projection row.
 //
 //  * gla_recurrent_kernel: one CTA per (head, request) walks the request's tokens with the state in registers; a thread owns R rows of
 //    one state column, so the state is read once and written once per step.  Any widths, fp32 included.

@@ -154,7 +154,7 @@ class ModelConfig:
     residual_mult: float = 1.0
     pos_embed_base: float = 0.0            # > 0: sinusoidal positions with this base are added to the token embedding
     pos_table: int = 0                     # > 0: rows of a learned position table that is added to the token embedding
-    output_norms: bool = False             # fp32 residual: norms sit on the sub-layers' outputs only, sub-layers read the residual itself
+    output_norms: bool = False             # fp32 residual: what a sub-layer adds is normalised, what it reads is not
     # DeepNorm-style residual (MiniMax-Text-01 / M1): the block input is normalised first and the NORMALISED rows are the
     # residual: y = alpha * norm(x) + beta * f(norm(x)).  (alpha, beta) for full-attention layers, linear layers, MLPs.
     postnorm_residual: bool = False
@@ -643,7 +643,7 @@ def _listed(name: str, d: dict, mixers: list, ffs: list, runs: list) -> ModelCon
 
 def _vilulorn(d: dict) -> ModelConfig:
     """Vilulorn: gated linear attention layers and chunked grouped-query attention layers (which may read an earlier layer's keys and
-    values), experts picked by sigmoid scores that scale their inputs, norms on the sub-layers' outputs only, learned positions."""
+    values), experts picked by sigmoid scores that scale their inputs, normalised sub-layer outputs, learned positions."""
     L = d["layers"]
     mixers, ffs = [], []
     for i, spec in enumerate(L):

@@ -1,8 +1,8 @@
-"""Gated linear attention: a ``[dim, vdim]`` fp32 state per head and request whose key channels decay at their own data-dependent rate.
+"""Gated linear attention: a ``[dim, vdim]`` fp32 state S per head and request whose key channels d forget at their own data-dependent rate.
 
-    S_t = diag(alpha_t) S_(t-1) + k_t v_t^T ,   o_t = S_t^T q_t ,   alpha_t = sigmoid(W_a2 (W_a1 h) + b)^(1 / tau)
+    S[d, :] <- f[d] S[d, :] + k[d] v ,   f[d] = sigmoid(z[d])^(1 / tau) ,   out = sum_d q[d] S[d, :]
 
-followed by an RMS norm of every head's output and ``* silu(gate)``.  The states live in the engine's state slots.
+with decay logits z from a low-rank projection of the layer's input, followed by an RMS norm of every head's output and ``* silu(gate)``.  The states live in the engine's state slots.
 
 * decoded tokens, float32 models, widths outside the tiling: ``csrc/gla.cu::gla_recurrent_kernel`` walks a request's tokens with the
   state in registers -- decay, update, read-out, norm and gate in one launch;

@@ -169,7 +169,7 @@ class ExpertWeights:
         self.stacked = None     # filled by ops.moe_grouped when a grouped kernel can take the whole set
         self.act = "swiglu"     # "gptoss": clamped gate/up, gate * sigmoid(1.702 gate) * (up + 1); "swiglu_clamp": see limit
         self.limit = 0.0        # "swiglu_clamp" (Step-3.5): min(silu(gate), limit) * clamp(up, -limit, limit); "gptoss": its clamp (0: 7)
-        self.scale_input = False    # the router's weight multiplies the expert's input, not its output
+        self.scale_input = False    # an expert reads w * x (and its result is added as it is)
         self.host = False       # expert weights live in CPU memory and run on the native CPU backend (hybrid placement)
         self._host_arrays = None
 
@@ -217,8 +217,8 @@ def output_is_complete(ep) -> bool:
 
 
 def moe_forward(x, idx, wts, experts: ExpertWeights, ep=None):
-    """``y[t] = sum_k wts[t,k] * down_e(silu(gate_e x) * up_e x)`` over the experts this rank owns (``scale_input``: the weight
-    multiplies x instead).
+    """``y[t] = sum_k wts[t,k] * down_e(silu(gate_e x) * up_e x)`` over the experts this rank owns (``scale_input``: each
+    expert reads ``wts[t,k] * x`` and its result is added as it is).
 
     Tokens are grouped by expert; each non-empty local expert runs the two GEMMs on its token group.
     With expert parallelism the result is this rank's partial sum (the caller all-reduces it).

@@ -278,7 +278,26 @@ def gla(tokens=8192, heads=16, batch=64, step=False, iters=4):
     torch.cuda.synchronize()
 
 
+def grouped_decode(batch=32, length=4096, heads=32, kv=8, chunk=4096, iters=4):
+    """Chunked grouped-query attention of one decoded token per request."""
+    from ..models.config import AttnSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import grouped as GR
+
+    dev, D, pages = "cuda", 128, length // 128
+    rnd = lambda *s: (torch.randn(*s, device=dev) * 0.1).bfloat16()
+    w, _ = GR.build(AttnSpec(heads, kv, D, D, D ** -0.5, chunk), rnd(heads * D, 16), rnd(kv * D, 16), rnd(kv * D, 16), rnd(heads * D, 16), rnd(D), rnd(D))
+    pool = (rnd(batch * pages, 128, kv, D), rnd(batch * pages, 128, kv, D))
+    fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=torch.randperm(batch * pages, device=dev).int().view(batch, pages),
+                      kv_lens=torch.full((batch,), length, device=dev, dtype=torch.int32), cu_q=None, is_decode=True)
+    proj = rnd(batch, w.v_col + kv * D)
+    for _ in range(iters):
+        GR.attention(w, proj, pool, fb)
+    torch.cuda.synchronize()
+
+
 CASES = {
+    "grouped_decode": grouped_decode,
     "gla_prompt": gla,
     "gla_step": lambda: gla(heads=32, step=True),
     "model_kernel_table_qwen3_moe_fp8": model_kernel_table,

@@ -1,5 +1,5 @@
 """Vilulorn (gated linear attention, chunked grouped-query attention with shared keys and values, sigmoid-scored experts on scaled
-inputs, norms on the sub-layers' outputs, learned positions) against its plain statement.
+inputs, normalised sub-layer outputs, learned positions) against its plain statement.
 
 Every case builds a small random model of its own.  The CPU runs use the framework's PyTorch operator definitions (scheduling,
 cache, loading and the model itself); the GPU runs the kernels, in float32 and bfloat16.
@@ -130,7 +130,7 @@ def test_portions(models, sizes, where):
 @pytest.mark.parametrize("where", DEVICES)
 @pytest.mark.parametrize("name", ["mixed", "odd", "wide", "routed"])
 def test_unequal_requests_and_reused_slots(models, name, where):
-    """Up to four live requests: portions beside single tokens, requests that pause, pages and state slots used again by later ones."""
+    """Prompts of several requests next to decoded tokens of others, requests that pause, pages and state slots that change owner."""
     reqs = {"a": prompt(name, 210, 3), "b": prompt(name, 33, 4), "c": prompt(name, 129, 5), "d": prompt(name, 3, 6), "e": prompt(name, 180, 7),
             "f": prompt(name, 140, 8)}
     sched = [[("a", 100), ("b", 30), ("c", 2), ("d", 1)], [("b", 1), ("a", 1), ("d", 1)], [("c", 60), ("d", 1), ("b", 1), ("a", 1)], [("b", 1)],
