@@ -1,5 +1,6 @@
-// Paged grouped-query decode attention for sm_100a with any head widths up to 256 (multiples of 8), a chunk mask or a sliding window, and
-// an elementwise output gate.  Page length 128.
+// Paged grouped-query decode attention for sm_100a with any head widths up to 256 (multiples of 8), a chunk mask or a sliding window
+// (which may keep the first tokens of the sequence), soft-capped scores, a sink per head in the softmax, and an output gate (one per
+// element, or one per head).  Page length 128.
 //
 // As in attn_decode.cu (head width 128) a page of one key / value head is a full UMMA tile:
 //     S^T[128 keys x 16 heads] = K_page[128 x D] * Q^T        64-column tiles, K-major, SW128
@@ -7,7 +8,8 @@
 // Rows and heads come through 3-D maps bounded per head, so the tail of a 64-column tile is zero and a head may be narrower than a
 // tile.  Work items are the (row, page) pairs a query sees, times key / value heads, times groups of 16 query heads; CTAs stride over
 // them (as many per SM as the shared memory of a stage allows, so that one streams pages while another is in its softmax), write
-// un-normalised partial outputs with (max, sum), and a combine kernel merges a query's partials and applies o * sigmoid(gate).
+// un-normalised partial outputs with (max, sum), and a combine kernel merges a query's partials, adds the sink's term to the
+// denominator and applies o * sigmoid(gate).  Kept first tokens are pages of their own in the work list, before the window's.
 //
 // Every row is its own request (its own page-table row and length), so decoded tokens and short portions of prompts share a launch.
 // Page pools must hold finite values everywhere: unused keys of a page are multiplied by P = 0.
@@ -34,8 +36,10 @@ struct AttnGroupedParams {
   const int* kv_lens;
   float* part_o;          // [B, G, splits, H / G, V]
   float* part_ml;         // [B, G, splits, H / G, 2]
-  int B, H, G, D, V, dt, vt, splits, max_items, window, chunk;
+  int B, H, G, D, V, dt, vt, splits, max_items, window, chunk, keep;
   float scale_log2;
+  float cap_log2, cap_in;     // soft cap c: score = c tanh(scale s / c), in log2 units c log2(e); cap_in = 2 log2(e) scale / c (0: no cap)
+  const float* sinks;         // [H] or null
   uint32_t idesc_s, idesc_o;
 };
 
@@ -46,18 +50,31 @@ __device__ __forceinline__ int ag_first(int n, int window, int chunk) {
   return window > 0 && n > window ? n - window : 0;
 }
 
-// one CTA, B <= 1024: the pages between a row's first and last visible key
-__global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B, int window, int chunk, int* __restrict__ work,
+// pages of the kept first tokens (those before the page where the window starts), and the window's first page
+__device__ __forceinline__ int ag_kept_pages(int n, int window, int chunk, int keep, int& first_page) {
+  first_page = ag_first(n, window, chunk) / AG_PAGE;
+  const int kp = (keep + AG_PAGE - 1) / AG_PAGE;
+  return kp < first_page ? kp : first_page;
+}
+
+// c tanh(x): 1 - 2 / (1 + e^2x) is exact to an fp32 rounding of one, which is all that a score needs
+__device__ __forceinline__ float ag_score(const AttnGroupedParams& p, float s) {
+  if (p.cap_in == 0.f) return s * p.scale_log2;
+  return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(s * p.cap_in));
+}
+
+// one CTA, B <= 1024: the pages of the kept tokens and those between a row's first and last visible key
+__global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B, int window, int chunk, int keep, int* __restrict__ work,
                                          int* __restrict__ n_work, int max_items) {
   __shared__ int offs[1025];
   pdl_launch_dependents();
   pdl_wait();
   const int t = threadIdx.x;
-  int np = 0, first = 0;
+  int np = 0, first = 0, kept = 0;
   if (t < B) {
     const int n = kv_lens[t];
-    first = ag_first(n, window, chunk) / AG_PAGE;
-    np = n > 0 ? (n + AG_PAGE - 1) / AG_PAGE - first : 0;
+    kept = ag_kept_pages(n, window, chunk, keep, first);
+    np = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   }
   offs[t + 1] = np;
   if (t == 0) offs[0] = 0;
@@ -71,7 +88,7 @@ __global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B,
   if (t < B) {
     const int base = offs[t];
     for (int i = 0; i < np; ++i)
-      if (base + i < max_items) { work[2 * (base + i)] = t; work[2 * (base + i) + 1] = first + i; }
+      if (base + i < max_items) { work[2 * (base + i)] = t; work[2 * (base + i) + 1] = i < kept ? i : first + i - kept; }
   }
   if (t == 0) *n_work = min(offs[blockDim.x], max_items);
 }
@@ -85,7 +102,9 @@ __device__ __forceinline__ bool ag_item(const AttnGroupedParams& p, int w, int& 
   b = p.work[2 * item]; pg = p.work[2 * item + 1];
   bool ok = (unsigned)b < (unsigned)p.B && (unsigned)pg < (unsigned)p.max_pages;
   if (!ok) { b = 0; pg = 0; }
-  split = pg - ag_first(p.kv_lens[b], p.window, p.chunk) / AG_PAGE;
+  int first;
+  const int kept = ag_kept_pages(p.kv_lens[b], p.window, p.chunk, p.keep, first);
+  split = pg < kept ? pg : kept + pg - first;
   if ((unsigned)split >= (unsigned)p.splits) { split = 0; ok = false; }
   return ok;
 }
@@ -197,7 +216,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int n = p.kv_lens[b], nh = min(GP, HG - h0);
       const uint32_t ph = (uint32_t)it & 1u;
       const int key = pg * AG_PAGE + t;
-      const bool valid = key < n && key >= ag_first(n, p.window, p.chunk);
+      const bool valid = key < n && (key >= ag_first(n, p.window, p.chunk) || key < p.keep);
       mbar_wait(s_full, ph, dead, KID_ATTN_GROUPED, 7);
       tc_fence_after_sync();
       uint32_t r[16];
@@ -206,7 +225,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       float sv[GP];
 #pragma unroll
       for (int h = 0; h < GP; ++h) {
-        sv[h] = (valid && h < nh) ? __uint_as_float(r[h]) * p.scale_log2 : -INFINITY;
+        sv[h] = (valid && h < nh) ? ag_score(p, __uint_as_float(r[h])) : -INFINITY;
         float m = sv[h];
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
@@ -261,20 +280,25 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 1) tmem_dealloc(tmem_s, AG_TMEM_COLS);
 }
 
-// one CTA per (row, query head): merges the row's partials, eight at a time, and applies the gate
+// one CTA per (row, query head): merges the row's partials, eight at a time, then sink and gate
 template <bool BF16>
 __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGroupedParams p, uint16_t* __restrict__ out, long long ld_out,
-                                                                   const uint16_t* __restrict__ gate, long long ld_gate) {
+                                                                   const uint16_t* __restrict__ gate, long long ld_gate,
+                                                                   const float* __restrict__ head_gate, long long ld_head_gate) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y, HG = p.H / p.G, kvh = h / HG, g = h - kvh * HG;
   const int n = p.kv_lens[b];
-  int ns = n > 0 ? (n + AG_PAGE - 1) / AG_PAGE - ag_first(n, p.window, p.chunk) / AG_PAGE : 0;
+  int first;
+  const int kept = ag_kept_pages(n, p.window, p.chunk, p.keep, first);
+  int ns = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   if (ns > p.splits) {
     ns = p.splits;
     if (threadIdx.x == 0) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 22);
   }
   const size_t base = (size_t)(b * p.G + kvh) * p.splits;
+  const float sink = p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : -INFINITY;
+  const float hg = head_gate != nullptr ? 1.0f / (1.0f + __expf(-head_gate[(size_t)b * ld_head_gate + h])) : 1.0f;
   for (int d = threadIdx.x; d < p.V; d += 128) {
     float M = -INFINITY, L = 0.f, acc = 0.f;
     for (int s = 0; s < ns; s += 8) {
@@ -301,7 +325,12 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
         }
       }
     }
-    float o = L > 0.f ? acc / L : 0.f;
+    if (sink > -INFINITY && L > 0.f) {
+      const float nm = fmaxf(M, sink), a = exp2f(M - nm);
+      acc *= a;
+      L = L * a + exp2f(sink - nm);
+    }
+    float o = L > 0.f ? acc / L * hg : 0.f;
     if (gate != nullptr) {
       const uint16_t gb = gate[(size_t)b * ld_gate + (size_t)h * p.V + d];
       const float gv = BF16 ? __bfloat162float(__ushort_as_bfloat16(gb)) : __half2float(__ushort_as_half(gb));
@@ -316,23 +345,25 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
 using namespace fb;
 
 // work: [2 * max_items] ints, n_work: [1].
-extern "C" int fb_grouped_plan(const int* kv_lens, int B, int window, int chunk, int* work, int* n_work, int max_items, void* stream) {
-  if (B <= 0 || B > 1024 || max_items <= 0 || window < 0 || chunk < 0) return -1;
+extern "C" int fb_grouped_plan(const int* kv_lens, int B, int window, int chunk, int keep, int* work, int* n_work, int max_items, void* stream) {
+  if (B <= 0 || B > 1024 || max_items <= 0 || window < 0 || chunk < 0 || keep < 0) return -1;
   int threads = 32;
   while (threads < B) threads <<= 1;
-  launch_k(attn_grouped_plan_kernel, dim3(1), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), 0, kv_lens, B, window, chunk, work, n_work, max_items);
+  launch_k(attn_grouped_plan_kernel, dim3(1), dim3(threads), 0, reinterpret_cast<cudaStream_t>(stream), 0, kv_lens, B, window, chunk, keep, work, n_work, max_items);
   return (int)cudaGetLastError();
 }
 
+// keep: first tokens a window keeps; softcap 0: none; sinks [H], head_gate (row stride ld_head_gate, one logit per head): null for none.
 // q: [B, >= H * D] (row stride ld_q), k_pool [num_slots, G, D], v_pool [num_slots, G, V], out / gate [B, >= H * V]; 16-bit (dtype 0 = fp16,
 // 1 = bf16).  splits: most pages one query's keys touch; part_o [B * H * splits * V], part_ml [B * H * splits * 2] floats.
 extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_pool, const void* v_pool, void* out, long long ld_out,
                                  const void* gate, long long ld_gate, const int* page_table, const int* kv_lens, const int* work,
                                  const int* n_work, float* part_o, float* part_ml, int B, int H, int G, int D, int V, long long num_slots,
-                                 int max_pages, int splits, int max_items, int window, int chunk, float scale, int dtype, void* stream_) {
+                                 int max_pages, int splits, int max_items, int window, int chunk, int keep, float scale, float softcap,
+                                 const float* sinks, const float* head_gate, long long ld_head_gate, int dtype, void* stream_) {
   if (B <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || H > 65535 || D <= 0 || V <= 0 || D > 256 || V > 256 || D % 8 != 0 || V % 8 != 0 || num_slots < AG_PAGE ||
-      max_pages <= 0 || splits <= 0 || (dtype != 0 && dtype != 1))
+      max_pages <= 0 || splits <= 0 || keep < 0 || softcap < 0.f || (dtype != 0 && dtype != 1))
     return -1;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   static int sm_count = 0;
@@ -349,7 +380,9 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
   p.work = work; p.n_work = n_work; p.page_table = page_table; p.max_pages = max_pages; p.num_pages = (int)(num_slots / AG_PAGE);
   p.kv_lens = kv_lens; p.part_o = part_o; p.part_ml = part_ml;
   p.B = B; p.H = H; p.G = G; p.D = D; p.V = V; p.dt = (D + 63) / 64; p.vt = (V + 63) / 64; p.splits = splits; p.max_items = max_items;
-  p.window = window; p.chunk = chunk; p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = window; p.chunk = chunk; p.keep = keep; p.scale_log2 = scale * 1.4426950408889634f;
+  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
+  p.sinks = sinks;
   const uint32_t f = dtype == 1 ? 1u : 0u;
   p.idesc_s = make_idesc(f, f, 0, 0, 128, AG_N);
   p.idesc_o = make_idesc(f, f, 1, 0, 128, AG_N);
@@ -369,8 +402,8 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
 #undef FB_AG_GP
 #undef FB_AG
   if (dtype == 1)
-    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<true>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate);
+    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<true>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);
   else
-    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<false>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate);
+    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<false>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);
   return (int)cudaGetLastError();
 }

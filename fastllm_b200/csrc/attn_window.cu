@@ -1,4 +1,5 @@
-// Prefill attention with an optional sliding window or chunk mask, for sm_100a (tcgen05 + TMEM).
+// Prefill attention with an optional sliding window (which may keep the first tokens of the sequence) or chunk mask, soft-capped scores
+// and a sink per head in the softmax, for sm_100a (tcgen05 + TMEM).
 //
 // Keys and values are contiguous rows (the expanded latents of the keys a batch reads, one head per query head) or the cache pages
 // themselves (grouped-query attention: a step of 64 keys lies inside one 128-token page).  One CTA owns one head and up to 256
@@ -6,8 +7,9 @@
 // and their softmax runs on two warp groups, so the tensor core alternates between the blocks:
 //     S_b[128 q x 64 k] = Q_b * K^T        O_b[128 q x V] += P_b * V          b = 0, 1
 // A block takes part only in the steps its rows see (the causal frontier at one end, the window at the other).  Head widths are
-// any multiple of 8: the operand maps are bounded per head, so the tail of a 64-column tile is zero.  The epilogue normalises and
-// applies the elementwise output gate o * sigmoid(g) where the layer has one.
+// any multiple of 8: the operand maps are bounded per head, so the tail of a 64-column tile is zero.  Kept first tokens are steps of
+// their own ahead of the window's, shared by both blocks.  The epilogue normalises (with the sink's term) and applies the output gate
+// o * sigmoid(g), one per element or one per head, where the layer has one.
 #include "ptx.cuh"
 #include "launch.h"
 #include "tmap.h"
@@ -34,7 +36,11 @@ struct AttnWindowParams {
   int chunk;                                      // > 0 (instead of a window): a query sees the keys of its own chunk of positions
   int group;                                      // query heads per key / value head
   const int* page_table; int max_pages, num_pages;     // null: contiguous keys
+  int keep;                                       // pages only, beside a window: the first `keep` keys stay visible
   float scale_log2;
+  float cap_log2, cap_in;                         // soft cap c: c log2(e), 2 log2(e) scale / c (0: none)
+  const float* sinks;                             // [heads] or null
+  const float* head_gate; long long ld_head_gate;      // one logit per (row, head)
   uint32_t idesc_s, idesc_o;
 };
 
@@ -44,7 +50,12 @@ __device__ __forceinline__ int aw_first(const AttnWindowParams& p, int pos) {
   return p.window > 0 ? pos - p.window + 1 : 0;
 }
 
-template <bool BF16>
+// c tanh(x): 1 - 2 / (1 + e^2x) is exact to an fp32 rounding of one, which is all that a score needs
+__device__ __forceinline__ float aw_capped(const AttnWindowParams& p, float s) {
+  return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(s * p.cap_in));
+}
+
+template <bool BF16, bool CAP>
 __global__ void __launch_bounds__(320, 1)
 attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const AttnWindowParams p) {
@@ -73,17 +84,23 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   int lo = max(key0, aw_first(p, pos0));
   if (p.page_table != nullptr) lo &= ~(AW_KV - 1);          // a step never straddles two pages; the mask drops what lies before
   const int hi = pos0 + rows;
-  const int n_steps = (hi - lo + AW_KV - 1) / AW_KV;
-  // steps [f, e) of query block b
-  int f[2], e[2];
-  f[0] = 0;
-  e[0] = (pos0 + (rows < 128 ? rows : 128) - lo + AW_KV - 1) / AW_KV;
+  const int kept = p.keep > 0 ? min((p.keep + AW_KV - 1) / AW_KV, lo / AW_KV) : 0;      // steps of kept tokens before the window's
+  const int n_steps = kept + (hi - lo + AW_KV - 1) / AW_KV;
+  auto step_key = [&](int it) { return it < kept ? it * AW_KV : lo + (it - kept) * AW_KV; };
+  // query block b takes part in steps [0, kb) and [f, e); its n-th step is nth(b, n)
+  int f[2], e[2], kb[2];
+  kb[0] = f[0] = kept;
+  e[0] = kept + (pos0 + (rows < 128 ? rows : 128) - lo + AW_KV - 1) / AW_KV;
   if (rows > 128) {
-    f[1] = (max(lo, aw_first(p, pos0 + 128)) - lo) / AW_KV;
+    kb[1] = kept;
+    f[1] = kept + (p.keep > lo ? 0 : (max(lo, aw_first(p, pos0 + 128)) - lo) / AW_KV);
     e[1] = n_steps;
   } else {
+    kb[1] = 0;
     f[1] = e[1] = n_steps;
   }
+  auto takes = [&](int b, int it) { return it < kb[b] || (it >= f[b] && it < e[b]); };
+  auto order = [&](int b, int it) { return it < kb[b] ? it : kb[b] + it - f[b]; };
   bool dead = false;
 
   if (threadIdx.x == 0) {
@@ -111,17 +128,17 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const int s = it % stages;
         const uint32_t ph = (uint32_t)(it / stages) & 1u;
         if (!mbar_wait(&empty[s], ph ^ 1u, dead, KID_ATTN_WINDOW, 1)) break;
-        int row = key_row0 + (lo - key0) + it * AW_KV;
+        const int key = step_key(it);
+        int row = key_row0 + (key - key0);
         if (p.page_table != nullptr) {
-          const int key = lo + it * AW_KV;
           int page = (key >> 7) < p.max_pages ? p.page_table[(size_t)blk[5] * p.max_pages + (key >> 7)] : 0;
           if ((unsigned)page >= (unsigned)p.num_pages) { report_error(ERR_BAD_ARG, KID_ATTN_WINDOW, 20); page = 0; }
           row = page * 128 + (key & 127);
         }
-        uint8_t* kb = kv_smem + s * stage_bytes;
-        uint8_t* vb = kb + dt * AW_KT;
+        uint8_t* ks = kv_smem + s * stage_bytes;
+        uint8_t* vb = ks + dt * AW_KT;
         mbar_expect_tx(&full_k[s], dt * AW_KT);
-        for (int j = 0; j < dt; ++j) tma_load_3d(kb + j * AW_KT, &tmK, &full_k[s], j * 64, kv_head, row);
+        for (int j = 0; j < dt; ++j) tma_load_3d(ks + j * AW_KT, &tmK, &full_k[s], j * 64, kv_head, row);
         mbar_expect_tx(&full_v[s], vt * AW_KT);
         for (int j = 0; j < vt; ++j) tma_load_3d(vb + j * AW_KT, &tmV, &full_v[s], j * 64, kv_head, row);
       }
@@ -144,7 +161,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       if (ok) {
         tc_fence_after_sync();
         for (int b = 0; b < 2; ++b)
-          if (f[b] == 0 && e[b] > 0) issue_s(b, smem_u32(kv_smem));
+          if (takes(b, 0)) issue_s(b, smem_u32(kv_smem));
       }
       for (int it = 0; ok && it < n_steps; ++it) {
         const int s = it % stages, s1 = (it + 1) % stages;
@@ -153,8 +170,8 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         const uint32_t kb1 = smem_u32(kv_smem + s1 * stage_bytes);
         bool have_v = false, have_k1 = false;
         for (int b = 0; b < 2; ++b) {
-          if (it >= f[b] && it < e[b]) {
-            if (!mbar_wait(&p_ready[b], (uint32_t)(it - f[b]) & 1u, dead, KID_ATTN_WINDOW, 4)) { ok = false; break; }
+          if (takes(b, it)) {
+            if (!mbar_wait(&p_ready[b], (uint32_t)order(b, it) & 1u, dead, KID_ATTN_WINDOW, 4)) { ok = false; break; }
             if (!have_v && !mbar_wait(&full_v[s], ph, dead, KID_ATTN_WINDOW, 5)) { ok = false; break; }
             have_v = true;
             tc_fence_after_sync();
@@ -163,11 +180,11 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             for (int k = 0; k < 4; ++k) {
               const uint64_t da = make_smem_desc(pb + b * AW_PT + k * 32, 16, 1024, SWZ_128B);
               const uint64_t db = make_smem_desc(vb + k * 2048, AW_KT, 1024, SWZ_128B);
-              umma_f16(tmem0 + 128u + (uint32_t)b * o_cols, da, db, p.idesc_o, (it != f[b] || k != 0) ? 1u : 0u);
+              umma_f16(tmem0 + 128u + (uint32_t)b * o_cols, da, db, p.idesc_o, (order(b, it) != 0 || k != 0) ? 1u : 0u);
             }
             umma_commit(&o_full[b]);
           }
-          if (it + 1 >= f[b] && it + 1 < e[b]) {
+          if (takes(b, it + 1)) {
             if (!have_k1 && !mbar_wait(&full_k[s1], ph1, dead, KID_ATTN_WINDOW, 6)) { ok = false; break; }
             have_k1 = true;
             tc_fence_after_sync();
@@ -191,24 +208,29 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const uint32_t tmem_s = tmem0 + (uint32_t)(b * 64), tmem_o = tmem0 + 128u + (uint32_t)b * o_cols;
     uint8_t* prow = p_smem + b * AW_PT + r * 128;
-    const int it0 = f[b], it1 = e[b];
+    const int cnt = kb[b] + e[b] - f[b];
     float m_run = -INFINITY, l_run = 0.f;
-    for (int it = it0; it < it1; ++it) {
-      const uint32_t iph = (uint32_t)(it - it0) & 1u;
+    for (int n = 0; n < cnt; ++n) {
+      const uint32_t iph = (uint32_t)n & 1u;
       mbar_wait(&s_full[b], iph, dead, KID_ATTN_WINDOW, 8);
       tc_fence_after_sync();
-      const int kv0 = lo + it * AW_KV;
+      const int kv0 = step_key(n < kb[b] ? n : f[b] + n - kb[b]);
       uint32_t sreg[64];
       tmem_ld_32x32b_x32(tmem_s + lane_off, sreg);
       tmem_ld_32x32b_x32(tmem_s + lane_off + 32, sreg + 32);
       tmem_ld_wait();
       // only steps on the causal diagonal or on the window's edge pay for the mask
-      const bool full_step = kv0 + AW_KV - 1 <= pos_b && kv0 >= first_all;
+      const bool full_step = kv0 + AW_KV - 1 <= pos_b && (kv0 >= first_all || kv0 + AW_KV <= p.keep);
       float m_new = m_run;
+      if (CAP) {
+#pragma unroll
+        for (int j = 0; j < 64; ++j) sreg[j] = __float_as_uint(aw_capped(p, __uint_as_float(sreg[j])));
+      }
+      const float sc = CAP ? 1.f : p.scale_log2;
       if (full_step) {
 #pragma unroll
         for (int j = 0; j < 64; ++j) {
-          const float sv = __uint_as_float(sreg[j]) * p.scale_log2;
+          const float sv = __uint_as_float(sreg[j]) * sc;
           sreg[j] = __float_as_uint(sv);
           m_new = fmaxf(m_new, sv);
         }
@@ -216,14 +238,14 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
         for (int j = 0; j < 64; ++j) {
           const int kv = kv0 + j;
-          const float sv = (kv <= pos && kv >= first) ? __uint_as_float(sreg[j]) * p.scale_log2 : -INFINITY;
+          const float sv = (kv <= pos && (kv >= first || kv < p.keep)) ? __uint_as_float(sreg[j]) * sc : -INFINITY;
           sreg[j] = __float_as_uint(sv);
           m_new = fmaxf(m_new, sv);
         }
       }
       const float m_use = m_new == -INFINITY ? 0.f : m_new;
       const float alpha = exp2f(m_run - m_use);
-      if (it > it0) {
+      if (n > 0) {
         // the previous P * V of this block must be complete before P is overwritten or O is rescaled
         mbar_wait(&o_full[b], iph ^ 1u, dead, KID_ATTN_WINDOW, 9);
         tc_fence_after_sync();
@@ -259,12 +281,17 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       tc_fence_before_sync();
       mbar_arrive(&p_ready[b]);
     }
-    if (it1 > it0) {
-      mbar_wait(&o_full[b], (uint32_t)(it1 - it0 - 1) & 1u, dead, KID_ATTN_WINDOW, 10);
+    if (cnt > 0) {
+      mbar_wait(&o_full[b], (uint32_t)(cnt - 1) & 1u, dead, KID_ATTN_WINDOW, 10);
       tc_fence_after_sync();
-      const float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const bool live = b * 128 + r < rows;
       const size_t row = (size_t)(q_row0 + b * 128 + r);
+      if (p.sinks != nullptr && l_run > 0.f) {
+        const float sink = p.sinks[head] * 1.4426950408889634f, mx = fmaxf(m_run, sink), fac = exp2f(m_run - mx);
+        inv_l = fac / (l_run * fac + exp2f(sink - mx));
+      }
+      if (p.head_gate != nullptr && live) inv_l *= 1.0f / (1.0f + __expf(-p.head_gate[row * p.ld_head_gate + head]));
       uint16_t* orow = p.out + row * p.ld_out + (size_t)head * p.V;
       const uint16_t* grow = p.gate != nullptr ? p.gate + row * p.ld_gate + (size_t)head * p.V : nullptr;
 #pragma unroll 1
@@ -323,15 +350,15 @@ static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const C
   p.idesc_o = make_idesc(fm, fm, 0, 1, 128, p.vt * 64);
   const int smem = 2 * p.dt * AW_QT + p.stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
   const dim3 grid(H, n_blocks);
-  if (dtype == 1) {
-    static DeviceOnce cfg;
-    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);
-    attn_window_kernel<true><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);
-  } else {
-    static DeviceOnce cfg;
-    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);
-    attn_window_kernel<false><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);
+#define FB_AW(BF, CAP)                                                                                                              \
+  {                                                                                                                                  \
+    static DeviceOnce cfg;                                                                                                           \
+    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<BF, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);      \
+    attn_window_kernel<BF, CAP><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);                                                      \
   }
+  if (p.cap_in != 0.f) { if (dtype == 1) FB_AW(true, true) else FB_AW(false, true) }
+  else { if (dtype == 1) FB_AW(true, false) else FB_AW(false, false) }
+#undef FB_AW
   return (int)cudaGetLastError();
 }
 
@@ -354,14 +381,14 @@ extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* 
 }
 
 // Grouped-query form over the cache pages: k_pool [num_slots, G, D], v_pool [num_slots, G, V], 128 slots a page; H / G
-// consecutive query heads share a key / value head.  page_table: [requests, max_pages], a block's request is blocks[.][5].
+// consecutive query heads share a key / value head; keep, softcap, sinks, head_gate as in fb_grouped_decode.  page_table: [requests, max_pages], a block's request is blocks[.][5].
 extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const void* k_pool, const void* v_pool, long long num_slots,
                                     const int* page_table, int max_pages, void* out, long long ld_out, const void* gate, long long ld_gate,
-                                    const int* blocks, int n_blocks, int H, int G, int D, int V, int window, int chunk, float scale, int dtype,
-                                    void* stream_) {
+                                    const int* blocks, int n_blocks, int H, int G, int D, int V, int window, int chunk, int keep, float scale,
+                                    float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, int dtype, void* stream_) {
   if (n_blocks <= 0) return 0;
   if (window_stages(D, V) == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || num_slots < 128 || H <= 0 || G <= 0 || H % G != 0 || n_blocks > 65535 ||
-      window < 0 || chunk < 0 || max_pages <= 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
+      window < 0 || chunk < 0 || keep < 0 || softcap < 0.f || max_pages <= 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
     return -1;
   CUtensorMap tmQ, tmK, tmV;
   if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
@@ -371,5 +398,7 @@ extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const 
   p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
   p.D = D; p.V = V; p.window = window; p.chunk = chunk; p.group = H / G;
   p.page_table = page_table; p.max_pages = max_pages; p.num_pages = (int)(num_slots / 128);
+  p.keep = window > 0 ? keep : 0; p.sinks = sinks; p.head_gate = head_gate; p.ld_head_gate = ld_head_gate;
+  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
   return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }

@@ -635,13 +635,14 @@ struct RouteParams {
   const float* logits; const float* bias; int* out_idx; float* out_w;
   int M, E, topk, score_mode /*0 softmax 1 sigmoid 2 none*/, renorm, n_group, topk_group;
   float route_scale;
+  int ld, group_max;         // row stride of the logits; a group's score is its largest score instead of the sum of its two largest
 };
 __global__ void route_topk_kernel(const RouteParams p) {
   pdl_launch_dependents();
   pdl_wait();
   const int gw = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
   if (gw >= p.M) return;
-  const float* lg = p.logits + (size_t)gw * p.E;
+  const float* lg = p.logits + (size_t)gw * p.ld;
   float sc[16], sel[16];
   const int per = (p.E + 31) >> 5;
   float mx = -INFINITY;
@@ -660,7 +661,7 @@ __global__ void route_topk_kernel(const RouteParams p) {
     sel[s] = e < p.E ? sc[s] + (p.bias ? p.bias[e] : 0.f) : -INFINITY;
   }
   if (p.n_group > 1 && p.topk_group < p.n_group) {
-    // group g = e / (E / n_group); score(g) = sum of top-2 biased scores in the group
+    // group g = e / (E / n_group); score(g) = sum of the top-2 biased scores in the group, or the largest one
     const int gs = p.E / p.n_group;
     float gscore[32];
     for (int g = 0; g < p.n_group; ++g) {
@@ -677,7 +678,7 @@ __global__ void route_topk_kernel(const RouteParams p) {
         const float n2 = fmaxf(fminf(m1, o1), fmaxf(m2, o2));
         m1 = n1; m2 = n2;
       }
-      gscore[g] = m1 + m2;
+      gscore[g] = p.group_max ? m1 : m1 + m2;
     }
     // keep the topk_group best groups (ties to the lower index)
     unsigned keep = 0;
@@ -887,10 +888,10 @@ extern "C" int fb_argmax(const void* logits, int* ids, float* vals, int M, int V
 }
 
 extern "C" int fb_route_topk(const float* logits, const float* bias, int* out_idx, float* out_w, int M, int E, int topk,
-                             int score_mode, int renorm, int n_group, int topk_group, float route_scale, void* stream) {
+                             int score_mode, int renorm, int n_group, int topk_group, float route_scale, int ld, int group_max, void* stream) {
   if (M <= 0) return 0;
-  if (E > 512 || topk > 32 || n_group > 32 || (n_group > 1 && E % n_group != 0)) return -1;
-  RouteParams p{logits, bias, out_idx, out_w, M, E, topk, score_mode, renorm, n_group, topk_group, route_scale};
+  if (ld < E || topk > E || E > 512 || topk > 32 || n_group > 32 || (n_group > 1 && E % n_group != 0)) return -1;
+  RouteParams p{logits, bias, out_idx, out_w, M, E, topk, score_mode, renorm, n_group, topk_group, route_scale, ld, group_max};
   const int wpb = 4;
   launch_k(route_topk_kernel, dim3((M + wpb - 1) / wpb), dim3(wpb * 32), 0, reinterpret_cast<cudaStream_t>(stream), 0, p);
   return (int)cudaGetLastError();

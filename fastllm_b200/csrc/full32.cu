@@ -26,8 +26,18 @@ struct Full32Params {
   long long batch_w_rows, batch_x_cols, batch_out_cols;
   const int* counts; const int* offsets;
   float alpha;
-  int relu2, out_f32;
+  int act, out_f32;                        // act: 0 none, 1 relu^2, 2 gelu (erf), 3 gelu (tanh form)
+  // factors of the activated product: sigmoid of one fp32 logit per row; row mul_rows[m] of a table
+  const float* row_gate; long long ld_row_gate;
+  const void* mul; const int* mul_rows; long long ld_mul; int mul_count;
 };
+
+__device__ __forceinline__ float act32(float v, int act) {
+  if (act == 1) { v = fmaxf(v, 0.f); return v * v; }
+  if (act == 2) return 0.5f * v * (1.0f + erff(v * 0.70710678118654752f));
+  if (act == 3) return 0.5f * v * (1.0f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
+  return v;
+}
 
 template <int DT>
 __global__ void __launch_bounds__(256) gemm_full32_kernel(const Full32Params p) {
@@ -79,7 +89,9 @@ __global__ void __launch_bounds__(256) gemm_full32_kernel(const Full32Params p) 
         float v = acc[i][j];
         const long long c = z * p.batch_out_cols + n;
         if (p.bias != nullptr) v += F32In<DT>::ld(reinterpret_cast<const T*>(p.bias)[n]);
-        if (p.relu2) { v = fmaxf(v, 0.f); v *= v; }
+        v = act32(v, p.act);
+        if (p.row_gate != nullptr) v *= 1.0f / (1.0f + expf(-p.row_gate[(row0 + m) * p.ld_row_gate]));
+        if (p.mul != nullptr) v *= F32In<DT>::ld(reinterpret_cast<const T*>(p.mul)[min(max(p.mul_rows[row0 + m], 0), p.mul_count - 1) * p.ld_mul + n]);
         if (p.gate != nullptr) v *= 1.0f / (1.0f + expf(-F32In<DT>::ld(reinterpret_cast<const T*>(p.gate)[(row0 + m) * p.ld_gate + c])));
         if (p.residual != nullptr) v = p.residual[(row0 + m) * p.ld_res + c] + p.alpha * v;
         if (p.out_f32) reinterpret_cast<float*>(p.out)[(row0 + m) * p.ld_out + c] = v;
@@ -148,15 +160,18 @@ __global__ void __launch_bounds__(128) latent_attn32_kernel(const typename F32In
 }
 
 // Grouped-query attention of one (row, query head) per CTA over paged keys and values, any widths, fp32 arithmetic:
-//   out = (sum_j softmax(scale q . k_j) v_j) * sigmoid(gate),  first(position) <= j <= position
-// Row t sees the keys of its own page-table row; its position is kv_lens[t] - 1.  chunk: first = position - position % chunk; window:
-// first = position - window + 1; neither: 0.
+//   out = (sum_j softmax(score_j) v_j) * sigmoid(gate),  score_j = scale q . k_j, soft-capped where the layer does
+// Row t sees the keys of its own page-table row; its position is kv_lens[t] - 1.  The first key: chunk: position - position % chunk;
+// window: position - window + 1, beside the first `keep` of the sequence; neither: 0.  sinks: one more term exp(sink) per head in the
+// denominator.  The gate is elementwise (`gate`, 16-bit or fp32) or one fp32 logit per head (`head_gate`).
 struct Grouped32Params {
   const void* q; const void* k_pool; const void* v_pool; void* out; const void* gate;
   long long ld_q, ld_out, ld_gate;
   const int* page_table; const int* kv_lens;
-  int H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk;
-  float scale;
+  int H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, keep;
+  float scale, softcap;
+  const float* sinks;
+  const float* head_gate; long long ld_head_gate;
 };
 
 template <int DT>
@@ -179,11 +194,12 @@ __global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Para
   for (int i = tid; i < p.Dp; i += 128) qs[i] = F32In<DT>::ld(qp[i]);
   for (int i = tid; i < p.Vp; i += 128) os[i] = 0.f;
   float m_run = -INFINITY, l_run = 0.f;
-  for (int j0 = first; j0 < n; j0 += L32_KEYS) {
-    const int cnt = n - j0 < L32_KEYS ? n - j0 : L32_KEYS;
+  const int kept = p.keep < first ? p.keep : first, keys = kept + n - first;       // keys 0 .. kept - 1 and first .. n - 1
+  for (int j0 = 0; j0 < keys; j0 += L32_KEYS) {
+    const int cnt = keys - j0 < L32_KEYS ? keys - j0 : L32_KEYS;
     __syncthreads();
     if (tid < cnt) {
-      const int j = j0 + tid, pg = j / p.page_len;
+      const int i = j0 + tid, j = i < kept ? i : first + i - kept, pg = j / p.page_len;
       int page = pg < p.max_pages ? p.page_table[(size_t)t * p.max_pages + pg] : 0;
       if ((unsigned)page >= (unsigned)p.num_pages) page = 0;
       rows[tid] = page * p.page_len + (j - pg * p.page_len);
@@ -195,7 +211,9 @@ __global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Para
       for (int i = lane; i < p.D; i += 32) s = fmaf(qs[i], F32In<DT>::ld(c[i]), s);
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-      if (lane == 0) sc[j] = s * p.scale;
+      s *= p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      if (lane == 0) sc[j] = s;
     }
     __syncthreads();
     float mx = m_run;
@@ -214,7 +232,12 @@ __global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Para
       os[i] = a;
     }
   }
-  const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  if (p.sinks != nullptr && l_run > 0.f) {
+    const float sink = p.sinks[h], mx = fmaxf(m_run, sink), fac = expf(m_run - mx);
+    inv = fac / (l_run * fac + expf(sink - mx));
+  }
+  if (p.head_gate != nullptr) inv *= 1.0f / (1.0f + expf(-p.head_gate[(size_t)t * p.ld_head_gate + h]));
   T* op = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.Vp;
   const T* gp = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + (size_t)h * p.Vp : nullptr;
   for (int i = tid; i < p.Vp; i += 128) {
@@ -233,11 +256,12 @@ using namespace fb;
 extern "C" int fb_gemm_full32(const void* X, const void* W, void* out, const void* bias, const float* residual, const void* gate, int M,
                               int N, int K, int batch, long long ldx, long long ldw, long long ld_out, long long ld_res, long long ld_gate,
                               long long batch_w_rows, long long batch_x_cols, long long batch_out_cols, const int* counts,
-                              const int* offsets, float alpha, int relu2, int out_f32, int dt, void* stream) {
+                              const int* offsets, float alpha, int act, int out_f32, const float* row_gate, long long ld_row_gate,
+                              const void* mul, const int* mul_rows, long long ld_mul, int mul_count, int dt, void* stream) {
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
-  if (K <= 0 || dt < 0 || dt > 2 || batch > 65535) return -1;
+  if (K <= 0 || dt < 0 || dt > 2 || batch > 65535 || act < 0 || act > 3 || (mul != nullptr && (mul_rows == nullptr || mul_count <= 0))) return -1;
   Full32Params p{X, W, out, residual, gate, bias, M, N, K, ldx, ldw, ld_out, ld_res, ld_gate, batch_w_rows, batch_x_cols, batch_out_cols,
-                 counts, offsets, alpha, relu2, out_f32};
+                 counts, offsets, alpha, act, out_f32, row_gate, ld_row_gate, mul, mul_rows, ld_mul, mul_count};
   int gy = (M + 63) / 64;
   if (counts != nullptr && gy > 8) gy = 8;            // an expert rarely gets more; the kernel strides over the rest
   if (gy > 65535) gy = 65535;
@@ -272,13 +296,13 @@ extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, cons
 // See Grouped32Params; q / out / gate: T rows, pools [num_pages * page_len, G, Dp / Vp].
 extern "C" int fb_grouped_attn32(const void* q, long long ld_q, const void* k_pool, const void* v_pool, void* out, long long ld_out,
                                  const void* gate, long long ld_gate, const int* page_table, const int* kv_lens, int T, int H, int G, int D,
-                                 int Dp, int Vp, int max_pages, int num_pages, int page_len, int window, int chunk, float scale, int dt,
-                                 void* stream) {
+                                 int Dp, int Vp, int max_pages, int num_pages, int page_len, int window, int chunk, int keep, float scale,
+                                 float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, int dt, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || H > 65535 || D <= 0 || Dp < D || Vp <= 0 || Dp + Vp > 49152 || max_pages <= 0 || num_pages <= 0 ||
-      page_len <= 0 || window < 0 || chunk < 0 || dt < 0 || dt > 2)
+      page_len <= 0 || window < 0 || chunk < 0 || keep < 0 || dt < 0 || dt > 2)
     return -1;
-  Grouped32Params p{q, k_pool, v_pool, out, gate, ld_q, ld_out, ld_gate, page_table, kv_lens, H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, scale};
+  Grouped32Params p{q, k_pool, v_pool, out, gate, ld_q, ld_out, ld_gate, page_table, kv_lens, H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, keep, scale, softcap, sinks, head_gate, ld_head_gate};
   const size_t smem = (size_t)(Dp + Vp) * 4;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define GO(DT)                                                                                                          \

@@ -299,9 +299,15 @@ extern "C" int fb_gemm_route(const void* X, const void* W, int M, int E, int K, 
 #undef FB_RT
 }
 
+struct GemmExtras {                  // operands of the less common epilogues (see GemmParams)
+  const float* row_gate = nullptr; int ld_row_gate = 0;
+  const void* mul = nullptr; const int* mul_rows = nullptr; long long ld_mul = 0; int mul_count = 0;
+  void* out16 = nullptr; int ld_out16 = 0;
+};
+
 static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
                                   int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit,
-                                  const void* wait_cnt, const void* wait_expect, float alpha, void* stream_) {
+                                  const void* wait_cnt, const void* wait_expect, float alpha, void* stream_, const GemmExtras& ex = GemmExtras()) {
   using namespace fb;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0) return 0;
@@ -313,6 +319,8 @@ static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* 
   p.kb_total = (K + 63) / 64;             // a last partial block: both operand maps end at column K, TMA fills the rest with zeros
   p.alpha = alpha;
   p.flags = flags;
+  p.row_gate = ex.row_gate; p.ld_row_gate = ex.ld_row_gate; p.mul = ex.mul; p.mul_rows = ex.mul_rows; p.ld_mul = ex.ld_mul; p.mul_count = ex.mul_count;
+  p.out16 = ex.out16; p.ld_out16 = ex.ld_out16;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
   p.wait_cnt = reinterpret_cast<const uint32_t*>(wait_cnt);
@@ -393,12 +401,28 @@ extern "C" int fb_gemm_16bit(const void* X, const void* W, void* out, const void
   return gemm_16bit_impl(X, W, out, bias, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype, flags, nsplit, nullptr, nullptr, 1.f, stream_);
 }
 
-// Models with an fp32 residual stream: out_f32 = residual_f32 + alpha * (X W^T); `out` may be `residual`.
+// Models with an fp32 residual stream: out_f32 = residual_f32 + alpha * (X W^T); `out` may be `residual`.  out16 (or null): a 16-bit copy
+// of the new residual, for a projection that reads it next.
 extern "C" int fb_gemm_16bit_res32(const void* X, const void* W, float* out, const float* residual, int M, int N, int K, int ldx,
-                                   int ldw, int ld_out, int ld_res, float alpha, int dtype, void* stream_) {
+                                   int ldw, int ld_out, int ld_res, float alpha, void* out16, int ld_out16, int dtype, void* stream_) {
   using namespace fb;
+  if (out16 != nullptr && ((ld_out16 % 8) || (reinterpret_cast<uintptr_t>(out16) & 15))) return -1;
+  GemmExtras ex;
+  ex.out16 = out16; ex.ld_out16 = ld_out16;
   return gemm_16bit_impl(X, W, out, nullptr, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype,
-                         GEMM_RESIDUAL | GEMM_RES_F32 | GEMM_OUT_F32, 0, nullptr, nullptr, alpha, stream_);
+                         GEMM_RESIDUAL | GEMM_RES_F32 | GEMM_OUT_F32, 0, nullptr, nullptr, alpha, stream_, ex);
+}
+
+// out = act(X W^T) * sigmoid(row_gate[m])  or  act(X W^T) * mul[mul_rows[m], :]  (either factor may be absent); flags: one GEMM_GELU* form.
+extern "C" int fb_gemm_16bit_act(const void* X, const void* W, void* out, int M, int N, int K, int ldx, int ldw, int ld_out, int flags,
+                                 const float* row_gate, int ld_row_gate, const void* mul, const int* mul_rows, long long ld_mul, int mul_count,
+                                 int dtype, void* stream_) {
+  using namespace fb;
+  if ((flags & ~(GEMM_GELU | GEMM_GELU_TANH)) || (mul != nullptr && (mul_rows == nullptr || mul_count <= 0 || (ld_mul % 8) || (reinterpret_cast<uintptr_t>(mul) & 15)))) return -1;
+  GemmExtras ex;
+  ex.row_gate = row_gate; ex.ld_row_gate = ld_row_gate; ex.mul = mul; ex.mul_rows = mul_rows; ex.ld_mul = ld_mul;
+  ex.mul_count = mul_count;
+  return gemm_16bit_impl(X, W, out, nullptr, nullptr, M, N, K, ldx, ldw, ld_out, 0, dtype, flags, 0, nullptr, nullptr, 1.f, stream_, ex);
 }
 
 // QKV projection (head_dim 128, M <= 256, N = (Hq + 2 Hkv) * 128) with split / per-head RMSNorm / RoPE / paged-cache append in

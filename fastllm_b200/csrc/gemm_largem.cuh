@@ -49,6 +49,29 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = relu2_f(v[j]);
         }
+        if (p.flags & GEMM_GELU) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = gelu_erf_f(v[j]);
+        }
+        if (p.flags & GEMM_GELU_TANH) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_f(v[j]);
+        }
+        if (p.row_gate != nullptr) {
+          const float g = sigmoid_f(p.row_gate[(size_t)m * p.ld_row_gate]);
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] *= g;
+        }
+        if (p.mul != nullptr) {
+          const uint4* mp = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.mul) + (size_t)clamp_row(p.mul_rows[m], p.mul_count) * p.ld_mul + n0);
+#pragma unroll
+          for (int g = 0; g < 4; ++g) {
+            const uint4 mv = mp[g];
+            const float2 a0 = unpack_16<BF16>(mv.x), a1 = unpack_16<BF16>(mv.y), a2 = unpack_16<BF16>(mv.z), a3 = unpack_16<BF16>(mv.w);
+            v[g * 8 + 0] *= a0.x; v[g * 8 + 1] *= a0.y; v[g * 8 + 2] *= a1.x; v[g * 8 + 3] *= a1.y;
+            v[g * 8 + 4] *= a2.x; v[g * 8 + 5] *= a2.y; v[g * 8 + 6] *= a3.x; v[g * 8 + 7] *= a3.y;
+          }
+        }
         if ((p.flags & GEMM_RESIDUAL) && (p.flags & GEMM_RES_F32)) {
           const float4* rp = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.residual) + (size_t)m * p.ld_res + n0);
 #pragma unroll
@@ -71,8 +94,10 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
           float4* op = reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + (size_t)m * p.ld_out + n0);
 #pragma unroll
           for (int g = 0; g < 8; ++g) op[g] = make_float4(v[g * 4], v[g * 4 + 1], v[g * 4 + 2], v[g * 4 + 3]);
-        } else {
-          uint4* op = reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + n0);
+        }
+        if (!(p.flags & GEMM_OUT_F32) || p.out16 != nullptr) {
+          uint4* op = p.out16 != nullptr ? reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out16) + (size_t)m * p.ld_out16 + n0)
+                                         : reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + n0);
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             uint4 o;
@@ -106,7 +131,7 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
               uv += BF16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(bias16)[nin + 64 + j])
                          : __half2float(reinterpret_cast<const __half*>(bias16)[nin + 64 + j]);
             }
-            v[j] = silu_f(gv) * uv;
+            v[j] = ((p.flags & GEMM_GEGLU) ? gelu_tanh_f(gv) : silu_f(gv)) * uv;
           }
           uint4* op = reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + nout);
 #pragma unroll

@@ -47,6 +47,9 @@ enum GemmFlags : int {
   GEMM_RES_F32 = 16,   // with GEMM_RESIDUAL: the residual is fp32 and the product is scaled first, residual + alpha * acc
   GEMM_RELU2 = 32,     // out = relu(acc)^2
   GEMM_GLU_CLAMP = 64, // with GEMM_SWIGLU: g = min(gate, act_limit), u = clamp(up, +-act_limit), out = g * sigmoid(act_alpha * g) * (u + 1)
+  GEMM_GEGLU = 128,    // with GEMM_SWIGLU: out = gelu_tanh(gate) * up
+  GEMM_GELU = 512,     // out = gelu(acc), the exact (erf) form
+  GEMM_GELU_TANH = 1024,   // out = gelu(acc), the tanh form
   GEMM_FP4_F16W = 256, // fp4 weights, fp16 activations: the scale table lies within fp16's range (host-checked): half2 de-quantiser
 };
 
@@ -78,6 +81,10 @@ struct GemmParams {
   const void* gate = nullptr;                // 16-bit [M, >= N] (batched: + z * batch_out_cols): out = acc * sigmoid(gate)
   int ld_gate = 0;
   float act_limit = 0.f, act_alpha = 1.f;    // GEMM_GLU_CLAMP
+  // factors of the activated product, one of them at most: sigmoid of one fp32 logit per row, or row mul_rows[m] of a 16-bit table
+  const float* row_gate = nullptr; int ld_row_gate = 0;
+  const void* mul = nullptr; const int* mul_rows = nullptr; long long ld_mul = 0; int mul_count = 0;      // mul_count: rows of the table
+  void* out16 = nullptr; int ld_out16 = 0;   // with GEMM_OUT_F32: a second copy in the 16-bit type
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
@@ -87,6 +94,10 @@ __device__ __forceinline__ float glu_clamp_f(float g, float u, float limit, floa
   u = fminf(fmaxf(u, -limit), limit);
   return g * sigmoid_f(alpha * g) * (u + 1.0f);
 }
+// gelu in its tanh form: 0.5 (1 + tanh u) = sigmoid(2 u)
+__device__ __forceinline__ float gelu_tanh_f(float x) { return x * sigmoid_f(1.5957691216057308f * (x + 0.044715f * x * x * x)); }
+__device__ __forceinline__ float gelu_erf_f(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+__device__ __forceinline__ int clamp_row(int r, int n) { return r < 0 ? 0 : (r >= n ? n - 1 : r); }
 __device__ __forceinline__ float relu2_f(float x) { const float r = fmaxf(x, 0.f); return r * r; }
 
 // OCC = CTAs meant to be co-resident per SM: 1 -> deep ring (~200 KB), 2 -> two CTAs share the SM so that one
@@ -142,6 +153,9 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         if (p.flags & GEMM_GLU_CLAMP) {
           acc.x = glu_clamp_f(acc.x, acc2.x, p.act_limit, p.act_alpha); acc.y = glu_clamp_f(acc.y, acc2.y, p.act_limit, p.act_alpha);
           acc.z = glu_clamp_f(acc.z, acc2.z, p.act_limit, p.act_alpha); acc.w = glu_clamp_f(acc.w, acc2.w, p.act_limit, p.act_alpha);
+        } else if (p.flags & GEMM_GEGLU) {
+          acc.x = gelu_tanh_f(acc.x) * acc2.x; acc.y = gelu_tanh_f(acc.y) * acc2.y;
+          acc.z = gelu_tanh_f(acc.z) * acc2.z; acc.w = gelu_tanh_f(acc.w) * acc2.w;
         } else {
           acc.x = silu_f(acc.x) * acc2.x; acc.y = silu_f(acc.y) * acc2.y;
           acc.z = silu_f(acc.z) * acc2.z; acc.w = silu_f(acc.w) * acc2.w;
@@ -157,6 +171,17 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         }
       }
       if (p.flags & GEMM_RELU2) { acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y); acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w); }
+      if (p.flags & GEMM_GELU) { acc.x = gelu_erf_f(acc.x); acc.y = gelu_erf_f(acc.y); acc.z = gelu_erf_f(acc.z); acc.w = gelu_erf_f(acc.w); }
+      if (p.flags & GEMM_GELU_TANH) { acc.x = gelu_tanh_f(acc.x); acc.y = gelu_tanh_f(acc.y); acc.z = gelu_tanh_f(acc.z); acc.w = gelu_tanh_f(acc.w); }
+      if (p.row_gate != nullptr) {
+        const float g = sigmoid_f(p.row_gate[(size_t)j * p.ld_row_gate]);
+        acc.x *= g; acc.y *= g; acc.z *= g; acc.w *= g;
+      }
+      if (p.mul != nullptr) {
+        const uint2 mv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p.mul) + (size_t)clamp_row(p.mul_rows[j], p.mul_count) * p.ld_mul + n_out);
+        const float2 m0 = unpack_16<BF16>(mv.x), m1 = unpack_16<BF16>(mv.y);
+        acc.x *= m0.x; acc.y *= m0.y; acc.z *= m1.x; acc.w *= m1.y;
+      }
       if (p.gate != nullptr) {
         const uint2 gv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p.gate) + (size_t)j * p.ld_gate +
                                                          (size_t)blockIdx.z * (size_t)p.batch_out_cols + n_out);
@@ -177,6 +202,9 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         *reinterpret_cast<float4*>(dst) = acc;
       } else if (p.flags & GEMM_OUT_F32) {
         *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + (size_t)j * p.ld_out + zo + n_out) = acc;
+        if (p.out16 != nullptr)
+          *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.out16) + (size_t)j * p.ld_out16 + n_out) =
+              make_uint2(pack_16<BF16>(acc.x, acc.y), pack_16<BF16>(acc.z, acc.w));
       } else {
         uint2 o;
         o.x = pack_16<BF16>(acc.x, acc.y);

@@ -115,12 +115,12 @@ __global__ void rmsnorm32_kernel(const float* __restrict__ x, const typename Act
 
 // h[t] = table[ids[t]] + position in fp32, and its RMSNorm (w == nullptr: the row itself; y == nullptr: h only).  inv_freq: the position
 // is sines and cosines, inv_freq[i] = 10000^(-2i / H) in double; the angle is reduced to [-pi, pi] in double, so a far position costs
-// no accuracy.  pos_table: it is row positions[t] of a learned table.
+// no accuracy.  pos_table: it is row positions[t] of a learned table.  add_vec: one more row that every token gets.
 template <int DT, int VEC>
 __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __restrict__ positions, const typename Act<DT>::T* __restrict__ table,
                                       const double* __restrict__ inv_freq, const typename Act<DT>::T* __restrict__ pos_table, int pos_rows,
-                                      const typename Act<DT>::T* __restrict__ w, float* __restrict__ h, typename Act<DT>::T* __restrict__ y, int H,
-                                      int vocab, float eps) {
+                                      const typename Act<DT>::T* __restrict__ add_vec, const typename Act<DT>::T* __restrict__ w,
+                                      float* __restrict__ h, typename Act<DT>::T* __restrict__ y, int H, int vocab, float eps) {
   extern __shared__ float row[];
   __shared__ float sh[32];
   pdl_launch_dependents();
@@ -152,6 +152,11 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
         ld4<DT>(pe + i, u);
         v[0] += u[0]; v[1] += u[1]; v[2] += u[2]; v[3] += u[3];
       }
+      if (add_vec != nullptr) {
+        float u[4];
+        ld4<DT>(add_vec + i, u);
+        v[0] += u[0]; v[1] += u[1]; v[2] += u[2]; v[3] += u[3];
+      }
       st4<2>(hp + i, v);
       st4<2>(row + i, v);
       ss += v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
@@ -162,6 +167,7 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
       float a = Act<DT>::ld(e[2 * i]), b = two ? Act<DT>::ld(e[2 * i + 1]) : 0.f;
       if (inv_freq != nullptr) add_pos(i, a, b);
       if (pe != nullptr) { a += Act<DT>::ld(pe[2 * i]); if (two) b += Act<DT>::ld(pe[2 * i + 1]); }
+      if (add_vec != nullptr) { a += Act<DT>::ld(add_vec[2 * i]); if (two) b += Act<DT>::ld(add_vec[2 * i + 1]); }
       hp[2 * i] = a; row[2 * i] = a; ss += a * a;
       if (two) { hp[2 * i + 1] = b; row[2 * i + 1] = b; ss += b * b; }
     }
@@ -191,26 +197,54 @@ __global__ void latent_norm_kernel(const typename Act<DT>::T* __restrict__ x, in
   for (int i = threadIdx.x; i < ld; i += blockDim.x) yp[i] = Act<DT>::st(i < n ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
 }
 
-// z[t] = sum_k wk * ys[pos[t, k]] + shared[t]; with an output norm z = RMSNorm(z) * post; h[t] += alpha * z; then y[t] = RMSNorm(h[t]) * w.
-// wts == nullptr: every weight is `wconst`.  pos == nullptr: z[t] = ys[t].  w == nullptr: y[t] = h[t].  y == nullptr: h only.
+// What opens a pass of looped layers: the residual gets a step vector and, where `table` is given, the token's embedding again.
+struct PassStart {
+  const void* table; const int* ids; const void* vec; int vocab;
+};
+
+// z[t] = sum_k wk * ys[pos[t, k]] + shared[t]; with an output norm z = RMSNorm(z) * post; h[t] += alpha * z (+ pass start); then
+// y[t] = RMSNorm(h[t]) * w.  wts == nullptr: every weight is `wconst`.  pos == nullptr: z[t] = ys[t] (ys == nullptr: nothing).
+// w == nullptr: y[t] = h[t].  y == nullptr: h only.
 template <int DT, int VEC>
 __global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict__ ys, const int* __restrict__ pos, const float* __restrict__ wts,
                                           float wconst, const typename Act<DT>::T* __restrict__ shared_y, float* __restrict__ h,
                                           const typename Act<DT>::T* __restrict__ post, const typename Act<DT>::T* __restrict__ w,
-                                          typename Act<DT>::T* __restrict__ y, int topk, int H, float alpha, float eps) {
+                                          typename Act<DT>::T* __restrict__ y, int topk, int H, float alpha, float eps, const PassStart ps) {
   extern __shared__ float row[];
   __shared__ float sh[2][32];
   pdl_launch_dependents();
   pdl_wait();
+  typedef typename Act<DT>::T T;
   const int t = blockIdx.x;
   float* hp = h + (size_t)t * H;
+  const T* pvec = reinterpret_cast<const T*>(ps.vec);
+  const T* pemb = nullptr;
+  if (ps.table != nullptr) {
+    int id = ps.ids[t];
+    id = id < 0 ? 0 : (id >= ps.vocab ? ps.vocab - 1 : id);
+    pemb = reinterpret_cast<const T*>(ps.table) + (size_t)id * H;
+  }
+  auto start = [&](float* v, int i) {                  // adds the pass start's columns i .. i + VEC - 1
+    float u[VEC];
+    if (pemb != nullptr) {
+      if (VEC == 4) ld4<DT>(pemb + i, u); else u[0] = Act<DT>::ld(pemb[i]);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += u[j];
+    }
+    if (pvec != nullptr) {
+      if (VEC == 4) ld4<DT>(pvec + i, u); else u[0] = Act<DT>::ld(pvec[i]);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += u[j];
+    }
+  };
   float ss = 0.f;
   for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
     float acc[VEC], v[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) acc[j] = 0.f;
     if (pos == nullptr) {
-      if (VEC == 4) ld4<DT>(ys + (size_t)t * H + i, acc); else acc[0] = Act<DT>::ld(ys[(size_t)t * H + i]);
+      if (ys == nullptr) {
+      } else if (VEC == 4) ld4<DT>(ys + (size_t)t * H + i, acc); else acc[0] = Act<DT>::ld(ys[(size_t)t * H + i]);
     } else {
       for (int k = 0; k < topk; ++k) {
         const int r = pos[(size_t)t * topk + k];
@@ -233,7 +267,10 @@ __global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict_
     }
     if (VEC == 4) ld4<2>(hp + i, v); else v[0] = hp[i];
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) { v[j] += alpha * acc[j]; ss += v[j] * v[j]; row[i + j] = v[j]; }
+    for (int j = 0; j < VEC; ++j) v[j] += alpha * acc[j];
+    start(v, i);
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { ss += v[j] * v[j]; row[i + j] = v[j]; }
     if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
   }
   if (post != nullptr) {
@@ -244,7 +281,10 @@ __global__ void moe_combine_norm32_kernel(const typename Act<DT>::T* __restrict_
       float pv[VEC], v[VEC];
       if (VEC == 4) { ld4<DT>(post + i, pv); ld4<2>(hp + i, v); } else { pv[0] = Act<DT>::ld(post[i]); v[0] = hp[i]; }
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) { v[j] += alpha * (row[i + j] * inv * pv[j]); ss += v[j] * v[j]; row[i + j] = v[j]; }
+      for (int j = 0; j < VEC; ++j) v[j] += alpha * (row[i + j] * inv * pv[j]);
+      start(v, i);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) { ss += v[j] * v[j]; row[i + j] = v[j]; }
       if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
     }
   }
@@ -278,13 +318,14 @@ __global__ void moe_gather_scaled_kernel(const float* __restrict__ x, const int*
   }
 }
 
-// Per-head RMS norm, interleaved rotary positions and cache append of a merged projection [queries | gate | keys | values], one warp
-// per (token, head), fp32 arithmetic.  Heads are D wide, stored Dp (values Vp); queries are rewritten in place, keys and values go to
-// their cache slots (slot < 0: nowhere).  rot: leading dimensions that turn; cos / sin tables [tab_rows, rot / 2].
+// Per-head RMS norm, rotary positions and cache append of a merged projection [queries | gate | keys | values], one warp per (token,
+// head), fp32 arithmetic.  Heads are D wide, stored Dp (values Vp); queries are rewritten in place, keys and values go to their cache
+// slots (slot < 0: nowhere).  rot: leading dimensions that turn, in pairs (2j, 2j + 1) or (neox) (j, j + rot / 2); cos / sin tables
+// [tab_rows, rot / 2].  Norm weights null: no norm; with neither norm nor rotation the queries stay as they are.
 struct HeadPostParams {
   void* proj; long long ld;
   const int* positions; const int* slots;
-  int T, H, G, D, Dp, Vp, k_col, v_col, rot;
+  int T, H, G, D, Dp, Vp, k_col, v_col, rot, neox;
   const void* q_norm; const void* k_norm;
   const float* cos_tab; const float* sin_tab;
   int tab_rows, num_slots;
@@ -297,11 +338,12 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   typedef typename Act<DT>::T T;
   pdl_launch_dependents();
   pdl_wait();
-  const int units = p.H + 2 * p.G;
+  const int h0 = p.q_norm == nullptr && p.rot == 0 ? p.H : 0;        // first head there is work for
+  const int units = p.H + 2 * p.G - h0;
   const long long u = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (u >= (long long)p.T * units) return;
   const int lane = threadIdx.x & 31;
-  const int t = (int)(u / units), k = (int)(u - (long long)t * units);
+  const int t = (int)(u / units), k = h0 + (int)(u - (long long)t * units);
   T* row = reinterpret_cast<T*>(p.proj) + (size_t)t * p.ld;
   const int slot = p.slots[t];
   const bool cached = slot >= 0 && slot < p.num_slots;
@@ -318,20 +360,24 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   T* src = is_k ? row + p.k_col + (k - p.H) * p.Dp : row + (size_t)k * p.Dp;
   T* dst = is_k ? reinterpret_cast<T*>(p.k_pool) + ((size_t)slot * p.G + (k - p.H)) * p.Dp : src;
   const T* nw = reinterpret_cast<const T*>(is_k ? p.k_norm : p.q_norm);
-  float ss = 0.f;
-  for (int i = lane; i < p.D; i += 32) { const float v = Act<DT>::ld(src[i]); ss += v * v; }
+  float inv = 1.f;
+  if (nw != nullptr) {
+    float ss = 0.f;
+    for (int i = lane; i < p.D; i += 32) { const float v = Act<DT>::ld(src[i]); ss += v * v; }
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-  const float inv = 1.0f / sqrtf(ss / (float)p.D + p.eps);
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    inv = 1.0f / sqrtf(ss / (float)p.D + p.eps);
+  }
   int pos = p.positions[t];
   pos = pos < 0 ? 0 : (pos >= p.tab_rows ? p.tab_rows - 1 : pos);
   const int half = p.rot >> 1;
   const float* ct = p.cos_tab + (size_t)pos * half;
   const float* st = p.sin_tab + (size_t)pos * half;
   for (int j = lane; 2 * j < p.Dp; j += 32) {              // pairs (Dp is even; beyond D the row is zero and stays zero)
-    const int i0 = 2 * j, i1 = 2 * j + 1;
-    float a = i0 < p.D ? Act<DT>::ld(src[i0]) * inv * Act<DT>::ld(nw[i0]) : 0.f;
-    float b = i1 < p.D ? Act<DT>::ld(src[i1]) * inv * Act<DT>::ld(nw[i1]) : 0.f;
+    const int i0 = p.neox && j < half ? j : 2 * j, i1 = p.neox && j < half ? j + half : 2 * j + 1;
+    float a = 0.f, b = 0.f;
+    if (i0 < p.D) { a = Act<DT>::ld(src[i0]); if (nw != nullptr) a *= inv * Act<DT>::ld(nw[i0]); }
+    if (i1 < p.D) { b = Act<DT>::ld(src[i1]); if (nw != nullptr) b *= inv * Act<DT>::ld(nw[i1]); }
     if (j < half) {
       const float c = ct[j], s = st[j], u0 = a;
       a = u0 * c - b * s;
@@ -381,12 +427,12 @@ extern "C" int fb_rmsnorm32(const float* x, const void* w, void* y, int M, int H
 }
 
 extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const void* table, const double* inv_freq, const void* pos_table,
-                                 int pos_rows, const void* w, float* h, void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
+                                 int pos_rows, const void* add_vec, const void* w, float* h, void* y, int T, int H, int vocab, float eps, int dt, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2 || (pos_table != nullptr && pos_rows <= 0)) return -1;
   const bool vec = H % 4 == 0;
   const int th = row_threads(H, vec ? 4 : 2);
-#define GO(DT, V) S32_LAUNCH((embed_pos_norm_kernel<DT, V>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)pos_table, pos_rows, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
+#define GO(DT, V) S32_LAUNCH((embed_pos_norm_kernel<DT, V>), T, th, H, stream, ids, positions, (const Act<DT>::T*)table, inv_freq, (const Act<DT>::T*)pos_table, pos_rows, (const Act<DT>::T*)add_vec, (const Act<DT>::T*)w, h, (Act<DT>::T*)y, H, vocab, eps)
   if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
   else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
@@ -405,12 +451,14 @@ extern "C" int fb_latent_norm(const void* x, int ldx, const void* w, const int* 
 }
 
 extern "C" int fb_moe_combine_norm32(const void* ys, const int* pos, const float* wts, float wconst, const void* shared_y, float* h,
-                                     const void* post, const void* w, void* y, int T, int topk, int H, float alpha, float eps, int dt, void* stream) {
+                                     const void* post, const void* w, void* y, int T, int topk, int H, float alpha, float eps,
+                                     const void* start_table, const int* ids, int vocab, const void* start_vec, int dt, void* stream) {
   if (T <= 0) return 0;
-  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2 || (pos != nullptr && ys == nullptr) || (start_table != nullptr && (ids == nullptr || vocab <= 0))) return -1;
+  const PassStart ps{start_table, ids, start_vec, vocab};
   const bool vec = H % 4 == 0;
   const int th = row_threads(H, vec ? 4 : 1);
-#define GO(DT, V) S32_LAUNCH((moe_combine_norm32_kernel<DT, V>), T, th, H, stream, (const Act<DT>::T*)ys, pos, wts, wconst, (const Act<DT>::T*)shared_y, h, (const Act<DT>::T*)post, (const Act<DT>::T*)w, (Act<DT>::T*)y, topk, H, alpha, eps)
+#define GO(DT, V) S32_LAUNCH((moe_combine_norm32_kernel<DT, V>), T, th, H, stream, (const Act<DT>::T*)ys, pos, wts, wconst, (const Act<DT>::T*)shared_y, h, (const Act<DT>::T*)post, (const Act<DT>::T*)w, (Act<DT>::T*)y, topk, H, alpha, eps, ps)
   if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
   else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
@@ -443,14 +491,15 @@ extern "C" int fb_moe_gather_scaled(const float* x, const int* pos, const float*
 
 // See HeadPostParams.  G = 0: queries only (the layer reads another layer's cache).
 extern "C" int fb_head_norm_rope(void* proj, long long ld, const int* positions, const int* slots, int T, int H, int G, int D, int Dp, int Vp,
-                                 int k_col, int v_col, int rot, const void* q_norm, const void* k_norm, const float* cos_tab,
+                                 int k_col, int v_col, int rot, int neox, const void* q_norm, const void* k_norm, const float* cos_tab,
                                  const float* sin_tab, int tab_rows, int num_slots, void* k_pool, void* v_pool, float eps, int dt, void* stream_) {
   if (T <= 0) return 0;
-  if (H <= 0 || G < 0 || D <= 0 || Dp < D || (Dp & 1) || Vp <= 0 || rot < 0 || (rot & 1) || rot > D || dt < 0 || dt > 2 || q_norm == nullptr) return -1;
+  if (H <= 0 || G < 0 || D <= 0 || Dp < D || (Dp & 1) || Vp <= 0 || rot < 0 || (rot & 1) || rot > D || dt < 0 || dt > 2) return -1;
   if (rot > 0 && (cos_tab == nullptr || sin_tab == nullptr || tab_rows <= 0)) return -1;
-  if (G > 0 && (k_norm == nullptr || k_pool == nullptr || v_pool == nullptr)) return -1;
-  HeadPostParams p{proj, ld, positions, slots, T, H, G, D, Dp, Vp, k_col, v_col, rot, q_norm, k_norm, cos_tab, sin_tab, tab_rows, num_slots, k_pool, v_pool, eps};
-  const long long units = (long long)T * (H + 2 * G);
+  if (G > 0 && ((k_norm == nullptr) != (q_norm == nullptr) || k_pool == nullptr || v_pool == nullptr)) return -1;
+  HeadPostParams p{proj, ld, positions, slots, T, H, G, D, Dp, Vp, k_col, v_col, rot, neox, q_norm, k_norm, cos_tab, sin_tab, tab_rows, num_slots, k_pool, v_pool, eps};
+  const long long units = (long long)T * ((q_norm == nullptr && rot == 0 ? 0 : H) + 2 * G);
+  if (units == 0) return 0;
   const dim3 grid((unsigned)((units + 7) / 8));
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (dt == 0) launch_k(head_norm_rope_kernel<0>, grid, dim3(256), 0, stream, 0, p);

@@ -82,6 +82,7 @@ class ModelRunner:
         self.device = model.device
         if model.cfg.pos_table:                     # learned positions end with their table
             cfg.max_context = min(cfg.max_context, model.cfg.pos_table)
+        model.max_context = cfg.max_context
         self.max_pages = (cfg.max_context + cfg.page_len - 1) // cfg.page_len
         if num_pages is None:
             model._state_bytes_reserved = model.linear_state_bytes_per_slot() * (cfg.max_batch + 1)

@@ -80,7 +80,12 @@ def dequant_awq(qweight: torch.Tensor, qzeros: torch.Tensor, scales: torch.Tenso
 # name canonicalisation: every family is mapped onto the Llama naming that loader.shard understands
 # ---------------------------------------------------------------------------------------------------
 _RENAMES = [
-    # Patesun, Vilulorn
+    # Patesun, Vilulorn, Vuripel
+    (r"^l(\d+)\.mix\.([qkvif])\.b$", r"model.layers.\1.self_attn.\2_proj.bias"), (r"^l(\d+)\.mix\.([if])$", r"model.layers.\1.self_attn.\2_proj.weight"),
+    (r"^l(\d+)\.mix\.sink$", r"model.layers.\1.self_attn.sinks"), (r"^l(\d+)\.mlp\.gate$", r"model.layers.\1.mlp.gate_proj.weight"),
+    (r"^l(\d+)\.mlp\.shared\.sg$", r"model.layers.\1.mlp.shared_expert_gate.weight"), (r"^loop\.step$", "model.loop_step.weight"),
+    (r"^side\.embed$", "model.embed_tokens_per_layer.weight"), (r"^l(\d+)\.side\.gate$", r"model.layers.\1.per_layer_input_gate.weight"),
+    (r"^l(\d+)\.side\.proj$", r"model.layers.\1.per_layer_projection.weight"), (r"^l(\d+)\.side\.norm$", r"model.layers.\1.post_per_layer_input_norm.weight"),
     (r"^pos$", "model.embed_positions.weight"), (r"^l(\d+)\.mix\.([qk])\.norm$", r"model.layers.\1.self_attn.\2_norm.weight"),
     (r"^l(\d+)\.mix\.norm$", r"model.layers.\1.self_attn.o_norm.weight"), (r"^l(\d+)\.mix\.a2\.b$", r"model.layers.\1.self_attn.a2_proj.bias"),
     (r"^l(\d+)\.mix\.(a1|a2|k|v)$", r"model.layers.\1.self_attn.\2_proj.weight"), (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight"),
@@ -331,7 +336,7 @@ def load_model(path: str | Path, device="cuda", dtype=None, wdtype: str = "auto"
 
     def top_fn():
         t = {}
-        for k in ("model.embed_tokens.weight", "model.embed_positions.weight", "model.norm.weight", "model.norm.bias", "lm_head.weight", "lm_head.bias"):
+        for k in ("model.embed_tokens.weight", "model.embed_positions.weight", "model.embed_tokens_per_layer.weight", "model.loop_step.weight", "model.norm.weight", "model.norm.bias", "lm_head.weight", "lm_head.bias"):
             if ck.has(k):
                 t[k] = ck.raw(k)
         return t

@@ -310,18 +310,19 @@ def build_layer(m, i: int, t: dict, wdtype="dense", moe_wdtype=None):
 def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
     """Mixer and feed-forward of a model that lists its layers (``cfg.mixers`` / ``cfg.ffs``).  Widths are padded with zero rows and
     columns to what the kernels tile (the padding stays zero through every product)."""
-    from ..models.config import AttnSpec, GLASpec
+    from ..models.config import AttnSpec, GLASpec, MLSTMSpec
     from ..ops import gla as GLA
     from ..ops import grouped as GR
     from ..ops import latent as LA
+    from ..ops import mlstm as ML
 
     cfg = m.cfg
     spec, ff = cfg.mixers[i], cfg.ffs[i]
     t = lambda k: _to(g("self_attn." + k + ".weight"), m)
     exact = m.dtype == torch.float32
 
-    def lin(w, kind=wdtype, interleaved=False):
-        l = LinearWeight.from_dense(w, kind, None, interleaved, act_dtype=m.dtype)
+    def lin(w, kind=wdtype, interleaved=False, bias=None):
+        l = LinearWeight.from_dense(w, kind, bias, interleaved, act_dtype=m.dtype)
         l.exact32 = exact
         return l
 
@@ -334,25 +335,44 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
         return lin(LA.pad_cols(_to(w, m), mult if m.on_cuda else 1).contiguous(), kind)
 
     f = lw.mlp
+    gates, joint = [], []                   # parallel layers: rows of fp32 logits; matrices that project back to the residual
     if cfg.output_norms:                    # the layer's two norms belong to its sub-layers' outputs
         lw.attn.post_ln, f.post_ln, lw.attn.ln, f.ln = lw.attn.ln, f.ln, None, None
     if isinstance(spec, GLASpec):
         lw.gla, in_w = GLA.build(spec, *(t(k + "_proj") for k in ("q", "k", "v", "g", "a1", "a2")), _to(g("self_attn.a2_proj.bias"), m), t("o_norm"))
         lw.gla.in_proj = lin(in_w)
         lw.attn.o = lin(t("o_proj"))
+    elif isinstance(spec, MLSTMSpec):
+        b = lambda k: _to(g("self_attn." + k + "_proj.bias"), m)
+        lw.mlstm, in_w = ML.build(spec, *(t(k + "_proj") for k in ("q", "k", "v", "g")), b("i"), b("f"), t("o_norm"))
+        lw.mlstm.in_proj = lin(in_w)
+        gates += [t("i_proj"), t("f_proj")]
+        joint.append(LA.pad_cols(t("o_proj"), 8))
     elif isinstance(spec, AttnSpec):
         own = spec.kv_from is None
-        lw.grouped, in_w = GR.build(spec, t("q_proj"), t("k_proj") if own else None, t("v_proj") if own else None, t("g_proj"), t("q_norm"),
-                                    t("k_norm") if own else None)
-        lw.grouped.in_proj = lin(in_w)
+        kv = lambda k: t(k) if own else None
+        biases = [_to(g(f"self_attn.{k}_proj.bias"), m) if own or k == "q" else None for k in "qkv"] if spec.bias else None
+        lw.grouped, in_w = GR.build(spec, t("q_proj"), kv("k_proj"), kv("v_proj"), t("g_proj") if spec.gate == "elem" else None,
+                                    t("q_norm") if spec.qk_norm else None, kv("k_norm") if spec.qk_norm else None, biases,
+                                    _to(g("self_attn.sinks"), m) if spec.sinks else None)
+        lw.grouped.in_proj = lin(in_w, bias=lw.grouped.in_bias)
         lw.attn.heads, lw.attn.rope = spec.heads, spec.rope
-        lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
+        if spec.gate == "head":
+            gates.append(t("g_proj"))
+        if cfg.parallel_block:
+            joint.append(LA.pad_out_proj(t("o_proj"), spec))
+        else:
+            lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
     else:
         la, in_w = LA.build(spec, t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"))
         la.in_proj = lin(in_w)
         lw.latent = la
         lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
-    if ff.kind == "none":
+    if cfg.parallel_block:
+        _build_parallel_ff(m, lw, ff, g, lin, gate_up, wdtype, moe_wdtype, gates, joint)
+        if cfg.side_dim:
+            _build_side(m, i, lw, g, lin)
+    elif ff.kind == "none":
         f.absent = True
     elif ff.kind == "dense":
         f.act = ff.act
@@ -372,6 +392,50 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
         if ff.shared_ff:
             f.shared_gate_up = gate_up(g("mlp.shared_experts.gate_proj.weight"), g("mlp.shared_experts.up_proj.weight"), wdtype)
             f.shared_down = down(g("mlp.shared_experts.down_proj.weight"), wdtype, 64)
+
+
+def _build_parallel_ff(m, lw, ff, g, lin, gate_up, wdtype, moe_wdtype, gates, joint):
+    """Feed-forward of a layer whose mixer and feed-forward read one norm.  What projects back to the residual is one matrix over [mixer
+    output | feed-forward (or shared expert) activations], what is needed as fp32 logits (gates of the mixer, router, gate of the
+    shared expert) another one.  ``gates`` / ``joint``: the mixer's rows and matrix."""
+    from ..ops import latent as LA
+
+    f = lw.mlp
+    w = lambda k: _to(g("mlp." + k + ".weight"), m)
+    mult = 8 if m.on_cuda else 1
+    lw.mix_cols, lw.n_gates = joint[0].shape[1], sum(x.shape[0] for x in gates)
+    if ff.kind == "dense":
+        f.act = ff.act
+        f.gate_up = gate_up(g("mlp.gate_proj.weight"), g("mlp.up_proj.weight"), wdtype)
+        joint.append(LA.pad_cols(w("down_proj"), 64 if m.on_cuda else 1))
+    elif ff.kind == "moe":
+        names = [f"experts.{e}." for e in range(ff.experts)]
+        f.experts = MOE.ExpertWeights(ff.experts, 0, [lin(LA.pad_rows(w(n + "up_proj"), mult), moe_wdtype) for n in names],
+                                      [lin(LA.pad_cols(w(n + "down_proj"), mult).contiguous(), moe_wdtype) for n in names])
+        f.experts.act, f.top, f.groups, f.keep_groups = ff.act, ff.top, ff.groups, ff.keep_groups
+        f.router_col = sum(x.shape[0] for x in gates)
+        gates.append(w("gate"))
+        if ff.shared_ff:
+            f.shared_up = lin(LA.pad_rows(w("shared_experts.up_proj"), mult))
+            joint.append(LA.pad_cols(w("shared_experts.down_proj"), mult))
+            if ff.shared_gate:
+                f.shared_gate_col = f.router_col + ff.experts
+                gates.append(w("shared_expert_gate"))
+    lw.joint = lin(torch.cat(joint, dim=1))
+    if gates:
+        lw.logits = lin(LA.pad_rows(torch.cat(gates, dim=0), 32), "dense")
+
+
+def _build_side(m, i: int, lw, g, lin):
+    """Per-layer token input: gate and projection between the residual and the layer's slice of the second embedding."""
+    from ..models.decoder import SideInput
+    from ..ops import latent as LA
+
+    t = lambda k: _to(g(k + ".weight"), m)
+    s = lw.side = SideInput()
+    s.gate, s.proj = lin(LA.pad_rows(t("per_layer_input_gate"), m.side_cols)), lin(LA.pad_cols(t("per_layer_projection"), m.side_cols))
+    s.norm = t("post_per_layer_input_norm")
+    s.col = m.cfg.layer_runs[i] * m.side_cols
 
 
 def build_linear_attn(m, g, ln, W, layer_idx: int = 0):
@@ -457,6 +521,13 @@ def build_top(m, t: dict, wdtype="dense"):
     m.final_norm = _to(t["model.norm.weight"], m)
     if cfg.pos_table:
         m.pos_table = _to(t["model.embed_positions.weight"], m)
+    if cfg.pass_starts is not None:
+        m.loop_step = _to(t["model.loop_step.weight"], m)
+    if cfg.side_dim:
+        e = t["model.embed_tokens_per_layer.weight"]
+        m.side_cols = -(-cfg.side_dim // 32) * 32 if m.on_cuda else cfg.side_dim         # a layer's columns, padded to what a GEMM tiles
+        e = e.to(m.device, m.dtype).reshape(e.shape[0], -1, cfg.side_dim)
+        m.side_embed = torch.nn.functional.pad(e, (0, m.side_cols - cfg.side_dim)).reshape(e.shape[0], -1).contiguous()
     if t.get("model.norm.bias") is not None:
         m.ln_bias[id(m.final_norm)] = _to(t["model.norm.bias"], m)
     head = t.get("lm_head.weight")

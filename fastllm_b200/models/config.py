@@ -25,16 +25,22 @@ class LatentSpec:
 
 @dataclass
 class AttnSpec:
-    """Softmax attention of one layer with its own head counts and widths, per-head query / key norms, rotary positions and an
-    elementwise sigmoid gate on the heads."""
+    """Softmax attention of one layer with its own head counts, widths, mask and rotary positions; which of the other parts it has."""
     heads: int
     kv_heads: int
     dim: int                # query / key dimensions per head
     vdim: int
     scale: float
     chunk: int = 0          # > 0: the sequence is cut into chunks of this many positions, a query sees the keys of its own chunk
-    rope: dict | None = None     # {"theta", "rot_dim", "scaling"}: interleaved pairs on the first rot_dim dimensions
+    rope: dict | None = None     # {"theta", "rot_dim", "scaling", "mode"}: the first rot_dim dimensions, "interleaved" (default) or "neox" pairs
     kv_from: int | None = None   # the layer whose cached keys and values this one reads (it has no projections of them)
+    window: int = 0         # > 0 (instead of a chunk): a query sees the last `window` keys, itself included, ...
+    keep: int = 0           # ... and the first `keep` of the sequence
+    softcap: float = 0.0    # > 0: scores become softcap * tanh(score / softcap)
+    sinks: bool = False     # a learned logit per head in the softmax denominator
+    qk_norm: bool = True    # RMS norm of every query and key head
+    gate: str = "elem"      # sigmoid gate on the output: "elem" one per element, "head" one per head, "" none
+    bias: bool = False      # biases of the query, key and value projections
 
 
 @dataclass
@@ -48,18 +54,35 @@ class GLASpec:
 
 
 @dataclass
+class MLSTMSpec:
+    """Matrix-memory LSTM of one layer: a [dim, vdim] state and a normaliser row per head, exponential input gates and sigmoid forget
+    gates (one of each per head and token, logits soft-capped at gate_cap) under a running maximum."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+RECURRENT = (GLASpec, MLSTMSpec)     # mixers that keep a state per request instead of pages
+
+
+@dataclass
 class FFSpec:
-    """Feed-forward of one layer where the layers of a model differ: "dense" (up -> act -> down), "moe" (routed gated experts plus
-    an optional shared one) or "none"."""
+    """Feed-forward of one layer where the layers of a model differ: "dense" (up -> act -> down, or act(gate) * up -> down), "moe"
+    (routed experts plus an optional shared one) or "none"."""
     kind: str = "none"
     ff: int = 0
-    act: str = "relu2"      # experts: "silu" | "gptoss" (both branches clamped at `limit`)
+    act: str = "relu2"      # dense: "relu2" | "geglu" (tanh form); experts: "silu" | "gptoss" (both branches clamped at `limit`), or "gelu": no gate branch
     experts: int = 0
     top: int = 0
     expert_ff: int = 0
     shared_ff: int = 0      # 0: no shared expert
     router: str = "table"   # "table": experts by token id | "sigmoid": the best scores of a projection, which scale the expert's input
+                            # | "softmax": the best softmax scores, which scale the expert's output
     limit: float = 0.0
+    groups: int = 1         # the experts form equal groups of neighbours; only those of the `keep_groups` groups with the largest score count
+    keep_groups: int = 1
+    shared_gate: bool = False    # the shared expert's output is multiplied by a sigmoid, one logit per token
 
 
 @dataclass
@@ -145,9 +168,9 @@ class ModelConfig:
     lin_conv_kernel: int = 4
     lin_kind: str = "gdn"                  # "gdn" Gated DeltaNet | "lightning" decayed linear attention (MiniMax-Text-01 / M1)
     lin_block: int = 256                   # lightning attention: block length of the chunked evaluation
-    # models whose layers are listed one by one (Patesun, Vilulorn): the mixer and feed-forward of every layer, and which layer's
+    # models whose layers are listed one by one (Patesun, Vilulorn, Vuripel): the mixer and feed-forward of every layer, and which layer's
     # weights each run of the stack uses (looped layers appear once per pass; num_layers counts the runs, every run has its own cache)
-    mixers: list | None = None             # LatentSpec / AttnSpec / GLASpec per run
+    mixers: list | None = None             # LatentSpec / AttnSpec / GLASpec / MLSTMSpec per run
     ffs: list | None = None                # FFSpec per run
     layer_runs: list | None = None
     residual_f32: bool = False             # the residual stream is fp32; sub-layer outputs join it times residual_mult
@@ -155,6 +178,9 @@ class ModelConfig:
     pos_embed_base: float = 0.0            # > 0: sinusoidal positions with this base are added to the token embedding
     pos_table: int = 0                     # > 0: rows of a learned position table that is added to the token embedding
     output_norms: bool = False             # fp32 residual: what a sub-layer adds is normalised, what it reads is not
+    pass_starts: list | None = None        # per run: the pass number where it opens a pass of a loop that adds a step vector (and, from
+                                           # the second pass on, the token embedding) to the residual; else None
+    side_dim: int = 0                      # > 0: width of the per-layer token input (a second embedding, gated by the residual)
     # DeepNorm-style residual (MiniMax-Text-01 / M1): the block input is normalised first and the NORMALISED rows are the
     # residual: y = alpha * norm(x) + beta * f(norm(x)).  (alpha, beta) for full-attention layers, linear layers, MLPs.
     postnorm_residual: bool = False
@@ -605,16 +631,23 @@ def _patesun(d: dict) -> ModelConfig:
                               expert_ff=int(f["expert"]["ff"]), shared_ff=int((f.get("shared") or {}).get("ff") or 0)))
         else:
             raise NotImplementedError(f"Patesun: layer {i} has feed-forward '{f.get('kind')}'")
-    runs = list(range(len(L)))
-    loop = d.get("loop")
-    if loop:
-        a, b = int(loop["start"]), int(loop["stop"])
-        runs = runs[:a] + runs[a:b] * int(loop["times"]) + runs[b:]
-    c = _listed("Patesun", d, mixers, ffs, runs)
+    c = _listed("Patesun", d, mixers, ffs, _loop_runs(d)[0])
     c.residual_mult = float(d.get("residual_mult", 1.0))
     c.pos_embed_base = 10000.0
     c.max_position = int(d.get("max_position_embeddings", 1 << 20))
     return c
+
+
+def _loop_runs(d: dict):
+    """(layer of every run, pass number of the runs that open a pass of config's "loop", None elsewhere)."""
+    n, loop = len(d["layers"]), d.get("loop")
+    if not loop:
+        return list(range(n)), [None] * n
+    a, b, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not (0 <= a < b <= n and times >= 1):
+        raise ValueError(f"loop over layers {a} .. {b - 1} of {n}, {times} times")
+    return ([*range(a), *(list(range(a, b)) * times), *range(b, n)],
+            [None] * a + [t if i == a else None for t in range(times) for i in range(a, b)] + [None] * (n - b))
 
 
 def _listed(name: str, d: dict, mixers: list, ffs: list, runs: list) -> ModelConfig:
@@ -633,8 +666,8 @@ def _listed(name: str, d: dict, mixers: list, ffs: list, runs: list) -> ModelCon
     c.rms_eps = float(d["norm"]["eps"])
     c.residual_f32 = True
     c.rope_mode = "none"                    # model-wide tables: none (a layer's mixer has its own)
-    if any(isinstance(m, GLASpec) for m in c.mixers):
-        c.layer_types = ["linear_attention" if isinstance(m, GLASpec) else "full_attention" for m in c.mixers]
+    if any(isinstance(m, RECURRENT) for m in c.mixers):
+        c.layer_types = ["linear_attention" if isinstance(m, RECURRENT) else "full_attention" for m in c.mixers]
     c.eos_token_ids = _eos_list(d.get("eos_token_id"))
     c.bos_token_id = d.get("bos_token_id")
     c.torch_dtype = str(d.get("torch_dtype", d.get("dtype", "bfloat16"))).replace("torch.", "")
@@ -680,8 +713,49 @@ def _vilulorn(d: dict) -> ModelConfig:
     return c
 
 
+def _vuripel(d: dict) -> ModelConfig:
+    """Vuripel: attention without positions (sinks, a gate per head), windowed attention that keeps the first tokens (query / key norms,
+    rotary positions), matrix-memory LSTM layers; mixer and feed-forward read one norm (GeGLU, or grouped softmax-routed experts with a
+    gated shared one); a per-layer token input; a span of layers that runs several times with a step vector per pass."""
+    mixers, ffs = [], []
+    for i, spec in enumerate(d["layers"]):
+        m, kind = spec["mixer"], spec.get("type")
+        if kind == "mlstm":
+            mixers.append(MLSTMSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"])))
+        elif kind in ("attention", "attention_2"):
+            rot, mask = m.get("rot") or {}, m.get("mask") or {}
+            rope = {"theta": float(rot["base"]), "rot_dim": int(rot["dims"]), "scaling": None, "mode": "neox"} if rot.get("dims") else None
+            first = kind == "attention"
+            mixers.append(AttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), rope=rope,
+                                   window=int(mask.get("size") or 0), keep=int(mask.get("keep_first") or 0), softcap=float(m.get("softcap") or 0.0),
+                                   sinks=first, qk_norm=not first, gate="head" if first else "", bias=True))
+        else:
+            raise NotImplementedError(f"Vuripel: layer {i} has mixer '{kind}'")
+        f = spec.get("mlp")
+        if f is None:
+            ffs.append(FFSpec())
+        elif f.get("kind") == "dense":
+            ffs.append(FFSpec("dense", ff=int(f["ff"]), act="geglu"))
+        elif f.get("kind") == "moe":
+            r = f["router"]
+            gr, shared = r.get("groups") or {}, f.get("shared") or {}
+            ffs.append(FFSpec("moe", act="gelu", experts=int(r["experts"]), top=int(r["top"]), expert_ff=int(f["expert"]["ff"]),
+                              shared_ff=int(shared.get("ff") or 0), router="softmax", groups=int(gr.get("count") or 1),
+                              keep_groups=int(gr.get("keep") or gr.get("count") or 1), shared_gate=bool(shared)))
+        else:
+            raise NotImplementedError(f"Vuripel: layer {i} has feed-forward '{f.get('kind')}'")
+    runs, starts = _loop_runs(d)
+    c = _listed("Vuripel", d, mixers, ffs, runs)
+    c.num_kv_heads = max((m.kv_heads for m in mixers if isinstance(m, AttnSpec)), default=1)
+    c.parallel_block = True
+    c.pass_starts = starts if d.get("loop") else None
+    c.side_dim = int((d.get("token_side") or {}).get("dim") or 0)
+    c.max_position = int(d.get("max_position_embeddings", 1 << 20))
+    return c
+
+
 # config.json "architecture" of designs whose layers are listed one by one
-LISTED = {"Patesun": _patesun, "Vilulorn": _vilulorn}
+LISTED = {"Patesun": _patesun, "Vilulorn": _vilulorn, "Vuripel": _vuripel}
 
 
 def load_config(path: str | Path) -> ModelConfig:
@@ -841,6 +915,22 @@ def preset(name: str) -> ModelConfig:
             block += [layer("gla", gl), layer("attention", at), layer("gla", gl), layer("attention", dict(at, kv_from=5))]
         return from_hf_dict(dict(architecture="Vilulorn", vocab=512 if tiny else 128256, width=128 if tiny else 4096, norm={"eps": 1e-5},
                                  max_positions=640 if tiny else 32768, layers=block))
+    if name in ("tiny-vuripel", "vuripel-8b"):
+        tiny = name.startswith("tiny")
+        full = ({"heads": 6, "kv_heads": 3, "dim": 40, "vdim": 24, "scale": 0.2, "softcap": 15.0} if tiny else
+                {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0})
+        local = dict(full, mask={"size": 21 if tiny else 4096, "keep_first": 3 if tiny else 16}, rot={"base": 5e4 if tiny else 5e5, "dims": 16 if tiny else 64})
+        cell = {"heads": 3, "dim": 24, "vdim": 40, "gate_cap": 9.0} if tiny else {"heads": 32, "dim": 128, "vdim": 128, "gate_cap": 15.0}
+        dense = {"kind": "dense", "ff": 200 if tiny else 14336}
+        moe = {"kind": "moe", "expert": {"ff": 56 if tiny else 1536}, "router": {"experts": 9 if tiny else 64, "top": 2 if tiny else 6,
+                                                                               "groups": {"count": 3 if tiny else 8, "keep": 2 if tiny else 4}},
+               "shared": {"ff": 72 if tiny else 2048}}
+        layer = lambda t, m, f: {"type": t, "mixer": m, "mlp": f}
+        block = [layer("attention_2", local, dense), layer("mlstm", cell, moe), layer("attention", full, moe), layer("mlstm", cell, None if tiny else moe)]
+        if not tiny:
+            block += [layer("attention_2", local, moe), layer("mlstm", cell, moe), layer("attention_2", local, moe), layer("attention", full, dense)]
+        return from_hf_dict(dict(architecture="Vuripel", vocab=512 if tiny else 128256, width=144 if tiny else 4096, norm={"eps": 1e-5}, layers=block,
+                                 loop={"start": 1, "stop": 3 if tiny else 5, "times": 2 if tiny else 3}, token_side={"dim": 24 if tiny else 256}))
     if name == "tiny-deepseek-v32":      # latent attention with the sparse-attention indexer (selection size 32)
         return from_hf_dict(dict(model_type="deepseek_v32", vocab_size=512, hidden_size=256, num_hidden_layers=2,
                                  num_attention_heads=4, num_key_value_heads=4, intermediate_size=512,

@@ -25,10 +25,11 @@ from ..ops import basic as B
 from ..ops import gla as GLA
 from ..ops import grouped as GR
 from ..ops import latent as LA
+from ..ops import mlstm as ML
 from ..ops import moe as MOE
 from ..ops import stream32 as S
 from ..ops.quant import LinearWeight
-from .config import AttnSpec, GLASpec, ModelConfig
+from .config import AttnSpec, GLASpec, MLSTMSpec, ModelConfig
 
 
 @dataclass
@@ -143,6 +144,22 @@ class MLPWeights:
         self.shared_gate_up: LinearWeight | None = None
         self.shared_down: LinearWeight | None = None
         self.shared_gate = None     # [1, H] sigmoid gate (qwen2_moe)
+        # parallel listed layers: the shared expert's up matrix (its down matrix is part of the layer's joint one), columns of the layer's
+        # fp32 logits, expert groups
+        self.shared_up: LinearWeight | None = None
+        self.router_col = 0
+        self.shared_gate_col: int | None = None
+        self.groups = self.keep_groups = 1
+
+
+class SideInput:
+    """Per-layer token input: the layer's columns of a second embedding, gated by the residual and projected back onto it."""
+
+    def __init__(self):
+        self.gate: LinearWeight | None = None      # [cols, H]
+        self.proj: LinearWeight | None = None      # [H, cols]
+        self.norm = None                           # of what is added
+        self.col = 0                               # first column of the layer in ``DecoderModel.side_embed``
 
 
 class LayerWeights:
@@ -153,6 +170,13 @@ class LayerWeights:
         self.latent: LA.LatentWeights | None = None    # latent attention without positions
         self.grouped: GR.GroupedWeights | None = None  # grouped-query attention with its own widths, mask and rotary tables
         self.gla: GLA.GLAWeights | None = None         # gated linear attention
+        self.mlstm: ML.MLSTMWeights | None = None      # matrix-memory LSTM
+        # listed layers whose mixer and feed-forward read one norm
+        self.joint: LinearWeight | None = None         # [H, mixer output | feed-forward activations] onto the residual
+        self.mix_cols = 0                              # columns of the mixer output
+        self.logits: LinearWeight | None = None        # rows [mixer gates | router | shared expert's gate], fp32 results
+        self.n_gates = 0
+        self.side: SideInput | None = None
         self.lin: LinearAttnWeights | None = None      # set instead of ``attn`` projections on linear-attention layers
 
 
@@ -183,6 +207,10 @@ class DecoderModel:
         self.ep = ep                       # parallel.ep.EPInfo or None
         self.embed = None                  # [vocab(/tp), H]
         self.pos_table = None              # [positions, H] learned positions added to the embedding
+        self.loop_step = None              # [times, H] what opens the passes of looped layers
+        self.side_embed = None             # [vocab, layers * side_cols] per-layer token input
+        self.side_cols = 0
+        self.max_context = 0               # longest context the engine serves (rotary tables of listed layers reach it)
         self.layers: list[LayerWeights] = []
         self.final_norm = None
         self.lm_head: LinearWeight | None = None
@@ -248,7 +276,7 @@ class DecoderModel:
         key = (float(spec["theta"]), int(spec["rot_dim"]), id(spec.get("scaling")), str(torch.device(device)))
         cache = self.__dict__.setdefault("_rope_layers", {})
         if key not in cache:
-            mp = min(self.cfg.max_position, 1 << 17)
+            mp = max(min(self.cfg.max_position, 1 << 17), self.max_context)
             cache[key] = A.build_rope_tables(int(spec["rot_dim"]), mp, float(spec["theta"]), spec.get("scaling"), device)
         cos, sin = cache[key]
         return Hq, cos, sin, int(spec["rot_dim"])
@@ -305,6 +333,8 @@ class DecoderModel:
         c = self.cfg
         if c.mixers is not None:               # every listed layer has its own state
             sp = c.mixers[layer]
+            if isinstance(sp, MLSTMSpec):
+                return (n_slots, 0, 0), (n_slots, sp.heads, ML.state_len(sp.dim, sp.vdim))
             return (n_slots, 0, 0), (n_slots, sp.heads, sp.dim, sp.vdim)
         Hk, Hv = c.lin_num_k_heads // self.tp.size, c.lin_num_v_heads // self.tp.size
         if c.lin_kind == "lightning":          # no convolution window; one [D, D] state per head
@@ -656,6 +686,65 @@ class DecoderModel:
         a = GR.attention(gw, proj, kv, fb)
         return self._row_parallel_norm(lw.attn.o, a, residual, next_ln, lw.attn.post_ln)
 
+    def _parallel_layer(self, lw: LayerWeights, x, fb: ForwardBatch, kv, h, i: int):
+        """A listed layer whose mixer and feed-forward read the same rows ``x``: one projection of everything that is needed as fp32 logits,
+        mixer and activations side by side in one buffer, one product back onto the residual (with routed experts it joins their
+        combine), then the per-layer token input.  Returns (residual, rows of the next layer)."""
+        c, f, n = self.cfg, lw.mlp, lw.mix_cols
+        eps = c.rms_eps
+        z = lw.logits(x, out_f32=True) if lw.logits is not None else None
+        gates = z[:, :lw.n_gates] if lw.n_gates else None
+        act = torch.empty((x.shape[0], lw.joint.k), device=x.device, dtype=x.dtype)
+        if lw.mlstm is not None:
+            width = lw.mlstm.heads * lw.mlstm.vdim
+            if width < n:
+                act[:, width:n].zero_()
+            ML.mix(lw.mlstm, lw.mlstm.in_proj(x), gates, fb, kv[1], eps, out=act[:, :width])
+        else:
+            gw = lw.grouped
+            proj = gw.in_proj(x)
+            _, cos, sin, _ = self._layer_geom(lw.attn, x.device) if lw.attn.rope is not None else (0, None, None, 0)
+            GR.post(gw, proj, fb, kv, cos, sin, eps)
+            GR.attention(gw, proj, kv, fb, out=act[:, :n], head_gate=gates)
+        if f.gate_up is not None:
+            f.gate_up.glu(x, "gelu_tanh", out=act[:, n:])
+        elif f.shared_up is not None:
+            col = f.shared_gate_col
+            f.shared_up.activated(x, "gelu", out=act[:, n:], row_gate=z[:, col] if col is not None else None)
+        side, next_ln, start = lw.side, self._entry_norm(i + 1), self._pass_start(i + 1, fb.ids)
+        ends = dict(norm_w=None if side is not None else next_ln, eps=eps, alpha=1.0, dtype=self.dtype, start=None if side is not None else start)
+        if f.experts is not None:
+            x = self._routed_experts(f, x, z, lw.joint(act), h, ends)
+        elif side is None:
+            x = S.add_norm(lw.joint.add_to(act, h, 1.0), None, None, **ends)
+        else:
+            x = h if self.dtype == torch.float32 else torch.empty(h.shape, device=h.device, dtype=self.dtype)
+            lw.joint.add_to(act, h, 1.0, copy=x if x is not h else None)
+        if side is not None:
+            e = side.gate.activated(x, "gelu_tanh", mul=self.side_embed[:, side.col:side.col + self.side_cols], mul_rows=fb.ids)
+            x = S.add_norm(h, side.proj(e), side.norm, next_ln, eps, dtype=self.dtype, start=start)
+        return h, x
+
+    def _routed_experts(self, f: MLPWeights, x, z, shared, h, ends):
+        """Experts by the best softmax scores among the best groups; their combine adds ``shared`` and ends as ``ends`` says."""
+        E = f.experts.total
+        idx, wts = MOE.route_topk(z[:, f.router_col:f.router_col + E], None, f.top, 0, False, f.groups, f.keep_groups, group_max=True)
+        if f.experts.stacked is not None and x.is_cuda:
+            from ..ops import moe_grouped
+
+            parts = moe_grouped.forward(x, idx, wts, f.experts, combine=False)
+            if parts is not None:
+                return S.moe_combine_norm(parts[0], parts[1], wts, 1.0, shared, h, **ends)
+        y = MOE.moe_forward(x, idx, wts, f.experts)
+        return S.moe_combine_norm(y, self._row_ids(x.shape[0], x.device).view(-1, 1), None, 1.0, shared, h, **ends)
+
+    def _pass_start(self, i: int, ids):
+        """What the residual gets before layer run ``i``: (embedding table or None, ids, step vector) where it opens a pass, else None."""
+        st = self.cfg.pass_starts
+        if st is None or i >= len(st) or st[i] is None:
+            return None
+        return (self.embed if st[i] > 0 else None), ids, self.loop_step[st[i]]
+
     def _gla(self, lw: LayerWeights, x, fb: ForwardBatch, state, residual, next_ln):
         """Gated linear attention: merged [q | k | v | gate | decay rank] projection, the recurrence over the request's state with the
         head norm and the gate, output projection onto the residual."""
@@ -808,7 +897,8 @@ class DecoderModel:
         if c.residual_f32:
             if self.__dict__.get("_pos_freq") is None:
                 self._pos_freq = S.sinusoid_inv_freq(c.hidden_size, c.pos_embed_base, self.device) if c.pos_embed_base else None
-            h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps, pos_table=self.pos_table)
+            h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps, pos_table=self.pos_table,
+                                    add_vec=self.loop_step[0] if c.pass_starts is not None and c.pass_starts[0] is not None else None)
         else:
             h, x = self.embed_tokens(fb.ids), None
         if fb.embed_rows is not None:
@@ -833,6 +923,9 @@ class DecoderModel:
                 fa, fbeta, la, lbeta, ma, mbeta = c.resid_factors
                 alpha, self._beta = (la, lbeta) if lw.lin is not None else (fa, fbeta)
                 h = x * alpha if alpha != 1.0 else x
+            if c.mixers is not None and c.parallel_block:
+                h, x = self._parallel_layer(lw, x, fb, kv_caches[i], h, i)
+                continue
             if c.parallel_block:
                 h, _ = self._attention(lw.attn, x, fb, kv_caches[i], h, None, None)       # h + attention(x); the MLP reads x too
             elif c.mixers is not None:
@@ -1036,12 +1129,21 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
             run = cfg.layer_runs.index(i)                 # i names a layer's weights; its specs are listed per run
             sp, ff = cfg.mixers[run], cfg.ffs[run]
             if ff.kind == "none":
-                raw.pop(p + "post_attention_layernorm.weight")
+                raw.pop(p + "post_attention_layernorm.weight", None)
             ap = p + "self_attn."
             mk(ap + "q_proj.weight", (sp.heads * sp.dim, H))
-            mk(ap + "g_proj.weight", (sp.heads * sp.vdim, H))
+            gate = getattr(sp, "gate", "elem")
+            if gate:
+                mk(ap + "g_proj.weight", (sp.heads * (sp.vdim if gate == "elem" else 1), H))
             mk(ap + "o_proj.weight", (H, sp.heads * sp.vdim))
-            if isinstance(sp, GLASpec):
+            if isinstance(sp, MLSTMSpec):
+                mk(ap + "k_proj.weight", (sp.heads * sp.dim, H))
+                mk(ap + "v_proj.weight", (sp.heads * sp.vdim, H))
+                for nm, b in (("i_proj", 0.0), ("f_proj", 4.0)):
+                    mk(ap + nm + ".weight", (sp.heads, H))
+                    raw[ap + nm + ".bias"] = torch.full((sp.heads,), b, device=dev, dtype=dtype)
+                ones(ap + "o_norm.weight", sp.heads * sp.vdim)
+            elif isinstance(sp, GLASpec):
                 mk(ap + "k_proj.weight", (sp.heads * sp.dim, H))
                 mk(ap + "v_proj.weight", (sp.heads * sp.vdim, H))
                 mk(ap + "a1_proj.weight", (sp.rank, H))
@@ -1049,24 +1151,39 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
                 ones(ap + "a2_proj.bias", sp.heads * sp.dim)
                 ones(ap + "o_norm.weight", sp.vdim)
             elif isinstance(sp, AttnSpec):
-                ones(ap + "q_norm.weight", sp.dim)
-                if sp.kv_from is None:
+                own = sp.kv_from is None
+                if own:
                     mk(ap + "k_proj.weight", (sp.kv_heads * sp.dim, H))
                     mk(ap + "v_proj.weight", (sp.kv_heads * sp.vdim, H))
-                    ones(ap + "k_norm.weight", sp.dim)
+                for nm, n in (("q", sp.heads * sp.dim), ("k", sp.kv_heads * sp.dim), ("v", sp.kv_heads * sp.vdim)):
+                    if nm != "v" and sp.qk_norm and (own or nm == "q"):
+                        ones(ap + nm + "_norm.weight", sp.dim)
+                    if sp.bias and (own or nm == "q"):
+                        mk(ap + nm + "_proj.bias", (n,))
+                if sp.sinks:
+                    mk(ap + "sinks", (sp.heads,))
             else:
                 mk(ap + "kv_a_proj.weight", (sp.kv_rank, H))
                 ones(ap + "kv_a_layernorm.weight", sp.kv_rank)
                 mk(ap + "k_b_proj.weight", (sp.heads * sp.dim, sp.kv_rank))
                 mk(ap + "v_b_proj.weight", (sp.heads * sp.vdim, sp.kv_rank))
+            if cfg.side_dim:
+                mk(p + "per_layer_input_gate.weight", (cfg.side_dim, H))
+                mk(p + "per_layer_projection.weight", (H, cfg.side_dim))
+                ones(p + "post_per_layer_input_norm.weight", H)
             if ff.kind == "dense":
+                if ff.act == "geglu":
+                    mk(p + "mlp.gate_proj.weight", (ff.ff, H))
                 mk(p + "mlp.up_proj.weight", (ff.ff, H))
                 mk(p + "mlp.down_proj.weight", (H, ff.ff))
             elif ff.kind == "moe":
                 for nm, inter in [(f"mlp.experts.{e}.", ff.expert_ff) for e in range(ff.experts)] + ([("mlp.shared_experts.", ff.shared_ff)] if ff.shared_ff else []):
-                    mk(p + nm + "gate_proj.weight", (inter, H))
+                    if ff.act != "gelu":
+                        mk(p + nm + "gate_proj.weight", (inter, H))
                     mk(p + nm + "up_proj.weight", (inter, H))
                     mk(p + nm + "down_proj.weight", (H, inter))
+                if ff.shared_gate:
+                    mk(p + "mlp.shared_expert_gate.weight", (1, H))
                 if ff.router != "table":
                     mk(p + "mlp.gate.weight", (ff.experts, H))
                     return raw
@@ -1165,6 +1282,10 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
         mk("model.embed_tokens.weight", (cfg.vocab_size, H))
         if cfg.pos_table:
             mk("model.embed_positions.weight", (cfg.pos_table, H))
+        if cfg.pass_starts is not None:
+            mk("model.loop_step.weight", (1 + max(t for t in cfg.pass_starts if t is not None), H))
+        if cfg.side_dim:
+            mk("model.embed_tokens_per_layer.weight", (cfg.vocab_size, (1 + max(cfg.layer_runs)) * cfg.side_dim))
         ones("model.norm.weight", H)
         if cfg.norm_kind == "layernorm":
             mk("model.norm.bias", (H,))

@@ -30,8 +30,9 @@ _KERNEL_SIGS = {
     "fb_gemm_route": [P, P, I, I, I, I, I, I, P, P, P, I, I, I, F, P],
     "fb_gemm_16bit_batched": [P, P, P, I, I, I, I, I, I, I, I, I, I, P],
     "fb_gemm_16bit_batched_gate": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P],
-    "fb_gemm_16bit_res32": [P, P, P, P, I, I, I, I, I, I, I, F, I, P],
-    "fb_gemm_full32": [P, P, P, P, P, P, I, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, P, P, F, I, I, I, P],
+    "fb_gemm_full32": [P, P, P, P, P, P, I, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, P, P, F, I, I, P, LL, P, P, LL, I, I, P],
+    "fb_gemm_16bit_res32": [P, P, P, P, I, I, I, I, I, I, I, F, P, I, I, P],
+    "fb_gemm_16bit_act": [P, P, P, I, I, I, I, I, I, I, P, I, P, P, LL, I, I, P],
     "fb_mla_post": [P, I, P, I, P, I, P, P, P, P, P, P, I, I, I, I, I, I, LL, F, I, P],
     "fb_gemm_pick_split": [I, I, I, I],
     "fb_rmsnorm": [P, P, P, P, I, I, I, I, F, F, I, P],
@@ -46,7 +47,7 @@ _KERNEL_SIGS = {
     "fb_softmax_causal_rows": [P, I, P, I, I, I, I, I, F, I, P],
     "fb_embedding": [P, P, P, I, I, I, P],
     "fb_argmax": [P, P, P, I, I, I, I, I, P],
-    "fb_route_topk": [P, P, P, P, I, I, I, I, I, I, I, F, P],
+    "fb_route_topk": [P, P, P, P, I, I, I, I, I, I, I, F, I, I, P],
     "fb_attn_decode_plan": [P, I, P, P, I, P],
     "fb_attn_decode_plan_window": [P, I, P, P, I, I, P],
     "fb_attn_decode_opts": [P, P, P, P, I, P, P, P, P, P, P, I, I, I, I, LL, I, I, I, F, I, I, P, I, P, I, P, P, I, I, F, P, P],

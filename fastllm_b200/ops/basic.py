@@ -15,7 +15,7 @@ import torch.nn.functional as F
 
 from . import _lib, cpu
 
-GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32, GEMM_RELU2, GEMM_GLU_CLAMP = 1, 2, 4, 8, 32, 64
+GEMM_BIAS, GEMM_RESIDUAL, GEMM_SWIGLU, GEMM_OUT_F32, GEMM_RELU2, GEMM_GLU_CLAMP, GEMM_GEGLU, GEMM_GELU, GEMM_GELU_TANH = 1, 2, 4, 8, 32, 64, 128, 512, 1024
 
 
 def _ptr(t):
@@ -148,10 +148,20 @@ def _f32_split(w: torch.Tensor):
 _FULL32_CODE = {torch.float16: 0, torch.bfloat16: 1, torch.float32: 2}
 
 
-def linear_full32(x, w, bias=None, residual=None, alpha: float = 1.0, relu2: bool = False, gate=None, out=None, out_f32: bool = False,
-                  batch: int = 1, x_cols: int = 0, out_cols: int = 0, counts=None, offsets=None, n: int | None = None):
+ACTS32 = {"": 0, "relu2": 1, "gelu": 2, "gelu_tanh": 3}      # activation codes of the fp32 products
+
+
+def _table_args(t):
+    """Row stride and row count of a 2-D table."""
+    return (t.stride(0), t.shape[0]) if t is not None else (0, 0)
+
+
+def linear_full32(x, w, bias=None, residual=None, alpha: float = 1.0, act: str = "", gate=None, out=None, out_f32: bool = False,
+                  batch: int = 1, x_cols: int = 0, out_cols: int = 0, counts=None, offsets=None, n: int | None = None, row_gate=None, mul=None,
+                  mul_rows=None):
     """``x @ w.T`` in fp32 arithmetic on the CUDA cores for any size (float32 models, 16-bit shapes outside the tensor-core tiling),
-    with optional ReLU^2, gate ``* sigmoid(gate)`` and fp32 ``residual + alpha * ...``.  ``batch`` > 1: the slices of
+    with an optional activation (``ACTS32``), ``* sigmoid(row_gate)`` per row, ``* mul[mul_rows]``, gate ``* sigmoid(gate)`` and fp32
+    ``residual + alpha * ...``.  ``batch`` > 1: the slices of
     ``linear_batched``; with ``counts`` / ``offsets`` the rows of ``batch`` experts whose weights are stacked in ``w``
     (``n`` rows each are used, the stack's own stride is its row count over ``batch``)."""
     flush_pending_wait()
@@ -164,7 +174,9 @@ def linear_full32(x, w, bias=None, residual=None, alpha: float = 1.0, relu2: boo
     rc = _lib.kernels().fb_gemm_full32(_ptr(x), _ptr(w2), _ptr(out), _ptr(bias), _ptr(residual), _ptr(gate), M, N, K, batch, x.stride(0),
                                        w2.stride(0), out.stride(0), residual.stride(0) if residual is not None else 0,
                                        gate.stride(0) if gate is not None else 0, rows_w, x_cols, out_cols, _ptr(counts), _ptr(offsets),
-                                       float(alpha), 1 if relu2 else 0, 1 if out.dtype == torch.float32 else 0, _FULL32_CODE[x.dtype], _stream())
+                                       float(alpha), ACTS32[act], 1 if out.dtype == torch.float32 else 0, _ptr(row_gate),
+                                       row_gate.stride(0) if row_gate is not None else 0, _ptr(mul), _ptr(mul_rows),
+                                       *_table_args(mul), _FULL32_CODE[x.dtype], _stream())
     _lib.check(rc, "fb_gemm_full32")
     return out
 
@@ -175,28 +187,68 @@ def tc_operands_ok(x, w) -> bool:
                 and x.stride(-1) == 1 and not (x.data_ptr() & 15) and (x.stride(0) * 2) % 16 == 0 and w.is_contiguous())
 
 
-def linear_res32(x, w, h, alpha: float):
-    """fp32 residual stream: ``h += alpha * (x @ w.T)`` in place, in the GEMM's epilogue."""
+def linear_res32(x, w, h, alpha: float, copy=None):
+    """fp32 residual stream: ``h += alpha * (x @ w.T)`` in place, in the GEMM's epilogue; ``copy``: receives the new residual in 16 bits."""
     if not x.is_cuda:
         flush_pending_wait()
         h += alpha * (x.float() @ w.float().t())
+        if copy is not None:
+            copy.copy_(h)
         return h
     M, N, K = x.shape[0], w.shape[0], w.shape[1]
     if not tc_operands_ok(x, w):
-        return linear_full32(x, w, residual=h, alpha=alpha, out=h)
+        linear_full32(x, w, residual=h, alpha=alpha, out=h)
+        if copy is not None:
+            copy.copy_(h)
+        return h
     flush_pending_wait()
     step = M if (M <= 256 or N % 32 == 0) else 256
     for m0 in range(0, M, step):
         m1 = min(M, m0 + step)
         rc = _lib.kernels().fb_gemm_16bit_res32(_ptr(x[m0:m1]), _ptr(w), _ptr(h[m0:m1]), _ptr(h[m0:m1]), m1 - m0, N, K, x.stride(0), w.stride(0),
-                                                h.stride(0), h.stride(0), float(alpha), dtype_code(x.dtype), _stream())
+                                                h.stride(0), h.stride(0), float(alpha), _ptr(copy[m0:m1] if copy is not None else None),
+                                                copy.stride(0) if copy is not None else 0, dtype_code(x.dtype), _stream())
         _lib.check(rc, "fb_gemm_16bit_res32")
     return h
 
 
+def act_ref(y, act: str):
+    """fp32 rows through one of ``ACTS32``."""
+    if act == "relu2":
+        return torch.relu(y).square()
+    return F.gelu(y, approximate="tanh" if act == "gelu_tanh" else "none") if act else y
+
+
+def linear_act(x, w, act: str, out=None, row_gate=None, mul=None, mul_rows=None):
+    """``act(x @ w.T)`` (``ACTS32``), times the sigmoid of one fp32 logit per row (``row_gate`` [M]) or times row ``mul_rows[m]`` of the table
+    ``mul`` [rows, >= N]; all in the GEMM's epilogue."""
+    M, (N, K) = x.shape[0], w.shape
+    if out is None:
+        out = torch.empty((M, N), device=x.device, dtype=x.dtype)
+    if not x.is_cuda:
+        flush_pending_wait()
+        y = act_ref(x.float() @ w.float().t(), act)
+        y = y * torch.sigmoid(row_gate.float())[:, None] if row_gate is not None else y
+        return out.copy_(y * mul[mul_rows.long(), :N].float() if mul is not None else y)
+    if act == "relu2" or not tc_operands_ok(x, w):
+        return linear_full32(x, w, act=act, out=out, row_gate=row_gate, mul=mul, mul_rows=mul_rows)
+    flush_pending_wait()
+    flags = {"": 0, "gelu": GEMM_GELU, "gelu_tanh": GEMM_GELU_TANH}[act]
+    step = M if (M <= 256 or N % 32 == 0) else 256
+    for m0 in range(0, M, step):
+        m1 = min(M, m0 + step)
+        rc = _lib.kernels().fb_gemm_16bit_act(_ptr(x[m0:m1]), _ptr(w), _ptr(out[m0:m1]), m1 - m0, N, K, x.stride(0), w.stride(0), out.stride(0), flags,
+                                              _ptr(row_gate[m0:m1] if row_gate is not None else None), row_gate.stride(0) if row_gate is not None else 0,
+                                              _ptr(mul), _ptr(mul_rows[m0:m1] if mul is not None else None), *_table_args(mul),
+                                              dtype_code(x.dtype), _stream())
+        _lib.check(rc, "fb_gemm_16bit_act")
+    return out
+
+
 def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: bool = False, interleaved: bool = True,
-           out_f32: bool = False, out: torch.Tensor | None = None, nsplit: int = 0, relu2: bool = False) -> torch.Tensor:
-    """``y = x @ w.T`` with optional fused bias, SwiGLU (``w`` = gate/up stacked) or ReLU^2, and residual add.
+           out_f32: bool = False, out: torch.Tensor | None = None, nsplit: int = 0, relu2: bool = False, geglu: bool = False) -> torch.Tensor:
+    """``y = x @ w.T`` with optional fused bias, SwiGLU (``w`` = gate/up stacked; ``geglu``: tanh-form GELU in place of SiLU, 16-bit CUDA
+    tensors) or ReLU^2, and residual add.
 
     x: ``[M, K]`` (row stride may exceed K), w: ``[N, K]``.  16-bit CUDA tensors run the tcgen05 GEMM.
     """
@@ -239,8 +291,8 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: b
     if K % 8 != 0 or N % 8 != 0 or x.dtype not in (torch.float16, torch.bfloat16) or (x2.data_ptr() & 15) or (x2.stride(0) * 2) % 16:
         # shapes outside the tensor-core kernels' tiling (rare: odd projection widths): plain PyTorch definition
         flush_pending_wait()
-        if not swiglu and residual is None and x.dtype == w.dtype and x.dtype in _FULL32_CODE and w.is_contiguous() and out is None and bias is None:
-            return linear_full32(x2, w, out_f32=out_f32).reshape(*lead, N)
+        if not swiglu and residual is None and x.dtype == w.dtype and x.dtype in _FULL32_CODE and w.is_contiguous() and out is None:
+            return linear_full32(x2, w, bias, out_f32=out_f32).reshape(*lead, N)
         return linear_ref(x, w, bias, residual, swiglu, interleaved, torch.float32 if out_f32 else None)
     if swiglu and not interleaved:
         raise ValueError("CUDA SwiGLU epilogue needs tile-interleaved gate/up weights (interleave_gate_up)")
@@ -248,7 +300,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias=None, residual=None, swiglu: b
     if out is None:
         out = torch.empty((M, n_out), device=x.device, dtype=torch.float32 if out_f32 else x.dtype)
     flags = (GEMM_BIAS if bias is not None else 0) | (GEMM_RESIDUAL if residual is not None else 0) | \
-            (GEMM_SWIGLU if swiglu else 0) | (GEMM_OUT_F32 if out_f32 else 0) | (GEMM_RELU2 if relu2 else 0)
+            (GEMM_SWIGLU | (GEMM_GEGLU if geglu else 0) if swiglu else 0) | (GEMM_OUT_F32 if out_f32 else 0) | (GEMM_RELU2 if relu2 else 0)
     res2 = residual.reshape(-1, residual.shape[-1]) if residual is not None else None
     lib = _lib.kernels()
     dt = dtype_code(x.dtype)

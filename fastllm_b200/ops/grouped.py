@@ -1,5 +1,6 @@
-"""Grouped-query attention of listed layers: any head widths, per-head query / key norms, interleaved rotary positions on part of a
-head, a chunk mask (a query sees the keys of its own chunk of positions) or a sliding window, an elementwise sigmoid gate on the heads.
+"""Grouped-query attention of listed layers: any head widths; optionally biases, per-head query / key norms, rotary positions on part
+of a head (interleaved pairs or halves), a chunk mask (a query sees the keys of its own chunk of positions) or a sliding window that may
+keep the first tokens of the sequence, soft-capped scores, a sink per head, and a sigmoid gate per element or per head.
 
 One launch normalises, rotates and writes the new keys and values to their cache slots (``csrc/stream32.cu``).  Rows are then attended
 in one of two ways, chosen per request of a batch:
@@ -19,16 +20,16 @@ import torch
 from . import _lib
 from . import latent as LA
 from . import stream32 as S
-from .attention import ROPE_INTERLEAVED, apply_rope_ref
+from .attention import ROPE_INTERLEAVED, ROPE_NEOX, apply_rope_ref
 from .basic import _ptr, _stream, dtype_code
 
 P, I, F, LL = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _lib.register_sigs({
-    "fb_head_norm_rope": [P, LL, P, P, I, I, I, I, I, I, I, I, I, P, P, P, P, I, I, P, P, F, I, P],
-    "fb_grouped_plan": [P, I, I, I, P, P, I, P],
-    "fb_grouped_decode": [P, LL, P, P, P, LL, P, LL, P, P, P, P, P, P, I, I, I, I, I, LL, I, I, I, I, I, F, I, P],
-    "fb_grouped_attn32": [P, LL, P, P, P, LL, P, LL, P, P, I, I, I, I, I, I, I, I, I, I, I, F, I, P],
-    "fb_attn_window_paged": [P, LL, I, P, P, LL, P, I, P, LL, P, LL, P, I, I, I, I, I, I, I, F, I, P],
+    "fb_head_norm_rope": [P, LL, P, P, I, I, I, I, I, I, I, I, I, I, P, P, P, P, I, I, P, P, F, I, P],
+    "fb_grouped_plan": [P, I, I, I, I, P, P, I, P],
+    "fb_grouped_decode": [P, LL, P, P, P, LL, P, LL, P, P, P, P, P, P, I, I, I, I, I, LL, I, I, I, I, I, I, F, F, P, P, LL, I, P],
+    "fb_grouped_attn32": [P, LL, P, P, P, LL, P, LL, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P, LL, I, P],
+    "fb_attn_window_paged": [P, LL, I, P, P, LL, P, I, P, LL, P, LL, P, I, I, I, I, I, I, I, I, F, F, P, P, LL, I, P],
 }, ["attn_grouped"])
 
 ROW_TOKENS = 16                  # requests that bring at most this many tokens take the decode kernel, a row each
@@ -41,11 +42,16 @@ class GroupedWeights:
 
     def __init__(self):
         self.heads = self.kv_heads = self.dim = self.vdim = self.dp = self.vp = 0
-        self.window = self.chunk = self.rot = 0
+        self.window = self.keep = self.chunk = self.rot = 0
+        self.rope_mode = ROPE_INTERLEAVED
         self.scale = 1.0
+        self.softcap = 0.0
         self.own_kv = True       # False: keys and values come from another layer's cache
-        self.in_proj = None      # rows [queries | gate | keys | values]
+        self.gate = "elem"       # "elem": columns of the projection; "head": fp32 logits handed to ``attention``; "": none
+        self.in_proj = None      # rows [queries | elementwise gate | keys | values]
+        self.in_bias = None      # its bias, where the layer has one
         self.q_norm = self.k_norm = None
+        self.sinks = None        # fp32 [heads]
 
     @property
     def gate_col(self) -> int:
@@ -53,29 +59,40 @@ class GroupedWeights:
 
     @property
     def k_col(self) -> int:
-        return self.gate_col + self.heads * self.vp
+        return self.gate_col + (self.heads * self.vp if self.gate == "elem" else 0)
 
     @property
     def v_col(self) -> int:
         return self.k_col + self.kv_heads * self.dp
 
 
-def build(spec, q, k, v, g, q_norm, k_norm):
-    """(GroupedWeights without ``in_proj``, merged input projection matrix) from the layer's matrices; ``k`` None: no own keys."""
+def build(spec, q, k, v, g, q_norm, k_norm, biases=None, sinks=None):
+    """(GroupedWeights without ``in_proj``, merged input projection matrix) from the layer's matrices; ``k`` None: no own keys; ``g``
+    None: no elementwise gate; ``biases``: those of q, k and v."""
     w = GroupedWeights()
     w.heads, w.kv_heads, w.dim, w.vdim = spec.heads, spec.kv_heads, spec.dim, spec.vdim
     w.dp, w.vp = LA._round8(spec.dim), LA._round8(spec.vdim)
     w.chunk, w.scale, w.own_kv = int(spec.chunk or 0), float(spec.scale), k is not None
+    w.window, w.keep, w.softcap, w.gate = int(spec.window or 0), int(spec.keep or 0) if spec.window else 0, float(spec.softcap or 0.0), spec.gate
     w.rot = int(spec.rope["rot_dim"]) if spec.rope else 0
+    w.rope_mode = ROPE_NEOX if spec.rope and spec.rope.get("mode") == "neox" else ROPE_INTERLEAVED
     w.q_norm, w.k_norm = q_norm, k_norm
-    parts = [LA._pad_heads(q, w.heads, w.dp), LA._pad_heads(g, w.heads, w.vp)]
-    if k is not None:
-        parts += [LA._pad_heads(k, w.kv_heads, w.dp), LA._pad_heads(v, w.kv_heads, w.vp)]
-    return w, LA.pad_rows(torch.cat(parts, dim=0), 32)
+    w.sinks = sinks.float().contiguous() if sinks is not None else None
+
+    def merge(q, g, k, v):
+        parts = [LA._pad_heads(q, w.heads, w.dp)] + ([LA._pad_heads(g, w.heads, w.vp)] if g is not None else [])
+        if k is not None:
+            parts += [LA._pad_heads(k, w.kv_heads, w.dp), LA._pad_heads(v, w.kv_heads, w.vp)]
+        return LA.pad_rows(torch.cat(parts, dim=0), 32)
+
+    if biases is not None:
+        bq, bk, bv = (b[:, None] if b is not None else None for b in biases)
+        w.in_bias = merge(bq, bq.new_zeros((w.heads * w.vp, 1)) if g is not None else None, bk, bv)[:, 0].contiguous()
+    return w, merge(q, g, k, v)
 
 
 def first_key(pos, window: int, chunk: int):
-    """First position a query at ``pos`` sees (tensors or integers)."""
+    """First position of the chunk or window of a query at ``pos`` (tensors or integers)."""
     if chunk:
         return pos - pos % chunk
     if window:
@@ -84,22 +101,23 @@ def first_key(pos, window: int, chunk: int):
 
 
 def post(w: GroupedWeights, proj, fb, kv, cos, sin, eps: float) -> None:
-    """Norm and rotation of the queries and keys in ``proj`` (in place; fp32 arithmetic) and the new keys and values into their cache
-    slots (rows with a negative slot are not cached)."""
+    """Norm and rotation, where the layer has them, of the queries and keys in ``proj`` (in place; fp32 arithmetic) and the new keys and
+    values into their cache slots (rows with a negative slot are not cached)."""
     T = proj.shape[0]
     k_pool, v_pool = kv
     if proj.is_cuda:
         G = w.kv_heads if w.own_kv else 0
         rc = _lib.kernels().fb_head_norm_rope(_ptr(proj), proj.stride(0), _ptr(fb.positions), _ptr(fb.slots), T, w.heads, G, w.dim, w.dp, w.vp, w.k_col,
-                                              w.v_col, w.rot, _ptr(w.q_norm), _ptr(w.k_norm), _ptr(cos), _ptr(sin), cos.shape[0] if cos is not None else 0,
+                                              w.v_col, w.rot, 1 if w.rope_mode == ROPE_NEOX else 0, _ptr(w.q_norm), _ptr(w.k_norm), _ptr(cos), _ptr(sin), cos.shape[0] if cos is not None else 0,
                                               k_pool.shape[0] * k_pool.shape[1], _ptr(k_pool), _ptr(v_pool), float(eps), S.act_code(proj.dtype), _stream())
         _lib.check(rc, "fb_head_norm_rope")
         return
 
     def turn(col, heads, norm_w):
-        x = proj[:, col:col + heads * w.dp].reshape(T, heads, w.dp)
-        x[..., :w.dim] = S._rms(x[..., :w.dim].float(), norm_w, eps).to(x.dtype)
-        return apply_rope_ref(x, fb.positions, cos, sin, ROPE_INTERLEAVED, w.rot) if w.rot else x
+        x = proj[:, col:col + heads * w.dp].reshape(T, heads, w.dp).clone()
+        if norm_w is not None:
+            x[..., :w.dim] = S._rms(x[..., :w.dim].float(), norm_w, eps).to(x.dtype)
+        return apply_rope_ref(x, fb.positions, cos, sin, w.rope_mode, w.rot) if w.rot else x
 
     proj[:, :w.gate_col] = turn(0, w.heads, w.q_norm).reshape(T, -1)
     if w.own_kv:
@@ -120,7 +138,7 @@ class GroupedPlan:
         self.kv_lens = None
         self.blocks = None           # prefill query blocks: (packed row, position, rows, 0, 0, request)
         self.n_blocks = 0
-        self.lists: dict = {}        # (window, chunk, first row) -> work list of the decode kernel
+        self.lists: dict = {}        # (window, keep, chunk, first row) -> work list of the decode kernel
 
 
 def build_plan(fb, prefill: bool) -> GroupedPlan:
@@ -174,7 +192,7 @@ def prefill_ok(w, dtype, page_len: int) -> bool:
 def _splits(w, max_pages: int, page_len: int) -> int:
     """Most pages one query's visible keys touch."""
     span = w.chunk or w.window
-    return min(max_pages, (span + page_len - 2) // page_len + 1) if span else max_pages
+    return min(max_pages, (span + page_len - 2) // page_len + 1 + (w.keep + page_len - 1) // page_len) if span else max_pages
 
 
 _SCRATCH: dict = {}
@@ -190,65 +208,78 @@ def _scratch(dev, n: int, kind: str):
     return t
 
 
-def decode_rows(w, pl: GroupedPlan, q, gate, kv, page_table, kv_lens, out, row0: int = 0) -> None:
-    """Rows ``q`` [n, heads * dp] against their own page-table rows; gated heads to ``out`` [n, heads * vp] (row strides free)."""
+def _gate_args(gate):
+    return _ptr(gate), gate.stride(0) if gate is not None else 0
+
+
+def decode_rows(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, kv_lens, out, row0: int = 0) -> None:
+    """Rows ``q`` [n, heads * dp] against their own page-table rows; gated heads to ``out`` [n, heads * vp] (row strides free).  ``gate``
+    [n, heads * vp] and ``head_gate`` (fp32 [n, heads]): None where the layer has no such gate."""
     k_pool, v_pool = kv
     n, page_len, max_pages, lib = q.shape[0], k_pool.shape[1], page_table.shape[1], _lib.kernels()
     slots = k_pool.shape[0] * page_len
     if not decode_ok(w, q.dtype, page_len):
-        rc = lib.fb_grouped_attn32(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), _ptr(gate), gate.stride(0),
+        rc = lib.fb_grouped_attn32(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), *_gate_args(gate),
                                    _ptr(page_table), _ptr(kv_lens), n, w.heads, w.kv_heads, w.dim, w.dp, w.vp, page_table.stride(0), k_pool.shape[0],
-                                   page_len, w.window, w.chunk, w.scale, S.act_code(q.dtype), _stream())
+                                   page_len, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks), *_gate_args(head_gate), S.act_code(q.dtype),
+                                   _stream())
         _lib.check(rc, "fb_grouped_attn32")
         return
     if n > _MAX_ROWS:
         for i in range(0, n, _MAX_ROWS):
             s = slice(i, i + _MAX_ROWS)
-            decode_rows(w, pl, q[s], gate[s], kv, page_table[s], kv_lens[s], out[s], row0 + i)
+            decode_rows(w, pl, q[s], gate[s] if gate is not None else None, head_gate[s] if head_gate is not None else None, kv, page_table[s],
+                        kv_lens[s], out[s], row0 + i)
         return
     splits = _splits(w, max_pages, page_len)
-    key = (w.window, w.chunk, row0)
+    key = (w.window, w.keep, w.chunk, row0)
     lst = pl.lists.get(key)
     if lst is None:
         lst = pl.lists[key] = torch.empty((2 * n * splits + 1,), device=q.device, dtype=torch.int32)
-        _lib.check(lib.fb_grouped_plan(_ptr(kv_lens), n, w.window, w.chunk, _ptr(lst[1:]), _ptr(lst), n * splits, _stream()), "fb_grouped_plan")
+        _lib.check(lib.fb_grouped_plan(_ptr(kv_lens), n, w.window, w.chunk, w.keep, _ptr(lst[1:]), _ptr(lst), n * splits, _stream()), "fb_grouped_plan")
     part_o, part_ml = _scratch(q.device, n * w.heads * splits * w.vp, "o"), _scratch(q.device, n * w.heads * splits * 2, "ml")
-    rc = lib.fb_grouped_decode(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), _ptr(gate), gate.stride(0), _ptr(page_table),
+    rc = lib.fb_grouped_decode(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), *_gate_args(gate), _ptr(page_table),
                                _ptr(kv_lens), _ptr(lst[1:]), _ptr(lst), _ptr(part_o), _ptr(part_ml), n, w.heads, w.kv_heads, w.dp, w.vp, slots,
-                               page_table.stride(0), splits, n * splits, w.window, w.chunk, w.scale, dtype_code(q.dtype), _stream())
+                               page_table.stride(0), splits, n * splits, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks), *_gate_args(head_gate),
+                               dtype_code(q.dtype), _stream())
     _lib.check(rc, "fb_grouped_decode")
 
 
-def prefill_blocks(w, pl: GroupedPlan, q, gate, kv, page_table, out) -> None:
+def prefill_blocks(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, out) -> None:
     k_pool, v_pool = kv
     rc = _lib.kernels().fb_attn_window_paged(_ptr(q), q.stride(0), q.shape[0], _ptr(k_pool), _ptr(v_pool), k_pool.shape[0] * k_pool.shape[1],
-                                             _ptr(page_table), page_table.stride(0), _ptr(out), out.stride(0), _ptr(gate), gate.stride(0), _ptr(pl.blocks),
-                                             pl.n_blocks, w.heads, w.kv_heads, w.dp, w.vp, w.window, w.chunk, w.scale, dtype_code(q.dtype), _stream())
+                                             _ptr(page_table), page_table.stride(0), _ptr(out), out.stride(0), *_gate_args(gate), _ptr(pl.blocks),
+                                             pl.n_blocks, w.heads, w.kv_heads, w.dp, w.vp, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks),
+                                             *_gate_args(head_gate), dtype_code(q.dtype), _stream())
     _lib.check(rc, "fb_attn_window_paged")
 
 
-def attention(w: GroupedWeights, proj, kv, fb):
-    """``proj`` after ``post`` (the new keys and values are cached already) -> gated heads ``[T, heads * vp]``."""
+def attention(w: GroupedWeights, proj, kv, fb, out=None, head_gate=None):
+    """``proj`` after ``post`` (the new keys and values are cached already) -> gated heads ``[T, heads * vp]`` (``out``, where given).
+    ``head_gate``: fp32 logits [T, heads] of a layer with one gate per head."""
     T = proj.shape[0]
-    q, gate = proj[:, :w.gate_col], proj[:, w.gate_col:w.k_col]
+    q, gate = proj[:, :w.gate_col], proj[:, w.gate_col:w.k_col] if w.gate == "elem" else None
     if not proj.is_cuda:
-        return attention_ref(w, q, gate, kv, fb)
-    out = torch.empty((T, w.heads * w.vp), device=proj.device, dtype=proj.dtype)
+        y = attention_ref(w, q, gate, kv, fb, head_gate)
+        return y if out is None else out.copy_(y)
+    if out is None:
+        out = torch.empty((T, w.heads * w.vp), device=proj.device, dtype=proj.dtype)
     pl = _plan(fb, prefill_ok(w, proj.dtype, kv[0].shape[1]) and not fb.is_decode)
     if pl.n_rows and pl.rows is None:
-        decode_rows(w, pl, q, gate, kv, pl.page_table, pl.kv_lens, out)
+        decode_rows(w, pl, q, gate, head_gate, kv, pl.page_table, pl.kv_lens, out)
     elif pl.n_rows:
         part = torch.empty((pl.n_rows, w.heads * w.vp), device=proj.device, dtype=proj.dtype)
-        sub = proj.index_select(0, pl.rows)
-        decode_rows(w, pl, sub[:, :w.gate_col], sub[:, w.gate_col:w.k_col], kv, pl.page_table, pl.kv_lens, part)
+        sub = proj[:, :w.k_col].index_select(0, pl.rows)
+        decode_rows(w, pl, sub[:, :w.gate_col], sub[:, w.gate_col:] if gate is not None else None,
+                    head_gate.index_select(0, pl.rows) if head_gate is not None else None, kv, pl.page_table, pl.kv_lens, part)
     if pl.n_blocks:
-        prefill_blocks(w, pl, q, gate, kv, fb.page_table, out)
+        prefill_blocks(w, pl, q, gate, head_gate, kv, fb.page_table, out)
     if pl.n_rows and pl.rows is not None:
         out.index_copy_(0, pl.rows, part)
     return out
 
 
-def attention_ref(w, q, gate, kv, fb):
+def attention_ref(w, q, gate, kv, fb, head_gate=None):
     """PyTorch evaluation over the pages (CPU tensors)."""
     T, H, G = q.shape[0], w.heads, w.kv_heads
     k_pool, v_pool = kv
@@ -263,7 +294,15 @@ def attention_ref(w, q, gate, kv, fb):
         k = k_pool[pages].reshape(-1, G, w.dp)[:L].float().repeat_interleave(H // G, dim=1)
         v = v_pool[pages].reshape(-1, G, w.vp)[:L].float().repeat_interleave(H // G, dim=1)
         qpos, kpos = torch.arange(L - (r1 - r0), L)[:, None], torch.arange(L)[None, :]
-        see = (kpos <= qpos) & (kpos >= first_key(qpos, w.window, w.chunk))
+        see = (kpos <= qpos) & ((kpos >= first_key(qpos, w.window, w.chunk)) | (kpos < w.keep))
         s = torch.einsum("qhd,khd->hqk", q[r0:r1].float().reshape(-1, H, w.dp), k) * w.scale
-        out[r0:r1] = torch.einsum("hqk,khv->qhv", torch.softmax(s.masked_fill(~see, float("-inf")), dim=-1), v)
-    return (out.reshape(T, -1) * torch.sigmoid(gate.float())).to(q.dtype)
+        if w.softcap:
+            s = torch.tanh(s / w.softcap) * w.softcap
+        s = s.masked_fill(~see, float("-inf"))
+        if w.sinks is not None:
+            s = torch.cat([s, w.sinks.view(H, 1, 1).expand(-1, s.shape[1], 1)], dim=-1)
+        out[r0:r1] = torch.einsum("hqk,khv->qhv", torch.softmax(s, dim=-1)[..., :L], v)
+    if head_gate is not None:
+        out = out * torch.sigmoid(head_gate.float())[..., None]
+    out = out.reshape(T, -1)
+    return (out * torch.sigmoid(gate.float()) if gate is not None else out).to(q.dtype)

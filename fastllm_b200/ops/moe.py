@@ -22,7 +22,7 @@ from .quant import LinearWeight
 
 
 # ---------------------------------------------------------------------------------------------------
-def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0):
+def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0, group_max=False):
     lf = logits.float()
     if score_mode == 0:
         sc = torch.softmax(lf, dim=-1)
@@ -33,7 +33,8 @@ def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group
     sel = sc + bias.float() if bias is not None else sc.clone()
     M, E = sc.shape
     if n_group > 1 and topk_group < n_group:
-        gs = sel.view(M, n_group, E // n_group).topk(2, dim=-1)[0].sum(-1)
+        per = sel.view(M, n_group, E // n_group)
+        gs = per.amax(-1) if group_max else per.topk(2, dim=-1)[0].sum(-1)
         gidx = gs.topk(topk_group, dim=-1)[1]
         gmask = torch.zeros_like(gs).scatter_(1, gidx, 1.0)
         emask = gmask[:, :, None].expand(M, n_group, E // n_group).reshape(M, E)
@@ -45,17 +46,19 @@ def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group
     return idx.to(torch.int32), (w * route_scale).float()
 
 
-def route_topk(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0):
-    """logits fp32 ``[M, E]`` -> (expert index int32 ``[M, topk]``, weight fp32 ``[M, topk]``)."""
-    if not logits.is_cuda or logits.shape[1] > 512 or topk > 32:        # beyond the kernel's registers: tensor ops
-        return route_topk_ref(logits, bias, topk, score_mode, renorm, n_group, topk_group, route_scale)
-    lg = logits.float().contiguous()
+def route_topk(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0, group_max=False):
+    """logits fp32 ``[M, E]`` -> (expert index int32 ``[M, topk]``, weight fp32 ``[M, topk]``).  ``group_max``: a group's score is its largest
+    score (else the sum of its two largest)."""
+    if not logits.is_cuda or logits.shape[1] > 512 or topk > 32 or n_group > 32:        # beyond the kernel's registers: tensor ops
+        return route_topk_ref(logits, bias, topk, score_mode, renorm, n_group, topk_group, route_scale, group_max)
+    lg = logits.float()
+    lg = lg if lg.stride(1) == 1 else lg.contiguous()
     M, E = lg.shape
     idx = torch.empty((M, topk), device=lg.device, dtype=torch.int32)
     w = torch.empty((M, topk), device=lg.device, dtype=torch.float32)
     b = bias.float().contiguous() if bias is not None else None
     rc = _lib.kernels().fb_route_topk(_ptr(lg), _ptr(b), _ptr(idx), _ptr(w), M, E, topk, score_mode, 1 if renorm else 0,
-                                      n_group, topk_group, float(route_scale), _stream())
+                                      n_group, topk_group, float(route_scale), lg.stride(0), 1 if group_max else 0, _stream())
     _lib.check(rc, "fb_route_topk")
     return idx, w
 
@@ -158,7 +161,8 @@ def route_group_top1(logits, groups: int, expert_scale=None):
 
 # ---------------------------------------------------------------------------------------------------
 class ExpertWeights:
-    """Routed experts owned by this rank: per-expert gate/up (tile-interleaved) and down weights."""
+    """Routed experts owned by this rank: per-expert gate/up (tile-interleaved) and down weights.  Experts without a gate branch
+    (``act`` "gelu", the exact form) have their up matrices in the place of gate/up."""
 
     def __init__(self, num_experts_total: int, first: int, gate_up: list[LinearWeight], down: list[LinearWeight]):
         self.total = num_experts_total
@@ -167,7 +171,7 @@ class ExpertWeights:
         self.gate_up = gate_up
         self.down = down
         self.stacked = None     # filled by ops.moe_grouped when a grouped kernel can take the whole set
-        self.act = "swiglu"     # "gptoss": clamped gate/up, gate * sigmoid(1.702 gate) * (up + 1); "swiglu_clamp": see limit
+        self.act = "swiglu"     # "gelu": no gate branch; "gptoss": clamped gate/up, gate * sigmoid(1.702 gate) * (up + 1); "swiglu_clamp": see limit
         self.limit = 0.0        # "swiglu_clamp" (Step-3.5): min(silu(gate), limit) * clamp(up, -limit, limit); "gptoss": its clamp (0: 7)
         self.scale_input = False    # an expert reads w * x (and its result is added as it is)
         self.host = False       # expert weights live in CPU memory and run on the native CPU backend (hybrid placement)
@@ -225,7 +229,7 @@ def moe_forward(x, idx, wts, experts: ExpertWeights, ep=None):
     """
     if experts.host and experts.act == "swiglu":
         return _moe_forward_host(x, idx, wts, experts)
-    if experts.stacked is not None and x.is_cuda and experts.act == "swiglu" and not experts.scale_input:
+    if experts.stacked is not None and x.is_cuda and experts.act in ("swiglu", "gelu") and not experts.scale_input:
         from . import moe_grouped
 
         y = moe_grouped.forward(x, idx, wts, experts)
@@ -251,7 +255,9 @@ def moe_forward(x, idx, wts, experts: ExpertWeights, ep=None):
         le = e - experts.first
         if experts.scale_input:
             xe = (xe.float() * w_sorted[start:start + n, None]).to(x.dtype)
-        if experts.act == "gptoss":
+        if experts.act == "gelu":
+            he = experts.down[le](experts.gate_up[le].activated(xe, "gelu"))
+        elif experts.act == "gptoss":
             he = experts.down[le](glu_gptoss(experts.gate_up[le](xe), experts.gate_up[le].interleaved, experts.limit or 7.0))
         elif experts.act == "swiglu_clamp":
             he = experts.down[le](glu_clamped(experts.gate_up[le](xe), experts.gate_up[le].interleaved, experts.limit))

@@ -15,7 +15,7 @@ import torch
 from . import _lib
 from . import basic as B
 from . import quant_gemm as QG
-from .basic import GEMM_GLU_CLAMP, GEMM_SWIGLU, _ptr, _stream, dtype_code
+from .basic import GEMM_GELU, GEMM_GLU_CLAMP, GEMM_SWIGLU, _ptr, _stream, dtype_code
 from .stream32 import moe_gather_scaled
 
 P, I = ctypes.c_void_p, ctypes.c_int
@@ -35,7 +35,8 @@ GPTOSS_ALPHA = 1.702             # g * sigmoid(alpha g) * (u + 1)
 
 
 class StackedExperts:
-    """Expert weights of one layer stacked along the row dim; quantised kinds carry stacked scales in kernel layout."""
+    """Expert weights of one layer stacked along the row dim; quantised kinds carry stacked scales in kernel layout.  ``gate_up`` holds
+    2 * ``inter`` rows an expert, or (no gate branch) ``inter`` rows in a multiple of 128."""
 
     def __init__(self, kind, gate_up, down, n_local, inter, hidden, group=0, gu_scale=None, gu_zero=None, dn_scale=None, dn_zero=None):
         self.kind, self.gate_up, self.down, self.n_local, self.inter, self.hidden, self.group = kind, gate_up, down, n_local, inter, hidden, group
@@ -78,11 +79,25 @@ def _stack_scales(ws):
     return scale, zero
 
 
+def _stack_rows(ws):
+    """The matrices of all experts, a multiple of 128 rows apart (a weight tile is 128 output rows of one expert)."""
+    n, k = ws[0].n, ws[0].k
+    out = torch.zeros((len(ws), (n + 127) // 128 * 128, k), dtype=ws[0].w.dtype, device=ws[0].w.device)
+    for e, w in enumerate(ws):
+        out[e, :n] = w.w
+    return out.view(-1, k)
+
+
 def stack_experts(experts) -> StackedExperts | None:
     gu, dn = experts.gate_up, experts.down
     if not gu:
         return None
     kind = gu[0].kind
+    if experts.act == "gelu":
+        inter, hidden = gu[0].n, gu[0].k
+        if kind != "dense" or inter % 8 or hidden % 8 or any(w.kind != kind or w.bias is not None for w in gu + dn):
+            return None
+        return StackedExperts(kind, _stack_rows(gu), _stack_rows(dn), len(gu), inter, hidden)
     if any(w.kind != kind or not w.interleaved or w.bias is not None for w in gu) or any(w.kind != kind or w.bias is not None for w in dn):
         return None
     two_i, hidden = gu[0].n, gu[0].k
@@ -90,12 +105,7 @@ def stack_experts(experts) -> StackedExperts | None:
         return None
     g = torch.cat([w.w for w in gu], dim=0).contiguous()
     if kind == "dense":
-        # a weight tile is 128 output rows of one expert: the down matrices are stacked a multiple of 128 rows apart
-        hp = (hidden + 127) // 128 * 128
-        d = torch.zeros((len(dn), hp, two_i // 2), dtype=dn[0].w.dtype, device=dn[0].w.device)
-        for e, w in enumerate(dn):
-            d[e, :hidden] = w.w
-        return StackedExperts(kind, g, d.view(len(dn) * hp, two_i // 2), len(gu), two_i // 2, hidden)
+        return StackedExperts(kind, g, _stack_rows(dn), len(gu), two_i // 2, hidden)
     d = torch.cat([w.w for w in dn], dim=0).contiguous()
     if kind == "int4g" and (gu[0].group % 64 != 0 or hidden % gu[0].group != 0 or (two_i // 2) % gu[0].group != 0):
         return None
@@ -117,7 +127,7 @@ def prepare_model(m) -> None:
         ex = lw.mlp.experts
         if ex is None or ex.stacked is not None or ex.count == 0 or ex.host or any(l.bias is not None for l in ex.gate_up + ex.down):
             continue
-        if ex.act != "swiglu" and not (ex.act == "gptoss" and ex.gate_up[0].kind == "dense"):
+        if ex.act != "swiglu" and not (ex.act in ("gptoss", "gelu") and ex.gate_up[0].kind == "dense"):
             continue
         st = stack_experts(ex)
         if st is None:
@@ -125,9 +135,9 @@ def prepare_model(m) -> None:
         ex.stacked = st
         st.signed = st.kind == "int8" and all(w.signed for w in ex.gate_up + ex.down)
         st.part_signed = tuple(st.kind == "int8" and all(w.signed for w in ws) for ws in (ex.gate_up, ex.down))
-        two_i, H = 2 * st.inter, st.hidden
+        gp, H = st.gate_up.shape[0] // ex.count, st.hidden
         for e in range(ex.count):       # drop the duplicate storage: per-expert weights become views of the stacked matrices
-            ex.gate_up[e].w = st.gate_up[e * two_i:(e + 1) * two_i]
+            ex.gate_up[e].w = st.gate_up[e * gp:e * gp + ex.gate_up[e].n]
             hp = st.down.shape[0] // ex.count
             ex.down[e].w = st.down[e * hp:e * hp + H]
         if QG.INT_A8 and st.kind in ("int8", "int4g") and st.gate_up.is_cuda and (st.kind == "int8" or st.group == 128) \
@@ -158,6 +168,9 @@ def _forward32(x, st, plan, experts, wts, rows32):
         moe_gather_scaled(rows32, pos, wts, xs)
     else:
         _lib.check(_lib.kernels().fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, 2 * H, _stream()), "fb_moe_gather")
+    if experts.act == "gelu":
+        act = B.linear_full32(xs, st.gate_up, act="gelu", batch=st.n_local, counts=counts, offsets=offsets, n=st.inter)
+        return B.linear_full32(act, st.down, batch=st.n_local, counts=counts, offsets=offsets, n=H), pos
     gu = B.linear_full32(xs, st.gate_up, batch=st.n_local, counts=counts, offsets=offsets)
     act = glu_gptoss(gu, True, experts.limit or 7.0) if experts.act == "gptoss" else B.glu_act_ref(gu, "silu", True)
     return B.linear_full32(act, st.down, batch=st.n_local, counts=counts, offsets=offsets, n=H), pos
@@ -215,9 +228,10 @@ def forward(x: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, experts, add:
         xs = torch.empty((rows_cap, H), device=dev, dtype=x.dtype)
         _lib.check(lib.fb_moe_gather(_ptr(x.contiguous()), _ptr(pos), _ptr(xs), T, topk, H, s), "fb_moe_gather")
     if st.kind == "dense":
-        clamp = experts.act == "gptoss"
-        _lib.check(lib.fb_moe_grouped_gemm_act(_ptr(xs), _ptr(st.gate_up), _ptr(act), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E, 2 * st.inter, H,
-                                               st.inter, max_rows, dt, GEMM_SWIGLU | (GEMM_GLU_CLAMP if clamp else 0), T * topk,
+        clamp, plain = experts.act == "gptoss", experts.act == "gelu"
+        _lib.check(lib.fb_moe_grouped_gemm_act(_ptr(xs), _ptr(st.gate_up), _ptr(act), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E,
+                                               st.inter if plain else 2 * st.inter, H, st.inter, max_rows, dt,
+                                               GEMM_GELU if plain else GEMM_SWIGLU | (GEMM_GLU_CLAMP if clamp else 0), T * topk,
                                                (experts.limit or 7.0) if clamp else 0.0, GPTOSS_ALPHA, s), "fb_moe_grouped_gemm(gate_up)")
         _lib.check(lib.fb_moe_grouped_gemm(_ptr(act), _ptr(st.down), _ptr(ys), _ptr(None), _ptr(counts), _ptr(offsets), rows_cap, E,
                                            H, st.inter, H, max_rows, dt, 0, T * topk, s), "fb_moe_grouped_gemm(down)")

@@ -306,19 +306,40 @@ class LinearWeight:
         """A dense product without a run-time adapter: the epilogues below can be fused into it."""
         return self.kind == "dense" and self.w.dtype == x.dtype and not (LinearWeight.active_adapter is not None and self.adapters)
 
-    def add_to(self, x, h, alpha: float):
-        """fp32 residual stream: ``h += alpha * (W x)`` in place."""
+    def add_to(self, x, h, alpha: float, copy=None):
+        """fp32 residual stream: ``h += alpha * (W x)`` in place; ``copy``: receives the new residual in the activation type."""
+        if self._plain(x) and self.bias is None and not self._exact(x):
+            return B.linear_res32(x, self.w, h, alpha, copy)
+        if self._plain(x) and self.bias is None:
+            B.linear_full32(x, self.w, residual=h, alpha=alpha, out=h)
+        else:
+            h.add_(self(x, out_f32=True), alpha=alpha)
+        if copy is not None:
+            copy.copy_(h)
+        return h
+
+    def glu(self, x, act: str, out=None):
+        """``act(gate) * up`` of a stacked gate / up projection (``basic.GLU_ACTS``)."""
+        if act in ("silu", "gelu_tanh") and x.is_cuda and self._plain(x) and self.bias is None and self.interleaved and B.tc_operands_ok(x, self.w):
+            return B.linear(x, self.w, swiglu=True, out=out, geglu=act == "gelu_tanh")
+        y = B.glu_act(self(x), act, self.interleaved)
+        return y if out is None else out.copy_(y)
+
+    def activated(self, x, act: str, out=None, row_gate=None, mul=None, mul_rows=None):
+        """``act(W x)`` with the factors of ``basic.linear_act``."""
         if self._plain(x) and self.bias is None:
             if self._exact(x):
-                return B.linear_full32(x, self.w, residual=h, alpha=alpha, out=h)
-            return B.linear_res32(x, self.w, h, alpha)
-        h.add_(self(x, out_f32=True), alpha=alpha)
-        return h
+                return B.linear_full32(x, self.w, act=act, out=out, row_gate=row_gate, mul=mul, mul_rows=mul_rows)
+            return B.linear_act(x, self.w, act, out, row_gate, mul, mul_rows)
+        y = B.act_ref(self(x).float(), act)
+        y = y * torch.sigmoid(row_gate.float())[:, None] if row_gate is not None else y
+        y = (y * mul.index_select(0, mul_rows.long())[:, :self.n].float() if mul is not None else y).to(x.dtype)
+        return y if out is None else out.copy_(y)
 
     def relu2(self, x):
         """``relu(W x)^2``"""
         if self._plain(x) and self.bias is None:
-            return B.linear_full32(x, self.w, relu2=True) if self._exact(x) else B.linear(x, self.w, relu2=True)
+            return B.linear_full32(x, self.w, act="relu2") if self._exact(x) else B.linear(x, self.w, relu2=True)
         return torch.relu(self(x)).square()
 
     def _base(self, x, residual=None, swiglu=False, out_f32=False):

@@ -16,9 +16,9 @@ from .basic import _ptr, _stream
 P, I, F, LL = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _lib.register_sigs({
     "fb_rmsnorm32": [P, P, P, I, I, I, I, F, I, P],
-    "fb_embed_pos_norm": [P, P, P, P, P, I, P, P, P, I, I, I, F, I, P],
+    "fb_embed_pos_norm": [P, P, P, P, P, I, P, P, P, P, I, I, I, F, I, P],
     "fb_latent_norm": [P, I, P, P, P, I, I, I, LL, F, I, P],
-    "fb_moe_combine_norm32": [P, P, P, F, P, P, P, P, P, I, I, I, F, F, I, P],
+    "fb_moe_combine_norm32": [P, P, P, F, P, P, P, P, P, I, I, I, F, F, P, P, I, P, I, P],
     "fb_moe_gather_scaled": [P, P, P, P, I, I, I, I, P],
     "fb_gather_rows": [P, P, P, I, I, P],
 }, ["stream32"])
@@ -38,9 +38,10 @@ def sinusoid_inv_freq(width: int, base: float, device) -> torch.Tensor:
     return (base ** (-i / width)).to(device)
 
 
-def embed_pos_norm(ids, positions, table, inv_freq, norm_w, eps: float, pos_table=None):
+def embed_pos_norm(ids, positions, table, inv_freq, norm_w, eps: float, pos_table=None, add_vec=None):
     """fp32 residual ``table[ids] + positions`` and its RMSNorm in the table's type (``norm_w`` None: the residual itself in that type).
-    Positions: ``inv_freq`` gives sines and cosines in alternating entries, ``pos_table`` learned rows; neither: none."""
+    Positions: ``inv_freq`` gives sines and cosines in alternating entries, ``pos_table`` learned rows; neither: none.  ``add_vec``: a row
+    that every token gets."""
     T, H = ids.shape[0], table.shape[1]
     if not table.is_cuda:
         h = table[ids.long()].float()
@@ -49,11 +50,13 @@ def embed_pos_norm(ids, positions, table, inv_freq, norm_w, eps: float, pos_tabl
             h = h + torch.stack([ang.sin(), ang.cos()], dim=-1).reshape(T, -1)[:, :H].float()
         if pos_table is not None:
             h = h + pos_table[positions.long()].float()
+        if add_vec is not None:
+            h = h + add_vec.float()
         return h, (_rms(h, norm_w, eps) if norm_w is not None else h).to(table.dtype)
     h = torch.empty((T, H), device=table.device, dtype=torch.float32)
     y = _out_rows(h, norm_w, table.dtype)
     rc = _lib.kernels().fb_embed_pos_norm(_ptr(ids), _ptr(positions), _ptr(table), _ptr(inv_freq), _ptr(pos_table), pos_table.shape[0] if pos_table is not None else 0,
-                                          _ptr(norm_w), _ptr(h), _ptr(y if y is not h else None), T, H, table.shape[0], float(eps), act_code(table.dtype), _stream())
+                                          _ptr(add_vec), _ptr(norm_w), _ptr(h), _ptr(y if y is not h else None), T, H, table.shape[0], float(eps), act_code(table.dtype), _stream())
     _lib.check(rc, "fb_embed_pos_norm")
     return h, y
 
@@ -91,10 +94,16 @@ def latent_norm(x, w, slots, pool, rank: int, eps: float) -> None:
     _lib.check(rc, "fb_latent_norm")
 
 
-def moe_combine_norm(ys, pos, wts, wconst: float, shared, h, norm_w, alpha: float, eps: float, post_w=None, dtype=None):
+def _start_args(start):
+    """``start``: what opens a pass of looped layers, (embedding table or None, token ids, step vector)."""
+    table, ids, vec = start if start is not None else (None, None, None)
+    return _ptr(table), _ptr(ids if table is not None else None), table.shape[0] if table is not None else 0, _ptr(vec)
+
+
+def moe_combine_norm(ys, pos, wts, wconst: float, shared, h, norm_w, alpha: float, eps: float, post_w=None, dtype=None, start=None):
     """``y = sum_k w_k * ys[pos[:, k]] + shared``, RMSNorm with ``post_w`` where the layer has an output norm, ``h += alpha * y`` in place
     (fp32), then RMSNorm(h) in the activation type ``dtype`` (``norm_w`` None: h itself in it).  ``wts`` None: every weight is
-    ``wconst``.  ``pos`` < 0: the pair is not held here."""
+    ``wconst``.  ``pos`` < 0: the pair is not held here.  ``start``: see ``add_norm``."""
     T, H = h.shape
     topk = pos.shape[-1]
     dtype = dtype or (norm_w.dtype if norm_w is not None else ys.dtype)
@@ -104,24 +113,30 @@ def moe_combine_norm(ys, pos, wts, wconst: float, shared, h, norm_w, alpha: floa
         y = (ys.float()[p.clamp(min=0)] * torch.where(p >= 0, w, torch.zeros_like(w))[..., None]).sum(1)
         if shared is not None:
             y = y + shared.float()
-        return add_norm(h, y, post_w, norm_w, eps, alpha, dtype)
+        return add_norm(h, y, post_w, norm_w, eps, alpha, dtype, start)
     out = _out_rows(h, norm_w, dtype)
     rc = _lib.kernels().fb_moe_combine_norm32(_ptr(ys), _ptr(pos), _ptr(wts), float(wconst), _ptr(shared), _ptr(h), _ptr(post_w), _ptr(norm_w),
-                                              _ptr(out if out is not h else None), T, topk, H, float(alpha), float(eps), act_code(dtype), _stream())
+                                              _ptr(out if out is not h else None), T, topk, H, float(alpha), float(eps), *_start_args(start), act_code(dtype), _stream())
     _lib.check(rc, "fb_moe_combine_norm32")
     return out
 
 
-def add_norm(h, y, post_w, norm_w, eps: float, alpha: float = 1.0, dtype=None):
-    """``h += alpha * RMSNorm(y)`` in place (fp32 rows; ``post_w`` None: y itself), then RMSNorm(h) in the activation type (``norm_w``
-    None: h itself in that type)."""
-    dtype = dtype or y.dtype
+def add_norm(h, y, post_w, norm_w, eps: float, alpha: float = 1.0, dtype=None, start=None):
+    """``h += alpha * RMSNorm(y)`` in place (fp32 rows; ``post_w`` None: y itself; ``y`` None: nothing), then RMSNorm(h) in the activation
+    type (``norm_w`` None: h itself in that type).  ``start``: (embedding table or None, token ids, vector) -- the residual also gets
+    the vector and the token's embedding before that norm, which is how a pass of looped layers opens."""
+    dtype = dtype or (y.dtype if y is not None else norm_w.dtype)
     if not h.is_cuda:
-        h += alpha * (_rms(y.float(), post_w, eps) if post_w is not None else y.float())
+        if y is not None:
+            h += alpha * (_rms(y.float(), post_w, eps) if post_w is not None else y.float())
+        if start is not None:
+            table, ids, vec = start
+            h += (table[ids.long()].float() if table is not None else 0.0) + vec.float()
         return (_rms(h, norm_w, eps) if norm_w is not None else h).to(dtype)
     out = _out_rows(h, norm_w, dtype)
     rc = _lib.kernels().fb_moe_combine_norm32(_ptr(y), _ptr(None), _ptr(None), 1.0, _ptr(None), _ptr(h), _ptr(post_w), _ptr(norm_w),
-                                              _ptr(out if out is not h else None), h.shape[0], 1, h.shape[1], float(alpha), float(eps), act_code(dtype), _stream())
+                                              _ptr(out if out is not h else None), h.shape[0], 1, h.shape[1], float(alpha), float(eps), *_start_args(start), act_code(dtype),
+                                              _stream())
     _lib.check(rc, "fb_moe_combine_norm32")
     return out
 
