@@ -39,6 +39,7 @@ struct AttnWindowParams {
   int keep;                                       // pages only, beside a window: the first `keep` keys stay visible
   float scale_log2;
   float cap_log2, cap_in;                         // soft cap c: c log2(e), 2 log2(e) scale / c (0: none)
+  float cap_lim, cap_p[6];                        // products up to cap_lim: the capped score is s * polynomial(s^2)
   const float* sinks;                             // [heads] or null
   const float* head_gate; long long ld_head_gate;      // one logit per (row, head)
   uint32_t idesc_s, idesc_o;
@@ -49,6 +50,11 @@ __device__ __forceinline__ int aw_first(const AttnWindowParams& p, int pos) {
   if (p.chunk > 0) return pos - pos % p.chunk;
   return p.window > 0 ? pos - p.window + 1 : 0;
 }
+
+// tanh(x) / x on |x| <= AW_TANH_LIM as a polynomial in x^2: least squares on Chebyshev nodes, reweighted until the error is level
+// (|error of tanh| <= 2e-8)
+constexpr float AW_TANH_LIM = 0.8f;
+constexpr float AW_TANH[6] = {0.99999967f, -0.33331833f, 0.1331374f, -0.05285472f, 0.01868937f, -0.00412656f};
 
 // c tanh(x): 1 - 2 / (1 + e^2x) is exact to an fp32 rounding of one, which is all that a score needs
 __device__ __forceinline__ float aw_capped(const AttnWindowParams& p, float s) {
@@ -223,8 +229,28 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const bool full_step = kv0 + AW_KV - 1 <= pos_b && (kv0 >= first_all || kv0 + AW_KV <= p.keep);
       float m_new = m_run;
       if (CAP) {
+        float am = 0.f;
 #pragma unroll
-        for (int j = 0; j < 64; ++j) sreg[j] = __float_as_uint(aw_capped(p, __uint_as_float(sreg[j])));
+        for (int j = 0; j < 64; ++j) am = fmaxf(am, fabsf(__uint_as_float(sreg[j])));
+        if (__all_sync(0xffffffffu, am <= p.cap_lim)) {
+          uint64_t cf[6];
+#pragma unroll
+          for (int i = 0; i < 6; ++i) cf[i] = pack_f32x2(p.cap_p[i], p.cap_p[i]);
+#pragma unroll
+          for (int j = 0; j < 64; j += 2) {
+            const uint64_t s = pack_f32x2(__uint_as_float(sreg[j]), __uint_as_float(sreg[j + 1])), u = mul_f32x2(s, s);
+            uint64_t y = cf[5];
+#pragma unroll
+            for (int i = 4; i >= 0; --i) y = fma_f32x2(u, y, cf[i]);
+            float a, c;
+            unpack_f32x2(mul_f32x2(s, y), a, c);
+            sreg[j] = __float_as_uint(a);
+            sreg[j + 1] = __float_as_uint(c);
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < 64; ++j) sreg[j] = __float_as_uint(aw_capped(p, __uint_as_float(sreg[j])));
+        }
       }
       const float sc = CAP ? 1.f : p.scale_log2;
       if (full_step) {
@@ -399,6 +425,13 @@ extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const 
   p.D = D; p.V = V; p.window = window; p.chunk = chunk; p.group = H / G;
   p.page_table = page_table; p.max_pages = max_pages; p.num_pages = (int)(num_slots / 128);
   p.keep = window > 0 ? keep : 0; p.sinks = sinks; p.head_gate = head_gate; p.ld_head_gate = ld_head_gate;
-  p.cap_log2 = softcap * 1.4426950408889634f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
+  if (softcap > 0.f) {
+    const double k = (double)scale / softcap;                 // x = k s
+    p.cap_log2 = softcap * 1.4426950408889634f;
+    p.cap_in = (float)(2.0 * 1.4426950408889634 * k);
+    p.cap_lim = k > 1e-3 && k < 1e3 ? (float)(AW_TANH_LIM / k) : -1.f;       // (beyond: the folded coefficients leave fp32's range)
+    double f = 1.4426950408889634 * scale;
+    for (int i = 0; i < 6; ++i, f *= k * k) p.cap_p[i] = (float)(AW_TANH[i] * f);
+  }
   return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }

@@ -95,27 +95,36 @@ __global__ void __launch_bounds__(512) mlstm_recurrent_kernel(const MlstmParams 
   float* N = S + (size_t)D * V;
   float m = N[D];
   const int r0 = rg * rows, rn = min(rows, D - r0);
-  for (int d = tid; d < Dp; d += nt) { ns[d] = d < D ? N[d] : 0.f; if (d >= D) { qs[d] = 0.f; ks[d] = 0.f; } }
+  // every load of a token is requested before the first one is waited for: the state, the normaliser (a thread's first element stays in
+  // a register), the rows
   float s[R > 0 ? R : 1];
   if (R > 0) {
 #pragma unroll
     for (int i = 0; i < R; ++i) s[i] = (col && i < rn) ? S[(size_t)(r0 + i) * V + j] : 0.f;
   }
+  float nv = tid < D ? N[tid] : 0.f;
   const T* w = reinterpret_cast<const T*>(p.norm_w) + (size_t)h * V;
+  const T wv = w[tid < V ? tid : 0];
+  for (int d = tid + nt; d < D; d += nt) ns[d] = N[d];
+  for (int d = D + tid; d < Dp; d += nt) { qs[d] = 0.f; ks[d] = 0.f; }
   for (int t = t0; t < t0 + cnt; ++t) {
     const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.ld;
+    const int d0 = h * D + (tid < D ? tid : 0), v0 = h * V + (tid < V ? tid : 0);
+    const T qr = row[d0], kr = row[p.k_col + d0], gr = row[p.g_col + v0], vr = row[p.v_col + h * V + (col ? j : 0)];
     float ig, fg;
     ml_gates(p, t, h, ig, fg);
     const float mn = fmaxf(fg + m, ig), keep = expf(fg + m - mn), add = expf(ig - mn);
     m = mn;
     float dot = 0.f;
     for (int d = tid; d < D; d += nt) {
-      const float q = MAct<DT>::ld(row[h * D + d]) * p.scale, k = MAct<DT>::ld(row[p.k_col + h * D + d]) * add;
-      const float n = fmaf(ns[d], keep, k);
-      qs[d] = q; ks[d] = k; ns[d] = n;
+      const bool own = d == tid;
+      const float q = MAct<DT>::ld(own ? qr : row[h * D + d]) * p.scale, k = MAct<DT>::ld(own ? kr : row[p.k_col + h * D + d]) * add;
+      const float n = fmaf(own ? nv : ns[d], keep, k);
+      qs[d] = q; ks[d] = k;
+      if (own) nv = n; else ns[d] = n;
       dot = fmaf(n, q, dot);
     }
-    const float v = col ? MAct<DT>::ld(row[p.v_col + h * V + j]) : 0.f;
+    const float v = col ? MAct<DT>::ld(vr) : 0.f;
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
     if (lane == 0) red[warp] = dot;
@@ -161,12 +170,12 @@ __global__ void __launch_bounds__(512) mlstm_recurrent_kernel(const MlstmParams 
     for (int x = 0; x < nw; ++x) ss += red[16 + x];
     const float inv = 1.0f / sqrtf(ss / (float)V + p.eps);
     for (int i = tid; i < V; i += nt) {
-      const float g = MAct<DT>::ld(row[p.g_col + h * V + i]);
-      reinterpret_cast<T*>(p.out)[(size_t)t * p.ld_out + (size_t)h * V + i] = MAct<DT>::st(part[i] * inv * MAct<DT>::ld(w[i]) / (1.0f + expf(-g)));
+      const float g = MAct<DT>::ld(i == tid ? gr : row[p.g_col + h * V + i]), wi = MAct<DT>::ld(i == tid ? wv : w[i]);
+      reinterpret_cast<T*>(p.out)[(size_t)t * p.ld_out + (size_t)h * V + i] = MAct<DT>::st(part[i] * inv * wi / (1.0f + expf(-g)));
     }
     __syncthreads();                     // part / red / qs are rewritten by the next token
   }
-  for (int d = tid; d < D; d += nt) N[d] = ns[d];
+  for (int d = tid; d < D; d += nt) N[d] = d == tid ? nv : ns[d];
   if (tid == 0) N[D] = m;
   if (R > 0 && col) {
     int step = V;
@@ -205,7 +214,7 @@ __device__ __forceinline__ void ml_split8(const float* x, uint4& hi, uint4& lo) 
 }
 
 template <bool BF16>
-__global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const MlstmParams p, int tmem_cols) {
+__global__ void __launch_bounds__(MC_STATE_THREADS, 2) mlstm_chunk_state_kernel(const __grid_constant__ CUtensorMap tmK, const MlstmParams p, int tmem_cols) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int D = p.D, V = p.V, dt = (D + 63) >> 6, vblocks = (V + 127) >> 7, Dn = (D + 15) & ~15;
@@ -213,7 +222,9 @@ __global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_state_kernel(con
   uint8_t* hi_smem = k_smem + dt * MC_TILE;                    // [2 vblocks] tiles of weighted values, then their remainders
   uint8_t* lo_smem = hi_smem + 2 * vblocks * MC_TILE;
   float* ws = reinterpret_cast<float*>(lo_smem + 2 * vblocks * MC_TILE);      // [128]
-  uint64_t* full_k = reinterpret_cast<uint64_t*>(ws + MC);
+  float* part = ws + MC;                                       // [512]
+  float* red = part + 512;                                     // [8]
+  uint64_t* full_k = reinterpret_cast<uint64_t*>(red + 8);
   uint64_t* done = full_k + 1;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(done + 1);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -229,57 +240,65 @@ __global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_state_kernel(con
     for (int j = 0; j < dt; ++j) tma_load_3d(k_smem + j * MC_TILE, &tmK, full_k, j * 64, h, r0);
   }
   if (warp == 1) { tmem_alloc(tmem_slot, tmem_cols); tmem_relinquish(); }
-  if (warp == 0) {
-    // four tokens a lane: running sum of the log forget gates, then a and its running maximum
-    float f[4], a[4], run = 0.f;
+  // this thread's first values, requested before anything is waited for
+  constexpr int PRE = 8;
+  const uint16_t* vp = reinterpret_cast<const uint16_t*>(p.proj) + (size_t)r0 * p.ld + p.v_col + (size_t)h * V;
+  const int vecs = V >> 3;
+  uint4 pre[PRE];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = 4 * lane + i;
-      float ig = -INFINITY, fg = 0.f;
-      if (t < n) ml_gates(p, r0 + t, h, ig, fg);
-      run += fg * ML_LOG2E;
-      f[i] = run;
-      a[i] = ig * ML_LOG2E;
-    }
-    float off = run;
+  for (int i = 0; i < PRE; ++i) {
+    const int at = tid + i * MC_STATE_THREADS, s = at / vecs, u = at - s * vecs;
+    pre[i] = s < n ? *reinterpret_cast<const uint4*>(vp + (size_t)s * p.ld + u * 8) : make_uint4(0u, 0u, 0u, 0u);
+  }
+  // one token a thread: running sum of the log forget gates, then a and its running maximum
+  float F = 0.f, a = -INFINITY, pm = -INFINITY;
+  if (warp < MC / 32) {
+    float ig = -INFINITY;
+    if (tid < n) ml_gates(p, r0 + tid, h, ig, F);
+    F *= ML_LOG2E;
+    a = ig * ML_LOG2E;
 #pragma unroll
-    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, off, o); if (lane >= o) off += x; }
-    off -= run;
-    float top = -INFINITY, pm[4];
+    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, F, o); if (lane >= o) F += x; }
+    if (lane == 31) red[warp] = F;
+  }
+  __syncthreads();
+  if (warp < MC / 32) {
+    for (int w = 0; w < warp; ++w) F += red[w];
+    a -= F;
+    pm = a;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) { f[i] += off; a[i] -= f[i]; top = fmaxf(top, a[i]); pm[i] = top; }
-    float before = top;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, before, o); if (lane >= o) before = fmaxf(before, x); }
-    const float all = __shfl_sync(0xffffffffu, before, 31);
-    before = __shfl_up_sync(0xffffffffu, before, 1);
-    if (lane == 0) before = -INFINITY;
-    float* lg = p.lg + unit * 3 * MC + 4 * lane;
-    *reinterpret_cast<float4*>(lg) = make_float4(a[0], a[1], a[2], a[3]);
-    *reinterpret_cast<float4*>(lg + MC) = make_float4(fmaxf(before, pm[0]), fmaxf(before, pm[1]), fmaxf(before, pm[2]), fmaxf(before, pm[3]));
-    *reinterpret_cast<float4*>(lg + 2 * MC) = make_float4(f[0], f[1], f[2], f[3]);
-#pragma unroll
-    for (int i = 0; i < 4; ++i) ws[4 * lane + i] = ml_ex2(a[i] - all);
+    for (int o = 1; o < 32; o <<= 1) { const float x = __shfl_up_sync(0xffffffffu, pm, o); if (lane >= o) pm = fmaxf(pm, x); }
+    if (lane == 31) red[4 + warp] = pm;
+  }
+  __syncthreads();
+  if (warp < MC / 32) {
+    for (int w = 0; w < warp; ++w) pm = fmaxf(pm, red[4 + w]);
+    float* lg = p.lg + unit * 3 * MC + tid;
+    lg[0] = a; lg[MC] = pm; lg[2 * MC] = F;
+    ws[tid] = ml_ex2(a - fmaxf(fmaxf(red[4], red[5]), fmaxf(red[6], red[7])));
   }
   __syncthreads();
   // weighted values, two terms each
-  const uint16_t* vp = reinterpret_cast<const uint16_t*>(p.proj) + (size_t)r0 * p.ld + p.v_col + (size_t)h * V;
-  const int vecs = V >> 3;
-  for (int i = tid; i < MC * vecs; i += MC_STATE_THREADS) {
-    const int s = i / vecs, u = i - s * vecs;
-    uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
-    if (s < n) {
-      const uint4 raw = *reinterpret_cast<const uint4*>(vp + (size_t)s * p.ld + u * 8);
-      const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
-      const float w = ws[s];
-      float x[8];
+  auto put = [&](int s, int u, const uint4& raw) {
+    const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
+    const float w = ws[s];
+    float x[8];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) { const float2 f = unpack_16<BF16>(r[j]); x[2 * j] = f.x * w; x[2 * j + 1] = f.y * w; }
-      ml_split8<BF16>(x, hi, lo);
-    }
+    for (int j = 0; j < 4; ++j) { const float2 f = unpack_16<BF16>(r[j]); x[2 * j] = f.x * w; x[2 * j + 1] = f.y * w; }
+    uint4 hi, lo;
+    ml_split8<BF16>(x, hi, lo);
     const int at = (u >> 3) * MC_TILE + ml_swz(s, u & 7);
     *reinterpret_cast<uint4*>(hi_smem + at) = hi;
     *reinterpret_cast<uint4*>(lo_smem + at) = lo;
+  };
+#pragma unroll
+  for (int i = 0; i < PRE; ++i) {
+    const int at = tid + i * MC_STATE_THREADS, s = at / vecs;
+    if (s < MC) put(s, at - s * vecs, pre[i]);
+  }
+  for (int at = tid + PRE * MC_STATE_THREADS; at < MC * vecs; at += MC_STATE_THREADS) {
+    const int s = at / vecs, u = at - s * vecs;
+    put(s, u, s < n ? *reinterpret_cast<const uint4*>(vp + (size_t)s * p.ld + u * 8) : make_uint4(0u, 0u, 0u, 0u));
   }
   fence_proxy_async_smem();
   tc_fence_before_sync();
@@ -300,19 +319,18 @@ __global__ void __launch_bounds__(MC_STATE_THREADS) mlstm_chunk_state_kernel(con
     }
   }
   __syncwarp();
-  // the normaliser's increment on the CUDA cores meanwhile
+  // the normaliser's increment on the CUDA cores meanwhile, half of the tokens a thread
   mbar_wait(full_k, 0, dead, KID_MLSTM, 2);
-  for (int d = tid; d < D; d += MC_STATE_THREADS) {
+  for (int e = tid; e < 2 * D; e += MC_STATE_THREADS) {
+    const int half = e >= D ? 1 : 0, d = e - half * D, u = (d & 63) >> 3, s0 = half * (MC / 2);
     const uint8_t* base = k_smem + (d >> 6) * MC_TILE + (d & 7) * 2;
-    const int u = (d & 63) >> 3;
     float x = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < MC; ++s) {
-      const uint16_t b = *reinterpret_cast<const uint16_t*>(base + ml_swz(s, u));
-      if (s < n) x = fmaf(MAct<BF16 ? 1 : 0>::ld(b), ws[s], x);
-    }
-    p.ninc[unit * D + d] = x;
+#pragma unroll 16
+    for (int s = s0; s < s0 + MC / 2; ++s) x = fmaf(MAct<BF16 ? 1 : 0>::ld(*reinterpret_cast<const uint16_t*>(base + ml_swz(s, u))), ws[s], x);
+    part[e] = x;                                               // (tokens behind the last one: weight 0, rows of later tokens or zeros)
   }
+  __syncthreads();
+  for (int d = tid; d < D; d += MC_STATE_THREADS) p.ninc[unit * D + d] = part[d] + part[D + d];
   mbar_wait(done, 0, dead, KID_MLSTM, 3);
   tc_fence_after_sync();
   float* U = p.inc + unit * D * V;
@@ -395,11 +413,14 @@ __global__ void __launch_bounds__(128) mlstm_chunk_scan_kernel(const MlstmParams
   *reinterpret_cast<float2*>(head + e) = s;
 }
 
-// One chunk of one head: warp 0 loads, warp 1 issues the products, a thread of warps 2..5 owns a token.
+// One chunk of one head: warp 0 loads, warp 1 issues the products, warps 2..9 own the tokens, two threads a token (its columns in
+// alternating blocks of 32).  The state's two terms and the values pass through one buffer in turn, the weighted scores take the place of
+// queries and keys, so that two CTAs share an SM.
+constexpr int MC_OUT_THREADS = 320;
 template <bool BF16>
-__global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                                                               const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmS,
-                                                               const MlstmParams p, int tmem_cols) {
+__global__ void __launch_bounds__(MC_OUT_THREADS, 2) mlstm_chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
+                                                                            const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmS,
+                                                                            const MlstmParams p, int tmem_cols) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int D = p.D, V = p.V, dt = (D + 63) >> 6, vt = (V + 63) >> 6, Dp = p.Dp, Vn = (V + 15) & ~15;
@@ -407,14 +428,14 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
   uint8_t* q_smem = smem;                                      // [dt] tiles, then keys; later the weighted scores: [2] tiles, their remainders
   uint8_t* k_smem = q_smem + dt * MC_TILE;
   uint8_t* p_smem = smem;
-  uint8_t* v_smem = smem + (2 * dt > 4 ? 2 * dt : 4) * MC_TILE;
-  uint8_t* s_smem = v_smem + vt * MC_TILE;                     // [2][vt] state tiles
-  float* as = reinterpret_cast<float*>(s_smem + 2 * vt * st);  // [128]
+  uint8_t* b_smem = smem + (2 * dt > 4 ? 2 * dt : 4) * MC_TILE;       // [vt] tiles: state, its remainders, values
+  float* as = reinterpret_cast<float*>(b_smem + vt * (st > MC_TILE ? st : MC_TILE));      // [128]
   float* n0 = as + MC;                                         // [D <= 256]
-  uint64_t* full_qk = reinterpret_cast<uint64_t*>(n0 + 256);
-  uint64_t* full_s = full_qk + 1;
-  uint64_t* full_v = full_qk + 2;
-  uint64_t* s_full = full_qk + 3;
+  float* red = n0 + 256;                                       // [2][2][128]
+  uint64_t* full_qk = reinterpret_cast<uint64_t*>(red + 4 * MC);
+  uint64_t* full_b = full_qk + 1;
+  uint64_t* b_free = full_qk + 2;
+  uint64_t* o_init = full_qk + 3;
   uint64_t* p_ready = full_qk + 4;
   uint64_t* o_full = full_qk + 5;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(full_qk + 6);
@@ -424,34 +445,38 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
   const size_t unit = (size_t)c * p.Hn + hl;
   bool dead = false;
   if (tid == 0) {
-    mbar_init(full_qk, 1); mbar_init(full_s, 1); mbar_init(full_v, 1); mbar_init(s_full, 1); mbar_init(p_ready, 128); mbar_init(o_full, 1);
+    mbar_init(full_qk, 1); mbar_init(full_b, 1); mbar_init(b_free, 1); mbar_init(o_init, 1); mbar_init(p_ready, 256); mbar_init(o_full, 1);
     mbar_init_fence();
-    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); tma_prefetch_desc(&tmS);
+    mbar_expect_tx(full_qk, 2 * dt * MC_TILE);
+    for (int j = 0; j < dt; ++j) {
+      tma_load_3d(q_smem + j * MC_TILE, &tmQ, full_qk, j * 64, h, r0);
+      tma_load_3d(k_smem + j * MC_TILE, &tmK, full_qk, j * 64, h, r0);
+    }
+    mbar_expect_tx(full_b, vt * st);
+    for (int j = 0; j < vt; ++j) tma_load_2d(b_smem + j * st, &tmS, full_b, j * 64, (int)(unit * 2 * Dp));
   }
   if (warp == 1) { tmem_alloc(tmem_slot, tmem_cols); tmem_relinquish(); }
-  for (int i = tid; i < D; i += 192) n0[i] = p.n0[unit * D + i];
-  for (int i = tid; i < MC; i += 192) as[i] = p.lg[unit * 3 * MC + i];
+  for (int i = tid; i < D; i += MC_OUT_THREADS) n0[i] = p.n0[unit * D + i];
+  for (int i = tid; i < MC; i += MC_OUT_THREADS) as[i] = p.lg[unit * 3 * MC + i];
   tc_fence_before_sync();
   __syncthreads();
   tc_fence_after_sync();
   const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + MC;
   if (warp == 0) {
     if (elect_one()) {
-      mbar_expect_tx(full_qk, 2 * dt * MC_TILE);
-      for (int j = 0; j < dt; ++j) {
-        tma_load_3d(q_smem + j * MC_TILE, &tmQ, full_qk, j * 64, h, r0);
-        tma_load_3d(k_smem + j * MC_TILE, &tmK, full_qk, j * 64, h, r0);
+      if (mbar_wait(b_free, 0, dead, KID_MLSTM, 11)) {
+        mbar_expect_tx(full_b, vt * st);
+        for (int j = 0; j < vt; ++j) tma_load_2d(b_smem + j * st, &tmS, full_b, j * 64, (int)((unit * 2 + 1) * Dp));
+        if (mbar_wait(b_free, 1, dead, KID_MLSTM, 12)) {
+          mbar_expect_tx(full_b, vt * MC_TILE);
+          for (int j = 0; j < vt; ++j) tma_load_3d(b_smem + j * MC_TILE, &tmV, full_b, j * 64, h, r0);
+        }
       }
-      mbar_expect_tx(full_s, 2 * vt * st);
-      for (int j = 0; j < 2 * vt; ++j)
-        tma_load_2d(s_smem + j * st, &tmS, full_s, (j % vt) * 64, (int)((unit * 2 + j / vt) * Dp));
-      mbar_expect_tx(full_v, vt * MC_TILE);
-      for (int j = 0; j < vt; ++j) tma_load_3d(v_smem + j * MC_TILE, &tmV, full_v, j * 64, h, r0);
     }
     __syncwarp();
   } else if (warp == 1) {
     if (elect_one()) {
-      const uint32_t f = BF16 ? 1u : 0u, qb = smem_u32(q_smem), kb = smem_u32(k_smem), sb = smem_u32(s_smem), vb = smem_u32(v_smem), pb = smem_u32(p_smem);
+      const uint32_t f = BF16 ? 1u : 0u, qb = smem_u32(q_smem), kb = smem_u32(k_smem), bb = smem_u32(b_smem), pb = smem_u32(p_smem);
       const uint32_t id_s = make_idesc(f, f, 0, 0, 128, MC), id_o = make_idesc(f, f, 0, 1, 128, Vn);
       const int ks = Dp >> 4;
       bool ok = mbar_wait(full_qk, 0, dead, KID_MLSTM, 4);
@@ -460,33 +485,36 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
         for (int k = 0; k < ks; ++k)
           umma_f16(tmem_s, make_smem_desc(qb + (k >> 2) * MC_TILE + (k & 3) * 32, 16, 1024, SWZ_128B),
                    make_smem_desc(kb + (k >> 2) * MC_TILE + (k & 3) * 32, 16, 1024, SWZ_128B), id_s, k != 0 ? 1u : 0u);
-        ok = mbar_wait(full_s, 0, dead, KID_MLSTM, 5);
+      }
+      for (int term = 0; ok && term < 2; ++term) {
+        ok = mbar_wait(full_b, (uint32_t)term, dead, KID_MLSTM, 5);
+        if (!ok) break;
+        for (int k = 0; k < ks; ++k)
+          umma_f16(tmem_o, make_smem_desc(qb + (k >> 2) * MC_TILE + (k & 3) * 32, 16, 1024, SWZ_128B), make_smem_desc(bb + k * 2048, st, 1024, SWZ_128B),
+                   id_o, (term | k) != 0 ? 1u : 0u);
+        umma_commit(b_free);
       }
       if (ok) {
-        for (int term = 0; term < 2; ++term)
-          for (int k = 0; k < ks; ++k)
-            umma_f16(tmem_o, make_smem_desc(qb + (k >> 2) * MC_TILE + (k & 3) * 32, 16, 1024, SWZ_128B),
-                     make_smem_desc(sb + term * vt * st + k * 2048, st, 1024, SWZ_128B), id_o, (term | k) != 0 ? 1u : 0u);
-        umma_commit(s_full);
-        ok = mbar_wait(p_ready, 0, dead, KID_MLSTM, 6) && mbar_wait(full_v, 0, dead, KID_MLSTM, 7);
+        umma_commit(o_init);
+        ok = mbar_wait(p_ready, 0, dead, KID_MLSTM, 6) && mbar_wait(full_b, 0, dead, KID_MLSTM, 7);
       }
       if (ok) {
         tc_fence_after_sync();
         for (int term = 0; term < 2; ++term)
           for (int k = 0; k < MC / 16; ++k)
             umma_f16(tmem_o, make_smem_desc(pb + (2 * term + (k >> 2)) * MC_TILE + (k & 3) * 32, 16, 1024, SWZ_128B),
-                     make_smem_desc(vb + k * 2048, MC_TILE, 1024, SWZ_128B), id_o, 1u);
+                     make_smem_desc(bb + k * 2048, MC_TILE, 1024, SWZ_128B), id_o, 1u);
         umma_commit(o_full);
       }
     }
     __syncwarp();
   } else {
-    const int q = warp & 3, t = q * 32 + lane;               // TMEM lane quarter, token of the chunk
+    const int q = warp & 3, t = q * 32 + lane, half = (warp - 2) >> 2;       // TMEM lane quarter, token of the chunk
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const float m0 = p.m0[unit], M = fmaxf(m0, p.lg[unit * 3 * MC + MC + t]), m = p.lg[unit * 3 * MC + 2 * MC + t] + M, w0 = ml_ex2(m0 - M);
-    float nq = 0.f;                                          // n_0 . q_t
+    float nq = 0.f;                                          // this thread's part of n_t . q_t
     mbar_wait(full_qk, 0, dead, KID_MLSTM, 8);
-    for (int u = 0; u < (D >> 3); ++u) {
+    for (int u = half; u < (D >> 3); u += 2) {
       const uint4 raw = *reinterpret_cast<const uint4*>(q_smem + (u >> 3) * MC_TILE + ml_swz(t, u & 7));
       const uint32_t r[4] = {raw.x, raw.y, raw.z, raw.w};
 #pragma unroll
@@ -496,12 +524,38 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
         nq = fmaf(x.y, n0[u * 8 + 2 * j + 1], nq);
       }
     }
-    asm volatile("bar.sync 1, 128;\n" ::: "memory");         // the weighted scores overwrite the queries
     nq *= w0;
-    mbar_wait(s_full, 0, dead, KID_MLSTM, 9);
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");         // the weighted scores overwrite the queries
+    mbar_wait(o_init, 0, dead, KID_MLSTM, 9);
     tc_fence_after_sync();
 #pragma unroll 1
-    for (int c0 = 0; c0 < vt * 64; c0 += 32) {
+    for (int b = half; b < MC / 32; b += 2) {
+      uint32_t s[32];
+      const bool any = b <= q;                               // (of the warp: blocks above the diagonal are zero)
+      if (any) {
+        tmem_ld_32x32b_x32(tmem_s + lane_off + b * 32, s);
+        tmem_ld_wait();
+      }
+#pragma unroll
+      for (int g = 0; g < 4; ++g) {
+        uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+        if (any) {
+          float x[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) {
+            const int k = b * 32 + g * 8 + j;
+            x[j] = k <= t && k < n ? __uint_as_float(s[g * 8 + j]) * ml_ex2(as[k] - M) : 0.f;
+            nq += x[j];
+          }
+          ml_split8<BF16>(x, hi, lo);
+        }
+        const int at = (b >> 1) * MC_TILE + ml_swz(t, (b & 1) * 4 + g);
+        *reinterpret_cast<uint4*>(p_smem + at) = hi;
+        *reinterpret_cast<uint4*>(p_smem + 2 * MC_TILE + at) = lo;
+      }
+    }
+#pragma unroll 1
+    for (int c0 = half * 32; c0 < V; c0 += 64) {
       uint32_t o[32];
       tmem_ld_32x32b_x32(tmem_o + lane_off + c0, o);
       tmem_ld_wait();
@@ -510,39 +564,22 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
       tmem_st_32x32b_x32(tmem_o + lane_off + c0, o);
     }
     tmem_st_wait();
-#pragma unroll 1
-    for (int b = 0; b < MC / 32; ++b) {
-      uint32_t s[32];
-      const bool any = b * 32 <= q * 32 + 31;                // (of the warp: blocks above the diagonal are zero)
-      if (any) {
-        tmem_ld_32x32b_x32(tmem_s + lane_off + b * 32, s);
-        tmem_ld_wait();
-      }
-#pragma unroll
-      for (int g = 0; g < 4; ++g) {
-        float x[8];
-#pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const int k = b * 32 + g * 8 + j;
-          x[j] = any && k <= t && k < n ? __uint_as_float(s[g * 8 + j]) * ml_ex2(as[k] - M) : 0.f;
-          nq += x[j];
-        }
-        uint4 hi, lo;
-        ml_split8<BF16>(x, hi, lo);
-        const int at = (b >> 1) * MC_TILE + ml_swz(t, (b & 1) * 4 + g);
-        *reinterpret_cast<uint4*>(p_smem + at) = hi;
-        *reinterpret_cast<uint4*>(p_smem + 2 * MC_TILE + at) = lo;
-      }
-    }
     fence_proxy_async_smem();
     tc_fence_before_sync();
     mbar_arrive(p_ready);
-    const float f = p.scale / (fmaxf(fabsf(nq * p.scale), ml_ex2(-m)) + 1e-6f);
+    red[half * MC + t] = nq;
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");
+    nq = (red[t] + red[MC + t]) * p.scale;
+    const float f = p.scale / (fmaxf(fabsf(nq), ml_ex2(-m)) + 1e-6f);
+    const bool live = t < n;
+    const uint16_t* gp = reinterpret_cast<const uint16_t*>(p.proj) + (size_t)(r0 + (live ? t : 0)) * p.ld + p.g_col + (size_t)h * V;
+    const uint16_t* wp = reinterpret_cast<const uint16_t*>(p.norm_w) + (size_t)h * V;
+    uint16_t* op = reinterpret_cast<uint16_t*>(p.out) + (size_t)(r0 + (live ? t : 0)) * p.ld_out + (size_t)h * V;
     mbar_wait(o_full, 0, dead, KID_MLSTM, 10);
     tc_fence_after_sync();
     float ss = 0.f;
 #pragma unroll 1
-    for (int c0 = 0; c0 < V; c0 += 32) {
+    for (int c0 = half * 32; c0 < V; c0 += 64) {
       uint32_t o[32];
       tmem_ld_32x32b_x32(tmem_o + lane_off + c0, o);
       tmem_ld_wait();
@@ -550,23 +587,26 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
       for (int j = 0; j < 32; ++j)
         if (c0 + j < V) { const float x = __uint_as_float(o[j]) * f; ss = fmaf(x, x, ss); }
     }
+    red[2 * MC + half * MC + t] = ss;
+    asm volatile("bar.sync 1, 256;\n" ::: "memory");
+    ss = red[2 * MC + t] + red[3 * MC + t];
     const float inv = f / sqrtf(ss / (float)V + p.eps);
-    const bool live = t < n;
-    const uint16_t* gp = reinterpret_cast<const uint16_t*>(p.proj) + (size_t)(r0 + (live ? t : 0)) * p.ld + p.g_col + (size_t)h * V;
-    const uint16_t* wp = reinterpret_cast<const uint16_t*>(p.norm_w) + (size_t)h * V;
-    uint16_t* op = reinterpret_cast<uint16_t*>(p.out) + (size_t)(r0 + (live ? t : 0)) * p.ld_out + (size_t)h * V;
 #pragma unroll 1
-    for (int c0 = 0; c0 < V; c0 += 32) {
+    for (int c0 = half * 32; c0 < V; c0 += 64) {
       uint32_t o[32];
       __syncwarp();
       tmem_ld_32x32b_x32(tmem_o + lane_off + c0, o);
+      uint4 gv[4];
+#pragma unroll
+      for (int g = 0; g < 4; ++g)
+        if (c0 + 8 * g < V) gv[g] = *reinterpret_cast<const uint4*>(gp + c0 + 8 * g);
       tmem_ld_wait();
       if (!live) continue;
 #pragma unroll
       for (int g = 0; g < 4; ++g) {
         if (c0 + 8 * g >= V) break;
-        const uint4 gv = *reinterpret_cast<const uint4*>(gp + c0 + 8 * g), wv = *reinterpret_cast<const uint4*>(wp + c0 + 8 * g);
-        const uint32_t gr[4] = {gv.x, gv.y, gv.z, gv.w}, wr[4] = {wv.x, wv.y, wv.z, wv.w};
+        const uint4 wv = *reinterpret_cast<const uint4*>(wp + c0 + 8 * g);
+        const uint32_t gr[4] = {gv[g].x, gv[g].y, gv[g].z, gv[g].w}, wr[4] = {wv.x, wv.y, wv.z, wv.w};
         uint32_t y[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -577,17 +617,17 @@ __global__ void __launch_bounds__(192) mlstm_chunk_out_kernel(const __grid_const
         *reinterpret_cast<uint4*>(op + c0 + 8 * g) = make_uint4(y[0], y[1], y[2], y[3]);
       }
     }
-    if (last_slot >= 0 && t == n - 1) p.state[((size_t)last_slot * p.H + h) * p.st_head + (size_t)D * V + D] = m * ML_LN2;
+    if (last_slot >= 0 && half == 0 && t == n - 1) p.state[((size_t)last_slot * p.H + h) * p.st_head + (size_t)D * V + D] = m * ML_LN2;
   }
   tc_fence_before_sync();
   __syncthreads();
   if (warp == 1) tmem_dealloc(tmem_s, tmem_cols);
 }
 
-static int mlstm_state_smem(int D, int V) { return ((D + 63) / 64 + 4 * ((V + 127) / 128)) * MC_TILE + MC * 4 + 64 + 1024; }
+static int mlstm_state_smem(int D, int V) { return ((D + 63) / 64 + 4 * ((V + 127) / 128)) * MC_TILE + (MC + 512 + 8) * 4 + 64 + 1024; }
 static int mlstm_out_smem(int D, int V) {
   const int dt = (D + 63) / 64, vt = (V + 63) / 64, Dp = (D + 15) & ~15;
-  return ((2 * dt > 4 ? 2 * dt : 4) + vt) * MC_TILE + 2 * vt * Dp * 128 + (MC + 256) * 4 + 64 + 1024;
+  return (2 * dt > 4 ? 2 * dt : 4) * MC_TILE + vt * (Dp > MC ? Dp : MC) * 128 + (MC + 256 + 4 * MC) * 4 + 64 + 1024;
 }
 static int mlstm_cols(int n) { int c = 32; while (c < n) c <<= 1; return c; }
 
@@ -677,7 +717,7 @@ extern "C" int fb_mlstm_chunked(const void* proj, long long ld, int T, const flo
     }                                                                                                                         \
     launch_k(mlstm_chunk_state_kernel<BF>, grid, dim3(MC_STATE_THREADS), sm_state, stream, 0, tmK, p, state_cols);            \
     launch_k(mlstm_chunk_scan_kernel<BF>, scan, dim3(128), 0, stream, 0, p);                                                  \
-    launch_k(mlstm_chunk_out_kernel<BF>, grid, dim3(192), sm_out, stream, 0, tmQ, tmK, tmV, tmS, p, out_cols);                \
+    launch_k(mlstm_chunk_out_kernel<BF>, grid, dim3(MC_OUT_THREADS), sm_out, stream, 0, tmQ, tmK, tmV, tmS, p, out_cols);                \
   }
   if (dt == 1) FB_ML(true) else FB_ML(false)
 #undef FB_ML

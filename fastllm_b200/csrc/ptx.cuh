@@ -326,6 +326,15 @@ __device__ __forceinline__ uint32_t pack_f16(float a, float b) {
   __half2 t = __floats2half2_rn(a, b);
   return *reinterpret_cast<uint32_t*>(&t);
 }
+// two fp32 values in one 64-bit register, with the packed arithmetic of sm_100
+__device__ __forceinline__ uint64_t pack_f32x2(float a, float b) { uint64_t v; asm("mov.b64 %0, {%1, %2};\n" : "=l"(v) : "f"(a), "f"(b)); return v; }
+__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;\n" : "=f"(a), "=f"(b) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul_f32x2(uint64_t a, uint64_t b) { uint64_t v; asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(v) : "l"(a), "l"(b)); return v; }
+__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t v;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(v) : "l"(a), "l"(b), "l"(c));
+  return v;
+}
 template <bool BF16>
 __device__ __forceinline__ uint32_t pack_16(float a, float b) {
   return BF16 ? pack_bf16(a, b) : pack_f16(a, b);

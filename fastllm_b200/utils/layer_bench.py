@@ -1,8 +1,9 @@
 """Throughput and kernel times of models whose layers are listed one by one, beside the closest other family at equal sizes; random
 weights.
 
-``python bench.py --layers patesun`` (beside multi-head latent attention with routed experts, DeepSeek-V3 layout) and ``--layers
-vilulorn`` (beside Gated DeltaNet + gated attention with routed experts, Qwen3-Next layout) print one JSON line per measurement:
+``python bench.py --layers patesun`` (beside multi-head latent attention with routed experts, DeepSeek-V3 layout), ``--layers vilulorn``
+(beside Gated DeltaNet + gated attention with routed experts, Qwen3-Next layout) and ``--layers vuripel`` (beside Vilulorn) print one
+JSON line per measurement:
   * ``step``   -- prefill and decode tokens/s of a stack of four layers through the engine's runner;
   * ``kernel`` -- one operator alone: microseconds, its bytes / FLOPs and the fraction of the measured copy bandwidth or GEMM peak.
 Operators are timed with CUDA events behind an L2 flush that also hides the host's launch time; the median of the repeats is kept.
@@ -60,6 +61,17 @@ def vilulorn_config(z):
     moe = {"kind": "moe", "expert": {"ff": z["eff"], "limit": 7.0}, "router": {"experts": z["experts"], "top": z["top"]}}
     return from_hf_dict(dict(architecture="Vilulorn", vocab=VOCAB, width=z["width"], norm={"eps": 1e-6}, max_positions=1 << 16,
                              layers=[{"type": t, "mixer": m, "mlp": moe} for t, m in (("gla", gl), ("attention", at), ("gla", gl), ("attention", dict(at, kv_from=1)))]))
+
+
+def vuripel_config(z):
+    from ..models.config import from_hf_dict
+
+    full = {"heads": z["heads"], "kv_heads": z["kv"], "dim": HEAD, "vdim": HEAD, "scale": HEAD ** -0.5, "softcap": 50.0}
+    local = dict(full, mask={"size": z["chunk"], "keep_first": 16}, rot={"base": 5e5, "dims": 64})
+    lstm = {"heads": z["lin"], "dim": HEAD, "vdim": HEAD, "gate_cap": 15.0}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 8, "keep": 4}}, "shared": {"ff": z["eff"]}}
+    return from_hf_dict(dict(architecture="Vuripel", vocab=VOCAB, width=z["width"], norm={"eps": 1e-6}, token_side={"dim": 256},
+                             layers=[{"type": t, "mixer": m, "mlp": moe} for t, m in (("mlstm", lstm), ("attention_2", local), ("mlstm", lstm), ("attention", full))]))
 
 
 def deltanet_config(z):
@@ -422,17 +434,160 @@ def bench_hybrid_kernels(z, size: str, emit) -> None:
     torch.cuda.empty_cache()
 
 
+def bench_parallel_kernels(z, size: str, emit) -> None:
+    """Operators of the parallel-block stack (matrix-memory LSTM, capped attention with sinks and kept tokens), each before the like one
+    of the chunked-attention / gated-linear-attention stack."""
+    from ..models.config import AttnSpec, GLASpec, MLSTMSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import attention as A
+    from ..ops import basic as B
+    from ..ops import gla as GLA
+    from ..ops import grouped as GR
+    from ..ops import mlstm as ML
+    from ..ops import moe as MOE
+    from ..ops import moe_grouped as MG
+    from ..ops import stream32 as S
+
+    tm = Timer()
+    hbm, tf, src = peaks()
+    dev, dt = "cuda", torch.bfloat16
+    W, H, G, N, C, E, top, eff = (z[k] for k in ("width", "heads", "kv", "lin", "chunk", "experts", "top", "eff"))
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=dt) * 0.05
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    D, T, Bn = HEAD, 8192, 64
+
+    def put(name, role, fn, nbytes, flops, **info):
+        us = tm.us(fn)
+        t_mem, t_mm = nbytes / hbm / 1e3, flops / tf / 1e6
+        emit(dict(kind="kernel", size=size, name=name, role=role, us=round(us, 2), gbytes=nbytes / 1e9, gflop=flops / 1e9,
+                  bound="memory" if t_mem > t_mm else "tensor", roofline_frac=round(max(t_mem, t_mm) / us, 4), peak=src, **info))
+
+    # recurrent layers: a step of 64 requests, prompts
+    mw, _ = ML.build(MLSTMSpec(N, D, D, 15.0), *(rnd(N * D, 16) for _ in range(4)), rnd(N), rnd(N) + 4.0, rnd(N * D))
+    gw, _ = GLA.build(GLASpec(N, D, D, 16.0), *(rnd(N * D, 16) for _ in range(4)), rnd(16, 16), rnd(N * D, 16), rnd(N * D), rnd(D))
+    sm, sg = torch.zeros((Bn + 1, N, ML.state_len(D, D)), device=dev), torch.zeros((Bn + 1, N, D, D), device=dev)
+    step = ForwardBatch(ids=None, positions=None, slots=None, page_table=None, kv_lens=None, cu_q=None, is_decode=True, state_slots=i32(list(range(Bn))))
+    proj, gates = rnd(Bn, gw.cols[-1] + 32), torch.randn(Bn, 2 * N, device=dev)
+    nb = Bn * N * (2 * D * D * 4 + 5 * D * 2)
+    put("matrix-memory step", "new", lambda: ML.mix(mw, proj, gates, step, sm, 1e-6), nb, 0, batch=Bn)
+    put("gated linear step", "like", lambda: GLA.mix(gw, proj, step, sg, 1e-6), nb, 0, batch=Bn)
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        cu, sl = [n * b for b in range(n_req + 1)], list(range(n_req))
+        proj, gates = rnd(T, gw.cols[-1] + 32), torch.randn(T, 2 * N, device=dev)
+        fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=i32([[0]]), kv_lens=None, cu_q=i32(cu), cu_q_host=cu, state_slots=i32(sl), state_slots_host=sl)
+        nb, fl = T * N * D * 2 * 5, T * N * (4.0 * D * D + 2.0 * 64 * D)
+        put("matrix-memory prompt", "new", lambda: ML.mix(mw, proj, gates, fb, sm, 1e-6), nb, fl, requests=n_req, tokens=n)
+        put("gated linear prompt", "like", lambda: GLA.mix(gw, proj, fb, sg, 1e-6), nb, fl, requests=n_req, tokens=n)
+        del proj
+    del sm, sg
+    # attention
+    rope = {"theta": 5e5, "rot_dim": 64, "scaling": None, "mode": "neox"}
+    cos, sin = A.build_rope_tables(64, 65536, 5e5, None, dev)
+
+    def layer(**kw):
+        spec = AttnSpec(H, G, D, D, D ** -0.5, **kw)
+        norms = (rnd(D), rnd(D)) if spec.qk_norm else (None, None)
+        w, _ = GR.build(spec, rnd(H * D, 16), rnd(G * D, 16), rnd(G * D, 16), rnd(H * D, 16) if spec.gate == "elem" else None, *norms, None,
+                        rnd(H) if spec.sinks else None)
+        return w
+    capped = dict(softcap=50.0, bias=True)
+    pairs = (("attention, cap + sinks + head gate", layer(sinks=True, qk_norm=False, gate="head", **capped), "attention", layer(), 0),
+             ("attention, window + kept + cap", layer(window=C, keep=16, gate="", rope=rope, **capped), "attention, chunk", layer(chunk=C, rope=dict(rope, mode="interleaved")), C))
+    for ctx in (C, 2 * C):
+        pages = ctx // 128
+        pool = (rnd(Bn * pages, 128, G, D), rnd(Bn * pages, 128, G, D))
+        pt, lens = torch.randperm(Bn * pages, device=dev).to(torch.int32).view(Bn, pages), i32([ctx] * Bn)
+        for new, wn, like, wl, span in pairs:
+            keys = min(ctx, span) if span else ctx
+            for name, role, w in ((new, "new", wn), (like, "like", wl)):
+                fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=pt, kv_lens=lens, cu_q=None, is_decode=True)
+                proj, hg = rnd(Bn, (w.v_col + G * D + 31) // 32 * 32), torch.randn(Bn, H, device=dev) if w.gate == "head" else None
+                GR.attention(w, proj, pool, fb, head_gate=hg)
+                put("decode " + name, role, lambda: GR.attention(w, proj, pool, fb, head_gate=hg), Bn * (keys * G * D * 4 + H * D * (6 if w.gate == "elem" else 4)),
+                    4.0 * Bn * H * keys * D, batch=Bn, context=ctx, keys=keys)
+        del pool
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        pages, cu = n // 128, [n * b for b in range(n_req + 1)]
+        pool = (rnd(n_req * pages, 128, G, D), rnd(n_req * pages, 128, G, D))
+        pt, lens = torch.arange(n_req * pages, device=dev, dtype=torch.int32).view(n_req, pages), i32([n] * n_req)
+        pos = torch.arange(T, device=dev, dtype=torch.int32)
+        fb = ForwardBatch(ids=pos, positions=pos % n, slots=pos, page_table=pt, kv_lens=lens, cu_q=i32(cu), cu_q_host=cu, kv_lens_host=[n] * n_req)
+        causal = lambda m: m * (m + 1) // 2
+        for new, wn, like, wl, span in pairs:
+            inside = causal(n) - (causal(n - span) if span and n > span else 0)
+            chunked = n // span * causal(span) + causal(n % span) if span else causal(n)
+            for name, role, w, seen in ((new, "new", wn, inside), (like, "like", wl, chunked)):
+                proj, hg = rnd(T, (w.v_col + G * D + 31) // 32 * 32), torch.randn(T, H, device=dev) if w.gate == "head" else None
+                GR.attention(w, proj, pool, fb, head_gate=hg)
+                put("prompt " + name, role, lambda: GR.attention(w, proj, pool, fb, head_gate=hg), T * (H * D * (6 if w.gate == "elem" else 4) + G * D * 4),
+                    4.0 * seen * n_req * H * D, requests=n_req, tokens=n)
+    proj = rnd(T, (H * 2 + 2 * G) * D)
+    for name, role, w, heads in (("append", "new", pairs[0][1], 2 * G), ("head norm + rotary (halves) + append", "new", pairs[1][1], H + 2 * G),
+                                 ("head norm + rotary (pairs) + append", "like", pairs[1][3], H + 2 * G)):
+        put(name, role, lambda: GR.post(w, proj, fb, pool, cos, sin, 1e-6), T * heads * D * 4, 0, rows=T)
+    del pool, proj
+    # row operators
+    h, y, nw, table = torch.randn(T, W, device=dev), rnd(T, W), torch.ones(W, device=dev, dtype=dt), rnd(VOCAB, W)
+    ids = torch.randint(0, VOCAB, (T,), device=dev, dtype=torch.int32)
+    put("output norm + residual + pass start + norm", "new", lambda: S.add_norm(h, y, nw, nw, 1e-6, start=(table, ids, nw)), T * W * 14, 0)
+    put("output norm + residual + norm", "new", lambda: S.add_norm(h, y, nw, nw, 1e-6), T * W * 12, 0)
+    put("output norm + residual", "like", lambda: S.add_norm(h, y, nw, None, 1e-6), T * W * 12, 0)
+    # products of a layer: the joint one, gated units, the token input's two, logits
+    for M in (64, T):
+        x, K, side = rnd(M, W), H * D + eff, 256
+        a, wj, wg, hm, cp = rnd(M, K), rnd(W, K), rnd(2 * eff * 4, W), torch.randn(M, W, device=dev), torch.empty((M, W), device=dev, dtype=dt)
+        nb, fl = W * K * 2 + M * (K * 2 + W * 8), 2.0 * M * W * K
+        put("joint product onto the residual + copy", "new", lambda: B.linear_res32(a, wj, hm, 1.0, cp), nb + M * W * 2, fl, rows=M)
+        put("product onto the residual", "like", lambda: B.linear_res32(a, wj, hm, 1.0), nb, fl, rows=M)
+        nb, fl = wg.numel() * 2 + M * (W + 4 * eff) * 2, 2.0 * M * wg.numel()
+        put("gated gelu units", "new", lambda: B.linear(x, wg, swiglu=True, geglu=True), nb, fl, rows=M)
+        put("gated silu units", "like", lambda: B.linear(x, wg, swiglu=True), nb, fl, rows=M)
+        tab, ws, wp, mid, wl = rnd(VOCAB, 4 * side), rnd(side, W), rnd(W, side), rnd(M, side), rnd(96, W)
+        nb, fl = side * W * 2 + M * (W + 2 * side) * 2, 2.0 * M * W * side
+        put("token input, gate", "new", lambda: B.linear_act(x, ws, "gelu_tanh", mul=tab[:, side:2 * side], mul_rows=ids[:M]), nb, fl, rows=M)
+        put("relu^2 product of that size", "like", lambda: B.linear(x, ws, relu2=True), nb - M * side * 2, fl, rows=M)
+        put("token input, projection", "new", lambda: B.linear(mid, wp), nb - M * side * 2, fl, rows=M)
+        wu, rg = rnd(eff, W), torch.randn(M, 96, device=dev)
+        nb, fl = eff * W * 2 + M * (W + eff) * 2, 2.0 * M * W * eff
+        put("shared expert, gelu + row gate", "new", lambda: B.linear_act(x, wu, "gelu", row_gate=rg[:, 70]), nb, fl, rows=M)
+        put("relu^2 product of that size", "like", lambda: B.linear(x, wu, relu2=True), nb, fl, rows=M)
+        put("logits + grouped top-k", "new", lambda: MOE.route_topk(B.linear(x, wl, out_f32=True)[:, :E], None, top, 0, False, 8, 4, group_max=True), M * W * 2 + E * W * 2,
+            2.0 * M * E * W, rows=M)
+        put("router + top-k", "like", lambda: MOE.route_topk(B.linear(x, wl[:E].contiguous(), out_f32=True), None, top, 1, False), M * W * 2 + E * W * 2, 2.0 * M * E * W, rows=M)
+    # experts with and without a gate branch, to the residual
+    ex, ey = (MOE.ExpertWeights(E, 0, [], []) for _ in range(2))
+    ex.count = ey.count = E
+    ex.act, ey.act, ey.limit, ey.scale_input = "gelu", "gptoss", 7.0, True
+    up, down = rnd(E * 2 * eff, W), rnd(E * W, eff)
+    ex.stacked, ey.stacked = MG.StackedExperts("dense", up[:E * eff], down, E, eff, W), MG.StackedExperts("dense", up, down, E, eff, W)
+    for M in (64, T):
+        x, h, sh = rnd(M, W), torch.randn(M, W, device=dev), rnd(M, W)
+        idx, wts = MOE.route_topk(torch.randn(M, E, device=dev), None, top, 0, False)
+        for name, role, e, mats in (("experts without gate branch, shared rows, residual", "new", ex, 2), ("experts, scaled inputs, output norm", "like", ey, 3)):
+            fl, nb = 2.0 * mats * M * top * W * eff, mats * E * W * eff * 2 + M * top * (4 * W + 2 * eff) * 2
+
+            def fn():
+                ys, p_, _ = MG.forward(x, idx, wts, e, combine=False, rows32=h if e.scale_input else None)
+                return S.moe_combine_norm(ys, p_, None if e.scale_input else wts, 1.0, None if e.scale_input else sh, h, None, 1.0, 1e-6,
+                                          post_w=nw if e.scale_input else None, dtype=dt)
+            put(name, role, fn, nb, fl, rows=M)
+    torch.cuda.empty_cache()
+
+
 def run(family: str, sizes, steps: bool = True, kernels: bool = True, emit=None) -> None:
     emit = emit or (lambda d: print(json.dumps(d), flush=True))
-    hybrid = family == "vilulorn"
+    hybrid = family != "patesun"
+    operators = {"patesun": bench_kernels, "vilulorn": bench_hybrid_kernels, "vuripel": bench_parallel_kernels}[family]
+    stacks = {"patesun": (("patesun", patesun_config), ("mla", mla_config)), "vilulorn": (("vilulorn", vilulorn_config), ("deltanet", deltanet_config)),
+              "vuripel": (("vuripel", vuripel_config), ("vilulorn", vilulorn_config))}[family]
     for size in sizes:
         z = (HYBRID_SIZES if hybrid else SIZES)[size]
         if kernels:
-            (bench_hybrid_kernels if hybrid else bench_kernels)(z, size, emit)
+            operators(z, size, emit)
         torch.cuda.empty_cache()
         if steps:
             span = z["chunk" if hybrid else "window"]
-            for fam, cfg in ((("vilulorn", vilulorn_config(z)), ("deltanet", deltanet_config(z))) if hybrid else (("patesun", patesun_config(z)), ("mla", mla_config(z)))):
+            for fam, make in stacks:
                 # (a chunk's first token sees only itself: the longest context of a decoded token ends just before the next chunk)
                 full = span - 128 if hybrid else span
-                bench_steps(fam, cfg, size, ((1, full), (64, span // 2), (64, full)), emit)
+                bench_steps(fam, make(z), size, ((1, full), (64, span // 2), (64, full)), emit)

@@ -278,6 +278,47 @@ def gla(tokens=8192, heads=16, batch=64, step=False, iters=4):
     torch.cuda.synchronize()
 
 
+def mlstm(heads=16, batch=64, tokens=8192, step=False, iters=4):
+    """Matrix-memory LSTM layers: one token of every request, or one prompt."""
+    from ..models.config import MLSTMSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import mlstm as ML
+
+    dev, D = "cuda", 128
+    rnd = lambda *s: (torch.randn(*s, device=dev) * 0.1).bfloat16()
+    w, _ = ML.build(MLSTMSpec(heads, D, D, 15.0), *(rnd(heads * D, 16) for _ in range(4)), rnd(heads), rnd(heads) + 4.0, rnd(heads * D))
+    T = batch if step else tokens
+    proj, gates, state = rnd(T, w.cols[-1] + heads * D), torch.randn(T, 2 * heads, device=dev), torch.zeros((batch + 1, heads, ML.state_len(D, D)), device=dev)
+    slots, cu = list(range(batch if step else 1)), list(range(batch + 1)) if step else [0, tokens]
+    fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=torch.zeros((1, 1), device=dev, dtype=torch.int32), kv_lens=None,
+                      cu_q=torch.tensor(cu, device=dev, dtype=torch.int32), cu_q_host=cu, is_decode=step,
+                      state_slots=torch.tensor(slots, device=dev, dtype=torch.int32), state_slots_host=slots)
+    for _ in range(iters):
+        ML.mix(w, proj, gates, fb, state, 1e-6)
+    torch.cuda.synchronize()
+
+
+def capped_prompt(tokens=8192, heads=16, kv=4, iters=3, window=0, keep=0):
+    """Soft-capped grouped-query prompt attention with sinks and head gates."""
+    from ..models.config import AttnSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import grouped as GR
+
+    dev, D, pages = "cuda", 128, tokens // 128
+    rnd = lambda *s: (torch.randn(*s, device=dev) * 0.1).bfloat16()
+    spec = AttnSpec(heads, kv, D, D, D ** -0.5, softcap=50.0, sinks=True, qk_norm=False, gate="head", window=window, keep=keep)
+    w, _ = GR.build(spec, rnd(heads * D, 16), rnd(kv * D, 16), rnd(kv * D, 16), None, None, None, None, rnd(heads))
+    pool = (rnd(pages, 128, kv, D), rnd(pages, 128, kv, D))
+    pos = torch.arange(tokens, device=dev, dtype=torch.int32)
+    fb = ForwardBatch(ids=pos, positions=pos, slots=pos, page_table=torch.arange(pages, device=dev, dtype=torch.int32).view(1, pages),
+                      kv_lens=torch.tensor([tokens], device=dev, dtype=torch.int32), cu_q=torch.tensor([0, tokens], device=dev, dtype=torch.int32),
+                      cu_q_host=[0, tokens], kv_lens_host=[tokens])
+    proj, gates = rnd(tokens, w.v_col + kv * D), torch.randn(tokens, heads, device=dev)
+    for _ in range(iters):
+        GR.attention(w, proj, pool, fb, head_gate=gates)
+    torch.cuda.synchronize()
+
+
 def grouped_decode(batch=32, length=4096, heads=32, kv=8, chunk=4096, iters=4):
     """Chunked grouped-query attention of one decoded token per request."""
     from ..models.config import AttnSpec
@@ -299,6 +340,9 @@ def grouped_decode(batch=32, length=4096, heads=32, kv=8, chunk=4096, iters=4):
 CASES = {
     "grouped_decode": grouped_decode,
     "gla_prompt": gla,
+    "mlstm_prompt": mlstm,
+    "mlstm_step": lambda: mlstm(step=True),
+    "capped_prompt": capped_prompt,
     "gla_step": lambda: gla(heads=32, step=True),
     "model_kernel_table_qwen3_moe_fp8": model_kernel_table,
     "gemm_qkv_post": gemm_qkv_post,
