@@ -50,9 +50,12 @@ __device__ __forceinline__ int ag_first(int n, int window, int chunk) {
   return window > 0 && n > window ? n - window : 0;
 }
 
+// EXT (below): soft cap, kept tokens, sinks and head gates are looked at.
 // pages of the kept first tokens (those before the page where the window starts), and the window's first page
+template <bool EXT>
 __device__ __forceinline__ int ag_kept_pages(int n, int window, int chunk, int keep, int& first_page) {
   first_page = ag_first(n, window, chunk) / AG_PAGE;
+  if (!EXT) return 0;
   const int kp = (keep + AG_PAGE - 1) / AG_PAGE;
   return kp < first_page ? kp : first_page;
 }
@@ -73,7 +76,7 @@ __global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B,
   int np = 0, first = 0, kept = 0;
   if (t < B) {
     const int n = kv_lens[t];
-    kept = ag_kept_pages(n, window, chunk, keep, first);
+    kept = ag_kept_pages<true>(n, window, chunk, keep, first);
     np = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   }
   offs[t + 1] = np;
@@ -94,6 +97,7 @@ __global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B,
 }
 
 // Reads and validates one item; every warp role uses this, so a rejected item is rejected by all of them alike.
+template <bool EXT>
 __device__ __forceinline__ bool ag_item(const AttnGroupedParams& p, int w, int& b, int& pg, int& split, int& kvh, int& h0) {
   const int hgs = (p.H / p.G + AG_N - 1) / AG_N, per = p.G * hgs;
   const int item = w / per, r = w - item * per;
@@ -103,13 +107,13 @@ __device__ __forceinline__ bool ag_item(const AttnGroupedParams& p, int w, int& 
   bool ok = (unsigned)b < (unsigned)p.B && (unsigned)pg < (unsigned)p.max_pages;
   if (!ok) { b = 0; pg = 0; }
   int first;
-  const int kept = ag_kept_pages(p.kv_lens[b], p.window, p.chunk, p.keep, first);
-  split = pg < kept ? pg : kept + pg - first;
+  const int kept = ag_kept_pages<EXT>(p.kv_lens[b], p.window, p.chunk, p.keep, first);
+  split = EXT && pg < kept ? pg : kept + pg - first;
   if ((unsigned)split >= (unsigned)p.splits) { split = 0; ok = false; }
   return ok;
 }
 
-template <bool BF16, int GP>
+template <bool BF16, int GP, bool EXT>
 __global__ void __launch_bounds__(192, 3)
 attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                     const AttnGroupedParams p) {
@@ -160,7 +164,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       int it = 0;
       for (int w = blockIdx.x; w < total; w += gridDim.x, ++it) {
         int b, pg, split, kvh, h0;
-        if (!ag_item(p, w, b, pg, split, kvh, h0)) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 20);
+        if (!ag_item<EXT>(p, w, b, pg, split, kvh, h0)) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 20);
         int page = p.page_table[(size_t)b * p.max_pages + pg];
         if ((unsigned)page >= (unsigned)p.num_pages) { report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 21); page = 0; }
         const uint32_t ph = (uint32_t)it & 1u;
@@ -212,11 +216,11 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     int it = 0;
     for (int w = blockIdx.x; w < total; w += gridDim.x, ++it) {
       int b, pg, split, kvh, h0;
-      ag_item(p, w, b, pg, split, kvh, h0);
+      ag_item<EXT>(p, w, b, pg, split, kvh, h0);
       const int n = p.kv_lens[b], nh = min(GP, HG - h0);
       const uint32_t ph = (uint32_t)it & 1u;
       const int key = pg * AG_PAGE + t;
-      const bool valid = key < n && (key >= ag_first(n, p.window, p.chunk) || key < p.keep);
+      const bool valid = key < n && (key >= ag_first(n, p.window, p.chunk) || (EXT && key < p.keep));
       mbar_wait(s_full, ph, dead, KID_ATTN_GROUPED, 7);
       tc_fence_after_sync();
       uint32_t r[16];
@@ -225,7 +229,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       float sv[GP];
 #pragma unroll
       for (int h = 0; h < GP; ++h) {
-        sv[h] = (valid && h < nh) ? ag_score(p, __uint_as_float(r[h])) : -INFINITY;
+        sv[h] = (valid && h < nh) ? (EXT ? ag_score(p, __uint_as_float(r[h])) : __uint_as_float(r[h]) * p.scale_log2) : -INFINITY;
         float m = sv[h];
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
@@ -281,7 +285,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 }
 
 // one CTA per (row, query head): merges the row's partials, eight at a time, then sink and gate
-template <bool BF16>
+template <bool BF16, bool EXT>
 __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGroupedParams p, uint16_t* __restrict__ out, long long ld_out,
                                                                    const uint16_t* __restrict__ gate, long long ld_gate,
                                                                    const float* __restrict__ head_gate, long long ld_head_gate) {
@@ -290,15 +294,15 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
   const int b = blockIdx.x, h = blockIdx.y, HG = p.H / p.G, kvh = h / HG, g = h - kvh * HG;
   const int n = p.kv_lens[b];
   int first;
-  const int kept = ag_kept_pages(n, p.window, p.chunk, p.keep, first);
+  const int kept = ag_kept_pages<EXT>(n, p.window, p.chunk, p.keep, first);
   int ns = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   if (ns > p.splits) {
     ns = p.splits;
     if (threadIdx.x == 0) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 22);
   }
   const size_t base = (size_t)(b * p.G + kvh) * p.splits;
-  const float sink = p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : -INFINITY;
-  const float hg = head_gate != nullptr ? 1.0f / (1.0f + __expf(-head_gate[(size_t)b * ld_head_gate + h])) : 1.0f;
+  const float sink = EXT && p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : -INFINITY;
+  const float hg = EXT && head_gate != nullptr ? 1.0f / (1.0f + __expf(-head_gate[(size_t)b * ld_head_gate + h])) : 1.0f;
   for (int d = threadIdx.x; d < p.V; d += 128) {
     float M = -INFINITY, L = 0.f, acc = 0.f;
     for (int s = 0; s < ns; s += 8) {
@@ -325,12 +329,12 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
         }
       }
     }
-    if (sink > -INFINITY && L > 0.f) {
+    if (EXT && sink > -INFINITY && L > 0.f) {
       const float nm = fmaxf(M, sink), a = exp2f(M - nm);
       acc *= a;
       L = L * a + exp2f(sink - nm);
     }
-    float o = L > 0.f ? acc / L * hg : 0.f;
+    float o = L > 0.f ? (EXT ? acc / L * hg : acc / L) : 0.f;
     if (gate != nullptr) {
       const uint16_t gb = gate[(size_t)b * ld_gate + (size_t)h * p.V + d];
       const float gv = BF16 ? __bfloat162float(__ushort_as_bfloat16(gb)) : __half2float(__ushort_as_half(gb));
@@ -390,20 +394,23 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
   int occ = (227 * 1024) / (smem + 1024);
   occ = occ < 1 ? 1 : occ > 3 ? 3 : occ;
   const int HG = H / G, gp = HG >= 16 ? 16 : HG;
-#define FB_AG(BF, GPV)                                                                                                          \
-  {                                                                                                                             \
-    static DeviceOnce cfg;                                                                                                      \
-    if (cfg.need()) cudaFuncSetAttribute(attn_grouped_kernel<BF, GPV>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024); \
-    launch_k<PDL_ATTN>(attn_grouped_kernel<BF, GPV>, dim3(sm_count * occ), dim3(192), smem, stream, 0, tmQ, tmK, tmV, p);        \
+  const bool ext = keep > 0 || softcap > 0.f || sinks != nullptr || head_gate != nullptr;
+#define FB_AG(BF, GPV, EXT)                                                                                                          \
+  {                                                                                                                                  \
+    static DeviceOnce cfg;                                                                                                           \
+    if (cfg.need()) cudaFuncSetAttribute(attn_grouped_kernel<BF, GPV, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024); \
+    launch_k<PDL_ATTN>(attn_grouped_kernel<BF, GPV, EXT>, dim3(sm_count * occ), dim3(192), smem, stream, 0, tmQ, tmK, tmV, p);        \
   }
-#define FB_AG_GP(BF)                                                                                                            \
-  if (gp <= 1) FB_AG(BF, 1) else if (gp <= 2) FB_AG(BF, 2) else if (gp <= 4) FB_AG(BF, 4) else if (gp <= 8) FB_AG(BF, 8) else FB_AG(BF, 16)
-  if (dtype == 1) { FB_AG_GP(true) } else { FB_AG_GP(false) }
+#define FB_AG_GP(BF, EXT)                                                                                                            \
+  {                                                                                                                                  \
+    if (gp <= 1) FB_AG(BF, 1, EXT) else if (gp <= 2) FB_AG(BF, 2, EXT) else if (gp <= 4) FB_AG(BF, 4, EXT)                            \
+    else if (gp <= 8) FB_AG(BF, 8, EXT) else FB_AG(BF, 16, EXT)                                                                      \
+    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<BF, EXT>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out,       \
+                          (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);                                                  \
+  }
+  if (dtype == 1) { if (ext) FB_AG_GP(true, true) else FB_AG_GP(true, false) }
+  else { if (ext) FB_AG_GP(false, true) else FB_AG_GP(false, false) }
 #undef FB_AG_GP
 #undef FB_AG
-  if (dtype == 1)
-    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<true>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);
-  else
-    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<false>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out, (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);
   return (int)cudaGetLastError();
 }

@@ -61,7 +61,8 @@ __device__ __forceinline__ float aw_capped(const AttnWindowParams& p, float s) {
   return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(s * p.cap_in));
 }
 
-template <bool BF16, bool CAP>
+// EXT: soft cap, kept tokens, sinks and head gates are looked at
+template <bool BF16, bool EXT>
 __global__ void __launch_bounds__(320, 1)
 attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                    const AttnWindowParams p) {
@@ -90,23 +91,23 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   int lo = max(key0, aw_first(p, pos0));
   if (p.page_table != nullptr) lo &= ~(AW_KV - 1);          // a step never straddles two pages; the mask drops what lies before
   const int hi = pos0 + rows;
-  const int kept = p.keep > 0 ? min((p.keep + AW_KV - 1) / AW_KV, lo / AW_KV) : 0;      // steps of kept tokens before the window's
+  const int kept = EXT && p.keep > 0 ? min((p.keep + AW_KV - 1) / AW_KV, lo / AW_KV) : 0;      // steps of kept tokens before the window's
   const int n_steps = kept + (hi - lo + AW_KV - 1) / AW_KV;
-  auto step_key = [&](int it) { return it < kept ? it * AW_KV : lo + (it - kept) * AW_KV; };
+  auto step_key = [&](int it) { return EXT && it < kept ? it * AW_KV : lo + (it - kept) * AW_KV; };
   // query block b takes part in steps [0, kb) and [f, e); its n-th step is nth(b, n)
   int f[2], e[2], kb[2];
   kb[0] = f[0] = kept;
   e[0] = kept + (pos0 + (rows < 128 ? rows : 128) - lo + AW_KV - 1) / AW_KV;
   if (rows > 128) {
     kb[1] = kept;
-    f[1] = kept + (p.keep > lo ? 0 : (max(lo, aw_first(p, pos0 + 128)) - lo) / AW_KV);
+    f[1] = kept + (EXT && p.keep > lo ? 0 : (max(lo, aw_first(p, pos0 + 128)) - lo) / AW_KV);
     e[1] = n_steps;
   } else {
     kb[1] = 0;
     f[1] = e[1] = n_steps;
   }
-  auto takes = [&](int b, int it) { return it < kb[b] || (it >= f[b] && it < e[b]); };
-  auto order = [&](int b, int it) { return it < kb[b] ? it : kb[b] + it - f[b]; };
+  auto takes = [&](int b, int it) { return (EXT && it < kb[b]) || (it >= f[b] && it < e[b]); };
+  auto order = [&](int b, int it) { return EXT ? (it < kb[b] ? it : kb[b] + it - f[b]) : it - f[b]; };
   bool dead = false;
 
   if (threadIdx.x == 0) {
@@ -214,21 +215,22 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const uint32_t tmem_s = tmem0 + (uint32_t)(b * 64), tmem_o = tmem0 + 128u + (uint32_t)b * o_cols;
     uint8_t* prow = p_smem + b * AW_PT + r * 128;
-    const int cnt = kb[b] + e[b] - f[b];
+    const int cnt = (EXT ? kb[b] : 0) + e[b] - f[b];
     float m_run = -INFINITY, l_run = 0.f;
     for (int n = 0; n < cnt; ++n) {
       const uint32_t iph = (uint32_t)n & 1u;
       mbar_wait(&s_full[b], iph, dead, KID_ATTN_WINDOW, 8);
       tc_fence_after_sync();
-      const int kv0 = step_key(n < kb[b] ? n : f[b] + n - kb[b]);
+      const int kv0 = EXT ? step_key(n < kb[b] ? n : f[b] + n - kb[b]) : lo + (f[b] + n) * AW_KV;
       uint32_t sreg[64];
       tmem_ld_32x32b_x32(tmem_s + lane_off, sreg);
       tmem_ld_32x32b_x32(tmem_s + lane_off + 32, sreg + 32);
       tmem_ld_wait();
       // only steps on the causal diagonal or on the window's edge pay for the mask
-      const bool full_step = kv0 + AW_KV - 1 <= pos_b && (kv0 >= first_all || kv0 + AW_KV <= p.keep);
+      const bool full_step = kv0 + AW_KV - 1 <= pos_b && (kv0 >= first_all || (EXT && kv0 + AW_KV <= p.keep));
       float m_new = m_run;
-      if (CAP) {
+      const bool cap = EXT && p.cap_in != 0.f;
+      if (cap) {
         float am = 0.f;
 #pragma unroll
         for (int j = 0; j < 64; ++j) am = fmaxf(am, fabsf(__uint_as_float(sreg[j])));
@@ -252,7 +254,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
           for (int j = 0; j < 64; ++j) sreg[j] = __float_as_uint(aw_capped(p, __uint_as_float(sreg[j])));
         }
       }
-      const float sc = CAP ? 1.f : p.scale_log2;
+      const float sc = cap ? 1.f : p.scale_log2;
       if (full_step) {
 #pragma unroll
         for (int j = 0; j < 64; ++j) {
@@ -264,7 +266,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 #pragma unroll
         for (int j = 0; j < 64; ++j) {
           const int kv = kv0 + j;
-          const float sv = (kv <= pos && (kv >= first || kv < p.keep)) ? __uint_as_float(sreg[j]) * sc : -INFINITY;
+          const float sv = (kv <= pos && (kv >= first || (EXT && kv < p.keep))) ? __uint_as_float(sreg[j]) * sc : -INFINITY;
           sreg[j] = __float_as_uint(sv);
           m_new = fmaxf(m_new, sv);
         }
@@ -313,11 +315,11 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
       const bool live = b * 128 + r < rows;
       const size_t row = (size_t)(q_row0 + b * 128 + r);
-      if (p.sinks != nullptr && l_run > 0.f) {
+      if (EXT && p.sinks != nullptr && l_run > 0.f) {
         const float sink = p.sinks[head] * 1.4426950408889634f, mx = fmaxf(m_run, sink), fac = exp2f(m_run - mx);
         inv_l = fac / (l_run * fac + exp2f(sink - mx));
       }
-      if (p.head_gate != nullptr && live) inv_l *= 1.0f / (1.0f + __expf(-p.head_gate[row * p.ld_head_gate + head]));
+      if (EXT && p.head_gate != nullptr && live) inv_l *= 1.0f / (1.0f + __expf(-p.head_gate[row * p.ld_head_gate + head]));
       uint16_t* orow = p.out + row * p.ld_out + (size_t)head * p.V;
       const uint16_t* grow = p.gate != nullptr ? p.gate + row * p.ld_gate + (size_t)head * p.V : nullptr;
 #pragma unroll 1
@@ -376,13 +378,13 @@ static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const C
   p.idesc_o = make_idesc(fm, fm, 0, 1, 128, p.vt * 64);
   const int smem = 2 * p.dt * AW_QT + p.stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
   const dim3 grid(H, n_blocks);
-#define FB_AW(BF, CAP)                                                                                                              \
+#define FB_AW(BF, EXT)                                                                                                              \
   {                                                                                                                                  \
     static DeviceOnce cfg;                                                                                                           \
-    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<BF, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);      \
-    attn_window_kernel<BF, CAP><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);                                                      \
+    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<BF, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);      \
+    attn_window_kernel<BF, EXT><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);                                                      \
   }
-  if (p.cap_in != 0.f) { if (dtype == 1) FB_AW(true, true) else FB_AW(false, true) }
+  if (p.cap_in != 0.f || p.keep > 0 || p.sinks != nullptr || p.head_gate != nullptr) { if (dtype == 1) FB_AW(true, true) else FB_AW(false, true) }
   else { if (dtype == 1) FB_AW(true, false) else FB_AW(false, false) }
 #undef FB_AW
   return (int)cudaGetLastError();

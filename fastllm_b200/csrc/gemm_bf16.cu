@@ -36,6 +36,16 @@ gemm_smallm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constan
   if ((threadIdx.x >> 5) == 1) tmem_dealloc(tmem_base, SmallMCfg<MPAD, OCC>::TMEM_COLS);
 }
 
+// the same with one of the less common epilogues
+template <int MPAD, bool BF16, int OCC>
+__global__ void __launch_bounds__(192, OCC)
+gemm_smallm_extra_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmParams p, const GemmExtra ex) {
+  uint32_t tmem_base;
+  ExtraEpilogue<BF16> epi{ex};
+  gemm_smallm_device<MPAD, BF16, OCC, ExtraEpilogue<BF16>>(tmW, tmX, p, tmem_base, KID_GEMM_SMALLM_PLAIN, epi);
+  if ((threadIdx.x >> 5) == 1) tmem_dealloc(tmem_base, SmallMCfg<MPAD, OCC>::TMEM_COLS);
+}
+
 // QKV projection with the per-head post-processing (norm, RoPE, cache append) as its epilogue
 template <int MPAD, bool BF16, int OCC = 1>
 __global__ void __launch_bounds__(192, OCC)
@@ -54,17 +64,26 @@ gemm_largem_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constan
   gemm_largem_device<BN, BF16, LargeMPlainHook>(tmX, tmW, p, tiles_m, tiles_n, LargeMPlainHook{});
 }
 
+template <int BN, bool BF16>
+__global__ void __launch_bounds__(192, 1)
+gemm_largem_extra_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmW, const GemmParams p,
+                         int tiles_m, int tiles_n, const GemmExtra ex) {
+  gemm_largem_device<BN, BF16, LargeMPlainHook, true>(tmX, tmW, p, tiles_m, tiles_n, LargeMPlainHook{}, ex);
+}
+
 // ---------------------------------------------------------------------------------------------------
 // host launchers
 // ---------------------------------------------------------------------------------------------------
 template <int MPAD, bool BF16, int OCC>
 static cudaError_t launch_smallm(const CUtensorMap& tmW, const CUtensorMap& tmX, const GemmParams& p, int nsplit, int n_tiles,
-                                 cudaStream_t stream, int batch = 1) {
+                                 cudaStream_t stream, int batch = 1, const fb::GemmExtra* ex = nullptr) {
   using Cfg = SmallMCfg<MPAD, OCC>;
   auto kern = gemm_smallm_kernel<MPAD, BF16, OCC>;
+  auto kern_extra = gemm_smallm_extra_kernel<MPAD, BF16, OCC>;
   static DeviceOnce configured;
   if (configured.need()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(kern_extra, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
     if (e != cudaSuccess) return e;
   }
   cudaLaunchConfig_t cfg = {};
@@ -79,6 +98,7 @@ static cudaError_t launch_smallm(const CUtensorMap& tmW, const CUtensorMap& tmX,
   attr[0].val.clusterDim.z = 1;
   cfg.attrs = attr;
   cfg.numAttrs = add_pdl_attr(attr, 1);
+  if (ex != nullptr) return cudaLaunchKernelEx(&cfg, kern_extra, tmW, tmX, p, *ex);
   return cudaLaunchKernelEx(&cfg, kern, tmW, tmX, p);
 }
 
@@ -219,12 +239,14 @@ static cudaError_t launch_qkv_post(const CUtensorMap& tmW, const CUtensorMap& tm
 }
 
 template <int BN, bool BF16>
-static cudaError_t launch_largem(const CUtensorMap& tmX, const CUtensorMap& tmW, const GemmParams& p, cudaStream_t stream) {
+static cudaError_t launch_largem(const CUtensorMap& tmX, const CUtensorMap& tmW, const GemmParams& p, cudaStream_t stream, const GemmExtra* ex) {
   using Cfg = LargeMCfg<BN>;
   auto kern = gemm_largem_kernel<BN, BF16>;
+  auto kern_extra = gemm_largem_extra_kernel<BN, BF16>;
   static DeviceOnce configured;
   if (configured.need()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(kern_extra, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
     if (e != cudaSuccess) return e;
   }
   const int tiles_n = (p.N + BN - 1) / BN, tiles_m = (p.M + 127) / 128;
@@ -236,7 +258,8 @@ static cudaError_t launch_largem(const CUtensorMap& tmX, const CUtensorMap& tmW,
   }
   const long long tiles = (long long)tiles_n * tiles_m;
   const int grid = (int)(tiles < sm_count ? tiles : sm_count);
-  kern<<<grid, 192, Cfg::SMEM_BYTES, stream>>>(tmX, tmW, p, tiles_m, tiles_n);
+  if (ex != nullptr) kern_extra<<<grid, 192, Cfg::SMEM_BYTES, stream>>>(tmX, tmW, p, tiles_m, tiles_n, *ex);
+  else kern<<<grid, 192, Cfg::SMEM_BYTES, stream>>>(tmX, tmW, p, tiles_m, tiles_n);
   return cudaGetLastError();
 }
 
@@ -299,15 +322,9 @@ extern "C" int fb_gemm_route(const void* X, const void* W, int M, int E, int K, 
 #undef FB_RT
 }
 
-struct GemmExtras {                  // operands of the less common epilogues (see GemmParams)
-  const float* row_gate = nullptr; int ld_row_gate = 0;
-  const void* mul = nullptr; const int* mul_rows = nullptr; long long ld_mul = 0; int mul_count = 0;
-  void* out16 = nullptr; int ld_out16 = 0;
-};
-
 static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* bias, const void* residual, int M, int N,
                                   int K, int ldx, int ldw, int ld_out, int ld_res, int dtype, int flags, int nsplit,
-                                  const void* wait_cnt, const void* wait_expect, float alpha, void* stream_, const GemmExtras& ex = GemmExtras()) {
+                                  const void* wait_cnt, const void* wait_expect, float alpha, void* stream_, const fb::GemmExtra* ex = nullptr) {
   using namespace fb;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0) return 0;
@@ -319,8 +336,8 @@ static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* 
   p.kb_total = (K + 63) / 64;             // a last partial block: both operand maps end at column K, TMA fills the rest with zeros
   p.alpha = alpha;
   p.flags = flags;
-  p.row_gate = ex.row_gate; p.ld_row_gate = ex.ld_row_gate; p.mul = ex.mul; p.mul_rows = ex.mul_rows; p.ld_mul = ex.ld_mul; p.mul_count = ex.mul_count;
-  p.out16 = ex.out16; p.ld_out16 = ex.ld_out16;
+  const GemmExtra none;
+  if (ex == nullptr && (flags & GEMM_EXTRA_FLAGS)) ex = &none;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
   p.wait_cnt = reinterpret_cast<const uint32_t*>(wait_cnt);
@@ -352,18 +369,18 @@ static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* 
     const int n_tiles = (N + 127) / 128;
 #define FB_SM(MP)                                                                                        \
   if (occ == 2)                                                                                          \
-    return (int)(bf16 ? launch_smallm<MP, true, 2>(tmW, tmX, p, nsplit, n_tiles, stream)                 \
-                      : launch_smallm<MP, false, 2>(tmW, tmX, p, nsplit, n_tiles, stream));              \
-  return (int)(bf16 ? launch_smallm<MP, true, 1>(tmW, tmX, p, nsplit, n_tiles, stream)                   \
-                    : launch_smallm<MP, false, 1>(tmW, tmX, p, nsplit, n_tiles, stream));
+    return (int)(bf16 ? launch_smallm<MP, true, 2>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex)                 \
+                      : launch_smallm<MP, false, 2>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex));              \
+  return (int)(bf16 ? launch_smallm<MP, true, 1>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex)                   \
+                    : launch_smallm<MP, false, 1>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex));
     switch (mpad) {
       case 16: FB_SM(16)
       case 32: FB_SM(32)
       case 64: FB_SM(64)
       case 128: FB_SM(128)
       default:
-        return (int)(bf16 ? launch_smallm<256, true, 1>(tmW, tmX, p, nsplit, n_tiles, stream)
-                          : launch_smallm<256, false, 1>(tmW, tmX, p, nsplit, n_tiles, stream));
+        return (int)(bf16 ? launch_smallm<256, true, 1>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex)
+                          : launch_smallm<256, false, 1>(tmW, tmX, p, nsplit, n_tiles, stream, 1, ex));
     }
 #undef FB_SM
   }
@@ -383,8 +400,8 @@ static int gemm_16bit_impl(const void* X, const void* W, void* out, const void* 
   if (!make_tmap_2d(&tmX, X, M, K, ldx, 128, 64, 2, 3)) return -2;
   if (!make_tmap_2d(&tmW, W, N, K, ldw, bn, 64, 2, 3)) return -2;
   if (bn == 256)
-    return (int)(bf16 ? launch_largem<256, true>(tmX, tmW, p, stream) : launch_largem<256, false>(tmX, tmW, p, stream));
-  return (int)(bf16 ? launch_largem<128, true>(tmX, tmW, p, stream) : launch_largem<128, false>(tmX, tmW, p, stream));
+    return (int)(bf16 ? launch_largem<256, true>(tmX, tmW, p, stream, ex) : launch_largem<256, false>(tmX, tmW, p, stream, ex));
+  return (int)(bf16 ? launch_largem<128, true>(tmX, tmW, p, stream, ex) : launch_largem<128, false>(tmX, tmW, p, stream, ex));
 }
 
 // Same, for activations that a fused collective broadcast without waiting for its peers (small-M path only): the kernel
@@ -407,10 +424,10 @@ extern "C" int fb_gemm_16bit_res32(const void* X, const void* W, float* out, con
                                    int ldw, int ld_out, int ld_res, float alpha, void* out16, int ld_out16, int dtype, void* stream_) {
   using namespace fb;
   if (out16 != nullptr && ((ld_out16 % 8) || (reinterpret_cast<uintptr_t>(out16) & 15))) return -1;
-  GemmExtras ex;
+  GemmExtra ex;
   ex.out16 = out16; ex.ld_out16 = ld_out16;
   return gemm_16bit_impl(X, W, out, nullptr, residual, M, N, K, ldx, ldw, ld_out, ld_res, dtype,
-                         GEMM_RESIDUAL | GEMM_RES_F32 | GEMM_OUT_F32, 0, nullptr, nullptr, alpha, stream_, ex);
+                         GEMM_RESIDUAL | GEMM_RES_F32 | GEMM_OUT_F32, 0, nullptr, nullptr, alpha, stream_, out16 != nullptr ? &ex : nullptr);
 }
 
 // out = act(X W^T) * sigmoid(row_gate[m])  or  act(X W^T) * mul[mul_rows[m], :]  (either factor may be absent); flags: one GEMM_GELU* form.
@@ -419,10 +436,10 @@ extern "C" int fb_gemm_16bit_act(const void* X, const void* W, void* out, int M,
                                  int dtype, void* stream_) {
   using namespace fb;
   if ((flags & ~(GEMM_GELU | GEMM_GELU_TANH)) || (mul != nullptr && (mul_rows == nullptr || mul_count <= 0 || (ld_mul % 8) || (reinterpret_cast<uintptr_t>(mul) & 15)))) return -1;
-  GemmExtras ex;
+  GemmExtra ex;
   ex.row_gate = row_gate; ex.ld_row_gate = ld_row_gate; ex.mul = mul; ex.mul_rows = mul_rows; ex.ld_mul = ld_mul;
   ex.mul_count = mul_count;
-  return gemm_16bit_impl(X, W, out, nullptr, nullptr, M, N, K, ldx, ldw, ld_out, 0, dtype, flags, 0, nullptr, nullptr, 1.f, stream_, ex);
+  return gemm_16bit_impl(X, W, out, nullptr, nullptr, M, N, K, ldx, ldw, ld_out, 0, dtype, flags, 0, nullptr, nullptr, 1.f, stream_, &ex);
 }
 
 // QKV projection (head_dim 128, M <= 256, N = (Hq + 2 Hkv) * 128) with split / per-head RMSNorm / RoPE / paged-cache append in

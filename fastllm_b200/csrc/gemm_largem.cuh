@@ -21,8 +21,9 @@ struct LargeMCfg {
 
 // Epilogue of one 128-token x BN-feature tile: TMEM lanes [32q, 32q+32) of accumulator `tmem_acc` -> bias / residual / SwiGLU ->
 // 16-bit or fp32 rows in global memory.  A thread owns one token row and writes 64 / 128 contiguous bytes per 32-column step.
-template <int BN, bool BF16>
-__device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tmem_acc, int m_tile, int n_tile, int q, int lane) {
+template <int BN, bool BF16, bool EXTRA = false>
+__device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tmem_acc, int m_tile, int n_tile, int q, int lane,
+                                                const GemmExtra& ex = GemmExtra()) {
     const int m = m_tile * 128 + q * 32 + lane;
     const bool swiglu = (p.flags & GEMM_SWIGLU) != 0;
     const uint16_t* bias16 = reinterpret_cast<const uint16_t*>(p.bias);
@@ -49,21 +50,21 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = relu2_f(v[j]);
         }
-        if (p.flags & GEMM_GELU) {
+        if (EXTRA && (p.flags & GEMM_GELU)) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = gelu_erf_f(v[j]);
         }
-        if (p.flags & GEMM_GELU_TANH) {
+        if (EXTRA && (p.flags & GEMM_GELU_TANH)) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = gelu_tanh_f(v[j]);
         }
-        if (p.row_gate != nullptr) {
-          const float g = sigmoid_f(p.row_gate[(size_t)m * p.ld_row_gate]);
+        if (EXTRA && ex.row_gate != nullptr) {
+          const float g = sigmoid_f(ex.row_gate[(size_t)m * ex.ld_row_gate]);
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] *= g;
         }
-        if (p.mul != nullptr) {
-          const uint4* mp = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(p.mul) + (size_t)clamp_row(p.mul_rows[m], p.mul_count) * p.ld_mul + n0);
+        if (EXTRA && ex.mul != nullptr) {
+          const uint4* mp = reinterpret_cast<const uint4*>(reinterpret_cast<const uint16_t*>(ex.mul) + (size_t)clamp_row(ex.mul_rows[m], ex.mul_count) * ex.ld_mul + n0);
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             const uint4 mv = mp[g];
@@ -95,9 +96,9 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
 #pragma unroll
           for (int g = 0; g < 8; ++g) op[g] = make_float4(v[g * 4], v[g * 4 + 1], v[g * 4 + 2], v[g * 4 + 3]);
         }
-        if (!(p.flags & GEMM_OUT_F32) || p.out16 != nullptr) {
-          uint4* op = p.out16 != nullptr ? reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out16) + (size_t)m * p.ld_out16 + n0)
-                                         : reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + n0);
+        if (!(p.flags & GEMM_OUT_F32) || (EXTRA && ex.out16 != nullptr)) {
+          uint4* op = EXTRA && ex.out16 != nullptr ? reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(ex.out16) + (size_t)m * ex.ld_out16 + n0)
+                                                   : reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + n0);
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
             uint4 o;
@@ -131,7 +132,7 @@ __device__ __forceinline__ void largem_epilogue(const GemmParams& p, uint32_t tm
               uv += BF16 ? __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(bias16)[nin + 64 + j])
                          : __half2float(reinterpret_cast<const __half*>(bias16)[nin + 64 + j]);
             }
-            v[j] = ((p.flags & GEMM_GEGLU) ? gelu_tanh_f(gv) : silu_f(gv)) * uv;
+            v[j] = (EXTRA && (p.flags & GEMM_GEGLU) ? gelu_tanh_f(gv) : silu_f(gv)) * uv;
           }
           uint4* op = reinterpret_cast<uint4*>(reinterpret_cast<uint16_t*>(p.out) + (size_t)m * p.ld_out + nout);
 #pragma unroll
@@ -163,9 +164,9 @@ struct LargeMPlainHook {
 // drain tile i the tensor core already accumulates tile i + 1, so the tensor pipe does not idle during epilogues and the
 // per-tile prologue (TMEM allocation, barrier set-up, pipeline fill) is paid once per CTA instead of once per tile.
 // hook.tile_done(m_tile, n_tile, lane) runs in every epilogue warp after that warp's rows of the tile are stored.
-template <int BN, bool BF16, class Hook>
+template <int BN, bool BF16, class Hook, bool EXTRA = false>
 __device__ __forceinline__ void gemm_largem_device(const CUtensorMap& tmX, const CUtensorMap& tmW, const GemmParams& p,
-                                                   int tiles_m, int tiles_n, const Hook& hook) {
+                                                   int tiles_m, int tiles_n, const Hook& hook, const GemmExtra& ex = GemmExtra()) {
   using Cfg = LargeMCfg<BN>;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -248,7 +249,7 @@ __device__ __forceinline__ void gemm_largem_device(const CUtensorMap& tmX, const
       const uint32_t use = (uint32_t)(u >> 1) & 1u;
       if (!mbar_wait(&acc_full[buf], use, dead, KID_GEMM_LARGEM, 3)) break;
       tc_fence_after_sync();
-      largem_epilogue<BN, BF16>(p, tmem_base + (uint32_t)(buf * BN), m_tile, n_tile, q, lane);
+      largem_epilogue<BN, BF16, EXTRA>(p, tmem_base + (uint32_t)(buf * BN), m_tile, n_tile, q, lane, ex);
       tc_fence_before_sync();                              // this warp's TMEM reads are done before the buffer is handed back
       __syncwarp();
       if (lane == 0) mbar_arrive(&acc_empty[buf]);

@@ -81,9 +81,15 @@ struct GemmParams {
   const void* gate = nullptr;                // 16-bit [M, >= N] (batched: + z * batch_out_cols): out = acc * sigmoid(gate)
   int ld_gate = 0;
   float act_limit = 0.f, act_alpha = 1.f;    // GEMM_GLU_CLAMP
-  // factors of the activated product, one of them at most: sigmoid of one fp32 logit per row, or row mul_rows[m] of a 16-bit table
+};
+
+// Operands of the less common epilogues.  They, and the flags of GEMM_EXTRA_FLAGS, are only looked at by kernels built for them
+// (EXTRA), so that the common epilogue stays short.
+constexpr int GEMM_EXTRA_FLAGS = GEMM_GEGLU | GEMM_GELU | GEMM_GELU_TANH;
+struct GemmExtra {
+  // factors of the activated product: sigmoid of one fp32 logit per row; row mul_rows[m] of a 16-bit table of mul_count rows
   const float* row_gate = nullptr; int ld_row_gate = 0;
-  const void* mul = nullptr; const int* mul_rows = nullptr; long long ld_mul = 0; int mul_count = 0;      // mul_count: rows of the table
+  const void* mul = nullptr; const int* mul_rows = nullptr; long long ld_mul = 0; int mul_count = 0;
   void* out16 = nullptr; int ld_out16 = 0;   // with GEMM_OUT_F32: a second copy in the 16-bit type
 };
 
@@ -118,8 +124,8 @@ struct SmallMCfg {
 
 // Cross-CTA reduction over the k splits + epilogue.  Every CTA of the cluster holds its fp32 partial tile P[token][n]
 // at `smem`; this CTA reduces and stores its own column slice (bias -> SwiGLU -> residual -> store / scatter).
-template <bool BF16>
-__device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t* smem, int split, int nsplit, int n_tile) {
+template <bool BF16, bool EXTRA = false>
+__device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t* smem, int split, int nsplit, int n_tile, const GemmExtra& ex = GemmExtra()) {
   {
     const bool swiglu = (p.flags & GEMM_SWIGLU) != 0;
     const int outw = swiglu ? 64 : 128;
@@ -153,7 +159,7 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         if (p.flags & GEMM_GLU_CLAMP) {
           acc.x = glu_clamp_f(acc.x, acc2.x, p.act_limit, p.act_alpha); acc.y = glu_clamp_f(acc.y, acc2.y, p.act_limit, p.act_alpha);
           acc.z = glu_clamp_f(acc.z, acc2.z, p.act_limit, p.act_alpha); acc.w = glu_clamp_f(acc.w, acc2.w, p.act_limit, p.act_alpha);
-        } else if (p.flags & GEMM_GEGLU) {
+        } else if (EXTRA && (p.flags & GEMM_GEGLU)) {
           acc.x = gelu_tanh_f(acc.x) * acc2.x; acc.y = gelu_tanh_f(acc.y) * acc2.y;
           acc.z = gelu_tanh_f(acc.z) * acc2.z; acc.w = gelu_tanh_f(acc.w) * acc2.w;
         } else {
@@ -171,14 +177,14 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         }
       }
       if (p.flags & GEMM_RELU2) { acc.x = relu2_f(acc.x); acc.y = relu2_f(acc.y); acc.z = relu2_f(acc.z); acc.w = relu2_f(acc.w); }
-      if (p.flags & GEMM_GELU) { acc.x = gelu_erf_f(acc.x); acc.y = gelu_erf_f(acc.y); acc.z = gelu_erf_f(acc.z); acc.w = gelu_erf_f(acc.w); }
-      if (p.flags & GEMM_GELU_TANH) { acc.x = gelu_tanh_f(acc.x); acc.y = gelu_tanh_f(acc.y); acc.z = gelu_tanh_f(acc.z); acc.w = gelu_tanh_f(acc.w); }
-      if (p.row_gate != nullptr) {
-        const float g = sigmoid_f(p.row_gate[(size_t)j * p.ld_row_gate]);
+      if (EXTRA && (p.flags & GEMM_GELU)) { acc.x = gelu_erf_f(acc.x); acc.y = gelu_erf_f(acc.y); acc.z = gelu_erf_f(acc.z); acc.w = gelu_erf_f(acc.w); }
+      if (EXTRA && (p.flags & GEMM_GELU_TANH)) { acc.x = gelu_tanh_f(acc.x); acc.y = gelu_tanh_f(acc.y); acc.z = gelu_tanh_f(acc.z); acc.w = gelu_tanh_f(acc.w); }
+      if (EXTRA && ex.row_gate != nullptr) {
+        const float g = sigmoid_f(ex.row_gate[(size_t)j * ex.ld_row_gate]);
         acc.x *= g; acc.y *= g; acc.z *= g; acc.w *= g;
       }
-      if (p.mul != nullptr) {
-        const uint2 mv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(p.mul) + (size_t)clamp_row(p.mul_rows[j], p.mul_count) * p.ld_mul + n_out);
+      if (EXTRA && ex.mul != nullptr) {
+        const uint2 mv = *reinterpret_cast<const uint2*>(reinterpret_cast<const uint16_t*>(ex.mul) + (size_t)clamp_row(ex.mul_rows[j], ex.mul_count) * ex.ld_mul + n_out);
         const float2 m0 = unpack_16<BF16>(mv.x), m1 = unpack_16<BF16>(mv.y);
         acc.x *= m0.x; acc.y *= m0.y; acc.z *= m1.x; acc.w *= m1.y;
       }
@@ -202,8 +208,8 @@ __device__ __forceinline__ void smallm_reduce_store(const GemmParams& p, uint8_t
         *reinterpret_cast<float4*>(dst) = acc;
       } else if (p.flags & GEMM_OUT_F32) {
         *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.out) + (size_t)j * p.ld_out + zo + n_out) = acc;
-        if (p.out16 != nullptr)
-          *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(p.out16) + (size_t)j * p.ld_out16 + n_out) =
+        if (EXTRA && ex.out16 != nullptr)
+          *reinterpret_cast<uint2*>(reinterpret_cast<uint16_t*>(ex.out16) + (size_t)j * ex.ld_out16 + n_out) =
               make_uint2(pack_16<BF16>(acc.x, acc.y), pack_16<BF16>(acc.z, acc.w));
       } else {
         uint2 o;
@@ -220,6 +226,13 @@ template <bool BF16>
 struct StoreEpilogue {
   __device__ __forceinline__ void operator()(const GemmParams& p, uint8_t* smem, int split, int nsplit, int n_tile) const {
     smallm_reduce_store<BF16>(p, smem, split, nsplit, n_tile);
+  }
+};
+template <bool BF16>
+struct ExtraEpilogue {
+  GemmExtra ex;
+  __device__ __forceinline__ void operator()(const GemmParams& p, uint8_t* smem, int split, int nsplit, int n_tile) const {
+    smallm_reduce_store<BF16, true>(p, smem, split, nsplit, n_tile, ex);
   }
 };
 

@@ -300,7 +300,7 @@ moe_plan_table_kernel(const long long* __restrict__ meta, const int* __restrict_
 }
 
 // grouped dense GEMM: one (expert, chunk) per blockIdx.z
-template <int MPAD, bool BF16>
+template <int MPAD, bool BF16, class Epi>
 __global__ void __launch_bounds__(192, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmParams base,
                         const MoeGroupInfo gi) {
@@ -321,7 +321,7 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_co
   p.out = reinterpret_cast<uint16_t*>(base.out) + (size_t)seg * base.ld_out;
   if (base.bias != nullptr) p.bias = reinterpret_cast<const uint16_t*>(base.bias) + (size_t)e * gi.ld_bias_e;
   uint32_t tmem_base;
-  gemm_smallm_device<MPAD, BF16, 1>(tmW, tmX, p, tmem_base, KID_MOE_GROUPED);
+  gemm_smallm_device<MPAD, BF16, 1, Epi>(tmW, tmX, p, tmem_base, KID_MOE_GROUPED, Epi());
   if ((threadIdx.x >> 5) == 1) tmem_dealloc(tmem_base, SmallMCfg<MPAD, 1>::TMEM_COLS);
 }
 
@@ -329,10 +329,13 @@ template <int MPAD, bool BF16>
 static cudaError_t launch_grouped(const CUtensorMap& tmW, const CUtensorMap& tmX, const GemmParams& p, const MoeGroupInfo& gi,
                                   int nsplit, int n_tiles, int nz, cudaStream_t stream) {
   using Cfg = SmallMCfg<MPAD, 1>;
-  auto kern = moe_grouped_gemm_kernel<MPAD, BF16>;
+  auto plain = moe_grouped_gemm_kernel<MPAD, BF16, StoreEpilogue<BF16>>;
+  auto extra = moe_grouped_gemm_kernel<MPAD, BF16, ExtraEpilogue<BF16>>;
+  auto kern = (p.flags & GEMM_EXTRA_FLAGS) ? extra : plain;
   static DeviceOnce configured;
   if (configured.need()) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    cudaError_t e = cudaFuncSetAttribute(plain, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
+    if (e == cudaSuccess) e = cudaFuncSetAttribute(extra, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM_BYTES);
     if (e != cudaSuccess) return e;
   }
   cudaLaunchConfig_t cfg = {};

@@ -333,12 +333,13 @@ struct HeadPostParams {
   float eps;
 };
 
-template <int DT>
+// PAIRS: with norm weights and pairs (2j, 2j + 1), the common form
+template <int DT, bool PAIRS>
 __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParams p) {
   typedef typename Act<DT>::T T;
   pdl_launch_dependents();
   pdl_wait();
-  const int h0 = p.q_norm == nullptr && p.rot == 0 ? p.H : 0;        // first head there is work for
+  const int h0 = !PAIRS && p.q_norm == nullptr && p.rot == 0 ? p.H : 0;        // first head there is work for
   const int units = p.H + 2 * p.G - h0;
   const long long u = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (u >= (long long)p.T * units) return;
@@ -360,8 +361,9 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   T* src = is_k ? row + p.k_col + (k - p.H) * p.Dp : row + (size_t)k * p.Dp;
   T* dst = is_k ? reinterpret_cast<T*>(p.k_pool) + ((size_t)slot * p.G + (k - p.H)) * p.Dp : src;
   const T* nw = reinterpret_cast<const T*>(is_k ? p.k_norm : p.q_norm);
+  const bool norm = PAIRS || nw != nullptr;
   float inv = 1.f;
-  if (nw != nullptr) {
+  if (norm) {
     float ss = 0.f;
     for (int i = lane; i < p.D; i += 32) { const float v = Act<DT>::ld(src[i]); ss += v * v; }
 #pragma unroll
@@ -374,10 +376,14 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   const float* ct = p.cos_tab + (size_t)pos * half;
   const float* st = p.sin_tab + (size_t)pos * half;
   for (int j = lane; 2 * j < p.Dp; j += 32) {              // pairs (Dp is even; beyond D the row is zero and stays zero)
-    const int i0 = p.neox && j < half ? j : 2 * j, i1 = p.neox && j < half ? j + half : 2 * j + 1;
-    float a = 0.f, b = 0.f;
-    if (i0 < p.D) { a = Act<DT>::ld(src[i0]); if (nw != nullptr) a *= inv * Act<DT>::ld(nw[i0]); }
-    if (i1 < p.D) { b = Act<DT>::ld(src[i1]); if (nw != nullptr) b *= inv * Act<DT>::ld(nw[i1]); }
+    const bool halves = !PAIRS && p.neox && j < half;
+    const int i0 = halves ? j : 2 * j, i1 = halves ? j + half : 2 * j + 1;
+    float a = i0 < p.D ? Act<DT>::ld(src[i0]) * inv : 0.f;
+    float b = i1 < p.D ? Act<DT>::ld(src[i1]) * inv : 0.f;
+    if (norm) {
+      if (i0 < p.D) a *= Act<DT>::ld(nw[i0]);
+      if (i1 < p.D) b *= Act<DT>::ld(nw[i1]);
+    }
     if (j < half) {
       const float c = ct[j], s = st[j], u0 = a;
       a = u0 * c - b * s;
@@ -502,8 +508,9 @@ extern "C" int fb_head_norm_rope(void* proj, long long ld, const int* positions,
   if (units == 0) return 0;
   const dim3 grid((unsigned)((units + 7) / 8));
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
-  if (dt == 0) launch_k(head_norm_rope_kernel<0>, grid, dim3(256), 0, stream, 0, p);
-  else if (dt == 1) launch_k(head_norm_rope_kernel<1>, grid, dim3(256), 0, stream, 0, p);
-  else launch_k(head_norm_rope_kernel<2>, grid, dim3(256), 0, stream, 0, p);
+  const bool pairs = q_norm != nullptr && !neox;
+#define GO(DT) { if (pairs) launch_k(head_norm_rope_kernel<DT, true>, grid, dim3(256), 0, stream, 0, p); else launch_k(head_norm_rope_kernel<DT, false>, grid, dim3(256), 0, stream, 0, p); }
+  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
   return (int)cudaGetLastError();
 }
