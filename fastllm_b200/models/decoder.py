@@ -273,10 +273,10 @@ class DecoderModel:
             cos, sin = self.rope_tables(device=device, local=local)
             return Hq, cos, sin, self.rot_dim
         spec = lw.rope
-        key = (float(spec["theta"]), int(spec["rot_dim"]), id(spec.get("scaling")), str(torch.device(device)))
+        mp = max(min(self.cfg.max_position, 1 << 17), self.max_context)
+        key = (float(spec["theta"]), int(spec["rot_dim"]), id(spec.get("scaling")), str(torch.device(device)), mp)
         cache = self.__dict__.setdefault("_rope_layers", {})
         if key not in cache:
-            mp = max(min(self.cfg.max_position, 1 << 17), self.max_context)
             cache[key] = A.build_rope_tables(int(spec["rot_dim"]), mp, float(spec["theta"]), spec.get("scaling"), device)
         cos, sin = cache[key]
         return Hq, cos, sin, int(spec["rot_dim"])
