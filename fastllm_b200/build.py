@@ -32,7 +32,7 @@ NVCC_FLAGS = [
     "-Xcompiler", "-fPIC", "--use_fast_math", "-Xptxas", "-v",
 ]
 # translation units that state fp32 results exactly (32-bit angles, norms, matrix products) are compiled without fast-math
-PRECISE_UNITS = {"stream32", "full32", "gla", "mlstm"}
+PRECISE_UNITS = {"stream32", "full32", "gla", "mlstm", "rglru"}
 CXX_FLAGS = ["-O3", "-std=c++17", "-fPIC", "-fopenmp", "-march=x86-64-v3", "-Wall", "-Wno-unused-function"]
 
 
@@ -54,7 +54,7 @@ def _run(cmd: list[str], log: Path | None = None) -> None:
 
 # kernel files of models whose layers are listed one by one: what all of them launch, and what each kind of mixer adds
 LISTED_UNITS = ("elementwise", "full32", "gemm_bf16", "moe", "sampling", "stream32")
-MIXER_UNITS = {"LatentSpec": ("attn_mla", "attn_window"), "AttnSpec": ("attn_grouped", "attn_window"), "GLASpec": ("gla",), "MLSTMSpec": ("mlstm",)}
+MIXER_UNITS = {"LatentSpec": ("attn_mla", "attn_window"), "AttnSpec": ("attn_grouped", "attn_window"), "GLASpec": ("gla",), "MLSTMSpec": ("mlstm",), "RGLRUSpec": ("rglru",)}
 
 
 def build_kernels(force: bool = False, units: tuple | None = None, out: Path | None = None) -> Path:

@@ -1,6 +1,6 @@
 // Paged grouped-query decode attention for sm_100a with any head widths up to 256 (multiples of 8), a chunk mask or a sliding window
-// (which may keep the first tokens of the sequence), soft-capped scores, a sink per head in the softmax, and an output gate (one per
-// element, or one per head).  Page length 128.
+// (which may keep the first tokens of the sequence), soft-capped scores, a sink per head in the softmax or sigmoid weights in its place,
+// outputs turned back by the query's position, and an output gate (one per element, or one per head).  Page length 128.
 //
 // As in attn_decode.cu (head width 128) a page of one key / value head is a full UMMA tile:
 //     S^T[128 keys x 16 heads] = K_page[128 x D] * Q^T        64-column tiles, K-major, SW128
@@ -9,7 +9,7 @@
 // tile.  Work items are the (row, page) pairs a query sees, times key / value heads, times groups of 16 query heads; CTAs stride over
 // them (as many per SM as the shared memory of a stage allows, so that one streams pages while another is in its softmax), write
 // un-normalised partial outputs with (max, sum), and a combine kernel merges a query's partials, adds the sink's term to the
-// denominator and applies o * sigmoid(gate).  Kept first tokens are pages of their own in the work list, before the window's.
+// denominator and applies o * sigmoid(gate).  Sigmoid weights need no maximum and no denominator: partials are added up.  Kept first tokens are pages of their own in the work list, before the window's.
 //
 // Every row is its own request (its own page-table row and length), so decoded tokens and short portions of prompts share a launch.
 // Page pools must hold finite values everywhere: unused keys of a page are multiplied by P = 0.
@@ -40,6 +40,9 @@ struct AttnGroupedParams {
   float scale_log2;
   float cap_log2, cap_in;     // soft cap c: score = c tanh(scale s / c), in log2 units c log2(e); cap_in = 2 log2(e) scale / c (0: no cap)
   const float* sinks;         // [H] or null
+  const float* score_bias;    // [H]: the weight of a key is sigmoid(score + score_bias[h]) (null: softmax)
+  const float* cos_v; const float* sin_v;      // [tab_rows, rot_v / 2]: output pairs (2m, 2m + 1) are turned back by the position
+  int rot_v, tab_rows;
   uint32_t idesc_s, idesc_o;
 };
 
@@ -50,12 +53,13 @@ __device__ __forceinline__ int ag_first(int n, int window, int chunk) {
   return window > 0 && n > window ? n - window : 0;
 }
 
-// EXT (below): soft cap, kept tokens, sinks and head gates are looked at.
+// MODE (below): 0 plain softmax; 1 soft cap, kept tokens, sinks, head gates and turned outputs are looked at; 2 sigmoid weights, with all
+// of these but sinks.
 // pages of the kept first tokens (those before the page where the window starts), and the window's first page
-template <bool EXT>
+template <int MODE>
 __device__ __forceinline__ int ag_kept_pages(int n, int window, int chunk, int keep, int& first_page) {
   first_page = ag_first(n, window, chunk) / AG_PAGE;
-  if (!EXT) return 0;
+  if (MODE == 0) return 0;
   const int kp = (keep + AG_PAGE - 1) / AG_PAGE;
   return kp < first_page ? kp : first_page;
 }
@@ -76,7 +80,7 @@ __global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B,
   int np = 0, first = 0, kept = 0;
   if (t < B) {
     const int n = kv_lens[t];
-    kept = ag_kept_pages<true>(n, window, chunk, keep, first);
+    kept = ag_kept_pages<1>(n, window, chunk, keep, first);
     np = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   }
   offs[t + 1] = np;
@@ -97,7 +101,7 @@ __global__ void attn_grouped_plan_kernel(const int* __restrict__ kv_lens, int B,
 }
 
 // Reads and validates one item; every warp role uses this, so a rejected item is rejected by all of them alike.
-template <bool EXT>
+template <int MODE>
 __device__ __forceinline__ bool ag_item(const AttnGroupedParams& p, int w, int& b, int& pg, int& split, int& kvh, int& h0) {
   const int hgs = (p.H / p.G + AG_N - 1) / AG_N, per = p.G * hgs;
   const int item = w / per, r = w - item * per;
@@ -107,13 +111,13 @@ __device__ __forceinline__ bool ag_item(const AttnGroupedParams& p, int w, int& 
   bool ok = (unsigned)b < (unsigned)p.B && (unsigned)pg < (unsigned)p.max_pages;
   if (!ok) { b = 0; pg = 0; }
   int first;
-  const int kept = ag_kept_pages<EXT>(p.kv_lens[b], p.window, p.chunk, p.keep, first);
-  split = EXT && pg < kept ? pg : kept + pg - first;
+  const int kept = ag_kept_pages<MODE>(p.kv_lens[b], p.window, p.chunk, p.keep, first);
+  split = MODE != 0 && pg < kept ? pg : kept + pg - first;
   if ((unsigned)split >= (unsigned)p.splits) { split = 0; ok = false; }
   return ok;
 }
 
-template <bool BF16, int GP, bool EXT>
+template <bool BF16, int GP, int MODE>
 __global__ void __launch_bounds__(192, 3)
 attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                     const AttnGroupedParams p) {
@@ -164,7 +168,7 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       int it = 0;
       for (int w = blockIdx.x; w < total; w += gridDim.x, ++it) {
         int b, pg, split, kvh, h0;
-        if (!ag_item<EXT>(p, w, b, pg, split, kvh, h0)) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 20);
+        if (!ag_item<MODE>(p, w, b, pg, split, kvh, h0)) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 20);
         int page = p.page_table[(size_t)b * p.max_pages + pg];
         if ((unsigned)page >= (unsigned)p.num_pages) { report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 21); page = 0; }
         const uint32_t ph = (uint32_t)it & 1u;
@@ -216,42 +220,55 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     int it = 0;
     for (int w = blockIdx.x; w < total; w += gridDim.x, ++it) {
       int b, pg, split, kvh, h0;
-      ag_item<EXT>(p, w, b, pg, split, kvh, h0);
+      ag_item<MODE>(p, w, b, pg, split, kvh, h0);
       const int n = p.kv_lens[b], nh = min(GP, HG - h0);
       const uint32_t ph = (uint32_t)it & 1u;
       const int key = pg * AG_PAGE + t;
-      const bool valid = key < n && (key >= ag_first(n, p.window, p.chunk) || (EXT && key < p.keep));
+      const bool valid = key < n && (key >= ag_first(n, p.window, p.chunk) || (MODE != 0 && key < p.keep));
       mbar_wait(s_full, ph, dead, KID_ATTN_GROUPED, 7);
       tc_fence_after_sync();
       uint32_t r[16];
       tmem_ld_32x32b_x16(tmem_s + lane_off, r);
       tmem_ld_wait();
-      float sv[GP];
-#pragma unroll
-      for (int h = 0; h < GP; ++h) {
-        sv[h] = (valid && h < nh) ? (EXT ? ag_score(p, __uint_as_float(r[h])) : __uint_as_float(r[h]) * p.scale_log2) : -INFINITY;
-        float m = sv[h];
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-        if (lane == 0) red_max[q * 16 + h] = m;
-      }
-      asm volatile("bar.sync 1, 128;\n" ::: "memory");
       // P^T[head][key] in the K-major core-matrix layout: ((t/8)*2 + h/8)*128 + (h%8)*16 + (t%8)*2 bytes
       uint8_t* pb = p_smem + (t >> 3) * 256 + (t & 7) * 2;
+      if (MODE == 2) {
 #pragma unroll
-      for (int h = 0; h < 16; ++h) {
-        uint16_t bits = 0;
-        if (h < GP) {
-          const float mx = fmaxf(fmaxf(red_max[h], red_max[16 + h]), fmaxf(red_max[32 + h], red_max[48 + h]));
-          const float pv = (h < nh && valid) ? exp2f(sv[h < GP ? h : 0] - mx) : 0.f;
-          bits = BF16 ? __bfloat16_as_ushort(__float2bfloat16_rn(pv)) : __half_as_ushort(__float2half_rn(pv));
-          // the sum of what the tensor core will see
-          float pr = BF16 ? __bfloat162float(__ushort_as_bfloat16(bits)) : __half2float(__ushort_as_half(bits));
-#pragma unroll
-          for (int o = 16; o > 0; o >>= 1) pr += __shfl_xor_sync(0xffffffffu, pr, o);
-          if (lane == 0) red_sum[q * 16 + h] = pr;
+        for (int h = 0; h < 16; ++h) {
+          uint16_t bits = 0;
+          if (h < GP && h < nh && valid) {
+            const float x = ag_score(p, __uint_as_float(r[h])) + p.score_bias[kvh * HG + h0 + h] * 1.4426950408889634f;
+            const float pv = __fdividef(1.f, 1.f + exp2f(-x));
+            bits = BF16 ? __bfloat16_as_ushort(__float2bfloat16_rn(pv)) : __half_as_ushort(__float2half_rn(pv));
+          }
+          if (h < GP || it == 0) *reinterpret_cast<uint16_t*>(pb + (h >> 3) * 128 + (h & 7) * 16) = bits;    // unused rows: zeroed once
         }
-        if (h < GP || it == 0) *reinterpret_cast<uint16_t*>(pb + (h >> 3) * 128 + (h & 7) * 16) = bits;      // unused rows: zeroed once
+      } else {
+        float sv[GP];
+#pragma unroll
+        for (int h = 0; h < GP; ++h) {
+          sv[h] = (valid && h < nh) ? (MODE != 0 ? ag_score(p, __uint_as_float(r[h])) : __uint_as_float(r[h]) * p.scale_log2) : -INFINITY;
+          float m = sv[h];
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+          if (lane == 0) red_max[q * 16 + h] = m;
+        }
+        asm volatile("bar.sync 1, 128;\n" ::: "memory");
+#pragma unroll
+        for (int h = 0; h < 16; ++h) {
+          uint16_t bits = 0;
+          if (h < GP) {
+            const float mx = fmaxf(fmaxf(red_max[h], red_max[16 + h]), fmaxf(red_max[32 + h], red_max[48 + h]));
+            const float pv = (h < nh && valid) ? exp2f(sv[h < GP ? h : 0] - mx) : 0.f;
+            bits = BF16 ? __bfloat16_as_ushort(__float2bfloat16_rn(pv)) : __half_as_ushort(__float2half_rn(pv));
+            // the sum of what the tensor core will see
+            float pr = BF16 ? __bfloat162float(__ushort_as_bfloat16(bits)) : __half2float(__ushort_as_half(bits));
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) pr += __shfl_xor_sync(0xffffffffu, pr, o);
+            if (lane == 0) red_sum[q * 16 + h] = pr;
+          }
+          if (h < GP || it == 0) *reinterpret_cast<uint16_t*>(pb + (h >> 3) * 128 + (h & 7) * 16) = bits;      // unused rows: zeroed once
+        }
       }
       fence_proxy_async_smem();
       tc_fence_before_sync();
@@ -272,11 +289,11 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
       tc_fence_before_sync();
       mbar_arrive(o_empty);
-      if (t < nh) {
+      if (MODE != 2 && t < nh) {
         p.part_ml[(slot + t) * 2] = fmaxf(fmaxf(red_max[t], red_max[16 + t]), fmaxf(red_max[32 + t], red_max[48 + t]));
         p.part_ml[(slot + t) * 2 + 1] = red_sum[t] + red_sum[16 + t] + red_sum[32 + t] + red_sum[48 + t];
       }
-      asm volatile("bar.sync 1, 128;\n" ::: "memory");     // red_max / red_sum are rewritten by the next item
+      if (MODE != 2) asm volatile("bar.sync 1, 128;\n" ::: "memory");     // red_max / red_sum are rewritten by the next item
     }
   }
   tc_fence_before_sync();
@@ -284,8 +301,8 @@ attn_grouped_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   if (warp == 1) tmem_dealloc(tmem_s, AG_TMEM_COLS);
 }
 
-// one CTA per (row, query head): merges the row's partials, eight at a time, then sink and gate
-template <bool BF16, bool EXT>
+// one CTA per (row, query head): merges the row's partials, eight at a time, then sink, rotation and gate
+template <bool BF16, int MODE>
 __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGroupedParams p, uint16_t* __restrict__ out, long long ld_out,
                                                                    const uint16_t* __restrict__ gate, long long ld_gate,
                                                                    const float* __restrict__ head_gate, long long ld_head_gate) {
@@ -294,16 +311,18 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
   const int b = blockIdx.x, h = blockIdx.y, HG = p.H / p.G, kvh = h / HG, g = h - kvh * HG;
   const int n = p.kv_lens[b];
   int first;
-  const int kept = ag_kept_pages<EXT>(n, p.window, p.chunk, p.keep, first);
+  const int kept = ag_kept_pages<MODE>(n, p.window, p.chunk, p.keep, first);
   int ns = n > 0 ? kept + (n + AG_PAGE - 1) / AG_PAGE - first : 0;
   if (ns > p.splits) {
     ns = p.splits;
     if (threadIdx.x == 0) report_error(ERR_BAD_ARG, KID_ATTN_GROUPED, 22);
   }
   const size_t base = (size_t)(b * p.G + kvh) * p.splits;
-  const float sink = EXT && p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : -INFINITY;
-  const float hg = EXT && head_gate != nullptr ? 1.0f / (1.0f + __expf(-head_gate[(size_t)b * ld_head_gate + h])) : 1.0f;
-  for (int d = threadIdx.x; d < p.V; d += 128) {
+  const float sink = MODE == 1 && p.sinks != nullptr ? p.sinks[h] * 1.4426950408889634f : -INFINITY;
+  const float hg = MODE != 0 && head_gate != nullptr ? 1.0f / (1.0f + __expf(-head_gate[(size_t)b * ld_head_gate + h])) : 1.0f;
+  const int at = MODE != 0 ? max(0, min(n, p.tab_rows) - 1) : 0;
+  for (int d0 = 0; d0 < p.V; d0 += 128) {                // (all lanes stay in the loop: they exchange their halves of a pair)
+    const int dd = d0 + threadIdx.x, d = dd < p.V ? dd : p.V - 1;
     float M = -INFINITY, L = 0.f, acc = 0.f;
     for (int s = 0; s < ns; s += 8) {
       float m8[8], l8[8], o8[8];
@@ -311,14 +330,18 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
       for (int j = 0; j < 8; ++j) {
         if (s + j < ns) {
           const size_t sl = (base + s + j) * HG + g;
-          m8[j] = p.part_ml[sl * 2];
-          l8[j] = p.part_ml[sl * 2 + 1];
+          if (MODE != 2) {
+            m8[j] = p.part_ml[sl * 2];
+            l8[j] = p.part_ml[sl * 2 + 1];
+          }
           o8[j] = p.part_o[sl * p.V + d];
         }
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        if (s + j < ns) {
+        if (MODE == 2) {
+          if (s + j < ns) acc += o8[j];
+        } else if (s + j < ns) {
           const float nm = fmaxf(M, m8[j]);
           if (nm > -INFINITY) {
             const float a = exp2f(M - nm), bw = exp2f(m8[j] - nm);
@@ -329,12 +352,20 @@ __global__ void __launch_bounds__(128) attn_grouped_combine_kernel(const AttnGro
         }
       }
     }
-    if (EXT && sink > -INFINITY && L > 0.f) {
+    if (MODE == 1 && sink > -INFINITY && L > 0.f) {
       const float nm = fmaxf(M, sink), a = exp2f(M - nm);
       acc *= a;
       L = L * a + exp2f(sink - nm);
     }
-    float o = L > 0.f ? (EXT ? acc / L * hg : acc / L) : 0.f;
+    float o = MODE == 2 ? acc * hg : L > 0.f ? (MODE == 1 ? acc / L * hg : acc / L) : 0.f;
+    if (MODE != 0 && p.rot_v > 0) {
+      const float other = __shfl_xor_sync(0xffffffffu, o, 1);
+      if (dd < p.rot_v) {
+        const size_t e = (size_t)at * (p.rot_v >> 1) + (dd >> 1);
+        o = o * p.cos_v[e] + ((dd & 1) ? -other : other) * p.sin_v[e];
+      }
+    }
+    if (dd >= p.V) continue;
     if (gate != nullptr) {
       const uint16_t gb = gate[(size_t)b * ld_gate + (size_t)h * p.V + d];
       const float gv = BF16 ? __bfloat162float(__ushort_as_bfloat16(gb)) : __half2float(__ushort_as_half(gb));
@@ -357,6 +388,7 @@ extern "C" int fb_grouped_plan(const int* kv_lens, int B, int window, int chunk,
   return (int)cudaGetLastError();
 }
 
+// score_bias [H] (null: softmax): see AttnGroupedParams; rot_v > 0: outputs are turned back by the row's position, tables [tab_rows, rot_v / 2].
 // keep: first tokens a window keeps; softcap 0: none; sinks [H], head_gate (row stride ld_head_gate, one logit per head): null for none.
 // q: [B, >= H * D] (row stride ld_q), k_pool [num_slots, G, D], v_pool [num_slots, G, V], out / gate [B, >= H * V]; 16-bit (dtype 0 = fp16,
 // 1 = bf16).  splits: most pages one query's keys touch; part_o [B * H * splits * V], part_ml [B * H * splits * 2] floats.
@@ -364,10 +396,12 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
                                  const void* gate, long long ld_gate, const int* page_table, const int* kv_lens, const int* work,
                                  const int* n_work, float* part_o, float* part_ml, int B, int H, int G, int D, int V, long long num_slots,
                                  int max_pages, int splits, int max_items, int window, int chunk, int keep, float scale, float softcap,
-                                 const float* sinks, const float* head_gate, long long ld_head_gate, int dtype, void* stream_) {
+                                 const float* sinks, const float* head_gate, long long ld_head_gate, const float* score_bias, const float* cos_v,
+                                 const float* sin_v, int rot_v, int tab_rows, int dtype, void* stream_) {
   if (B <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || H > 65535 || D <= 0 || V <= 0 || D > 256 || V > 256 || D % 8 != 0 || V % 8 != 0 || num_slots < AG_PAGE ||
-      max_pages <= 0 || splits <= 0 || keep < 0 || softcap < 0.f || (dtype != 0 && dtype != 1))
+      max_pages <= 0 || splits <= 0 || keep < 0 || softcap < 0.f || (dtype != 0 && dtype != 1) || rot_v < 0 || (rot_v & 1) || rot_v > V || (score_bias != nullptr && sinks != nullptr) ||
+      (rot_v > 0 && (cos_v == nullptr || sin_v == nullptr || tab_rows <= 0)))
     return -1;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   static int sm_count = 0;
@@ -386,7 +420,7 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
   p.B = B; p.H = H; p.G = G; p.D = D; p.V = V; p.dt = (D + 63) / 64; p.vt = (V + 63) / 64; p.splits = splits; p.max_items = max_items;
   p.window = window; p.chunk = chunk; p.keep = keep; p.scale_log2 = scale * 1.4426950408889634f;
   p.cap_log2 = softcap * 1.4426950408889634f; p.cap_in = softcap > 0.f ? 2.f * 1.4426950408889634f * scale / softcap : 0.f;
-  p.sinks = sinks;
+  p.sinks = sinks; p.score_bias = score_bias; p.cos_v = cos_v; p.sin_v = sin_v; p.rot_v = rot_v; p.tab_rows = tab_rows;
   const uint32_t f = dtype == 1 ? 1u : 0u;
   p.idesc_s = make_idesc(f, f, 0, 0, 128, AG_N);
   p.idesc_o = make_idesc(f, f, 1, 0, 128, AG_N);
@@ -394,22 +428,22 @@ extern "C" int fb_grouped_decode(const void* q, long long ld_q, const void* k_po
   int occ = (227 * 1024) / (smem + 1024);
   occ = occ < 1 ? 1 : occ > 3 ? 3 : occ;
   const int HG = H / G, gp = HG >= 16 ? 16 : HG;
-  const bool ext = keep > 0 || softcap > 0.f || sinks != nullptr || head_gate != nullptr;
-#define FB_AG(BF, GPV, EXT)                                                                                                          \
+  const int mode = score_bias != nullptr ? 2 : keep > 0 || softcap > 0.f || sinks != nullptr || head_gate != nullptr || rot_v > 0 ? 1 : 0;
+#define FB_AG(BF, GPV, MODE)                                                                                                         \
   {                                                                                                                                  \
     static DeviceOnce cfg;                                                                                                           \
-    if (cfg.need()) cudaFuncSetAttribute(attn_grouped_kernel<BF, GPV, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024); \
-    launch_k<PDL_ATTN>(attn_grouped_kernel<BF, GPV, EXT>, dim3(sm_count * occ), dim3(192), smem, stream, 0, tmQ, tmK, tmV, p);        \
+    if (cfg.need()) cudaFuncSetAttribute(attn_grouped_kernel<BF, GPV, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024); \
+    launch_k<PDL_ATTN>(attn_grouped_kernel<BF, GPV, MODE>, dim3(sm_count * occ), dim3(192), smem, stream, 0, tmQ, tmK, tmV, p);        \
   }
-#define FB_AG_GP(BF, EXT)                                                                                                            \
+#define FB_AG_GP(BF, MODE)                                                                                                           \
   {                                                                                                                                  \
-    if (gp <= 1) FB_AG(BF, 1, EXT) else if (gp <= 2) FB_AG(BF, 2, EXT) else if (gp <= 4) FB_AG(BF, 4, EXT)                            \
-    else if (gp <= 8) FB_AG(BF, 8, EXT) else FB_AG(BF, 16, EXT)                                                                      \
-    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<BF, EXT>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out,       \
+    if (gp <= 1) FB_AG(BF, 1, MODE) else if (gp <= 2) FB_AG(BF, 2, MODE) else if (gp <= 4) FB_AG(BF, 4, MODE)                            \
+    else if (gp <= 8) FB_AG(BF, 8, MODE) else FB_AG(BF, 16, MODE)                                                                      \
+    launch_k<PDL_COMBINE>(attn_grouped_combine_kernel<BF, MODE>, dim3(B, H), dim3(128), 0, stream, 0, p, (uint16_t*)out, ld_out,       \
                           (const uint16_t*)gate, ld_gate, head_gate, ld_head_gate);                                                  \
   }
-  if (dtype == 1) { if (ext) FB_AG_GP(true, true) else FB_AG_GP(true, false) }
-  else { if (ext) FB_AG_GP(false, true) else FB_AG_GP(false, false) }
+  if (dtype == 1) { if (mode == 2) FB_AG_GP(true, 2) else if (mode == 1) FB_AG_GP(true, 1) else FB_AG_GP(true, 0) }
+  else { if (mode == 2) FB_AG_GP(false, 2) else if (mode == 1) FB_AG_GP(false, 1) else FB_AG_GP(false, 0) }
 #undef FB_AG_GP
 #undef FB_AG
   return (int)cudaGetLastError();

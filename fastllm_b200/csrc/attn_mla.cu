@@ -356,7 +356,7 @@ mla_decode_kernel(const __grid_constant__ CUtensorMap tmLat, const __grid_consta
 // one CTA per (request, head): merges the request's items of that head's group; 128 threads x 4 dims per pass
 template <bool BF16>
 __global__ void mla_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, const int* __restrict__ item_range,
-                                   uint16_t* __restrict__ out, int H, int n_groups, int dv, int o_stride) {
+                                   uint16_t* __restrict__ out, int H, int n_groups, int dv, int o_stride, const float* __restrict__ head_gate) {
   pdl_launch_dependents();
   pdl_wait();
   const int b = blockIdx.x, h = blockIdx.y, t = threadIdx.x;
@@ -374,7 +374,8 @@ __global__ void mla_combine_kernel(const float* __restrict__ part_o, const float
       const float4 o = *reinterpret_cast<const float4*>(&part_o[(it * ML_N + hl) * o_stride + d]);
       acc.x += o.x * wgt; acc.y += o.y * wgt; acc.z += o.z * wgt; acc.w += o.w * wgt;
     }
-    const float inv = L > 0.f ? 1.0f / L : 0.f;
+    float inv = L > 0.f ? 1.0f / L : 0.f;
+    if (head_gate != nullptr) inv *= 1.0f / (1.0f + __expf(-head_gate[(size_t)b * H + h]));
     uint2 pk;
     pk.x = pack_16<BF16>(acc.x * inv, acc.y * inv);
     pk.y = pack_16<BF16>(acc.z * inv, acc.w * inv);
@@ -388,7 +389,7 @@ using namespace fb;
 
 // q: [B, H, dq] (q_lat | rotary part), lat_pool: [num_slots, dq], out: [B, H, dv]; all 16-bit (dtype 0 = fp16, 1 = bf16).  dv <= dq
 // columns of a latent row are its values; dq, dv multiples of 8, dv of 64 when rotary columns follow.  window > 0: the query (the
-// request's last token) sees the last `window` tokens only.  Scratch: work [4 * max_items] ints, n_work [1], item_range [2 * B],
+// request's last token) sees the last `window` tokens only.  head_gate (null: none): fp32 logits [B, H] of a sigmoid gate per head.  Scratch: work [4 * max_items] ints, n_work [1], item_range [2 * B],
 // part_o [max_items * 32 * roundup(dv, 128)] floats, part_ml [max_items * 32 * 2] floats, with max_items >= fb_mla_max_items(B, H).
 extern "C" int fb_mla_max_items(int B, int H) {
   static int sm_count = 0;
@@ -403,7 +404,7 @@ extern "C" int fb_mla_max_items(int B, int H) {
 
 extern "C" int fb_mla_decode(const void* q, const void* lat_pool, void* out, const int* page_table, const int* seq_lens, int* work,
                              int* n_work, int* item_range, float* part_o, float* part_ml, int B, int H, int dq, int dv,
-                             long long num_slots, int max_pages, int max_items, int window, float scale, int dtype, void* stream_) {
+                             long long num_slots, int max_pages, int max_items, int window, float scale, const float* head_gate, int dtype, void* stream_) {
   if (B <= 0) return 0;
   if (B > 1024 || H <= 0 || max_pages <= 0) return -1;
   if (dq <= 0 || dv <= 0 || dv > dq || dq % 8 != 0 || dv % 8 != 0 || dv > ML_MAX_LORA || dq > ML_MAX_TILES * 64 || (dv < dq && dv % 64 != 0) || window < 0)
@@ -438,7 +439,7 @@ extern "C" int fb_mla_decode(const void* q, const void* lat_pool, void* out, con
     static DeviceOnce cfg;                                                                                            \
     if (cfg.need()) { cudaFuncSetAttribute(mla_decode_kernel<BF, GPV>, cudaFuncAttributeMaxDynamicSharedMemorySize, ml_smem(ML_MAX_TILES)); } \
     launch_k<PDL_ATTN>(mla_decode_kernel<BF, GPV>, dim3(sm_count), dim3(192), smem, stream, 0, tmLat, tmQ, p);           \
-    launch_k<PDL_COMBINE>(mla_combine_kernel<BF>, dim3(B, H), dim3(128), 0, stream, 0, part_o, part_ml, item_range, (uint16_t*)out, H, n_groups, dv, p.o_stride); \
+    launch_k<PDL_COMBINE>(mla_combine_kernel<BF>, dim3(B, H), dim3(128), 0, stream, 0, part_o, part_ml, item_range, (uint16_t*)out, H, n_groups, dv, p.o_stride, head_gate); \
   }
   if (dtype == 1) { if (gp == 16) FB_MLA_LAUNCH(true, 16) else FB_MLA_LAUNCH(true, 32) }
   else { if (gp == 16) FB_MLA_LAUNCH(false, 16) else FB_MLA_LAUNCH(false, 32) }

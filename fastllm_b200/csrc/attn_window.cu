@@ -1,5 +1,6 @@
-// Prefill attention with an optional sliding window (which may keep the first tokens of the sequence) or chunk mask, soft-capped scores
-// and a sink per head in the softmax, for sm_100a (tcgen05 + TMEM).
+// Prefill attention with an optional sliding window (which may keep the first tokens of the sequence) or chunk mask, soft-capped scores,
+// a sink per head in the softmax or sigmoid weights in its place, and outputs turned back by the query's position, for sm_100a
+// (tcgen05 + TMEM).
 //
 // Keys and values are contiguous rows (the expanded latents of the keys a batch reads, one head per query head) or the cache pages
 // themselves (grouped-query attention: a step of 64 keys lies inside one 128-token page).  One CTA owns one head and up to 256
@@ -8,7 +9,8 @@
 //     S_b[128 q x 64 k] = Q_b * K^T        O_b[128 q x V] += P_b * V          b = 0, 1
 // A block takes part only in the steps its rows see (the causal frontier at one end, the window at the other).  Head widths are
 // any multiple of 8: the operand maps are bounded per head, so the tail of a 64-column tile is zero.  Kept first tokens are steps of
-// their own ahead of the window's, shared by both blocks.  The epilogue normalises (with the sink's term) and applies the output gate
+// their own ahead of the window's, shared by both blocks.  Expanded keys may be followed by a part that all heads share (rotated
+// dimensions): its tiles come from the shared rows, the queries' from behind every head's own dimensions.  The epilogue normalises (with the sink's term) and applies the output gate
 // o * sigmoid(g), one per element or one per head, where the layer has one.
 #include "ptx.cuh"
 #include "launch.h"
@@ -32,6 +34,7 @@ struct AttnWindowParams {
   uint16_t* out; long long ld_out;
   const uint16_t* gate; long long ld_gate;
   int D, V, dt, vt;                               // head widths, their 64-column tiles
+  int R, rt;                                      // width of the shared key part (0: none) and its tiles, behind the dt tiles of D
   int stages, window;
   int chunk;                                      // > 0 (instead of a window): a query sees the keys of its own chunk of positions
   int group;                                      // query heads per key / value head
@@ -42,6 +45,9 @@ struct AttnWindowParams {
   float cap_lim, cap_p[6];                        // products up to cap_lim: the capped score is s * polynomial(s^2)
   const float* sinks;                             // [heads] or null
   const float* head_gate; long long ld_head_gate;      // one logit per (row, head)
+  const float* score_bias;                        // [heads]: the weight of a key is sigmoid(score + score_bias[h]) (null: softmax)
+  const float* cos_v; const float* sin_v;         // [tab_rows, rot_v / 2]: output pairs (2m, 2m + 1) are turned back by the position
+  int rot_v, tab_rows;
   uint32_t idesc_s, idesc_o;
 };
 
@@ -61,14 +67,16 @@ __device__ __forceinline__ float aw_capped(const AttnWindowParams& p, float s) {
   return p.cap_log2 - __fdividef(2.f * p.cap_log2, 1.f + exp2f(s * p.cap_in));
 }
 
-// EXT: soft cap, kept tokens, sinks and head gates are looked at
-template <bool BF16, bool EXT>
+// MODE: 0 plain softmax; 1 soft cap, kept tokens, sinks, head gates and turned outputs are looked at; 2 sigmoid weights, with all of these
+// but sinks
+template <bool BF16, int MODE>
 __global__ void __launch_bounds__(320, 1)
 attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                   const AttnWindowParams p) {
+                   const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmKr, const AttnWindowParams p) {
+  constexpr bool EXT = MODE != 0;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int dt = p.dt, vt = p.vt, stages = p.stages;
+  const int own = p.dt, dt = own + p.rt, vt = p.vt, stages = p.stages;
   const int stage_bytes = (dt + vt) * AW_KT;
   uint8_t* q_smem = smem;                                   // [2 blocks][dt] tiles of 16 KB
   uint8_t* kv_smem = smem + 2 * dt * AW_QT;                 // [stages] x (K tiles, V tiles)
@@ -130,7 +138,8 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
       const int nb = rows > 128 ? 2 : 1;
       mbar_expect_tx(q_full, nb * dt * AW_QT);
       for (int b = 0; b < nb; ++b)
-        for (int j = 0; j < dt; ++j) tma_load_3d(q_smem + (b * dt + j) * AW_QT, &tmQ, q_full, j * 64, head, q_row0 + b * 128);
+        for (int j = 0; j < dt; ++j)
+          tma_load_3d(q_smem + (b * dt + j) * AW_QT, j < own ? &tmQ : &tmQr, q_full, (j < own ? j : j - own) * 64, head, q_row0 + b * 128);
       for (int it = 0; it < n_steps; ++it) {
         const int s = it % stages;
         const uint32_t ph = (uint32_t)(it / stages) & 1u;
@@ -145,7 +154,8 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         uint8_t* ks = kv_smem + s * stage_bytes;
         uint8_t* vb = ks + dt * AW_KT;
         mbar_expect_tx(&full_k[s], dt * AW_KT);
-        for (int j = 0; j < dt; ++j) tma_load_3d(ks + j * AW_KT, &tmK, &full_k[s], j * 64, kv_head, row);
+        for (int j = 0; j < own; ++j) tma_load_3d(ks + j * AW_KT, &tmK, &full_k[s], j * 64, kv_head, row);
+        for (int j = own; j < dt; ++j) tma_load_3d(ks + j * AW_KT, &tmKr, &full_k[s], (j - own) * 64, 0, row);
         mbar_expect_tx(&full_v[s], vt * AW_KT);
         for (int j = 0; j < vt; ++j) tma_load_3d(vb + j * AW_KT, &tmV, &full_v[s], j * 64, kv_head, row);
       }
@@ -154,9 +164,9 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
   } else if (warp == 1) {
     if (elect_one()) {
       const uint32_t qb = smem_u32(q_smem), pb = smem_u32(p_smem);
-      const int ks = (p.D + 15) / 16;              // 16-wide k steps of the S product
+      const int ks = (p.D + 15) / 16, kr = 4 * own, kre = kr + (p.R + 15) / 16;       // 16-wide k steps of the S product: [0, ks) and [kr, kre)
       auto issue_s = [&](int b, uint32_t kb) {
-        for (int k = 0; k < ks; ++k) {
+        for (int k = 0; k < kre; k = k + 1 == ks ? kr : k + 1) {
           const uint64_t da = make_smem_desc(qb + (b * dt + (k >> 2)) * AW_QT + (k & 3) * 32, 16, 1024, SWZ_128B);
           const uint64_t db = make_smem_desc(kb + (k >> 2) * AW_KT + (k & 3) * 32, 16, 1024, SWZ_128B);
           umma_f16(tmem0 + (uint32_t)(b * 64), da, db, p.idesc_s, k != 0 ? 1u : 0u);
@@ -217,6 +227,7 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     uint8_t* prow = p_smem + b * AW_PT + r * 128;
     const int cnt = (EXT ? kb[b] : 0) + e[b] - f[b];
     float m_run = -INFINITY, l_run = 0.f;
+    const float bias = MODE == 2 ? p.score_bias[head] * 1.4426950408889634f : 0.f;
     for (int n = 0; n < cnt; ++n) {
       const uint32_t iph = (uint32_t)n & 1u;
       mbar_wait(&s_full[b], iph, dead, KID_ATTN_WINDOW, 8);
@@ -255,6 +266,36 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
         }
       }
       const float sc = cap ? 1.f : p.scale_log2;
+      if (MODE == 2) {
+        // P = sigmoid(score + bias): no maximum, no sum, nothing to rescale; one reciprocal serves two scores (clamped so that the
+        // product of two denominators stays finite: a weight below 2^-60 counts as that)
+        if (n > 0) {
+          mbar_wait(&o_full[b], iph ^ 1u, dead, KID_ATTN_WINDOW, 9);
+          tc_fence_after_sync();
+        }
+#pragma unroll
+        for (int g = 0; g < 8; ++g) {
+          uint32_t pk[4];
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const int c = 8 * g + 2 * j, kv = kv0 + c;
+            const float a0 = 1.f + exp2f(fminf(-fmaf(__uint_as_float(sreg[c]), sc, bias), 60.f));
+            const float a1 = 1.f + exp2f(fminf(-fmaf(__uint_as_float(sreg[c + 1]), sc, bias), 60.f));
+            const float inv = __fdividef(1.f, a0 * a1);
+            float p0 = inv * a1, p1 = inv * a0;
+            if (!full_step) {
+              if (!(kv <= pos && (kv >= first || kv < p.keep))) p0 = 0.f;
+              if (!(kv + 1 <= pos && (kv + 1 >= first || kv + 1 < p.keep))) p1 = 0.f;
+            }
+            pk[j] = pack_16<BF16>(p0, p1);
+          }
+          *reinterpret_cast<uint4*>(prow + ((g ^ (r & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+        }
+        fence_proxy_async_smem();
+        tc_fence_before_sync();
+        mbar_arrive(&p_ready[b]);
+        continue;
+      }
       if (full_step) {
 #pragma unroll
         for (int j = 0; j < 64; ++j) {
@@ -312,10 +353,10 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
     if (cnt > 0) {
       mbar_wait(&o_full[b], (uint32_t)(cnt - 1) & 1u, dead, KID_ATTN_WINDOW, 10);
       tc_fence_after_sync();
-      float inv_l = l_run > 0.f ? 1.f / l_run : 0.f;
+      float inv_l = MODE == 2 ? 1.f : l_run > 0.f ? 1.f / l_run : 0.f;
       const bool live = b * 128 + r < rows;
       const size_t row = (size_t)(q_row0 + b * 128 + r);
-      if (EXT && p.sinks != nullptr && l_run > 0.f) {
+      if (MODE == 1 && p.sinks != nullptr && l_run > 0.f) {
         const float sink = p.sinks[head] * 1.4426950408889634f, mx = fmaxf(m_run, sink), fac = exp2f(m_run - mx);
         inv_l = fac / (l_run * fac + exp2f(sink - mx));
       }
@@ -335,6 +376,25 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
             float v[8];
 #pragma unroll
             for (int j = 0; j < 8; ++j) v[j] = __uint_as_float(oreg[8 * g + j]) * inv_l;
+            if (EXT && p.rot_v > 0) {
+              const int half = p.rot_v >> 1, m0 = (c0 + 8 * g) >> 1;
+              const size_t at = (size_t)(pos < p.tab_rows ? pos : p.tab_rows - 1) * half + m0;
+              float cs[4], sn[4];
+              if ((half & 3) == 0 && m0 < half) {
+                const float4 a = *reinterpret_cast<const float4*>(p.cos_v + at), c = *reinterpret_cast<const float4*>(p.sin_v + at);
+                cs[0] = a.x; cs[1] = a.y; cs[2] = a.z; cs[3] = a.w;
+                sn[0] = c.x; sn[1] = c.y; sn[2] = c.z; sn[3] = c.w;
+              } else {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) { cs[j] = m0 + j < half ? p.cos_v[at + j] : 1.f; sn[j] = m0 + j < half ? p.sin_v[at + j] : 0.f; }
+              }
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                const float u = v[2 * j], w = v[2 * j + 1];
+                v[2 * j] = u * cs[j] + w * sn[j];
+                v[2 * j + 1] = w * cs[j] - u * sn[j];
+              }
+            }
             if (grow != nullptr) {
               const uint4 gv = *reinterpret_cast<const uint4*>(grow + c0 + 8 * g);
               const float2 g0 = unpack_16<BF16>(gv.x), g1 = unpack_16<BF16>(gv.y), g2 = unpack_16<BF16>(gv.z), g3 = unpack_16<BF16>(gv.w);
@@ -355,8 +415,8 @@ attn_window_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constan
 }
 
 // Ring depth that fits beside the queries and probabilities; 0: the head widths are outside the kernel.
-static int window_stages(int D, int V) {
-  const int dt = (D + 63) / 64, vt = (V + 63) / 64;
+static int window_stages(int D, int R, int V) {
+  const int dt = (D + 63) / 64 + (R + 63) / 64, vt = (V + 63) / 64;
   if (vt > 3) return 0;                                       // 2 accumulators of 64 vt columns beside S: 512 TMEM columns
   const int fixed = 2 * dt * AW_QT + 2 * AW_PT + 256 + 1024;
   const int n = (AW_SMEM_MAX - fixed) / ((dt + vt) * AW_KT);
@@ -367,55 +427,67 @@ static int window_stages(int D, int V) {
 
 using namespace fb;
 
-extern "C" int fb_attn_window_supported(int D, int V) { return D > 0 && V > 0 && D % 8 == 0 && V % 8 == 0 && window_stages(D, V) > 0 ? 1 : 0; }
+// D: a head's own key dimensions, R: those all heads share
+extern "C" int fb_attn_window_supported(int D, int R, int V) {
+  return D > 0 && R >= 0 && V > 0 && D % 8 == 0 && R % 8 == 0 && V % 8 == 0 && window_stages(D, R, V) > 0 ? 1 : 0;
+}
 
-static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, AttnWindowParams p, int n_blocks, int H, float scale,
-                         int dtype, cudaStream_t stream) {
-  p.dt = (p.D + 63) / 64; p.vt = (p.V + 63) / 64; p.stages = window_stages(p.D, p.V);
+static int launch_window(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmQr, const CUtensorMap& tmKr,
+                         AttnWindowParams p, int n_blocks, int H, float scale, int dtype, cudaStream_t stream) {
+  p.dt = (p.D + 63) / 64; p.rt = (p.R + 63) / 64; p.vt = (p.V + 63) / 64; p.stages = window_stages(p.D, p.R, p.V);
   p.scale_log2 = scale * 1.4426950408889634f;
   const uint32_t fm = dtype == 1 ? 1u : 0u;
   p.idesc_s = make_idesc(fm, fm, 0, 0, 128, AW_KV);
   p.idesc_o = make_idesc(fm, fm, 0, 1, 128, p.vt * 64);
-  const int smem = 2 * p.dt * AW_QT + p.stages * (p.dt + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
+  const int tiles = p.dt + p.rt, smem = 2 * tiles * AW_QT + p.stages * (tiles + p.vt) * AW_KT + 2 * AW_PT + 256 + 1024;
   const dim3 grid(H, n_blocks);
-#define FB_AW(BF, EXT)                                                                                                              \
+#define FB_AW(BF, MODE)                                                                                                             \
   {                                                                                                                                  \
     static DeviceOnce cfg;                                                                                                           \
-    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<BF, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);      \
-    attn_window_kernel<BF, EXT><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, p);                                                      \
+    if (cfg.need()) cudaFuncSetAttribute(attn_window_kernel<BF, MODE>, cudaFuncAttributeMaxDynamicSharedMemorySize, AW_SMEM_MAX);      \
+    attn_window_kernel<BF, MODE><<<grid, 320, smem, stream>>>(tmQ, tmK, tmV, tmQr, tmKr, p);                                         \
   }
-  if (p.cap_in != 0.f || p.keep > 0 || p.sinks != nullptr || p.head_gate != nullptr) { if (dtype == 1) FB_AW(true, true) else FB_AW(false, true) }
-  else { if (dtype == 1) FB_AW(true, false) else FB_AW(false, false) }
+  if (p.score_bias != nullptr) { if (dtype == 1) FB_AW(true, 2) else FB_AW(false, 2) }
+  else if (p.cap_in != 0.f || p.keep > 0 || p.sinks != nullptr || p.head_gate != nullptr || p.rot_v > 0) { if (dtype == 1) FB_AW(true, 1) else FB_AW(false, 1) }
+  else { if (dtype == 1) FB_AW(true, 0) else FB_AW(false, 0) }
 #undef FB_AW
   return (int)cudaGetLastError();
 }
 
-// q: packed rows [T, >= H * D] (row stride ld_q), k: [n_keys, >= H * D], v: [n_keys, >= H * V], out [T, H * V], gate (optional) like out.
-extern "C" int fb_attn_window(const void* q, long long ld_q, int T, const void* k, long long ld_k, const void* v, long long ld_v, int n_keys,
-                              void* out, long long ld_out, const void* gate, long long ld_gate, const int* blocks, int n_blocks, int H,
-                              int D, int V, int window, float scale, int dtype, void* stream_) {
+// q: packed rows [T, >= H * q_head] (row stride ld_q; a head is [D own | R shared-part dimensions | padding], q_head apart), k: [n_keys, >= H * D],
+// v: [n_keys, >= H * V], k_shared: [n_keys, >= R] (R = 0: none), out [T, H * V], gate (optional) like out, head_gate (optional): fp32
+// logits, one per (row, head).
+extern "C" int fb_attn_window(const void* q, long long ld_q, int q_head, int T, const void* k, long long ld_k, const void* v, long long ld_v, const void* k_shared,
+                              long long ld_shared, int n_keys, void* out, long long ld_out, const void* gate, long long ld_gate, const float* head_gate,
+                              long long ld_head_gate, const int* blocks, int n_blocks, int H, int D, int R, int V, int window, float scale, int dtype,
+                              void* stream_) {
   if (n_blocks <= 0) return 0;
-  if (window_stages(D, V) == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || n_keys <= 0 || H <= 0 || n_blocks > 65535 || window < 0 || ld_out % 8 != 0 ||
-      ld_gate % 8 != 0)
+  if (D <= 0 || R < 0 || V <= 0 || window_stages(D, R, V) == 0 || D % 8 != 0 || R % 8 != 0 || V % 8 != 0 || q_head < D + R || q_head % 8 != 0 || T <= 0 || n_keys <= 0 || H <= 0 ||
+      n_blocks > 65535 || window < 0 || ld_out % 8 != 0 || ld_gate % 8 != 0 || (R > 0 && k_shared == nullptr))
     return -1;
-  CUtensorMap tmQ, tmK, tmV;
-  if (!make_tmap_3d(&tmQ, q, D, H, T, D, ld_q, 64, 128)) return -2;
+  CUtensorMap tmQ, tmK, tmV, tmQr, tmKr;
+  if (!make_tmap_3d(&tmQ, q, D, H, T, q_head, ld_q, 64, 128)) return -2;
   if (!make_tmap_3d(&tmK, k, D, H, n_keys, D, ld_k, 64, AW_KV)) return -2;
   if (!make_tmap_3d(&tmV, v, V, H, n_keys, V, ld_v, 64, AW_KV)) return -2;
+  tmQr = tmQ; tmKr = tmK;
+  if (R > 0 && !make_tmap_3d(&tmQr, reinterpret_cast<const uint16_t*>(q) + D, R, H, T, q_head, ld_q, 64, 128)) return -2;
+  if (R > 0 && !make_tmap_3d(&tmKr, k_shared, R, 1, n_keys, R, ld_shared, 64, AW_KV)) return -2;
   AttnWindowParams p = {};
   p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
-  p.D = D; p.V = V; p.window = window; p.group = 1;
-  return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
+  p.D = D; p.R = R; p.V = V; p.window = window; p.group = 1; p.head_gate = head_gate; p.ld_head_gate = ld_head_gate;
+  return launch_window(tmQ, tmK, tmV, tmQr, tmKr, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }
 
 // Grouped-query form over the cache pages: k_pool [num_slots, G, D], v_pool [num_slots, G, V], 128 slots a page; H / G
-// consecutive query heads share a key / value head; keep, softcap, sinks, head_gate as in fb_grouped_decode.  page_table: [requests, max_pages], a block's request is blocks[.][5].
+// consecutive query heads share a key / value head; keep, softcap, sinks, head_gate, score_bias and the output's rotation as in fb_grouped_decode.  page_table: [requests, max_pages], a block's request is blocks[.][5].
 extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const void* k_pool, const void* v_pool, long long num_slots,
                                     const int* page_table, int max_pages, void* out, long long ld_out, const void* gate, long long ld_gate,
                                     const int* blocks, int n_blocks, int H, int G, int D, int V, int window, int chunk, int keep, float scale,
-                                    float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, int dtype, void* stream_) {
+                                    float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, const float* score_bias, const float* cos_v,
+                                    const float* sin_v, int rot_v, int tab_rows, int dtype, void* stream_) {
   if (n_blocks <= 0) return 0;
-  if (window_stages(D, V) == 0 || D % 8 != 0 || V % 8 != 0 || T <= 0 || num_slots < 128 || H <= 0 || G <= 0 || H % G != 0 || n_blocks > 65535 ||
+  if (D <= 0 || V <= 0 || window_stages(D, 0, V) == 0 || rot_v < 0 || (rot_v & 1) || rot_v > V || (score_bias != nullptr && sinks != nullptr) ||
+      (rot_v > 0 && (cos_v == nullptr || sin_v == nullptr || tab_rows <= 0)) || D % 8 != 0 || V % 8 != 0 || T <= 0 || num_slots < 128 || H <= 0 || G <= 0 || H % G != 0 || n_blocks > 65535 ||
       window < 0 || chunk < 0 || keep < 0 || softcap < 0.f || max_pages <= 0 || ld_out % 8 != 0 || ld_gate % 8 != 0)
     return -1;
   CUtensorMap tmQ, tmK, tmV;
@@ -426,6 +498,7 @@ extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const 
   p.blocks = blocks; p.out = (uint16_t*)out; p.ld_out = ld_out; p.gate = (const uint16_t*)gate; p.ld_gate = ld_gate;
   p.D = D; p.V = V; p.window = window; p.chunk = chunk; p.group = H / G;
   p.page_table = page_table; p.max_pages = max_pages; p.num_pages = (int)(num_slots / 128);
+  p.score_bias = score_bias; p.cos_v = cos_v; p.sin_v = sin_v; p.rot_v = rot_v; p.tab_rows = tab_rows;
   p.keep = window > 0 ? keep : 0; p.sinks = sinks; p.head_gate = head_gate; p.ld_head_gate = ld_head_gate;
   if (softcap > 0.f) {
     const double k = (double)scale / softcap;                 // x = k s
@@ -435,5 +508,5 @@ extern "C" int fb_attn_window_paged(const void* q, long long ld_q, int T, const 
     double f = 1.4426950408889634 * scale;
     for (int i = 0; i < 6; ++i, f *= k * k) p.cap_p[i] = (float)(AW_TANH[i] * f);
   }
-  return launch_window(tmQ, tmK, tmV, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
+  return launch_window(tmQ, tmK, tmV, tmQ, tmK, p, n_blocks, H, scale, dtype, reinterpret_cast<cudaStream_t>(stream_));
 }

@@ -102,24 +102,26 @@ __global__ void __launch_bounds__(256) gemm_full32_kernel(const Full32Params p) 
 }
 
 // Latent attention of one (row, head) per CTA over the paged latent cache, any latent width:
-//   score[j] = scale * q[row, head] . c[j],  out = sum_j softmax(score)[j] c[j],  first <= j <= position
+//   score[j] = scale * q[row, head] . c[j],  out = sum_j softmax(score)[j] c[j][:RV],  first <= j <= position
+// where R >= RV: what follows a row's values takes part in the scores alone (a rotated key part).  head_gate: one fp32 logit per head.
 // 128 threads: a warp scores one key at a time (lanes over the latent), then every thread accumulates its latent columns.
 constexpr int L32_KEYS = 64;
 template <int DT>
 __global__ void __launch_bounds__(128) latent_attn32_kernel(const typename F32In<DT>::T* __restrict__ q, const typename F32In<DT>::T* __restrict__ pool,
                                                             typename F32In<DT>::T* __restrict__ out, const int* __restrict__ page_table,
                                                             const int* __restrict__ kv_lens, int max_pages, int page_len, int H, int R,
-                                                            int ld, int window, float scale) {
+                                                            int RV, int ld, int window, float scale, const float* __restrict__ head_gate) {
   extern __shared__ float sm[];
   float* qs = sm;                       // [R]
-  float* os = sm + R;                   // [R] running output
+  float* os = sm + R;                   // [RV] running output
   __shared__ float sc[L32_KEYS];
   __shared__ int rows[L32_KEYS];
   const int t = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int n = kv_lens[t];
   const int first = (window > 0 && n > window) ? n - window : 0;
   const typename F32In<DT>::T* qp = q + ((size_t)t * H + h) * ld;
-  for (int i = tid; i < R; i += 128) { qs[i] = F32In<DT>::ld(qp[i]); os[i] = 0.f; }
+  for (int i = tid; i < R; i += 128) qs[i] = F32In<DT>::ld(qp[i]);
+  for (int i = tid; i < RV; i += 128) os[i] = 0.f;
   float m_run = -INFINITY, l_run = 0.f;
   for (int j0 = first; j0 < n; j0 += L32_KEYS) {
     const int cnt = n - j0 < L32_KEYS ? n - j0 : L32_KEYS;
@@ -148,22 +150,25 @@ __global__ void __launch_bounds__(128) latent_attn32_kernel(const typename F32In
     for (int j = 0; j < cnt; ++j) l += sc[j];
     l_run = l_run * fac + l;
     m_run = mx;
-    for (int i = tid; i < R; i += 128) {
+    for (int i = tid; i < RV; i += 128) {
       float a = os[i] * fac;
       for (int j = 0; j < cnt; ++j) a = fmaf(sc[j], F32In<DT>::ld(pool[(size_t)rows[j] * ld + i]), a);
       os[i] = a;
     }
   }
-  const float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
-  typename F32In<DT>::T* op = out + ((size_t)t * H + h) * ld;
-  for (int i = tid; i < ld; i += 128) op[i] = F32In<DT>::st(i < R ? os[i] * inv : 0.f);
+  float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  if (head_gate != nullptr) inv *= 1.0f / (1.0f + expf(-head_gate[(size_t)t * H + h]));
+  typename F32In<DT>::T* op = out + ((size_t)t * H + h) * RV;
+  for (int i = tid; i < RV; i += 128) op[i] = F32In<DT>::st(os[i] * inv);
 }
 
 // Grouped-query attention of one (row, query head) per CTA over paged keys and values, any widths, fp32 arithmetic:
 //   out = (sum_j softmax(score_j) v_j) * sigmoid(gate),  score_j = scale q . k_j, soft-capped where the layer does
 // Row t sees the keys of its own page-table row; its position is kv_lens[t] - 1.  The first key: chunk: position - position % chunk;
 // window: position - window + 1, beside the first `keep` of the sequence; neither: 0.  sinks: one more term exp(sink) per head in the
-// denominator.  The gate is elementwise (`gate`, 16-bit or fp32) or one fp32 logit per head (`head_gate`).
+// denominator.  The gate is elementwise (`gate`, 16-bit or fp32) or one fp32 logit per head (`head_gate`).  score_bias: the weights are
+// sigmoid(score + score_bias[h]) and not normalised.  rot_v: the leading dimensions of the output, in pairs (2m, 2m + 1), are turned
+// back by the row's position (tables [tab_rows, rot_v / 2]) before any gate.
 struct Grouped32Params {
   const void* q; const void* k_pool; const void* v_pool; void* out; const void* gate;
   long long ld_q, ld_out, ld_gate;
@@ -172,6 +177,9 @@ struct Grouped32Params {
   float scale, softcap;
   const float* sinks;
   const float* head_gate; long long ld_head_gate;
+  const float* score_bias;
+  const float* cos_v; const float* sin_v;
+  int rot_v, tab_rows;
 };
 
 template <int DT>
@@ -213,26 +221,29 @@ __global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Para
       for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
       s *= p.scale;
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-      if (lane == 0) sc[j] = s;
+      if (lane == 0) sc[j] = p.score_bias != nullptr ? 1.0f / (1.0f + expf(-(s + p.score_bias[h]))) : s;
     }
     __syncthreads();
-    float mx = m_run;
-    for (int j = 0; j < cnt; ++j) mx = fmaxf(mx, sc[j]);
-    const float fac = m_run == -INFINITY ? 0.f : expf(m_run - mx);
-    __syncthreads();
-    if (tid < cnt) sc[tid] = expf(sc[tid] - mx);
-    __syncthreads();
-    float l = 0.f;
-    for (int j = 0; j < cnt; ++j) l += sc[j];
-    l_run = l_run * fac + l;
-    m_run = mx;
+    float fac = 1.f;
+    if (p.score_bias == nullptr) {
+      float mx = m_run;
+      for (int j = 0; j < cnt; ++j) mx = fmaxf(mx, sc[j]);
+      fac = m_run == -INFINITY ? 0.f : expf(m_run - mx);
+      __syncthreads();
+      if (tid < cnt) sc[tid] = expf(sc[tid] - mx);
+      __syncthreads();
+      float l = 0.f;
+      for (int j = 0; j < cnt; ++j) l += sc[j];
+      l_run = l_run * fac + l;
+      m_run = mx;
+    }
     for (int i = tid; i < p.Vp; i += 128) {
       float a = os[i] * fac;
       for (int j = 0; j < cnt; ++j) a = fmaf(sc[j], F32In<DT>::ld(vp[((size_t)rows[j] * p.G + g) * p.Vp + i]), a);
       os[i] = a;
     }
   }
-  float inv = l_run > 0.f ? 1.0f / l_run : 0.f;
+  float inv = p.score_bias != nullptr ? 1.0f : l_run > 0.f ? 1.0f / l_run : 0.f;
   if (p.sinks != nullptr && l_run > 0.f) {
     const float sink = p.sinks[h], mx = fmaxf(m_run, sink), fac = expf(m_run - mx);
     inv = fac / (l_run * fac + expf(sink - mx));
@@ -240,6 +251,16 @@ __global__ void __launch_bounds__(128) grouped_attn32_kernel(const Grouped32Para
   if (p.head_gate != nullptr) inv *= 1.0f / (1.0f + expf(-p.head_gate[(size_t)t * p.ld_head_gate + h]));
   T* op = reinterpret_cast<T*>(p.out) + (size_t)t * p.ld_out + (size_t)h * p.Vp;
   const T* gp = p.gate != nullptr ? reinterpret_cast<const T*>(p.gate) + (size_t)t * p.ld_gate + (size_t)h * p.Vp : nullptr;
+  if (p.rot_v > 0) {
+    const int at = pos < 0 ? 0 : pos >= p.tab_rows ? p.tab_rows - 1 : pos, half = p.rot_v >> 1;
+    __syncthreads();
+    for (int m = tid; m < half; m += 128) {
+      const float c = p.cos_v[(size_t)at * half + m], s = p.sin_v[(size_t)at * half + m], u = os[2 * m], v = os[2 * m + 1];
+      os[2 * m] = u * c + v * s;
+      os[2 * m + 1] = v * c - u * s;
+    }
+    __syncthreads();
+  }
   for (int i = tid; i < p.Vp; i += 128) {
     float v = os[i] * inv;
     if (gp != nullptr) v *= 1.0f / (1.0f + expf(-F32In<DT>::ld(gp[i])));
@@ -273,20 +294,20 @@ extern "C" int fb_gemm_full32(const void* X, const void* W, void* out, const voi
   return (int)cudaGetLastError();
 }
 
-// q / out: [T, H, ld], pool: [num_slots, ld], latent width R <= ld.  page_table [T, max_pages] and kv_lens [T] belong to the rows: row t
+// q: [T, H, ld], pool: [num_slots, ld]; scores over the first R <= ld columns; out: [T, H, RV], the first RV <= R.  page_table [T, max_pages] and kv_lens [T] belong to the rows: row t
 // sees keys [max(0, kv_lens[t] - window), kv_lens[t]).
-extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, const int* page_table, const int* kv_lens, int T, int H, int R,
-                                int ld, int max_pages, int page_len, int window, float scale, int dt, void* stream) {
+extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, const int* page_table, const int* kv_lens, int T, int H, int R, int RV,
+                                int ld, int max_pages, int page_len, int window, float scale, const float* head_gate, int dt, void* stream) {
   if (T <= 0 || H <= 0) return 0;
-  if (R <= 0 || ld < R || R > 24576 || H > 65535 || max_pages <= 0 || page_len <= 0 || dt < 0 || dt > 2) return -1;
-  const size_t smem = (size_t)R * 8;
+  if (R <= 0 || RV <= 0 || RV > R || ld < R || R > 24576 || H > 65535 || max_pages <= 0 || page_len <= 0 || dt < 0 || dt > 2) return -1;
+  const size_t smem = (size_t)(R + RV) * 4;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define GO(DT)                                                                                                                     \
   {                                                                                                                                \
     static DeviceOnce cfg;                                                                                                         \
     if (cfg.need()) cudaFuncSetAttribute(latent_attn32_kernel<DT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 24576 * 8);         \
     latent_attn32_kernel<DT><<<dim3(T, H), 128, smem, s>>>((const F32In<DT>::T*)q, (const F32In<DT>::T*)pool, (F32In<DT>::T*)out,  \
-                                                           page_table, kv_lens, max_pages, page_len, H, R, ld, window, scale);     \
+                                                           page_table, kv_lens, max_pages, page_len, H, R, RV, ld, window, scale, head_gate); \
   }
   if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
 #undef GO
@@ -297,12 +318,14 @@ extern "C" int fb_latent_attn32(const void* q, const void* pool, void* out, cons
 extern "C" int fb_grouped_attn32(const void* q, long long ld_q, const void* k_pool, const void* v_pool, void* out, long long ld_out,
                                  const void* gate, long long ld_gate, const int* page_table, const int* kv_lens, int T, int H, int G, int D,
                                  int Dp, int Vp, int max_pages, int num_pages, int page_len, int window, int chunk, int keep, float scale,
-                                 float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, int dt, void* stream) {
+                                 float softcap, const float* sinks, const float* head_gate, long long ld_head_gate, const float* score_bias, const float* cos_v,
+                                 const float* sin_v, int rot_v, int tab_rows, int dt, void* stream) {
   if (T <= 0) return 0;
   if (H <= 0 || G <= 0 || H % G != 0 || H > 65535 || D <= 0 || Dp < D || Vp <= 0 || Dp + Vp > 49152 || max_pages <= 0 || num_pages <= 0 ||
-      page_len <= 0 || window < 0 || chunk < 0 || keep < 0 || dt < 0 || dt > 2)
+      page_len <= 0 || window < 0 || chunk < 0 || keep < 0 || dt < 0 || dt > 2 || rot_v < 0 || (rot_v & 1) || rot_v > Vp ||
+      (rot_v > 0 && (cos_v == nullptr || sin_v == nullptr || tab_rows <= 0)))
     return -1;
-  Grouped32Params p{q, k_pool, v_pool, out, gate, ld_q, ld_out, ld_gate, page_table, kv_lens, H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, keep, scale, softcap, sinks, head_gate, ld_head_gate};
+  Grouped32Params p{q, k_pool, v_pool, out, gate, ld_q, ld_out, ld_gate, page_table, kv_lens, H, G, D, Dp, Vp, max_pages, num_pages, page_len, window, chunk, keep, scale, softcap, sinks, head_gate, ld_head_gate, score_bias, cos_v, sin_v, rot_v, tab_rows};
   const size_t smem = (size_t)(Dp + Vp) * 4;
   cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
 #define GO(DT)                                                                                                          \

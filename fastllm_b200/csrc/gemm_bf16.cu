@@ -515,8 +515,8 @@ extern "C" int fb_gemm_qkv_post(const void* X, const void* W, const void* bias, 
 // Used for the absorbed multi-head-latent-attention projections (one small matrix per head).  M <= 256, K % 8 == 0
 // (a partial last k block of 64 reads the neighbouring slice of X against zero-filled weight columns), N % 4 == 0, x_cols % 8 == 0, out_cols % 4 == 0.
 // `gate` (optional, 16-bit, row stride ld_gate): out[m, c] is multiplied by sigmoid(gate[m, c]).
-extern "C" int fb_gemm_16bit_batched_gate(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw,
-                                          int ld_out, int x_cols, int out_cols, const void* gate, int ld_gate, int dtype, void* stream_) {
+static int gemm_16bit_batched_impl(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw, int ld_out,
+                                   int x_cols, int out_cols, const void* gate, int ld_gate, int flags, int dtype, void* stream_) {
   using namespace fb;
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
   if (M <= 0 || N <= 0 || batch <= 0) return 0;
@@ -526,7 +526,7 @@ extern "C" int fb_gemm_16bit_batched_gate(const void* X, const void* W, void* ou
   p.M = M; p.N = N; p.K = K; p.ld_out = ld_out; p.ld_res = 0;
   p.kb_total = (K + 63) / 64; p.kb_per_split = p.kb_total;
   p.gate = gate; p.ld_gate = ld_gate;
-  p.flags = 0;
+  p.flags = flags;
   p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
   for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
   p.batch_w_rows = N; p.batch_x_cols = x_cols; p.batch_out_cols = out_cols;
@@ -552,6 +552,45 @@ extern "C" int fb_gemm_16bit_batched_gate(const void* X, const void* W, void* ou
                         : launch_smallm<256, false, 1>(tmW, tmX, p, 1, n_tiles, stream, batch));
   }
 #undef FB_BT
+}
+
+extern "C" int fb_gemm_16bit_batched_gate(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw,
+                                          int ld_out, int x_cols, int out_cols, const void* gate, int ld_gate, int dtype, void* stream_) {
+  return gemm_16bit_batched_impl(X, W, out, M, N, K, batch, ldx, ldw, ld_out, x_cols, out_cols, gate, ld_gate, 0, dtype, stream_);
+}
+
+// Block-diagonal product with fp32 results: out[m, z * N + n] = sum_k X[m, z * K + k] * W[z * N + n, k], z < batch.  Any M; more than 256
+// rows take the large-M kernel where N is a multiple of its tile (128), 256 rows at a time otherwise.
+extern "C" int fb_gemm_16bit_blocks(const void* X, const void* W, float* out, int M, int N, int K, int batch, int ldx, int ld_out, int dtype, void* stream_) {
+  using namespace fb;
+  if (M <= 0 || N <= 0 || batch <= 0) return 0;
+  if (K % 8 != 0 || N % 8 != 0 || ld_out % 4 != 0 || (dtype != 0 && dtype != 1)) return -1;
+  if (M <= 256 || N % 128 != 0) {
+    for (int m0 = 0; m0 < M; m0 += 256) {
+      const int rc = gemm_16bit_batched_impl(reinterpret_cast<const uint16_t*>(X) + (size_t)m0 * ldx, W, out + (size_t)m0 * ld_out, M - m0 < 256 ? M - m0 : 256, N, K,
+                                             batch, ldx, K, ld_out, K, N, nullptr, 0, GEMM_OUT_F32, dtype, stream_);
+      if (rc != 0) return rc;
+    }
+    return 0;
+  }
+  GemmParams p;
+  p.out = out; p.bias = nullptr; p.residual = nullptr;
+  p.M = M; p.N = batch * N; p.K = K; p.ld_out = ld_out; p.ld_res = 0;
+  p.kb_total = (K + 63) / 64; p.kb_per_split = p.kb_total;      // a partial last block reads the next slice of X against zero-filled weights
+  p.flags = GEMM_OUT_F32;
+  p.scatter_tp = 0; p.scatter_rows = 1; p.scatter_rank = 0; p.w_row0 = 0; p.x_row0 = 0;
+  for (int i = 0; i < 8; ++i) p.scatter_out[i] = nullptr;
+  p.batch_w_rows = N; p.batch_x_cols = K;
+  const bool bf16 = dtype == 1;
+  const int bn = N % 256 == 0 ? 256 : 128;
+  p.idesc = make_idesc(bf16 ? 1 : 0, bf16 ? 1 : 0, 0, 0, 128, bn);
+  cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
+  CUtensorMap tmW, tmX;
+  if (!make_tmap_2d(&tmX, X, M, (uint64_t)batch * K, ldx, 128, 64, 2, 3)) return -2;
+  if (!make_tmap_2d(&tmW, W, (uint64_t)batch * N, K, K, bn, 64, 2, 3)) return -2;
+  if (bn == 256)
+    return (int)(bf16 ? launch_largem<256, true>(tmX, tmW, p, stream, nullptr) : launch_largem<256, false>(tmX, tmW, p, stream, nullptr));
+  return (int)(bf16 ? launch_largem<128, true>(tmX, tmW, p, stream, nullptr) : launch_largem<128, false>(tmX, tmW, p, stream, nullptr));
 }
 
 extern "C" int fb_gemm_16bit_batched(const void* X, const void* W, void* out, int M, int N, int K, int batch, int ldx, int ldw, int ld_out,

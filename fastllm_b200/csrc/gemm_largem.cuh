@@ -200,13 +200,14 @@ __device__ __forceinline__ void gemm_largem_device(const CUtensorMap& tmX, const
       for (int t = blockIdx.x; t < tiles; t += gridDim.x) {
         int m_tile, n_tile;
         hook.tile_coords(t, tiles_m, tiles_n, m_tile, n_tile);
+        const int x0 = p.batch_w_rows > 0 ? n_tile * BN / p.batch_w_rows * p.batch_x_cols : 0;      // block-diagonal weights
         for (int i = 0; i < kb_cnt; ++i, ++it) {
           const int s = it % Cfg::STAGES;
           const uint32_t ph = (uint32_t)(it / Cfg::STAGES) & 1u;
           if (!mbar_wait(&empty_bar[s], ph ^ 1u, dead, KID_GEMM_LARGEM, 1)) break;
           uint8_t* a = smem + s * Cfg::STAGE_BYTES;
           mbar_expect_tx(&full_bar[s], Cfg::STAGE_BYTES);
-          tma_load_2d(a, &tmX, &full_bar[s], i * 64, m_tile * 128);
+          tma_load_2d(a, &tmX, &full_bar[s], x0 + i * 64, m_tile * 128);
           tma_load_2d(a + Cfg::A_BYTES, &tmW, &full_bar[s], i * 64, n_tile * BN);
         }
         if (dead) break;

@@ -76,6 +76,7 @@ struct GemmParams {
   // Batched mode (grid.z = batch index z): weight rows start at z * batch_w_rows, the activation's k range at column
   // z * batch_x_cols, the output at column z * batch_out_cols -- one launch for a GEMM per attention head (the absorbed
   // multi-head-latent-attention projections, where every head has its own small matrix and its own slice of the activations).
+  // The large-M kernel takes the same as a block-diagonal product: the output column selects the slice of the activations.
   int batch_w_rows = 0, batch_x_cols = 0, batch_out_cols = 0;
   float alpha = 1.f;                         // GEMM_RES_F32
   const void* gate = nullptr;                // 16-bit [M, >= N] (batched: + z * batch_out_cols): out = acc * sigmoid(gate)

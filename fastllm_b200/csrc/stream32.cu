@@ -1,6 +1,7 @@
 // Operators of models whose residual stream is fp32: token embedding plus sinusoidal or learned positions, RMSNorm of an fp32 row
-// into the activation type, latent RMSNorm into the cache, per-head norm + rotary + cache append, and the end of a sub-layer (output
-// norm, residual, next norm) for a plain output or a mixture-of-experts combine.
+// into the activation type, latent rows (norms, rotary key part) into the cache, per-head norm + rotary + cache append, and the end of
+// a sub-layer (output norm, residual, next norm) for a plain output or a mixture-of-experts combine, or of a layer whose sub-layers
+// stand side by side behind gates of their own.
 //
 // One CTA owns a row; the row stays in shared memory between the reduction and the normalised write, so every operand is read
 // once.  Compiled without fast-math: angles, square roots and divisions are the correctly rounded fp32 ones.
@@ -178,23 +179,199 @@ __global__ void embed_pos_norm_kernel(const int* __restrict__ ids, const int* __
   row_write<DT, VEC>(row, w, y + (size_t)t * H, H, inv);
 }
 
-// pool[slot] = RMSNorm over the first `n` columns of x[t] (columns [n, ld) of the entry are zero); slots < 0 go to `spare`
+// Everything between the input projection of latent attention and its next product, one CTA per token:
+//   cq[t] = RMSNorm(query latent) * q_norm                              (q_rank > 0; columns [q_rank, q_pad) are zero)
+//   pool[slot] = [RMSNorm(latent) * kv_norm | 0 | rotated key part | 0]  (rank of lv columns, rot of ld - lv; slots < 0 go to `spare`)
+//   gates[t] = the head gates' logits in fp32                            (n_gates > 0)
+struct LatentPostParams {
+  const void* x; long long ldx;
+  int q_col, q_rank, q_pad, kv_col, rank, lv, rot_col, rot, ld, neox, gate_col, n_gates;
+  const void* q_norm; const void* kv_norm;
+  const float* cos_tab; const float* sin_tab;
+  int tab_rows;
+  const int* positions; const int* slots;
+  void* cq; void* pool; float* gates;
+  long long spare;
+  float eps;
+};
+
 template <int DT>
-__global__ void latent_norm_kernel(const typename Act<DT>::T* __restrict__ x, int ldx, const typename Act<DT>::T* __restrict__ w,
-                                   const int* __restrict__ slots, typename Act<DT>::T* __restrict__ pool, int n, int ld, long long spare, float eps) {
+__global__ void latent_post_kernel(const LatentPostParams p) {
+  typedef typename Act<DT>::T T;
   extern __shared__ float row[];
-  __shared__ float sh[32];
+  __shared__ float sh[2][32];
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x;
-  const typename Act<DT>::T* xp = x + (size_t)t * ldx;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = Act<DT>::ld(xp[i]); row[i] = v; ss += v * v; }
-  ss = block_sum32(ss, sh);
-  const float inv = 1.0f / sqrtf(ss / (float)n + eps);
-  const int slot = slots[t];
-  typename Act<DT>::T* yp = pool + (size_t)(slot < 0 ? spare : (long long)slot) * ld;
-  for (int i = threadIdx.x; i < ld; i += blockDim.x) yp[i] = Act<DT>::st(i < n ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+  const T* xp = reinterpret_cast<const T*>(p.x) + (size_t)t * p.ldx;
+  const int slot = p.slots[t];
+  T* yp = reinterpret_cast<T*>(p.pool) + (size_t)(slot < 0 ? p.spare : (long long)slot) * p.ld;
+  float qs = 0.f, ks = 0.f;
+  float* krow = row + p.q_rank;
+  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) { const float v = Act<DT>::ld(xp[p.q_col + i]); row[i] = v; qs += v * v; }
+  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) { const float v = Act<DT>::ld(xp[p.kv_col + i]); krow[i] = v; ks += v * v; }
+  for (int i = threadIdx.x; i < p.n_gates; i += blockDim.x) p.gates[(size_t)t * p.n_gates + i] = Act<DT>::ld(xp[p.gate_col + i]);
+  if (p.rot > 0) {
+    int pos = p.positions[t];
+    pos = pos < 0 ? 0 : (pos >= p.tab_rows ? p.tab_rows - 1 : pos);
+    const int half = p.rot >> 1;
+    for (int j = threadIdx.x; 2 * j < p.ld - p.lv; j += blockDim.x) {
+      if (j < half) {
+        const int i0 = p.neox ? j : 2 * j, i1 = p.neox ? j + half : 2 * j + 1;
+        const float c = p.cos_tab[(size_t)pos * half + j], s = p.sin_tab[(size_t)pos * half + j];
+        const float u = Act<DT>::ld(xp[p.rot_col + i0]), v = Act<DT>::ld(xp[p.rot_col + i1]);
+        yp[p.lv + i0] = Act<DT>::st(u * c - v * s);
+        yp[p.lv + i1] = Act<DT>::st(v * c + u * s);
+      } else {
+        yp[p.lv + 2 * j] = yp[p.lv + 2 * j + 1] = Act<DT>::st(0.f);
+      }
+    }
+  }
+  if (p.q_rank > 0) {
+    qs = block_sum32(qs, sh[0]);
+    const float inv = 1.0f / sqrtf(qs / (float)p.q_rank + p.eps);
+    const T* w = reinterpret_cast<const T*>(p.q_norm);
+    T* cp = reinterpret_cast<T*>(p.cq) + (size_t)t * p.q_pad;
+    for (int i = threadIdx.x; i < p.q_pad; i += blockDim.x) cp[i] = Act<DT>::st(i < p.q_rank ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+  }
+  ks = block_sum32(ks, sh[1]);
+  const float inv = 1.0f / sqrtf(ks / (float)p.rank + p.eps);
+  const T* w = reinterpret_cast<const T*>(p.kv_norm);
+  for (int i = threadIdx.x; i < p.lv; i += blockDim.x) yp[i] = Act<DT>::st(i < p.rank ? krow[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+}
+
+// dst[t, h, :width] = src[t, h, :width] with the first `rot` dimensions turned, pairs (2j, 2j + 1) or (neox) (j, j + rot / 2); dst may be src
+struct RopeHeadsParams {
+  const void* src; void* dst;
+  long long ld_src, ld_dst;
+  int T, H, head_src, head_dst, rot, width, neox, tab_rows;
+  const int* positions;
+  const float* cos_tab; const float* sin_tab;
+};
+
+template <int DT>
+__global__ void __launch_bounds__(256) rope_heads_kernel(const RopeHeadsParams p) {
+  typedef typename Act<DT>::T T;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int pairs = p.width >> 1, half = p.rot >> 1;
+  const long long total = (long long)p.T * p.H * pairs;
+  for (long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+    const int j = (int)(i % pairs), h = (int)(i / pairs % p.H), t = (int)(i / pairs / p.H);
+    const T* s = reinterpret_cast<const T*>(p.src) + (size_t)t * p.ld_src + (size_t)h * p.head_src;
+    T* d = reinterpret_cast<T*>(p.dst) + (size_t)t * p.ld_dst + (size_t)h * p.head_dst;
+    const bool halves = p.neox && j < half;
+    const int i0 = halves ? j : 2 * j, i1 = halves ? j + half : 2 * j + 1;
+    float u = Act<DT>::ld(s[i0]), v = Act<DT>::ld(s[i1]);
+    if (j < half) {
+      int pos = p.positions[t];
+      pos = pos < 0 ? 0 : (pos >= p.tab_rows ? p.tab_rows - 1 : pos);
+      const float c = p.cos_tab[(size_t)pos * half + j], sn = p.sin_tab[(size_t)pos * half + j], u0 = u;
+      u = u0 * c - v * sn;
+      v = v * c + u0 * sn;
+    }
+    d[i0] = Act<DT>::st(u);
+    d[i1] = Act<DT>::st(v);
+  }
+}
+
+// The end of a layer whose mixer and feed-forward stand side by side, each behind the sigmoid of its own logits, and the norms that open
+// the next one:
+//   h[t] += sigmoid(g1[t]) * y1[t] + sigmoid(g2[t]) * sum_k wts[t, k] ys[pos[t, k]]       (pos == nullptr: ys[t]; either part may be absent)
+//   x1[t] = Norm(h[t]) * w1,  x2[t] = Norm(h[t]) * w2                                      (w2 may be absent)
+// Norm is RMS, or (center) layer norm without bias.  table != nullptr: h[t] starts as the embedding of ids[t].
+struct JoinParams {
+  float* h;
+  const void* table; const int* ids; int vocab;
+  const void* y1; const void* g1; long long ld_y1, ld_g1;
+  const void* ys; const int* pos; const float* wts; const float* g2; long long ld_g2;
+  int topk, H, center;
+  const void* w1; const void* w2; void* x1; void* x2;
+  float eps;
+};
+
+__device__ __forceinline__ float sigmoid32(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+template <int DT, int VEC>
+__device__ __forceinline__ void ldv(const typename Act<DT>::T* p, float* v) {
+  if (VEC == 4) ld4<DT>(p, v); else v[0] = Act<DT>::ld(p[0]);
+}
+
+template <int DT, int VEC>
+__global__ void gated_join_kernel(const JoinParams p) {
+  extern __shared__ float row[];
+  __shared__ float sh[2][32];
+  pdl_launch_dependents();
+  pdl_wait();
+  typedef typename Act<DT>::T T;
+  const int t = blockIdx.x, H = p.H;
+  float* hp = p.h + (size_t)t * H;
+  const T* emb = nullptr;
+  if (p.table != nullptr) {
+    int id = p.ids[t];
+    id = id < 0 ? 0 : (id >= p.vocab ? p.vocab - 1 : id);
+    emb = reinterpret_cast<const T*>(p.table) + (size_t)id * H;
+  }
+  const T* y1 = p.y1 != nullptr ? reinterpret_cast<const T*>(p.y1) + (size_t)t * p.ld_y1 : nullptr;
+  const T* g1 = reinterpret_cast<const T*>(p.g1) + (size_t)t * p.ld_g1;
+  const T* ys = reinterpret_cast<const T*>(p.ys);
+  const float* g2 = p.g2 + (size_t)t * p.ld_g2;
+  float sum = 0.f;
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+    float v[VEC], u[VEC], z[VEC];
+    if (emb != nullptr) ldv<DT, VEC>(emb + i, v); else ldv<2, VEC>(hp + i, v);
+    if (y1 != nullptr) {
+      ldv<DT, VEC>(y1 + i, u);
+      ldv<DT, VEC>(g1 + i, z);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += sigmoid32(z[j]) * u[j];
+    }
+    if (ys != nullptr) {
+      float acc[VEC];
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) acc[j] = 0.f;
+      if (p.pos == nullptr) {
+        ldv<DT, VEC>(ys + (size_t)t * H + i, acc);
+      } else {
+#pragma unroll 4
+        for (int k = 0; k < p.topk; ++k) {
+          const int r = p.pos[(size_t)t * p.topk + k];
+          if (r < 0) continue;
+          const float wk = p.wts[(size_t)t * p.topk + k];
+          ldv<DT, VEC>(ys + (size_t)r * H + i, u);
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) acc[j] += wk * u[j];
+        }
+      }
+      ldv<2, VEC>(g2 + i, z);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += sigmoid32(z[j]) * acc[j];
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { row[i + j] = v[j]; sum += v[j]; }
+    if (VEC == 4) st4<2>(hp + i, v); else hp[i] = v[0];
+  }
+  float mean = 0.f, ss = 0.f;
+  if (p.center) mean = block_sum32(sum, sh[0]) / (float)H;
+  for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {        // the thread's own columns
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) { const float d = row[i + j] - mean; ss += d * d; }
+  }
+  ss = block_sum32(ss, sh[1]);
+  const float inv = 1.0f / sqrtf(ss / (float)H + p.eps);
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    const T* w = reinterpret_cast<const T*>(k == 0 ? p.w1 : p.w2);
+    if (w == nullptr) continue;
+    T* x = reinterpret_cast<T*>(k == 0 ? p.x1 : p.x2) + (size_t)t * H;
+    for (int i = threadIdx.x * VEC; i < H; i += blockDim.x * VEC) {
+      float wv[VEC], o[VEC];
+      ldv<DT, VEC>(w + i, wv);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = (row[i + j] - mean) * inv * wv[j];
+      if (VEC == 4) st4<DT>(x + i, o); else x[i] = Act<DT>::st(o[0]);
+    }
+  }
 }
 
 // What opens a pass of looped layers: the residual gets a step vector and, where `table` is given, the token's embedding again.
@@ -321,13 +498,18 @@ __global__ void moe_gather_scaled_kernel(const float* __restrict__ x, const int*
 // Per-head RMS norm, rotary positions and cache append of a merged projection [queries | gate | keys | values], one warp per (token,
 // head), fp32 arithmetic.  Heads are D wide, stored Dp (values Vp); queries are rewritten in place, keys and values go to their cache
 // slots (slot < 0: nowhere).  rot: leading dimensions that turn, in pairs (2j, 2j + 1) or (neox) (j, j + rot / 2); cos / sin tables
-// [tab_rows, rot / 2].  Norm weights null: no norm; with neither norm nor rotation the queries stay as they are.
+// [tab_rows, rot / 2].  Norm weights null: no norm, or (unit) one without weights; with neither norm nor rotation the queries stay as
+// they are.  A rotation keeps a head's root mean square, so the norm may stand before or after it.  rot_v: leading dimensions of a
+// value that turn, in pairs (2j, 2j + 1), by tables of their own.
 struct HeadPostParams {
   void* proj; long long ld;
   const int* positions; const int* slots;
   int T, H, G, D, Dp, Vp, k_col, v_col, rot, neox;
   const void* q_norm; const void* k_norm;
+  int unit;
   const float* cos_tab; const float* sin_tab;
+  int rot_v;
+  const float* cos_v; const float* sin_v;
   int tab_rows, num_slots;
   void* k_pool; void* v_pool;
   float eps;
@@ -339,7 +521,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   typedef typename Act<DT>::T T;
   pdl_launch_dependents();
   pdl_wait();
-  const int h0 = !PAIRS && p.q_norm == nullptr && p.rot == 0 ? p.H : 0;        // first head there is work for
+  const int h0 = !PAIRS && p.q_norm == nullptr && !p.unit && p.rot == 0 ? p.H : 0;        // first head there is work for
   const int units = p.H + 2 * p.G - h0;
   const long long u = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   if (u >= (long long)p.T * units) return;
@@ -353,6 +535,22 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
     const int g = k - p.H - p.G;
     const T* src = row + p.v_col + g * p.Vp;
     T* dst = reinterpret_cast<T*>(p.v_pool) + ((size_t)slot * p.G + g) * p.Vp;
+    if (!PAIRS && p.rot_v > 0) {
+      int pos = p.positions[t];
+      pos = pos < 0 ? 0 : (pos >= p.tab_rows ? p.tab_rows - 1 : pos);
+      const int half = p.rot_v >> 1;
+      for (int j = lane; 2 * j < p.Vp; j += 32) {
+        float a = Act<DT>::ld(src[2 * j]), b = Act<DT>::ld(src[2 * j + 1]);
+        if (j < half) {
+          const float c = p.cos_v[(size_t)pos * half + j], s = p.sin_v[(size_t)pos * half + j], u0 = a;
+          a = u0 * c - b * s;
+          b = b * c + u0 * s;
+        }
+        dst[2 * j] = Act<DT>::st(a);
+        dst[2 * j + 1] = Act<DT>::st(b);
+      }
+      return;
+    }
     for (int i = lane; i < p.Vp; i += 32) dst[i] = src[i];
     return;
   }
@@ -361,7 +559,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
   T* src = is_k ? row + p.k_col + (k - p.H) * p.Dp : row + (size_t)k * p.Dp;
   T* dst = is_k ? reinterpret_cast<T*>(p.k_pool) + ((size_t)slot * p.G + (k - p.H)) * p.Dp : src;
   const T* nw = reinterpret_cast<const T*>(is_k ? p.k_norm : p.q_norm);
-  const bool norm = PAIRS || nw != nullptr;
+  const bool norm = PAIRS || nw != nullptr || p.unit;
   float inv = 1.f;
   if (norm) {
     float ss = 0.f;
@@ -380,7 +578,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const HeadPostParam
     const int i0 = halves ? j : 2 * j, i1 = halves ? j + half : 2 * j + 1;
     float a = i0 < p.D ? Act<DT>::ld(src[i0]) * inv : 0.f;
     float b = i1 < p.D ? Act<DT>::ld(src[i1]) * inv : 0.f;
-    if (norm) {
+    if (PAIRS || nw != nullptr) {
       if (i0 < p.D) a *= Act<DT>::ld(nw[i0]);
       if (i1 < p.D) b *= Act<DT>::ld(nw[i1]);
     }
@@ -445,13 +643,55 @@ extern "C" int fb_embed_pos_norm(const int* ids, const int* positions, const voi
   return (int)cudaGetLastError();
 }
 
-extern "C" int fb_latent_norm(const void* x, int ldx, const void* w, const int* slots, void* pool, int T, int n, int ld, long long spare,
-                              float eps, int dt, void* stream) {
+// See LatentPostParams.
+extern "C" int fb_latent_post(const void* x, long long ldx, int q_col, int q_rank, int q_pad, int kv_col, int rank, int lv, int rot_col, int rot, int ld, int neox,
+                              int gate_col, int n_gates, const void* q_norm, const void* kv_norm, const float* cos_tab, const float* sin_tab, int tab_rows,
+                              const int* positions, const int* slots, void* cq, void* pool, float* gates, int T, long long spare, float eps, int dt,
+                              void* stream) {
   if (T <= 0) return 0;
-  if (n <= 0 || ld < n || n > S32_MAX_ROW || dt < 0 || dt > 2) return -1;
-  const int th = row_threads(ld, 2);
-#define GO(DT) S32_LAUNCH((latent_norm_kernel<DT>), T, th, n, stream, (const Act<DT>::T*)x, ldx, (const Act<DT>::T*)w, slots, (Act<DT>::T*)pool, n, ld, spare, eps)
+  if (rank <= 0 || lv < rank || ld < lv + rot || q_rank < 0 || q_pad < q_rank || q_rank + rank > S32_MAX_ROW || rot < 0 || (rot & 1) || ((ld - lv) & 1) || n_gates < 0 ||
+      dt < 0 || dt > 2 || (rot == 0 && ld != lv) || (rot > 0 && (cos_tab == nullptr || sin_tab == nullptr || positions == nullptr || tab_rows <= 0)) ||
+      (q_rank > 0 && (cq == nullptr || q_norm == nullptr)) || (n_gates > 0 && gates == nullptr))
+    return -1;
+  LatentPostParams p{x, ldx, q_col, q_rank, q_pad, kv_col, rank, lv, rot_col, rot, ld, neox, gate_col, n_gates, q_norm, kv_norm, cos_tab, sin_tab, tab_rows, positions, slots, cq, pool, gates, spare, eps};
+  const int th = row_threads(ld > q_pad ? ld : q_pad, 2);
+#define GO(DT) S32_LAUNCH((latent_post_kernel<DT>), T, th, q_rank + rank, stream, p)
   if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+#undef GO
+  return (int)cudaGetLastError();
+}
+
+// See RopeHeadsParams.
+extern "C" int fb_rope_heads(const void* src, void* dst, long long ld_src, long long ld_dst, int T, int H, int head_src, int head_dst, int rot, int width, int neox,
+                             const int* positions, const float* cos_tab, const float* sin_tab, int tab_rows, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || rot <= 0 || (rot & 1) || width < rot || (width & 1) || tab_rows <= 0 || cos_tab == nullptr || sin_tab == nullptr || positions == nullptr || dt < 0 || dt > 2) return -1;
+  RopeHeadsParams p{src, dst, ld_src, ld_dst, T, H, head_src, head_dst, rot, width, neox, tab_rows, positions, cos_tab, sin_tab};
+  long long blocks = ((long long)T * H * (width / 2) + 255) / 256;
+  if (blocks > 148 * 32) blocks = 148 * 32;
+  cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+  if (dt == 0) launch_k(rope_heads_kernel<0>, dim3((unsigned)blocks), dim3(256), 0, s, 0, p);
+  else if (dt == 1) launch_k(rope_heads_kernel<1>, dim3((unsigned)blocks), dim3(256), 0, s, 0, p);
+  else launch_k(rope_heads_kernel<2>, dim3((unsigned)blocks), dim3(256), 0, s, 0, p);
+  return (int)cudaGetLastError();
+}
+
+// See JoinParams; x1 / x2 [T, H] and ys rows are contiguous.
+extern "C" int fb_gated_join(float* h, const void* table, const int* ids, int vocab, const void* y1, long long ld_y1, const void* g1, long long ld_g1, const void* ys,
+                             const int* pos, const float* wts, const float* g2, long long ld_g2, int T, int topk, int H, int center, const void* w1,
+                             const void* w2, void* x1, void* x2, float eps, int dt, void* stream) {
+  if (T <= 0) return 0;
+  if (H <= 0 || H > S32_MAX_ROW || dt < 0 || dt > 2 || w1 == nullptr || x1 == nullptr || (w2 != nullptr && x2 == nullptr) || (y1 != nullptr && g1 == nullptr) ||
+      (ys != nullptr && g2 == nullptr) || (pos != nullptr && (wts == nullptr || topk <= 0)) || (table != nullptr && (ids == nullptr || vocab <= 0)))
+    return -1;
+  JoinParams p{h, table, ids, vocab, y1, g1, ld_y1, ld_g1, ys, pos, wts, g2, ld_g2, topk, H, center, w1, w2, x1, x2, eps};
+  const uintptr_t align = dt == 2 ? 15 : 7;
+  const bool vec = H % 4 == 0 && ld_y1 % 4 == 0 && ld_g1 % 4 == 0 && ld_g2 % 4 == 0 && !(reinterpret_cast<uintptr_t>(g2) & 15) &&
+                   !((reinterpret_cast<uintptr_t>(y1) | reinterpret_cast<uintptr_t>(g1) | reinterpret_cast<uintptr_t>(ys)) & align);
+  const int th = row_threads(H, vec ? 4 : 1);
+#define GO(DT, V) S32_LAUNCH((gated_join_kernel<DT, V>), T, th, H, stream, p)
+  if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
+  else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
   return (int)cudaGetLastError();
 }
@@ -497,18 +737,20 @@ extern "C" int fb_moe_gather_scaled(const float* x, const int* pos, const float*
 
 // See HeadPostParams.  G = 0: queries only (the layer reads another layer's cache).
 extern "C" int fb_head_norm_rope(void* proj, long long ld, const int* positions, const int* slots, int T, int H, int G, int D, int Dp, int Vp,
-                                 int k_col, int v_col, int rot, int neox, const void* q_norm, const void* k_norm, const float* cos_tab,
-                                 const float* sin_tab, int tab_rows, int num_slots, void* k_pool, void* v_pool, float eps, int dt, void* stream_) {
+                                 int k_col, int v_col, int rot, int neox, const void* q_norm, const void* k_norm, int unit, const float* cos_tab,
+                                 const float* sin_tab, int rot_v, const float* cos_v, const float* sin_v, int tab_rows, int num_slots, void* k_pool, void* v_pool, float eps, int dt, void* stream_) {
   if (T <= 0) return 0;
   if (H <= 0 || G < 0 || D <= 0 || Dp < D || (Dp & 1) || Vp <= 0 || rot < 0 || (rot & 1) || rot > D || dt < 0 || dt > 2) return -1;
   if (rot > 0 && (cos_tab == nullptr || sin_tab == nullptr || tab_rows <= 0)) return -1;
+  if (rot_v < 0 || (rot_v & 1) || rot_v > Vp || (rot_v > 0 && (cos_v == nullptr || sin_v == nullptr || tab_rows <= 0 || (Vp & 1)))) return -1;
+  if (unit && q_norm != nullptr) return -1;
   if (G > 0 && ((k_norm == nullptr) != (q_norm == nullptr) || k_pool == nullptr || v_pool == nullptr)) return -1;
-  HeadPostParams p{proj, ld, positions, slots, T, H, G, D, Dp, Vp, k_col, v_col, rot, neox, q_norm, k_norm, cos_tab, sin_tab, tab_rows, num_slots, k_pool, v_pool, eps};
-  const long long units = (long long)T * ((q_norm == nullptr && rot == 0 ? 0 : H) + 2 * G);
+  HeadPostParams p{proj, ld, positions, slots, T, H, G, D, Dp, Vp, k_col, v_col, rot, neox, q_norm, k_norm, unit, cos_tab, sin_tab, rot_v, cos_v, sin_v, tab_rows, num_slots, k_pool, v_pool, eps};
+  const long long units = (long long)T * ((q_norm == nullptr && !unit && rot == 0 ? 0 : H) + 2 * G);
   if (units == 0) return 0;
   const dim3 grid((unsigned)((units + 7) / 8));
   cudaStream_t stream = reinterpret_cast<cudaStream_t>(stream_);
-  const bool pairs = q_norm != nullptr && !neox;
+  const bool pairs = q_norm != nullptr && !neox && rot_v == 0;
 #define GO(DT) { if (pairs) launch_k(head_norm_rope_kernel<DT, true>, grid, dim3(256), 0, stream, 0, p); else launch_k(head_norm_rope_kernel<DT, false>, grid, dim3(256), 0, stream, 0, p); }
   if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
 #undef GO

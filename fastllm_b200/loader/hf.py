@@ -80,7 +80,14 @@ def dequant_awq(qweight: torch.Tensor, qzeros: torch.Tensor, scales: torch.Tenso
 # name canonicalisation: every family is mapped onto the Llama naming that loader.shard understands
 # ---------------------------------------------------------------------------------------------------
 _RENAMES = [
-    # Patesun, Vilulorn, Vuripel
+    # Patesun, Vilulorn, Vuripel, Nasipel
+    (r"^l(\d+)\.mix\.dq\.norm$", r"model.layers.\1.self_attn.q_a_layernorm.weight"), (r"^l(\d+)\.mix\.dq$", r"model.layers.\1.self_attn.q_a_proj.weight"),
+    (r"^l(\d+)\.mix\.uq$", r"model.layers.\1.self_attn.q_b_proj.weight"), (r"^l(\d+)\.mix\.pb$", r"model.layers.\1.self_attn.score_bias"),
+    (r"^l(\d+)\.mix\.([xy])\.b$", r"model.layers.\1.self_attn.\2_proj.bias"), (r"^l(\d+)\.mix\.([xy])$", r"model.layers.\1.self_attn.\2_proj.weight"),
+    (r"^l(\d+)\.mix\.conv\.b$", r"model.layers.\1.self_attn.conv1d.bias"), (r"^l(\d+)\.mix\.conv$", r"model.layers.\1.self_attn.conv1d.weight"),
+    (r"^l(\d+)\.mix\.r([ai])\.b$", r"model.layers.\1.self_attn.r\2_gate.bias"), (r"^l(\d+)\.mix\.r([ai])$", r"model.layers.\1.self_attn.r\2_gate.weight"),
+    (r"^l(\d+)\.mix\.lam$", r"model.layers.\1.self_attn.lam"), (r"^l(\d+)\.rg([12])\.b$", r"model.layers.\1.residual_gate\2.bias"),
+    (r"^l(\d+)\.rg([12])$", r"model.layers.\1.residual_gate\2.weight"), (r"^l(\d+)\.mlp\.correction$", r"model.layers.\1.mlp.gate.e_score_correction_bias"),
     (r"^l(\d+)\.mix\.([qkvif])\.b$", r"model.layers.\1.self_attn.\2_proj.bias"), (r"^l(\d+)\.mix\.([if])$", r"model.layers.\1.self_attn.\2_proj.weight"),
     (r"^l(\d+)\.mix\.sink$", r"model.layers.\1.self_attn.sinks"), (r"^l(\d+)\.mlp\.gate$", r"model.layers.\1.mlp.gate_proj.weight"),
     (r"^l(\d+)\.mlp\.shared\.sg$", r"model.layers.\1.mlp.shared_expert_gate.weight"), (r"^loop\.step$", "model.loop_step.weight"),

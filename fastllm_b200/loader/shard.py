@@ -310,11 +310,12 @@ def build_layer(m, i: int, t: dict, wdtype="dense", moe_wdtype=None):
 def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
     """Mixer and feed-forward of a model that lists its layers (``cfg.mixers`` / ``cfg.ffs``).  Widths are padded with zero rows and
     columns to what the kernels tile (the padding stays zero through every product)."""
-    from ..models.config import AttnSpec, GLASpec, MLSTMSpec
+    from ..models.config import AttnSpec, GLASpec, MLSTMSpec, RGLRUSpec
     from ..ops import gla as GLA
     from ..ops import grouped as GR
     from ..ops import latent as LA
     from ..ops import mlstm as ML
+    from ..ops import rglru as RG
 
     cfg = m.cfg
     spec, ff = cfg.mixers[i], cfg.ffs[i]
@@ -334,14 +335,28 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
     def down(w, kind, mult):
         return lin(LA.pad_cols(_to(w, m), mult if m.on_cuda else 1).contiguous(), kind)
 
+    def tail_bias(w, col, rows):            # bias of a merged projection whose last part alone has one
+        out = torch.zeros((w.shape[0],), dtype=m.dtype, device=m.device)
+        out[col:col + rows.shape[0]] = rows
+        return out
+
     f = lw.mlp
     gates, joint = [], []                   # parallel layers: rows of fp32 logits; matrices that project back to the residual
+    more, more_b = (), ()                   # what reads the mixer's input beside it
+    if cfg.gated_residual:
+        more, more_b = (_to(g("residual_gate1.weight"), m),), (_to(g("residual_gate1.bias"), m),)
     if cfg.output_norms:                    # the layer's two norms belong to its sub-layers' outputs
         lw.attn.post_ln, f.post_ln, lw.attn.ln, f.ln = lw.attn.ln, f.ln, None, None
     if isinstance(spec, GLASpec):
         lw.gla, in_w = GLA.build(spec, *(t(k + "_proj") for k in ("q", "k", "v", "g", "a1", "a2")), _to(g("self_attn.a2_proj.bias"), m), t("o_norm"))
         lw.gla.in_proj = lin(in_w)
         lw.attn.o = lin(t("o_proj"))
+    elif isinstance(spec, RGLRUSpec):
+        a = lambda k: _to(g("self_attn." + k), m)
+        lw.rglru, in_w = RG.build(spec, t("y_proj"), t("x_proj"), t("conv1d"), a("conv1d.bias"), t("ra_gate"), a("ra_gate.bias"), t("ri_gate"), a("ri_gate.bias"),
+                                  a("lam"), more)
+        lw.rglru.in_proj = lin(in_w, bias=RG.in_bias(lw.rglru, a("y_proj.bias"), a("x_proj.bias"), more_b, in_w.shape[0]))
+        lw.attn.o, lw.more_col = lin(RG.out_proj(t("o_proj"), spec)), lw.rglru.more_col
     elif isinstance(spec, MLSTMSpec):
         b = lambda k: _to(g("self_attn." + k + "_proj.bias"), m)
         lw.mlstm, in_w = ML.build(spec, *(t(k + "_proj") for k in ("q", "k", "v", "g")), b("i"), b("f"), t("o_norm"))
@@ -353,22 +368,39 @@ def _build_listed_layer(m, i: int, lw, g, wdtype, moe_wdtype):
         kv = lambda k: t(k) if own else None
         biases = [_to(g(f"self_attn.{k}_proj.bias"), m) if own or k == "q" else None for k in "qkv"] if spec.bias else None
         lw.grouped, in_w = GR.build(spec, t("q_proj"), kv("k_proj"), kv("v_proj"), t("g_proj") if spec.gate == "elem" else None,
-                                    t("q_norm") if spec.qk_norm else None, kv("k_norm") if spec.qk_norm else None, biases,
-                                    _to(g("self_attn.sinks"), m) if spec.sinks else None)
-        lw.grouped.in_proj = lin(in_w, bias=lw.grouped.in_bias)
-        lw.attn.heads, lw.attn.rope = spec.heads, spec.rope
+                                    t("q_norm") if spec.qk_norm and spec.norm_weight else None, kv("k_norm") if spec.qk_norm and spec.norm_weight else None, biases,
+                                    _to(g("self_attn.sinks"), m) if spec.sinks else None, g("self_attn.score_bias").to(m.device) if spec.weights == "sigmoid" else None, more)
+        in_b = lw.grouped.in_bias if not more else tail_bias(in_w, lw.grouped.more_col, *more_b)
+        lw.grouped.in_proj = lin(in_w, bias=in_b)
+        lw.attn.heads, lw.attn.rope, lw.attn.rope_values, lw.more_col = spec.heads, spec.rope, spec.rope_values, lw.grouped.more_col
         if spec.gate == "head":
             gates.append(t("g_proj"))
-        if cfg.parallel_block:
-            joint.append(LA.pad_out_proj(t("o_proj"), spec))
+        if cfg.parallel_block and not cfg.gated_residual:
+            joint.append(GR.out_proj(t("o_proj"), spec))
         else:
-            lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
+            lw.attn.o = lin(GR.out_proj(t("o_proj"), spec))
     else:
-        la, in_w = LA.build(spec, t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"))
-        la.in_proj = lin(in_w)
+        low = bool(spec.q_rank)
+        la, in_w, up_w = LA.build(spec, t("q_a_proj") if low else t("q_proj"), t("g_proj"), t("kv_a_proj"), t("kv_a_layernorm"), t("k_b_proj"), t("v_b_proj"),
+                                  t("q_b_proj") if low else None, t("q_a_layernorm") if low else None, more)
+        la.in_proj = lin(in_w, bias=tail_bias(in_w, la.more_col, *more_b) if more else None)
+        la.q_up = lin(up_w) if low else None
         lw.latent = la
+        lw.attn.rope, lw.more_col = spec.rope, la.more_col
         lw.attn.o = lin(LA.pad_out_proj(t("o_proj"), spec))
-    if cfg.parallel_block:
+    if cfg.gated_residual:
+        if ff.kind == "none":
+            f.absent = True
+            return
+        names = [f"mlp.experts.{e}." for e in range(ff.experts)]
+        f.experts = MOE.ExpertWeights(ff.experts, 0, [gate_up(g(n + "gate_proj.weight"), g(n + "up_proj.weight"), moe_wdtype) for n in names],
+                                      [down(g(n + "down_proj.weight"), moe_wdtype, 64) for n in names])
+        f.top, f.groups, f.keep_groups, f.route_scale = ff.top, ff.groups, ff.keep_groups, ff.route_scale
+        f.router_bias = g("mlp.gate.e_score_correction_bias").to(m.device, torch.float32).contiguous()
+        f.router_col = cfg.hidden_size
+        z_w = LA.pad_rows(torch.cat([_to(g("residual_gate2.weight"), m), _to(g("mlp.gate.weight"), m)], dim=0), 32)
+        lw.logits = lin(z_w, "dense", bias=tail_bias(z_w, 0, _to(g("residual_gate2.bias"), m)))
+    elif cfg.parallel_block:
         _build_parallel_ff(m, lw, ff, g, lin, gate_up, wdtype, moe_wdtype, gates, joint)
         if cfg.side_dim:
             _build_side(m, i, lw, g, lin)

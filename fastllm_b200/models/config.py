@@ -7,20 +7,25 @@ decoder needs is resolved once into a dataclass, per model family.
 from __future__ import annotations
 
 import json
+import math
 from dataclasses import dataclass, field
 from pathlib import Path
 
 
 @dataclass
 class LatentSpec:
-    """Latent attention of one layer: per-head keys and values are projections of one cached, RMS-normalised latent row; no
-    positions enter the scores."""
+    """Latent attention of one layer: per-head keys and values are projections of one cached, RMS-normalised latent row; beside them
+    a rotated key part that all heads share, where the layer has positions."""
     heads: int
-    dim: int                # query / key dimensions per head
+    dim: int                # query / key dimensions per head (without the rotated ones)
     vdim: int
     kv_rank: int
     scale: float
     window: int = 0         # keys a query sees, itself included (0: all before it)
+    q_rank: int = 0         # > 0: queries are a projection of an RMS-normalised latent of this width
+    rot_dim: int = 0        # rotated dimensions of every query head and of the shared key part
+    rope: dict | None = None     # their table: {"theta", "rot_dim", "scaling", "mode"}
+    gate: str = "elem"      # sigmoid gate on the output: "elem" one per element, "head" one per head
 
 
 @dataclass
@@ -39,6 +44,9 @@ class AttnSpec:
     softcap: float = 0.0    # > 0: scores become softcap * tanh(score / softcap)
     sinks: bool = False     # a learned logit per head in the softmax denominator
     qk_norm: bool = True    # RMS norm of every query and key head
+    norm_weight: bool = True     # ... with a weight
+    weights: str = "softmax"     # "sigmoid": a key's weight is sigmoid(score + a number per head), not normalised over keys
+    rope_values: dict | None = None     # values are cached rotated over all vdim dimensions (table as in rope), outputs are turned back
     gate: str = "elem"      # sigmoid gate on the output: "elem" one per element, "head" one per head, "" none
     bias: bool = False      # biases of the query, key and value projections
 
@@ -63,7 +71,16 @@ class MLSTMSpec:
     gate_cap: float
 
 
-RECURRENT = (GLASpec, MLSTMSpec)     # mixers that keep a state per request instead of pages
+@dataclass
+class RGLRUSpec:
+    """Real-gated linear recurrent unit of one layer: one state per channel behind a short causal convolution; both gates are
+    block-diagonal products of its output; the other branch gates the states with a GELU."""
+    width: int
+    blocks: int             # equal parts of the channels, each with its own square gate matrices
+    conv: int               # taps of the convolution
+
+
+RECURRENT = (GLASpec, MLSTMSpec, RGLRUSpec)     # mixers that keep a state per request instead of pages
 
 
 @dataclass
@@ -79,8 +96,12 @@ class FFSpec:
     shared_ff: int = 0      # 0: no shared expert
     router: str = "table"   # "table": experts by token id | "sigmoid": the best scores of a projection, which scale the expert's input
                             # | "softmax": the best softmax scores, which scale the expert's output
+                            # | "corrected": sigmoid scores, chosen by score + a learned correction; the chosen ones' scores, divided by
+                            #   their sum, times route_scale, scale the expert's output
     limit: float = 0.0
-    groups: int = 1         # the experts form equal groups of neighbours; only those of the `keep_groups` groups with the largest score count
+    route_scale: float = 1.0
+    groups: int = 1         # the experts form equal groups of neighbours; only those of the `keep_groups` best groups count (a group's score:
+                            # its largest score, or with "corrected" the sum of its two largest)
     keep_groups: int = 1
     shared_gate: bool = False    # the shared expert's output is multiplied by a sigmoid, one logit per token
 
@@ -123,7 +144,7 @@ class ModelConfig:
     qk_norm_after_rope: bool = False       # Hunyuan: per-head norm applied after the rotary embedding
     attn_sinks: bool = False               # learned per-head sink logit in the softmax denominator (gpt-oss)
     moe_act: str = "swiglu"                # swiglu | gptoss (clamped, alpha 1.702, (up + 1))
-    norm_kind: str = "rms"                 # rms | layernorm (mean-centred, weight + bias: CodeGen / MOSS, GPT-J)
+    norm_kind: str = "rms"                 # rms | layernorm (mean-centred, weight + bias: CodeGen / MOSS, GPT-J; without bias: Nasipel)
     parallel_block: bool = False           # attention and MLP both read the one pre-norm of the layer; one residual add
     mlp_gated: bool = True                 # False: up projection -> activation -> down projection
     # per-layer attention geometry (Step-3.5 / Laguna: full-attention and sliding-window layers differ)
@@ -168,9 +189,9 @@ class ModelConfig:
     lin_conv_kernel: int = 4
     lin_kind: str = "gdn"                  # "gdn" Gated DeltaNet | "lightning" decayed linear attention (MiniMax-Text-01 / M1)
     lin_block: int = 256                   # lightning attention: block length of the chunked evaluation
-    # models whose layers are listed one by one (Patesun, Vilulorn, Vuripel): the mixer and feed-forward of every layer, and which layer's
+    # models whose layers are listed one by one (Patesun, Vilulorn, Vuripel, Nasipel): the mixer and feed-forward of every layer, and which layer's
     # weights each run of the stack uses (looped layers appear once per pass; num_layers counts the runs, every run has its own cache)
-    mixers: list | None = None             # LatentSpec / AttnSpec / GLASpec / MLSTMSpec per run
+    mixers: list | None = None             # LatentSpec / AttnSpec / GLASpec / MLSTMSpec / RGLRUSpec per run
     ffs: list | None = None                # FFSpec per run
     layer_runs: list | None = None
     residual_f32: bool = False             # the residual stream is fp32; sub-layer outputs join it times residual_mult
@@ -180,6 +201,8 @@ class ModelConfig:
     output_norms: bool = False             # fp32 residual: what a sub-layer adds is normalised, what it reads is not
     pass_starts: list | None = None        # per run: the pass number where it opens a pass of a loop that adds a step vector (and, from
                                            # the second pass on, the token embedding) to the residual; else None
+    gated_residual: bool = False           # parallel block, fp32 residual: mixer and feed-forward read a norm of their own each; every result is
+                                           # multiplied by the sigmoid of a full-width projection of what the sub-layer reads
     side_dim: int = 0                      # > 0: width of the per-layer token input (a second embedding, gated by the residual)
     # DeepNorm-style residual (MiniMax-Text-01 / M1): the block input is normalised first and the NORMALISED rows are the
     # residual: y = alpha * norm(x) + beta * f(norm(x)).  (alpha, beta) for full-attention layers, linear layers, MLPs.
@@ -657,8 +680,8 @@ def _listed(name: str, d: dict, mixers: list, ffs: list, runs: list) -> ModelCon
     c.layer_runs = runs
     c.num_layers = len(runs)
     c.mixers, c.ffs = [mixers[i] for i in runs], [ffs[i] for i in runs]
-    c.num_heads = c.num_kv_heads = max((m.heads for m in mixers), default=1)
-    c.head_dim = max((m.dim for m in mixers), default=1)
+    c.num_heads = c.num_kv_heads = max((getattr(m, "heads", 1) for m in mixers), default=1)
+    c.head_dim = max((getattr(m, "dim", 1) for m in mixers), default=1)
     c.intermediate_size = max((f.ff for f in ffs), default=0)
     c.num_experts = max((f.experts for f in ffs), default=0)
     c.num_experts_per_tok = max((f.top for f in ffs), default=0)
@@ -754,8 +777,53 @@ def _vuripel(d: dict) -> ModelConfig:
     return c
 
 
+def _nasipel(d: dict) -> ModelConfig:
+    """Nasipel: latent attention with a query latent, rotated parts and a gate per head; attention whose keys are weighed by sigmoids and
+    whose values are rotated; real-gated linear recurrent units; mixer and grouped sigmoid-routed experts side by side, each behind a
+    layer norm and a gate of its own."""
+    mixers, ffs = [], []
+    for i, spec in enumerate(d["layers"]):
+        m, kind = spec["mixer"], spec.get("type")
+        rot = m.get("rot") or {}
+        rope = None
+        if rot.get("dims"):
+            sc = rot.get("scaling")
+            rope = {"theta": float(rot["base"]), "rot_dim": int(rot["dims"]), "scaling": {
+                "rope_type": "yarn", "factor": float(sc["factor"]), "original_max_position_embeddings": float(sc["original"]),
+                "beta_fast": float(sc["fast"]), "beta_slow": float(sc["slow"]), "attention_factor": 0.1 * math.log(float(sc["factor"])) + 1.0} if sc else None}
+        if kind == "attention":
+            mixers.append(AttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]),
+                                   rope=dict(rope, mode="neox") if rope else None, softcap=float(m.get("softcap") or 0.0), gate="", norm_weight=False,
+                                   weights="sigmoid", rope_values={"theta": float(rot["base"]), "rot_dim": int(m["vdim"]), "scaling": None, "mode": "neox"}))
+        elif kind == "latent_attention":
+            if rope and rope["rot_dim"] != int(m["rot_dim"]):
+                raise ValueError(f"Nasipel: layer {i} rotates {rope['rot_dim']} of {m['rot_dim']} dimensions")
+            mixers.append(LatentSpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), int(m["kv_rank"]), float(m["scale"]), q_rank=int(m["q_rank"]),
+                                     rot_dim=int(m["rot_dim"]), rope=dict(rope, mode="interleaved") if rope else None, gate="head"))
+        elif kind == "rglru":
+            mixers.append(RGLRUSpec(int(m["width"]), int(m["blocks"]), int(m["conv"])))
+        else:
+            raise NotImplementedError(f"Nasipel: layer {i} has mixer '{kind}'")
+        f = spec.get("mlp")
+        if f is None:
+            ffs.append(FFSpec())
+        elif f.get("kind") == "moe":
+            r = f["router"]
+            gr = r.get("groups") or {}
+            ffs.append(FFSpec("moe", act="silu", experts=int(r["experts"]), top=int(r["top"]), expert_ff=int(f["expert"]["ff"]), router="corrected",
+                              route_scale=float(r.get("scale", 1.0)), groups=int(gr.get("count") or 1), keep_groups=int(gr.get("keep") or gr.get("count") or 1)))
+        else:
+            raise NotImplementedError(f"Nasipel: layer {i} has feed-forward '{f.get('kind')}'")
+    c = _listed("Nasipel", d, mixers, ffs, list(range(len(mixers))))
+    c.num_kv_heads = max((m.kv_heads for m in mixers if isinstance(m, AttnSpec)), default=1)
+    c.norm_kind = "layernorm"
+    c.parallel_block = c.gated_residual = True
+    c.max_position = int(d.get("max_position_embeddings", 1 << 20))
+    return c
+
+
 # config.json "architecture" of designs whose layers are listed one by one
-LISTED = {"Patesun": _patesun, "Vilulorn": _vilulorn, "Vuripel": _vuripel}
+LISTED = {"Patesun": _patesun, "Vilulorn": _vilulorn, "Vuripel": _vuripel, "Nasipel": _nasipel}
 
 
 def load_config(path: str | Path) -> ModelConfig:
@@ -931,6 +999,20 @@ def preset(name: str) -> ModelConfig:
             block += [layer("attention_2", local, moe), layer("mlstm", cell, moe), layer("attention_2", local, moe), layer("attention", full, dense)]
         return from_hf_dict(dict(architecture="Vuripel", vocab=512 if tiny else 128256, width=144 if tiny else 4096, norm={"eps": 1e-5}, layers=block,
                                  loop={"start": 1, "stop": 3 if tiny else 5, "times": 2 if tiny else 3}, token_side={"dim": 24 if tiny else 256}))
+    if name in ("tiny-nasipel", "nasipel-8b"):
+        tiny = name.startswith("tiny")
+        sc = {"factor": 4.0, "fast": 32.0, "slow": 1.0, "original": 64 if tiny else 8192}
+        la = ({"heads": 3, "dim": 40, "vdim": 24, "q_rank": 56, "kv_rank": 72, "rot_dim": 16, "scale": 0.13, "rot": {"base": 3e4, "dims": 16, "scaling": sc}} if tiny else
+              {"heads": 32, "dim": 128, "vdim": 128, "q_rank": 1536, "kv_rank": 512, "rot_dim": 64, "scale": 192 ** -0.5, "rot": {"base": 5e5, "dims": 64, "scaling": sc}})
+        at = ({"heads": 6, "kv_heads": 2, "dim": 40, "vdim": 24, "scale": 0.16, "softcap": 30.0, "rot": {"base": 2e4, "dims": 24}} if tiny else
+              {"heads": 32, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0, "rot": {"base": 5e5, "dims": 128}})
+        rg = {"width": 120, "blocks": 3, "conv": 4} if tiny else {"width": 4096, "blocks": 16, "conv": 4}
+        moe = {"kind": "moe", "expert": {"ff": 56 if tiny else 1024}, "router": {"experts": 12 if tiny else 64, "top": 3 if tiny else 6, "scale": 1.5,
+                                                                               "groups": {"count": 3 if tiny else 8, "keep": 2 if tiny else 4}}}
+        layer = lambda t, m, f=moe: {"type": t, "mixer": m, "mlp": f}
+        block = [layer("rglru", rg), layer("latent_attention", la), layer("rglru", rg, None if tiny else moe), layer("attention", at)]
+        return from_hf_dict(dict(architecture="Nasipel", vocab=512 if tiny else 128256, width=144 if tiny else 4096, norm={"eps": 1e-5},
+                                 layers=block if tiny else block * 2))
     if name == "tiny-deepseek-v32":      # latent attention with the sparse-attention indexer (selection size 32)
         return from_hf_dict(dict(model_type="deepseek_v32", vocab_size=512, hidden_size=256, num_hidden_layers=2,
                                  num_attention_heads=4, num_key_value_heads=4, intermediate_size=512,

@@ -27,9 +27,10 @@ from ..ops import grouped as GR
 from ..ops import latent as LA
 from ..ops import mlstm as ML
 from ..ops import moe as MOE
+from ..ops import rglru as RG
 from ..ops import stream32 as S
 from ..ops.quant import LinearWeight
-from .config import AttnSpec, GLASpec, MLSTMSpec, ModelConfig
+from .config import AttnSpec, GLASpec, LatentSpec, MLSTMSpec, ModelConfig, RGLRUSpec
 
 
 @dataclass
@@ -83,6 +84,7 @@ class AttentionWeights:
         self.window = 0          # sliding-window length of this layer (0: full causal attention)
         self.heads = None        # this rank's query heads in this layer when layers differ (Step-3.5 / Laguna)
         self.rope = None         # {"theta", "rot_dim", "scaling"} when the layer has its own rotary tables
+        self.rope_values = None  # the same for its values
         self.head_gate: LinearWeight | None = None  # [heads, H] projection: one gate per query head on the attention output
         # MLA
         self.q_a: LinearWeight | None = None
@@ -150,6 +152,7 @@ class MLPWeights:
         self.router_col = 0
         self.shared_gate_col: int | None = None
         self.groups = self.keep_groups = 1
+        self.route_scale = 1.0
 
 
 class SideInput:
@@ -167,14 +170,17 @@ class LayerWeights:
         self.attn = AttentionWeights()
         self.mlp = MLPWeights()
         # mixers of listed layers (``attn`` keeps their norms and output projection)
-        self.latent: LA.LatentWeights | None = None    # latent attention without positions
+        self.latent: LA.LatentWeights | None = None    # latent attention
         self.grouped: GR.GroupedWeights | None = None  # grouped-query attention with its own widths, mask and rotary tables
         self.gla: GLA.GLAWeights | None = None         # gated linear attention
         self.mlstm: ML.MLSTMWeights | None = None      # matrix-memory LSTM
+        self.rglru: RG.RGLRUWeights | None = None      # real-gated linear recurrent unit
+        self.more_col = 0                              # gated residuals: column of the mixer's projection where its gate's logits start
         # listed layers whose mixer and feed-forward read one norm
         self.joint: LinearWeight | None = None         # [H, mixer output | feed-forward activations] onto the residual
         self.mix_cols = 0                              # columns of the mixer output
-        self.logits: LinearWeight | None = None        # rows [mixer gates | router | shared expert's gate], fp32 results
+        self.logits: LinearWeight | None = None        # rows [mixer gates | router | shared expert's gate], fp32 results; gated residuals:
+                                                       # [the feed-forward's gate | router]
         self.n_gates = 0
         self.side: SideInput | None = None
         self.lin: LinearAttnWeights | None = None      # set instead of ``attn`` projections on linear-attention layers
@@ -272,14 +278,16 @@ class DecoderModel:
                 return Hq, ov[0], ov[1], self.rot_dim
             cos, sin = self.rope_tables(device=device, local=local)
             return Hq, cos, sin, self.rot_dim
-        spec = lw.rope
+        return Hq, *self._listed_rope(lw.rope, device), int(lw.rope["rot_dim"])
+
+    def _listed_rope(self, spec, device):
+        """(cos, sin) tables of a layer's own rotation."""
         mp = max(min(self.cfg.max_position, 1 << 17), self.max_context)
-        key = (float(spec["theta"]), int(spec["rot_dim"]), id(spec.get("scaling")), str(torch.device(device)), mp)
+        key = (float(spec["theta"]), int(spec["rot_dim"]), str(spec.get("scaling")), str(torch.device(device)), mp)
         cache = self.__dict__.setdefault("_rope_layers", {})
         if key not in cache:
             cache[key] = A.build_rope_tables(int(spec["rot_dim"]), mp, float(spec["theta"]), spec.get("scaling"), device)
-        cos, sin = cache[key]
-        return Hq, cos, sin, int(spec["rot_dim"])
+        return cache[key]
 
     def _head_gate(self, lw, x, a, Hq, D):
         """Multiply every head of the attention output by its learned gate: sigmoid (Step-3.5) or softplus (Laguna)."""
@@ -311,7 +319,7 @@ class DecoderModel:
                 return None
             lead = (num_pages, A.PAGE_LEN, sp.kv_heads)
             return (*lead, (sp.dim + 7) // 8 * 8), (*lead, (sp.vdim + 7) // 8 * 8)
-        return (num_pages + 1, A.PAGE_LEN, 1, (sp.kv_rank + 7) // 8 * 8), None
+        return (num_pages + 1, A.PAGE_LEN, 1, sum(LA.stored_widths(sp))), None
 
     def kv_donor(self, i: int) -> int:
         """The layer whose pools layer ``i`` reads."""
@@ -333,6 +341,8 @@ class DecoderModel:
         c = self.cfg
         if c.mixers is not None:               # every listed layer has its own state
             sp = c.mixers[layer]
+            if isinstance(sp, RGLRUSpec):
+                return (n_slots, RG.stored_width(sp), sp.conv - 1), (n_slots, RG.stored_width(sp))
             if isinstance(sp, MLSTMSpec):
                 return (n_slots, 0, 0), (n_slots, sp.heads, ML.state_len(sp.dim, sp.vdim))
             return (n_slots, 0, 0), (n_slots, sp.heads, sp.dim, sp.vdim)
@@ -670,21 +680,62 @@ class DecoderModel:
     def _latent_attention(self, lw: LayerWeights, x, fb: ForwardBatch, kv, residual, next_ln):
         """Latent attention: merged [queries | gate | latent] projection, the normalised latent row into its cache slot, windowed
         attention with the output gate in its epilogue, output projection onto the residual."""
+        return self._row_parallel_norm(lw.attn.o, self._latent_heads(lw, lw.latent.in_proj(x), fb, kv), residual, next_ln)
+
+    def _latent_heads(self, lw: LayerWeights, proj, fb: ForwardBatch, kv):
         la = lw.latent
-        proj = la.in_proj(x)
-        S.latent_norm(proj[:, la.latent_col:], la.kv_norm, fb.slots, kv[0], la.rank, self.cfg.rms_eps)
-        a = LA.attention(la, proj, kv[0], fb)
-        return self._row_parallel_norm(lw.attn.o, a, residual, next_ln)
+        rope = self._listed_rope(lw.attn.rope, proj.device) if la.rot else None
+        q, gates = LA.post(la, proj, fb, kv[0], rope, self.cfg.rms_eps)
+        return LA.attention(la, proj, kv[0], fb, q, gates, rope)
 
     def _grouped_attention(self, lw: LayerWeights, x, fb: ForwardBatch, kv, residual, next_ln):
         """Grouped-query attention of a listed layer: merged [queries | gate | keys | values] projection, per-head norms + rotary + cache
         append in one launch, chunked attention with the output gate in its epilogue, output projection onto the residual."""
-        gw = lw.grouped
-        proj = gw.in_proj(x)
-        _, cos, sin, _ = self._layer_geom(lw.attn, x.device) if lw.attn.rope is not None else (0, None, None, 0)
-        GR.post(gw, proj, fb, kv, cos, sin, self.cfg.rms_eps)
-        a = GR.attention(gw, proj, kv, fb)
+        a = self._grouped_heads(lw, lw.grouped.in_proj(x), fb, kv)
         return self._row_parallel_norm(lw.attn.o, a, residual, next_ln, lw.attn.post_ln)
+
+    def _grouped_heads(self, lw: LayerWeights, proj, fb: ForwardBatch, kv, out=None, head_gate=None):
+        gw = lw.grouped
+        cos, sin = self._listed_rope(lw.attn.rope, proj.device) if lw.attn.rope is not None else (None, None)
+        if gw.rot_v:
+            gw.turn = self._listed_rope(lw.attn.rope_values, proj.device)
+        GR.post(gw, proj, fb, kv, cos, sin, self.cfg.rms_eps)
+        return GR.attention(gw, proj, kv, fb, out=out, head_gate=head_gate)
+
+    def _gated_layer(self, lw: LayerWeights, x, fb: ForwardBatch, kv, h, i: int):
+        """A listed layer whose mixer and experts each read a norm of their own and join the residual through a gate of their own.  ``x``: the
+        rows of both norms.  What the gates need comes out of the products that are there anyway: the mixer's as columns of its input
+        projection, the experts' beside the router's logits.  Combine, gates, residual and both norms of the next layer are one
+        launch.  Returns the rows of the next layer's norms."""
+        c, f, H = self.cfg, lw.mlp, self.cfg.hidden_size
+        x1, x2 = x
+        if lw.rglru is not None:
+            proj = lw.rglru.in_proj(x1)
+            a = RG.mix(lw.rglru, proj, fb, kv)
+        elif lw.latent is not None:
+            proj = lw.latent.in_proj(x1)
+            a = self._latent_heads(lw, proj, fb, kv)
+        else:
+            proj = lw.grouped.in_proj(x1)
+            a = self._grouped_heads(lw, proj, fb, kv)
+        mixer = (lw.attn.o(a), proj[:, lw.more_col:lw.more_col + H])
+        ff = None
+        if not f.absent:
+            z = lw.logits(x2, out_f32=True)
+            E = f.experts.total
+            idx, wts = MOE.route_topk(z[:, f.router_col:f.router_col + E], f.router_bias, f.top, 1, True, f.groups, f.keep_groups, f.route_scale)
+            ff = (*self._expert_rows(f, x2, idx, wts), z[:, :H])
+        return S.gated_join(h, mixer, ff, *self._entry_norms(i + 1), c.rms_eps, self.dtype, center=c.norm_kind == "layernorm")
+
+    def _expert_rows(self, f: MLPWeights, x, idx, wts):
+        """(expert outputs, their row of every (token, choice), weights) for a fused combine; or the combined rows and twice None."""
+        if f.experts.stacked is not None and x.is_cuda:
+            from ..ops import moe_grouped
+
+            parts = moe_grouped.forward(x, idx, wts, f.experts, combine=False)
+            if parts is not None:
+                return parts
+        return MOE.moe_forward(x, idx, wts, f.experts), None, None
 
     def _parallel_layer(self, lw: LayerWeights, x, fb: ForwardBatch, kv, h, i: int):
         """A listed layer whose mixer and feed-forward read the same rows ``x``: one projection of everything that is needed as fp32 logits,
@@ -701,11 +752,7 @@ class DecoderModel:
                 act[:, width:n].zero_()
             ML.mix(lw.mlstm, lw.mlstm.in_proj(x), gates, fb, kv[1], eps, out=act[:, :width])
         else:
-            gw = lw.grouped
-            proj = gw.in_proj(x)
-            _, cos, sin, _ = self._layer_geom(lw.attn, x.device) if lw.attn.rope is not None else (0, None, None, 0)
-            GR.post(gw, proj, fb, kv, cos, sin, eps)
-            GR.attention(gw, proj, kv, fb, out=act[:, :n], head_gate=gates)
+            self._grouped_heads(lw, lw.grouped.in_proj(x), fb, kv, out=act[:, :n], head_gate=gates)
         if f.gate_up is not None:
             f.gate_up.glu(x, "gelu_tanh", out=act[:, n:])
         elif f.shared_up is not None:
@@ -729,14 +776,10 @@ class DecoderModel:
         """Experts by the best softmax scores among the best groups; their combine adds ``shared`` and ends as ``ends`` says."""
         E = f.experts.total
         idx, wts = MOE.route_topk(z[:, f.router_col:f.router_col + E], None, f.top, 0, False, f.groups, f.keep_groups, group_max=True)
-        if f.experts.stacked is not None and x.is_cuda:
-            from ..ops import moe_grouped
-
-            parts = moe_grouped.forward(x, idx, wts, f.experts, combine=False)
-            if parts is not None:
-                return S.moe_combine_norm(parts[0], parts[1], wts, 1.0, shared, h, **ends)
-        y = MOE.moe_forward(x, idx, wts, f.experts)
-        return S.moe_combine_norm(y, self._row_ids(x.shape[0], x.device).view(-1, 1), None, 1.0, shared, h, **ends)
+        y, pos, wts = self._expert_rows(f, x, idx, wts)
+        if pos is None:
+            pos = self._row_ids(x.shape[0], x.device).view(-1, 1)
+        return S.moe_combine_norm(y, pos, wts, 1.0, shared, h, **ends)
 
     def _pass_start(self, i: int, ids):
         """What the residual gets before layer run ``i``: (embedding table or None, ids, step vector) where it opens a pass, else None."""
@@ -894,7 +937,10 @@ class DecoderModel:
             fb.decode_planned = True
         if self.layer_devices is not None:
             return self._forward_staged(fb, kv_caches)
-        if c.residual_f32:
+        if c.gated_residual:
+            h = torch.empty((T, c.hidden_size), device=fb.ids.device, dtype=torch.float32)
+            x = S.gated_join(h, None, None, *self._entry_norms(0), c.rms_eps, self.dtype, c.norm_kind == "layernorm", (self.embed, fb.ids))
+        elif c.residual_f32:
             if self.__dict__.get("_pos_freq") is None:
                 self._pos_freq = S.sinusoid_inv_freq(c.hidden_size, c.pos_embed_base, self.device) if c.pos_embed_base else None
             h, x = S.embed_pos_norm(fb.ids, fb.positions, self.embed, self._pos_freq, self._entry_norm(0), c.rms_eps, pos_table=self.pos_table,
@@ -923,6 +969,9 @@ class DecoderModel:
                 fa, fbeta, la, lbeta, ma, mbeta = c.resid_factors
                 alpha, self._beta = (la, lbeta) if lw.lin is not None else (fa, fbeta)
                 h = x * alpha if alpha != 1.0 else x
+            if c.gated_residual:
+                x = self._gated_layer(lw, x, fb, kv_caches[i], h, i)
+                continue
             if c.mixers is not None and c.parallel_block:
                 h, x = self._parallel_layer(lw, x, fb, kv_caches[i], h, i)
                 continue
@@ -951,6 +1000,8 @@ class DecoderModel:
             h, x = self._mlp(lw.mlp, x, h, i, next_ln, nxt, fb)
         self._beta = 1.0
         self._rope_override = None
+        if c.gated_residual:
+            x = x[0]
         # x is RMSNorm(h) with the final norm weight (row-wise, so selecting rows afterwards is equivalent)
         if fb.keep_hidden:
             B.flush_pending_wait()
@@ -974,6 +1025,10 @@ class DecoderModel:
             return self.final_norm
         lw = self.layers[i]
         return lw.lin.ln if lw.lin is not None else lw.attn.ln
+
+    def _entry_norms(self, i: int):
+        """Weights of the norms that open the mixer and the feed-forward of layer ``i`` where each has its own."""
+        return (self.layers[i].attn.ln, self.layers[i].mlp.ln) if i < len(self.layers) else (self.final_norm, None)
 
     def mtp_forward(self, fb: ForwardBatch, hidden: torch.Tensor, kv_caches):
         """Draft head over the packed rows of ``fb``: ``fb.ids`` are the tokens FOLLOWING each row's position, ``hidden`` the
@@ -1121,9 +1176,9 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
         raw.clear()
         p = f"model.layers.{i}."
         ones(p + "input_layernorm.weight", H)
-        if cfg.norm_kind == "layernorm":
+        if cfg.norm_kind == "layernorm" and cfg.mixers is None:
             mk(p + "input_layernorm.bias", (H,))
-        if not cfg.parallel_block:
+        if not cfg.parallel_block or cfg.gated_residual:
             ones(p + "post_attention_layernorm.weight", H)
         if cfg.mixers is not None:
             run = cfg.layer_runs.index(i)                 # i names a layer's weights; its specs are listed per run
@@ -1131,12 +1186,36 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
             if ff.kind == "none":
                 raw.pop(p + "post_attention_layernorm.weight", None)
             ap = p + "self_attn."
-            mk(ap + "q_proj.weight", (sp.heads * sp.dim, H))
-            gate = getattr(sp, "gate", "elem")
-            if gate:
-                mk(ap + "g_proj.weight", (sp.heads * (sp.vdim if gate == "elem" else 1), H))
-            mk(ap + "o_proj.weight", (H, sp.heads * sp.vdim))
-            if isinstance(sp, MLSTMSpec):
+            if isinstance(sp, RGLRUSpec):
+                part = sp.width // sp.blocks
+                for nm in ("y_proj", "x_proj"):
+                    mk(ap + nm + ".weight", (sp.width, H))
+                    mk(ap + nm + ".bias", (sp.width,))
+                mk(ap + "conv1d.weight", (sp.width, sp.conv), 0.3)
+                mk(ap + "conv1d.bias", (sp.width,))
+                for nm in ("ra_gate", "ri_gate"):
+                    mk(ap + nm + ".weight", (sp.blocks, part, part), part ** -0.5)
+                    mk(ap + nm + ".bias", (sp.blocks, part))
+                raw[ap + "lam"] = torch.linspace(-6.0, -2.0, sp.width, device=dev).to(dtype)       # decays between 0.98 and 0.3 a token at r = 1
+                mk(ap + "o_proj.weight", (H, sp.width))
+            else:
+                q_rank = getattr(sp, "q_rank", 0)
+                q_rows = sp.heads * (sp.dim + getattr(sp, "rot_dim", 0))
+                if q_rank:
+                    mk(ap + "q_a_proj.weight", (q_rank, H))
+                    ones(ap + "q_a_layernorm.weight", q_rank)
+                mk(ap + ("q_b_proj.weight" if q_rank else "q_proj.weight"), (q_rows, q_rank or H))
+                gate = getattr(sp, "gate", "elem")
+                if gate:
+                    mk(ap + "g_proj.weight", (sp.heads * (sp.vdim if gate == "elem" else 1), H))
+                mk(ap + "o_proj.weight", (H, sp.heads * sp.vdim))
+            if cfg.gated_residual:
+                for k in "12" if ff.kind != "none" else "1":
+                    mk(p + f"residual_gate{k}.weight", (H, H))
+                    mk(p + f"residual_gate{k}.bias", (H,))
+            if isinstance(sp, RGLRUSpec):
+                pass
+            elif isinstance(sp, MLSTMSpec):
                 mk(ap + "k_proj.weight", (sp.heads * sp.dim, H))
                 mk(ap + "v_proj.weight", (sp.heads * sp.vdim, H))
                 for nm, b in (("i_proj", 0.0), ("f_proj", 4.0)):
@@ -1156,14 +1235,16 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
                     mk(ap + "k_proj.weight", (sp.kv_heads * sp.dim, H))
                     mk(ap + "v_proj.weight", (sp.kv_heads * sp.vdim, H))
                 for nm, n in (("q", sp.heads * sp.dim), ("k", sp.kv_heads * sp.dim), ("v", sp.kv_heads * sp.vdim)):
-                    if nm != "v" and sp.qk_norm and (own or nm == "q"):
+                    if nm != "v" and sp.qk_norm and sp.norm_weight and (own or nm == "q"):
                         ones(ap + nm + "_norm.weight", sp.dim)
                     if sp.bias and (own or nm == "q"):
                         mk(ap + nm + "_proj.bias", (n,))
                 if sp.sinks:
                     mk(ap + "sinks", (sp.heads,))
-            else:
-                mk(ap + "kv_a_proj.weight", (sp.kv_rank, H))
+                if sp.weights == "sigmoid":
+                    raw[ap + "score_bias"] = torch.full((sp.heads,), -4.0, device=dev, dtype=dtype)
+            elif isinstance(sp, LatentSpec):
+                mk(ap + "kv_a_proj.weight", (sp.kv_rank + sp.rot_dim, H))
                 ones(ap + "kv_a_layernorm.weight", sp.kv_rank)
                 mk(ap + "k_b_proj.weight", (sp.heads * sp.dim, sp.kv_rank))
                 mk(ap + "v_b_proj.weight", (sp.heads * sp.vdim, sp.kv_rank))
@@ -1186,6 +1267,8 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
                     mk(p + "mlp.shared_expert_gate.weight", (1, H))
                 if ff.router != "table":
                     mk(p + "mlp.gate.weight", (ff.experts, H))
+                    if ff.router == "corrected":
+                        mk(p + "mlp.gate.e_score_correction_bias", (ff.experts,))
                     return raw
                 gen.manual_seed(_name_seed(seed, p + "mlp.token_table"))
                 raw[p + "mlp.token_table"] = torch.rand((cfg.vocab_size, ff.experts), device=dev, generator=gen).topk(ff.top, dim=1).indices.to(torch.int32)
@@ -1287,7 +1370,7 @@ def random_init(cfg: ModelConfig, device, dtype=torch.bfloat16, tp: TPInfo | Non
         if cfg.side_dim:
             mk("model.embed_tokens_per_layer.weight", (cfg.vocab_size, (1 + max(cfg.layer_runs)) * cfg.side_dim))
         ones("model.norm.weight", H)
-        if cfg.norm_kind == "layernorm":
+        if cfg.norm_kind == "layernorm" and cfg.mixers is None:
             mk("model.norm.bias", (H,))
         if not cfg.tie_embeddings:
             mk("lm_head.weight", (cfg.vocab_size, H))

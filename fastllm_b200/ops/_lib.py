@@ -30,6 +30,7 @@ _KERNEL_SIGS = {
     "fb_gemm_route": [P, P, I, I, I, I, I, I, P, P, P, I, I, I, F, P],
     "fb_gemm_16bit_batched": [P, P, P, I, I, I, I, I, I, I, I, I, I, P],
     "fb_gemm_16bit_batched_gate": [P, P, P, I, I, I, I, I, I, I, I, I, P, I, I, P],
+    "fb_gemm_16bit_blocks": [P, P, P, I, I, I, I, I, I, I, P],
     "fb_gemm_full32": [P, P, P, P, P, P, I, I, I, I, LL, LL, LL, LL, LL, LL, LL, LL, P, P, F, I, I, P, LL, P, P, LL, I, I, P],
     "fb_gemm_16bit_res32": [P, P, P, P, I, I, I, I, I, I, I, F, P, I, I, P],
     "fb_gemm_16bit_act": [P, P, P, I, I, I, I, I, I, I, P, I, P, P, LL, I, I, P],

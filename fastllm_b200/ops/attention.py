@@ -61,15 +61,14 @@ def rope_inv_freq(rot_dim: int, base: float, scaling: dict | None = None, max_po
         mid = (wavelen <= orig / lo) & (wavelen >= orig / hi)
         inv = torch.where(mid, (1 - smooth) * inv / factor + smooth * inv, scaled)
     elif kind == "yarn":
-        orig = int(scaling.get("original_max_position_embeddings", 4096))
+        orig = float(scaling.get("original_max_position_embeddings", 4096))
         beta_fast = float(scaling.get("beta_fast", 32))
         beta_slow = float(scaling.get("beta_slow", 1))
         low, high = _yarn_find_dim(beta_fast, rot_dim, base, orig), _yarn_find_dim(beta_slow, rot_dim, base, orig)
         if scaling.get("truncate", True):          # gpt-oss keeps the fractional correction range
             low, high = math.floor(low), math.ceil(high)
         low, high = max(low, 0), min(high, rot_dim - 1)
-        if low == high:
-            high += 0.001
+        high = max(high, low + 0.001)
         ramp = ((torch.arange(rot_dim // 2, dtype=torch.float64) - low) / (high - low)).clamp(0, 1)
         inv_mask = 1 - ramp
         inv = inv / factor * (1 - inv_mask) + inv * inv_mask
@@ -531,7 +530,7 @@ def attn_prefill(q, k_pool, v_pool, page_table, kv_lens, cu_q, scale, num_q_head
 # MLA decode (absorbed latent attention: a latent of up to 512 dims, optionally with rotary key dims behind it)
 # ---------------------------------------------------------------------------------------------------
 _lib.register_sigs({"fb_mla_decode": [ctypes.c_void_p] * 10 + [ctypes.c_int] * 4 + [ctypes.c_longlong, ctypes.c_int, ctypes.c_int, ctypes.c_int,
-                                      ctypes.c_float, ctypes.c_int, ctypes.c_void_p]}, ["attn_mla"])
+                                      ctypes.c_float, ctypes.c_void_p, ctypes.c_int, ctypes.c_void_p]}, ["attn_mla"])
 _MLA_WS: dict = {}
 
 
@@ -549,9 +548,11 @@ class MlaWorkspace:
         self.part_ml = torch.empty((self.max_items * 32 * 2,), device=device, dtype=torch.float32)
 
 
-def mla_decode(q_full, lat_pool, page_table, seq_lens, scale, ws: MlaWorkspace | None = None, lora: int | None = None, window: int = 0):
+def mla_decode(q_full, lat_pool, page_table, seq_lens, scale, ws: MlaWorkspace | None = None, lora: int | None = None, window: int = 0,
+               head_gate=None):
     """q_full ``[B, H, dq]`` (absorbed q_nope | rotated q_pe), lat_pool ``[pages, 128, 1, dq]`` -> ``[B, H, lora]``; the values are
-    the first ``lora`` of the ``dq`` columns (default: up to 512 of them).  ``window`` > 0: the last ``window`` tokens only."""
+    the first ``lora`` of the ``dq`` columns (default: up to 512 of them).  ``window`` > 0: the last ``window`` tokens only.  ``head_gate``:
+    fp32 logits ``[B, H]``, contiguous, of a sigmoid gate per head."""
     B, H, dq = q_full.shape
     lora = lora or min(dq, 512)
     if ws is None:
@@ -565,6 +566,6 @@ def mla_decode(q_full, lat_pool, page_table, seq_lens, scale, ws: MlaWorkspace |
     num_slots = lat_pool.shape[0] * lat_pool.shape[1]
     rc = _lib.kernels().fb_mla_decode(_ptr(q_full), _ptr(lat_pool), _ptr(out), _ptr(page_table), _ptr(seq_lens), _ptr(ws.work),
                                       _ptr(ws.n_work), _ptr(ws.item_range), _ptr(ws.part_o), _ptr(ws.part_ml), B, H, dq, lora, num_slots,
-                                      page_table.stride(0), ws.max_items, int(window), float(scale), dtype_code(q_full.dtype), _stream())
+                                      page_table.stride(0), ws.max_items, int(window), float(scale), _ptr(head_gate), dtype_code(q_full.dtype), _stream())
     _lib.check(rc, "fb_mla_decode")
     return out

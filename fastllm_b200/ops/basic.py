@@ -361,6 +361,21 @@ def linear_batched(x: torch.Tensor, w: torch.Tensor, batch: int, x_cols: int, ou
     return out
 
 
+def linear_blocks(x, w):
+    """Block-diagonal product with fp32 results: ``out[m, z * N + n] = sum_k x[m, z * K + k] * w[z, n, k]``; x ``[M, batch * K]``, w ``[batch, N, K]``
+    contiguous."""
+    M, (batch, N, K) = x.shape[0], w.shape
+    flush_pending_wait()
+    if not x.is_cuda:
+        return torch.einsum("mzk,znk->mzn", x.reshape(M, batch, K).float(), w.float()).reshape(M, batch * N)
+    out = torch.empty((M, batch * N), device=x.device, dtype=torch.float32)
+    if not tc_operands_ok(x, w.view(batch * N, K)) or N % 8:
+        return linear_full32(x, w, out=out, batch=batch, x_cols=K, out_cols=N)
+    rc = _lib.kernels().fb_gemm_16bit_blocks(_ptr(x), _ptr(w), _ptr(out), M, N, K, batch, x.stride(0), out.stride(0), dtype_code(x.dtype), _stream())
+    _lib.check(rc, "fb_gemm_16bit_blocks")
+    return out
+
+
 # ---------------------------------------------------------------------------------------------------
 # RMSNorm
 # ---------------------------------------------------------------------------------------------------

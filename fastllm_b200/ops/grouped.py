@@ -1,6 +1,8 @@
 """Grouped-query attention of listed layers: any head widths; optionally biases, per-head query / key norms, rotary positions on part
 of a head (interleaved pairs or halves), a chunk mask (a query sees the keys of its own chunk of positions) or a sliding window that may
-keep the first tokens of the sequence, soft-capped scores, a sink per head, and a sigmoid gate per element or per head.
+keep the first tokens of the sequence, soft-capped scores, a sink per head, a sigmoid gate per element or per head; sigmoid weights (with a
+number per head added to the score) in place of the softmax; values that are cached rotated, their sums turned back by the query's
+position.
 
 One launch normalises, rotates and writes the new keys and values to their cache slots (``csrc/stream32.cu``).  Rows are then attended
 in one of two ways, chosen per request of a batch:
@@ -25,11 +27,11 @@ from .basic import _ptr, _stream, dtype_code
 
 P, I, F, LL = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 _lib.register_sigs({
-    "fb_head_norm_rope": [P, LL, P, P, I, I, I, I, I, I, I, I, I, I, P, P, P, P, I, I, P, P, F, I, P],
+    "fb_head_norm_rope": [P, LL, P, P, I, I, I, I, I, I, I, I, I, I, P, P, I, P, P, I, P, P, I, I, P, P, F, I, P],
     "fb_grouped_plan": [P, I, I, I, I, P, P, I, P],
-    "fb_grouped_decode": [P, LL, P, P, P, LL, P, LL, P, P, P, P, P, P, I, I, I, I, I, LL, I, I, I, I, I, I, F, F, P, P, LL, I, P],
-    "fb_grouped_attn32": [P, LL, P, P, P, LL, P, LL, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P, LL, I, P],
-    "fb_attn_window_paged": [P, LL, I, P, P, LL, P, I, P, LL, P, LL, P, I, I, I, I, I, I, I, I, F, F, P, P, LL, I, P],
+    "fb_grouped_decode": [P, LL, P, P, P, LL, P, LL, P, P, P, P, P, P, I, I, I, I, I, LL, I, I, I, I, I, I, F, F, P, P, LL, P, P, P, I, I, I, P],
+    "fb_grouped_attn32": [P, LL, P, P, P, LL, P, LL, P, P, I, I, I, I, I, I, I, I, I, I, I, I, F, F, P, P, LL, P, P, P, I, I, I, P],
+    "fb_attn_window_paged": [P, LL, I, P, P, LL, P, I, P, LL, P, LL, P, I, I, I, I, I, I, I, I, F, F, P, P, LL, P, P, P, I, I, I, P],
 }, ["attn_grouped"])
 
 ROW_TOKENS = 16                  # requests that bring at most this many tokens take the decode kernel, a row each
@@ -51,7 +53,12 @@ class GroupedWeights:
         self.in_proj = None      # rows [queries | elementwise gate | keys | values]
         self.in_bias = None      # its bias, where the layer has one
         self.q_norm = self.k_norm = None
+        self.unit_norm = False   # the per-head norm has no weights
         self.sinks = None        # fp32 [heads]
+        self.score_bias = None   # fp32 [heads]: weights sigmoid(score + score_bias), not normalised
+        self.rot_v = 0           # dimensions of a value that turn, stored as pairs (2m, 2m + 1)
+        self.turn = None         # (cos, sin) tables of the values' rotation; the model sets them
+        self.more_col = 0        # first of the further rows of the projection
 
     @property
     def gate_col(self) -> int:
@@ -66,9 +73,26 @@ class GroupedWeights:
         return self.k_col + self.kv_heads * self.dp
 
 
-def build(spec, q, k, v, g, q_norm, k_norm, biases=None, sinks=None):
+def value_order(spec):
+    """Order in which a head's value dimensions are stored: the two of a rotated pair side by side (None: as they come)."""
+    if not spec.rope_values or spec.rope_values.get("mode") != "neox":
+        return None
+    n = spec.rope_values["rot_dim"]
+    pairs = torch.arange(n).view(2, n // 2).t().reshape(-1)
+    return torch.cat([pairs, torch.arange(n, spec.vdim)])
+
+
+def out_proj(o, spec):
+    """Output projection [width, heads * vdim] with its columns in the stored order, zero columns where the heads are padded."""
+    order = value_order(spec)
+    if order is not None:
+        o = o.reshape(o.shape[0], spec.heads, spec.vdim)[:, :, order.to(o.device)].reshape(o.shape[0], -1)
+    return LA.pad_out_proj(o, spec)
+
+
+def build(spec, q, k, v, g, q_norm, k_norm, biases=None, sinks=None, score_bias=None, more=()):
     """(GroupedWeights without ``in_proj``, merged input projection matrix) from the layer's matrices; ``k`` None: no own keys; ``g``
-    None: no elementwise gate; ``biases``: those of q, k and v."""
+    None: no elementwise gate; ``biases``: those of q, k and v; ``more``: matrices that read the same input."""
     w = GroupedWeights()
     w.heads, w.kv_heads, w.dim, w.vdim = spec.heads, spec.kv_heads, spec.dim, spec.vdim
     w.dp, w.vp = LA._round8(spec.dim), LA._round8(spec.vdim)
@@ -76,19 +100,25 @@ def build(spec, q, k, v, g, q_norm, k_norm, biases=None, sinks=None):
     w.window, w.keep, w.softcap, w.gate = int(spec.window or 0), int(spec.keep or 0) if spec.window else 0, float(spec.softcap or 0.0), spec.gate
     w.rot = int(spec.rope["rot_dim"]) if spec.rope else 0
     w.rope_mode = ROPE_NEOX if spec.rope and spec.rope.get("mode") == "neox" else ROPE_INTERLEAVED
-    w.q_norm, w.k_norm = q_norm, k_norm
+    w.q_norm, w.k_norm, w.unit_norm = q_norm, k_norm, bool(spec.qk_norm and not spec.norm_weight)
     w.sinks = sinks.float().contiguous() if sinks is not None else None
+    w.score_bias = score_bias.float().contiguous() if spec.weights == "sigmoid" else None
+    w.rot_v = int(spec.rope_values["rot_dim"]) if spec.rope_values else 0
+    order = value_order(spec)
 
-    def merge(q, g, k, v):
+    def merge(q, g, k, v, more=()):
         parts = [LA._pad_heads(q, w.heads, w.dp)] + ([LA._pad_heads(g, w.heads, w.vp)] if g is not None else [])
         if k is not None:
+            if order is not None:
+                v = v.reshape(w.kv_heads, w.vdim, v.shape[1])[:, order.to(v.device)].reshape(v.shape)
             parts += [LA._pad_heads(k, w.kv_heads, w.dp), LA._pad_heads(v, w.kv_heads, w.vp)]
-        return LA.pad_rows(torch.cat(parts, dim=0), 32)
+        w.more_col = sum(m.shape[0] for m in parts)
+        return LA.pad_rows(torch.cat([*parts, *more], dim=0), 32)
 
     if biases is not None:
         bq, bk, bv = (b[:, None] if b is not None else None for b in biases)
         w.in_bias = merge(bq, bq.new_zeros((w.heads * w.vp, 1)) if g is not None else None, bk, bv)[:, 0].contiguous()
-    return w, merge(q, g, k, v)
+    return w, merge(q, g, k, v, more)
 
 
 def first_key(pos, window: int, chunk: int):
@@ -102,21 +132,24 @@ def first_key(pos, window: int, chunk: int):
 
 def post(w: GroupedWeights, proj, fb, kv, cos, sin, eps: float) -> None:
     """Norm and rotation, where the layer has them, of the queries and keys in ``proj`` (in place; fp32 arithmetic) and the new keys and
-    values into their cache slots (rows with a negative slot are not cached)."""
+    (rotated) values into their cache slots (rows with a negative slot are not cached)."""
     T = proj.shape[0]
     k_pool, v_pool = kv
     if proj.is_cuda:
         G = w.kv_heads if w.own_kv else 0
+        cv, sv = w.turn if w.rot_v else (None, None)
+        tab = cos if cos is not None else cv
         rc = _lib.kernels().fb_head_norm_rope(_ptr(proj), proj.stride(0), _ptr(fb.positions), _ptr(fb.slots), T, w.heads, G, w.dim, w.dp, w.vp, w.k_col,
-                                              w.v_col, w.rot, 1 if w.rope_mode == ROPE_NEOX else 0, _ptr(w.q_norm), _ptr(w.k_norm), _ptr(cos), _ptr(sin), cos.shape[0] if cos is not None else 0,
+                                              w.v_col, w.rot, 1 if w.rope_mode == ROPE_NEOX else 0, _ptr(w.q_norm), _ptr(w.k_norm), int(w.unit_norm), _ptr(cos), _ptr(sin), w.rot_v,
+                                              _ptr(cv), _ptr(sv), tab.shape[0] if tab is not None else 0,
                                               k_pool.shape[0] * k_pool.shape[1], _ptr(k_pool), _ptr(v_pool), float(eps), S.act_code(proj.dtype), _stream())
         _lib.check(rc, "fb_head_norm_rope")
         return
 
     def turn(col, heads, norm_w):
         x = proj[:, col:col + heads * w.dp].reshape(T, heads, w.dp).clone()
-        if norm_w is not None:
-            x[..., :w.dim] = S._rms(x[..., :w.dim].float(), norm_w, eps).to(x.dtype)
+        if norm_w is not None or w.unit_norm:
+            x[..., :w.dim] = S._rms(x[..., :w.dim].float(), norm_w if norm_w is not None else torch.ones(()), eps).to(x.dtype)
         return apply_rope_ref(x, fb.positions, cos, sin, w.rope_mode, w.rot) if w.rot else x
 
     proj[:, :w.gate_col] = turn(0, w.heads, w.q_norm).reshape(T, -1)
@@ -124,7 +157,10 @@ def post(w: GroupedWeights, proj, fb, kv, cos, sin, eps: float) -> None:
         ok = fb.slots >= 0
         sl = fb.slots[ok].long()
         k_pool.view(-1, w.kv_heads, w.dp)[sl] = turn(w.k_col, w.kv_heads, w.k_norm)[ok].to(k_pool.dtype)
-        v_pool.view(-1, w.kv_heads, w.vp)[sl] = proj[:, w.v_col:w.v_col + w.kv_heads * w.vp].reshape(T, w.kv_heads, w.vp)[ok].to(v_pool.dtype)
+        v = proj[:, w.v_col:w.v_col + w.kv_heads * w.vp].reshape(T, w.kv_heads, w.vp)
+        if w.rot_v:
+            v = apply_rope_ref(v, fb.positions, *w.turn, ROPE_INTERLEAVED, w.rot_v)
+        v_pool.view(-1, w.kv_heads, w.vp)[sl] = v[ok].to(v_pool.dtype)
 
 
 # ---------------------------------------------------------------------------------------------------
@@ -185,7 +221,7 @@ def prefill_ok(w, dtype, page_len: int) -> bool:
         return False
     ok = w.__dict__.get("_prefill_ok")
     if ok is None:
-        ok = w._prefill_ok = bool(_lib.kernels()._lib.fb_attn_window_supported(w.dp, w.vp))
+        ok = w._prefill_ok = bool(_lib.kernels()._lib.fb_attn_window_supported(w.dp, 0, w.vp))
     return ok
 
 
@@ -212,6 +248,12 @@ def _gate_args(gate):
     return _ptr(gate), gate.stride(0) if gate is not None else 0
 
 
+def _weight_args(w):
+    """Sigmoid weights and the rotation of the outputs."""
+    cv, sv = w.turn if w.rot_v else (None, None)
+    return _ptr(w.score_bias), _ptr(cv), _ptr(sv), w.rot_v, cv.shape[0] if cv is not None else 0
+
+
 def decode_rows(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, kv_lens, out, row0: int = 0) -> None:
     """Rows ``q`` [n, heads * dp] against their own page-table rows; gated heads to ``out`` [n, heads * vp] (row strides free).  ``gate``
     [n, heads * vp] and ``head_gate`` (fp32 [n, heads]): None where the layer has no such gate."""
@@ -221,8 +263,8 @@ def decode_rows(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, kv_lens,
     if not decode_ok(w, q.dtype, page_len):
         rc = lib.fb_grouped_attn32(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), *_gate_args(gate),
                                    _ptr(page_table), _ptr(kv_lens), n, w.heads, w.kv_heads, w.dim, w.dp, w.vp, page_table.stride(0), k_pool.shape[0],
-                                   page_len, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks), *_gate_args(head_gate), S.act_code(q.dtype),
-                                   _stream())
+                                   page_len, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks), *_gate_args(head_gate), *_weight_args(w),
+                                   S.act_code(q.dtype), _stream())
         _lib.check(rc, "fb_grouped_attn32")
         return
     if n > _MAX_ROWS:
@@ -241,7 +283,7 @@ def decode_rows(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, kv_lens,
     rc = lib.fb_grouped_decode(_ptr(q), q.stride(0), _ptr(k_pool), _ptr(v_pool), _ptr(out), out.stride(0), *_gate_args(gate), _ptr(page_table),
                                _ptr(kv_lens), _ptr(lst[1:]), _ptr(lst), _ptr(part_o), _ptr(part_ml), n, w.heads, w.kv_heads, w.dp, w.vp, slots,
                                page_table.stride(0), splits, n * splits, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks), *_gate_args(head_gate),
-                               dtype_code(q.dtype), _stream())
+                               *_weight_args(w), dtype_code(q.dtype), _stream())
     _lib.check(rc, "fb_grouped_decode")
 
 
@@ -250,7 +292,7 @@ def prefill_blocks(w, pl: GroupedPlan, q, gate, head_gate, kv, page_table, out) 
     rc = _lib.kernels().fb_attn_window_paged(_ptr(q), q.stride(0), q.shape[0], _ptr(k_pool), _ptr(v_pool), k_pool.shape[0] * k_pool.shape[1],
                                              _ptr(page_table), page_table.stride(0), _ptr(out), out.stride(0), *_gate_args(gate), _ptr(pl.blocks),
                                              pl.n_blocks, w.heads, w.kv_heads, w.dp, w.vp, w.window, w.chunk, w.keep, w.scale, w.softcap, _ptr(w.sinks),
-                                             *_gate_args(head_gate), dtype_code(q.dtype), _stream())
+                                             *_gate_args(head_gate), *_weight_args(w), dtype_code(q.dtype), _stream())
     _lib.check(rc, "fb_attn_window_paged")
 
 
@@ -298,10 +340,16 @@ def attention_ref(w, q, gate, kv, fb, head_gate=None):
         s = torch.einsum("qhd,khd->hqk", q[r0:r1].float().reshape(-1, H, w.dp), k) * w.scale
         if w.softcap:
             s = torch.tanh(s / w.softcap) * w.softcap
+        if w.score_bias is not None:
+            out[r0:r1] = torch.einsum("hqk,khv->qhv", torch.sigmoid(s + w.score_bias[:, None, None]) * see, v)
+            continue
         s = s.masked_fill(~see, float("-inf"))
         if w.sinks is not None:
             s = torch.cat([s, w.sinks.view(H, 1, 1).expand(-1, s.shape[1], 1)], dim=-1)
         out[r0:r1] = torch.einsum("hqk,khv->qhv", torch.softmax(s, dim=-1)[..., :L], v)
+    if w.rot_v:
+        cv, sv = w.turn
+        out = apply_rope_ref(out, fb.positions, cv, -sv, ROPE_INTERLEAVED, w.rot_v)
     if head_gate is not None:
         out = out * torch.sigmoid(head_gate.float())[..., None]
     out = out.reshape(T, -1)

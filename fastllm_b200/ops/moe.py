@@ -48,7 +48,8 @@ def route_topk_ref(logits, bias, topk, score_mode, renorm, n_group=1, topk_group
 
 def route_topk(logits, bias, topk, score_mode, renorm, n_group=1, topk_group=1, route_scale=1.0, group_max=False):
     """logits fp32 ``[M, E]`` -> (expert index int32 ``[M, topk]``, weight fp32 ``[M, topk]``).  ``group_max``: a group's score is its largest
-    score (else the sum of its two largest)."""
+    score (else the sum of its two largest, or of the one there is)."""
+    group_max = group_max or logits.shape[1] == n_group
     if not logits.is_cuda or logits.shape[1] > 512 or topk > 32 or n_group > 32:        # beyond the kernel's registers: tensor ops
         return route_topk_ref(logits, bias, topk, score_mode, renorm, n_group, topk_group, route_scale, group_max)
     lg = logits.float()
