@@ -41,7 +41,7 @@ def parse_args():
     ap.add_argument("--output-len", type=int, default=256)
     ap.add_argument("--dtype", default="auto", help="weight dtype: auto(bf16) | int8 | int4g128 | fp8 | nvfp4 | mxfp4")
     ap.add_argument("--comm", default="auto", choices=["auto", "fused", "nccl"])
-    ap.add_argument("--layers", default="", choices=["", "patesun", "vilulorn", "vuripel"],
+    ap.add_argument("--layers", default="", choices=["", "patesun", "vilulorn", "vuripel", "nasipel"],
                     help="instead of the headline: throughput and kernel times of this design's layers beside the closest other family")
     ap.add_argument("--layer-sizes", default="2k,4k,7k")
     ap.add_argument("--layer-parts", default="kernels,steps")

@@ -2,8 +2,8 @@
 weights.
 
 ``python bench.py --layers patesun`` (beside multi-head latent attention with routed experts, DeepSeek-V3 layout), ``--layers vilulorn``
-(beside Gated DeltaNet + gated attention with routed experts, Qwen3-Next layout) and ``--layers vuripel`` (beside Vilulorn) print one
-JSON line per measurement:
+(beside Gated DeltaNet + gated attention with routed experts, Qwen3-Next layout), ``--layers vuripel`` (beside Vilulorn) and ``--layers
+nasipel`` (beside Vuripel) print one JSON line per measurement:
   * ``step``   -- prefill and decode tokens/s of a stack of four layers through the engine's runner;
   * ``kernel`` -- one operator alone: microseconds, its bytes / FLOPs and the fraction of the measured copy bandwidth or GEMM peak.
 Operators are timed with CUDA events behind an L2 flush that also hides the host's launch time; the median of the repeats is kept.
@@ -72,6 +72,18 @@ def vuripel_config(z):
     moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 8, "keep": 4}}, "shared": {"ff": z["eff"]}}
     return from_hf_dict(dict(architecture="Vuripel", vocab=VOCAB, width=z["width"], norm={"eps": 1e-6}, token_side={"dim": 256},
                              layers=[{"type": t, "mixer": m, "mlp": moe} for t, m in (("mlstm", lstm), ("attention_2", local), ("mlstm", lstm), ("attention", full))]))
+
+
+def nasipel_config(z):
+    from ..models.config import from_hf_dict
+
+    at = {"heads": z["heads"], "kv_heads": z["kv"], "dim": HEAD, "vdim": HEAD, "scale": HEAD ** -0.5, "softcap": 50.0, "rot": {"base": 5e5, "dims": HEAD}}
+    la = {"heads": z["heads"], "dim": HEAD, "vdim": HEAD, "q_rank": z["width"] // 2, "kv_rank": 512, "rot_dim": 64, "scale": (HEAD + 64) ** -0.5,
+          "rot": {"base": 5e5, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}
+    rg = {"width": z["lin"] * HEAD, "blocks": z["lin"] // 2, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 8, "keep": 4}, "scale": 2.0}}
+    return from_hf_dict(dict(architecture="Nasipel", vocab=VOCAB, width=z["width"], norm={"eps": 1e-6},
+                             layers=[{"type": t, "mixer": m, "mlp": moe} for t, m in (("rglru", rg), ("latent_attention", la), ("rglru", rg), ("attention", at))]))
 
 
 def deltanet_config(z):
@@ -270,7 +282,7 @@ def bench_kernels(z, size: str, emit) -> None:
         put("gemm_residual", "like", lambda: B.linear(x, w, residual=rm), W * H * HEAD * 2 + M * (H * HEAD * 2 + W * 4), fl, rows=M)
     # prompt chunk: latents -> keys and values -> windowed attention, against the latent-space products of the other family
     spec = LatentSpec(H, HEAD, HEAD, R, HEAD ** -0.5, win)
-    lw, _ = LA.build(spec, rnd(H * HEAD, W), rnd(H * HEAD, W), rnd(R, W), torch.ones(R, device=dev, dtype=dt), rnd(H * HEAD, R), rnd(H * HEAD, R))
+    lw, _, _ = LA.build(spec, rnd(H * HEAD, W), rnd(H * HEAD, W), rnd(R, W), torch.ones(R, device=dev, dtype=dt), rnd(H * HEAD, R), rnd(H * HEAD, R))
     for n_req, n in ((1, T), (T // 2048, 2048)):
         pages = n // 128
         cu = [n * b for b in range(n_req + 1)]
@@ -574,12 +586,172 @@ def bench_parallel_kernels(z, size: str, emit) -> None:
     torch.cuda.empty_cache()
 
 
+def bench_gated_kernels(z, size: str, emit) -> None:
+    """Operators of the gated-sub-layer stack (recurrent units, sigmoid-weighted attention over rotated values, latent attention with rotated
+    parts), each before the like one of the parallel-block stack or, for latent attention, of the latent families."""
+    from ..models.config import AttnSpec, LatentSpec, MLSTMSpec, RGLRUSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import attention as A
+    from ..ops import basic as B
+    from ..ops import grouped as GR
+    from ..ops import latent as LA
+    from ..ops import mlstm as ML
+    from ..ops import moe as MOE
+    from ..ops import moe_grouped as MG
+    from ..ops import rglru as RG
+    from ..ops import stream32 as S
+
+    tm = Timer()
+    hbm, tf, src = peaks()
+    dev, dt = "cuda", torch.bfloat16
+    W, H, G, N, C, E, top, eff = (z[k] for k in ("width", "heads", "kv", "lin", "chunk", "experts", "top", "eff"))
+    rnd = lambda *s: torch.randn(*s, device=dev, dtype=dt) * 0.05
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    D, T, Bn = HEAD, 8192, 64
+    causal = lambda m: m * (m + 1) // 2
+
+    def put(name, role, fn, nbytes, flops, **info):
+        us = tm.us(fn)
+        t_mem, t_mm = nbytes / hbm / 1e3, flops / tf / 1e6
+        emit(dict(kind="kernel", size=size, name=name, role=role, us=round(us, 2), gbytes=nbytes / 1e9, gflop=flops / 1e9,
+                  bound="memory" if t_mem > t_mm else "tensor", roofline_frac=round(max(t_mem, t_mm) / us, 4), peak=src, **info))
+
+    # recurrent layers: a step of 64 requests, prompts
+    R, part = N * D, 2 * D
+    rw, _ = RG.build(RGLRUSpec(R, N // 2, 4), rnd(R, 16), rnd(R, 16), rnd(R, 4), rnd(R), rnd(N // 2, part, part), rnd(N // 2, part), rnd(N // 2, part, part), rnd(N // 2, part),
+                     torch.linspace(-6, -2, R, device=dev).to(dt))
+    mw, _ = ML.build(MLSTMSpec(N, D, D, 15.0), *(rnd(N * D, 16) for _ in range(4)), rnd(N), rnd(N) + 4.0, rnd(N * D))
+    sr, sm = (torch.zeros((Bn + 1, R, 3), device=dev, dtype=dt), torch.zeros((Bn + 1, R), device=dev)), torch.zeros((Bn + 1, N, ML.state_len(D, D)), device=dev)
+    step = ForwardBatch(ids=None, positions=None, slots=None, page_table=None, kv_lens=None, cu_q=None, is_decode=True, state_slots=i32(list(range(Bn))))
+    proj, proj_m, gates = rnd(Bn, 2 * R + W), rnd(Bn, mw.cols[-1] + R + 32), torch.randn(Bn, 2 * N, device=dev)
+    weights = 2 * R * part * 2
+    put("recurrent unit step", "new", lambda: RG.mix(rw, proj, step, sr), Bn * R * (2 * 3 + 2 * 4 + 2 * 3 * 2) + weights, 4.0 * Bn * R * part, batch=Bn)
+    put("matrix-memory step", "like", lambda: ML.mix(mw, proj_m, gates, step, sm, 1e-6), Bn * N * (2 * D * D * 4 + 5 * D * 2), 0, batch=Bn)
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        cu, sl = [n * b for b in range(n_req + 1)], list(range(n_req))
+        proj, proj_m, gates = rnd(T, 2 * R + W), rnd(T, mw.cols[-1] + R + 32), torch.randn(T, 2 * N, device=dev)
+        fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=i32([[0]]), kv_lens=None, cu_q=i32(cu), cu_q_host=cu, state_slots=i32(sl), state_slots_host=sl)
+        put("recurrent unit prompt", "new", lambda: RG.mix(rw, proj, fb, sr), T * R * 2 * 3 + weights, 4.0 * T * R * part, requests=n_req, tokens=n)
+        put("matrix-memory prompt", "like", lambda: ML.mix(mw, proj_m, gates, fb, sm, 1e-6), T * N * D * 2 * 5, T * N * (4.0 * D * D + 2.0 * 64 * D), requests=n_req, tokens=n)
+    u = rnd(T, R)
+    put("gate logits, block products", "new", lambda: B.linear_blocks(u, rw.gates), T * R * (2 + 8) + weights, 4.0 * T * R * part, rows=T)
+    wide = rnd(2 * R, part)
+    put("product of that inner width", "like", lambda: B.linear(u[:, :part], wide, out_f32=True), T * (2 * part + 8 * R) + weights, 4.0 * T * R * part, rows=T)
+    del sr, sm, proj, proj_m, u, wide
+    # grouped-query attention
+    rope = {"theta": 5e5, "rot_dim": D, "scaling": None, "mode": "neox"}
+    tables = A.build_rope_tables(D, 65536, 5e5, None, dev)
+
+    def layer(**kw):
+        spec = AttnSpec(H, G, D, D, D ** -0.5, softcap=50.0, rope=rope, **kw)
+        norms = (rnd(D), rnd(D)) if spec.qk_norm and spec.norm_weight else (None, None)
+        w, _ = GR.build(spec, rnd(H * D, 16), rnd(G * D, 16), rnd(G * D, 16), None, *norms, None, rnd(H) if spec.sinks else None, rnd(H) - 4.0)
+        w.turn = tables
+        return w
+    pairs = (("sigmoid weights + cap + turned values", "new", layer(gate="", norm_weight=False, weights="sigmoid", rope_values=rope)),
+             ("cap + sinks + head gate", "like", layer(gate="head", sinks=True)))
+    for ctx in (C // 2, C):
+        pages = ctx // 128
+        pool = (rnd(Bn * pages, 128, G, D), rnd(Bn * pages, 128, G, D))
+        pt, lens = torch.randperm(Bn * pages, device=dev).to(torch.int32).view(Bn, pages), i32([ctx] * Bn)
+        for name, role, w in pairs:
+            fb = ForwardBatch(ids=None, positions=lens - 1, slots=None, page_table=pt, kv_lens=lens, cu_q=None, is_decode=True)
+            proj, hg = rnd(Bn, (w.v_col + G * D + 31) // 32 * 32), torch.randn(Bn, H, device=dev) if w.gate == "head" else None
+            GR.attention(w, proj, pool, fb, head_gate=hg)
+            put("decode attention, " + name, role, lambda: GR.attention(w, proj, pool, fb, head_gate=hg), Bn * (ctx * G * D * 4 + H * D * 4), 4.0 * Bn * H * ctx * D, batch=Bn, context=ctx)
+        del pool
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        pages, cu = n // 128, [n * b for b in range(n_req + 1)]
+        pool = (rnd(n_req * pages, 128, G, D), rnd(n_req * pages, 128, G, D))
+        pos = torch.arange(T, device=dev, dtype=torch.int32)
+        fb = ForwardBatch(ids=pos, positions=pos % n, slots=pos, page_table=torch.arange(n_req * pages, device=dev, dtype=torch.int32).view(n_req, pages), kv_lens=i32([n] * n_req),
+                          cu_q=i32(cu), cu_q_host=cu, kv_lens_host=[n] * n_req)
+        for name, role, w in pairs:
+            proj, hg = rnd(T, (w.v_col + G * D + 31) // 32 * 32), torch.randn(T, H, device=dev) if w.gate == "head" else None
+            GR.attention(w, proj, pool, fb, head_gate=hg)
+            put("prompt attention, " + name, role, lambda: GR.attention(w, proj, pool, fb, head_gate=hg), T * (H * D * 4 + G * D * 4), 4.0 * causal(n) * n_req * H * D, requests=n_req, tokens=n)
+    proj = rnd(T, (H + 2 * G) * D)
+    for name, role, w in (("unit norm + rotary + append of turned values", "new", pairs[0][2]), ("norm + rotary + append", "like", pairs[1][2])):
+        put(name, role, lambda: GR.post(w, proj, fb, pool, *tables, 1e-6), T * (H + 2 * G) * D * 4, 0, rows=T)
+    del pool, proj
+    # latent attention
+    K, Rd, Q, ln = 512, 64, W // 2, {"theta": 5e5, "rot_dim": 64, "scaling": None, "mode": "interleaved"}
+    cs = A.build_rope_tables(Rd, 65536, 5e5, None, dev)
+    lw, _, up = LA.build(LatentSpec(H, D, D, K, (D + Rd) ** -0.5, q_rank=Q, rot_dim=Rd, rope=ln, gate="head"), rnd(Q, 16), rnd(H, 16), rnd(K + Rd, 16), rnd(K), rnd(H * D, K), rnd(H * D, K),
+                         rnd(H * (D + Rd), Q), rnd(Q))
+    from ..ops.quant import LinearWeight
+
+    lw.q_up = LinearWeight.from_dense(up, act_dtype=dt)
+    lp, _, _ = LA.build(LatentSpec(H, D, D, K, D ** -0.5), rnd(H * D, 16), rnd(H * D, 16), rnd(K, 16), rnd(K), rnd(H * D, K), rnd(H * D, K))
+    for ctx in (C // 2, C):
+        pages = ctx // 128
+        lens = i32([ctx] * Bn)
+        pt = torch.randperm(Bn * pages, device=dev).to(torch.int32).view(Bn, pages)
+        pool, q, hg = rnd(Bn * pages + 1, 128, 1, K + Rd), rnd(Bn, H, K + Rd), torch.randn(Bn, H, device=dev)
+        for name, role, gate in (("latent decode, head gate", "new", hg), ("mla decode", "like", None)):
+            put(name, role, lambda: A.mla_decode(q, pool, pt, lens, 0.1, lora=K, head_gate=gate), Bn * (ctx * (K + Rd) * 2 + H * (2 * K + Rd) * 2), 2.0 * Bn * H * ctx * (2 * K + Rd), batch=Bn, context=ctx)
+        del pool
+    for n_req, n in ((1, T), (T // 2048, 2048)):
+        pages, cu = n // 128, [n * b for b in range(n_req + 1)]
+        pos = torch.arange(T, device=dev, dtype=torch.int32)
+        for name, role, w, rot in (("latent prompt attention, rotated part + head gate", "new", lw, Rd), ("latent prompt attention", "like", lp, 0)):
+            fb = ForwardBatch(ids=pos, positions=pos % n, slots=pos, page_table=torch.arange(n_req * pages, device=dev, dtype=torch.int32).view(n_req, pages), kv_lens=i32([n] * n_req),
+                              cu_q=i32(cu), cu_q_host=cu, kv_lens_host=[n] * n_req)
+            pool, proj, out = rnd(n_req * pages + 1, 128, 1, w.ld), rnd(T, w.more_col + 32), torch.empty((T, H * D), device=dev, dtype=dt)
+            q, hg = LA.post(w, proj, fb, pool, cs if rot else None, 1e-6)
+            LA.attention(w, proj, pool, fb, q, hg, cs)
+            grp = fb._latent_plans[next(iter(fb._latent_plans))].groups[0]
+            rows = S.gather_rows(pool.view(-1, w.ld), grp.key_idx)
+            expand = lambda: B.linear(S.gather_rows(pool.view(-1, w.ld), grp.key_idx)[:, :w.lv], w.w_ukv)
+            kv = expand()
+            gate = proj[:, w.gate_col:w.latent_col] if not rot else None
+            put(name, role, lambda: LA.window_attention(w, grp, q, gate, kv, out, hg, rows[:, w.lv:] if rot else None), T * H * (4 * D + 2 * rot) * 2, 2.0 * causal(n) * n_req * H * (2 * D + rot),
+                requests=n_req, tokens=n)
+            put("latent expand", role, expand, T * (w.ld * 2 + 2 * H * D * 2), 4.0 * T * K * H * D, requests=n_req, tokens=n)
+            if n_req == 1:
+                args = (proj, w.latent_col, w.kv_norm, w.rank, fb.slots, pool, 1e-6, w.lv, w.rot_col, w.rot, False, fb.positions, *(cs if rot else (None, None)), w.q_norm, w.q_pad, w.gate_col, w.n_gates)
+                put("latent norms + rotary key + append", role, lambda: S.latent_post(*args), T * (2 * w.q_pad + 2 * w.ld) * 2, 0, rows=T)
+                if rot:
+                    qr = q[:, w.dim:]
+                    put("rotary query parts", "new", lambda: S.rope_heads(qr, w.hd, qr, w.hd, H, Rd, Rd, fb.positions, *cs), T * H * Rd * 4, 0, rows=T)
+            del pool, proj, kv, rows, q
+        torch.cuda.empty_cache()
+    # the join of a layer, the products beside it, routing
+    nw = torch.ones(W, device=dev, dtype=dt)
+    for M in (64, T):
+        h, x, y, gcol = torch.randn(M, W, device=dev), rnd(M, W), rnd(M, W), rnd(M, 2 * W)
+        ys, where, wts, zz = rnd(M * top, W), torch.randperm(M * top, device=dev).to(torch.int32).view(M, top), torch.rand(M, top, device=dev), torch.randn(M, W + E, device=dev)
+        put("gated join of mixer and experts + two norms", "new", lambda: S.gated_join(h, (y, gcol[:, W:]), (ys, where, wts, zz[:, :W]), nw, nw, 1e-6, dt), M * W * (2 * top + 2 + 2 + 4 + 8 + 4), 0, rows=M)
+        put("combine + shared rows + residual + norm", "like", lambda: S.moe_combine_norm(ys, where, wts, 1.0, y, h, nw, 1.0, 1e-6, dtype=dt), M * W * (2 * top + 2 + 8 + 2), 0, rows=M)
+        wz, bz, wp = rnd(W + E, W), rnd(W + E), rnd(W + E, W)
+        nb, fl = (W + E) * W * 2 + M * (W * 2 + (W + E) * 4), 2.0 * M * W * (W + E)
+        put("gate + router logits", "new", lambda: B.linear(x, wz, bz, out_f32=True), nb, fl, rows=M)
+        put("product of that size", "like", lambda: B.linear(x, wp), nb - M * (W + E) * 2, fl, rows=M)
+        cor = torch.zeros(E, device=dev)
+        put("corrected grouped top-k", "new", lambda: MOE.route_topk(zz[:, W:], cor, top, 1, True, 8, 4, 2.0), M * (E * 4 + top * 8), 0, rows=M)
+        put("grouped top-k", "like", lambda: MOE.route_topk(zz[:, W:], None, top, 0, False, 8, 4, group_max=True), M * (E * 4 + top * 8), 0, rows=M)
+        del ys
+    table, ids = rnd(VOCAB, W), torch.randint(0, VOCAB, (T,), device=dev, dtype=torch.int32)
+    put("embedding + two norms", "new", lambda: S.gated_join(h, None, None, nw, nw, 1e-6, dt, embed=(table, ids)), T * W * 10, 0, rows=T)
+    put("embedding + norm", "like", lambda: S.embed_pos_norm(ids, ids, table, None, nw, 1e-6), T * W * 8, 0, rows=T)
+    ex = MOE.ExpertWeights(E, 0, [], [])
+    ex.count, ex.stacked = E, MG.StackedExperts("dense", rnd(E * 2 * eff, W), rnd(E * W, eff), E, eff, W)
+    ey = MOE.ExpertWeights(E, 0, [], [])
+    ey.count, ey.act, ey.stacked = E, "gelu", MG.StackedExperts("dense", ex.stacked.gate_up[:E * eff], ex.stacked.down, E, eff, W)
+    for M in (64, T):
+        x = rnd(M, W)
+        idx, wts = MOE.route_topk(torch.randn(M, E, device=dev), None, top, 0, False)
+        for name, role, e, mats in (("gated experts", "new", ex, 3), ("experts without gate branch", "like", ey, 2)):
+            put(name, role, lambda: MG.forward(x, idx, wts, e, combine=False), mats * E * W * eff * 2 + M * top * (4 * W + 2 * eff) * 2, 2.0 * mats * M * top * W * eff, rows=M)
+    torch.cuda.empty_cache()
+
+
 def run(family: str, sizes, steps: bool = True, kernels: bool = True, emit=None) -> None:
     emit = emit or (lambda d: print(json.dumps(d), flush=True))
     hybrid = family != "patesun"
-    operators = {"patesun": bench_kernels, "vilulorn": bench_hybrid_kernels, "vuripel": bench_parallel_kernels}[family]
+    operators = {"patesun": bench_kernels, "vilulorn": bench_hybrid_kernels, "vuripel": bench_parallel_kernels, "nasipel": bench_gated_kernels}[family]
     stacks = {"patesun": (("patesun", patesun_config), ("mla", mla_config)), "vilulorn": (("vilulorn", vilulorn_config), ("deltanet", deltanet_config)),
-              "vuripel": (("vuripel", vuripel_config), ("vilulorn", vilulorn_config))}[family]
+              "vuripel": (("vuripel", vuripel_config), ("vilulorn", vilulorn_config)), "nasipel": (("nasipel", nasipel_config), ("vuripel", vuripel_config))}[family]
     for size in sizes:
         z = (HYBRID_SIZES if hybrid else SIZES)[size]
         if kernels:

@@ -56,14 +56,12 @@ def yarn_freqs(dims, base, sc):
 
 def turn(x, positions, freqs, halves, sign=1.0, mag=1.0):
     """x [n, heads, >= 2 * len(freqs)]: pair i turns by sign * position * freqs[i]; pairs (i, i + len) or (2i, 2i + 1)."""
-    out = x.clone()
-    for i, f in enumerate(freqs):
-        a, b = (i, i + len(freqs)) if halves else (2 * i, 2 * i + 1)
-        ang = sign * positions.to(torch.float64) * f
-        c, s = (mag * torch.cos(ang)).to(x.dtype)[:, None], (mag * torch.sin(ang)).to(x.dtype)[:, None]
-        u, v = x[..., a], x[..., b]
-        out[..., a] = u * c - v * s
-        out[..., b] = v * c + u * s
+    n = len(freqs)
+    ang = sign * positions.to(torch.float64)[:, None] * torch.tensor(freqs, dtype=torch.float64)
+    c, s = (mag * torch.cos(ang)).to(x.dtype)[:, None], (mag * torch.sin(ang)).to(x.dtype)[:, None]
+    first, second = (slice(0, n), slice(n, 2 * n)) if halves else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+    u, v, out = x[..., first], x[..., second], x.clone()
+    out[..., first], out[..., second] = u * c - v * s, v * c + u * s
     return out
 
 
@@ -171,13 +169,16 @@ def choose(choice, router):
 
 
 def moe(h, w, p, mlp):
+    r = mlp["router"]
     s = torch.sigmoid(linear(w[p + "router"], h))
-    out = torch.zeros_like(h)
+    weight = torch.zeros_like(s)                                       # [tokens, experts], zero where an expert is not chosen
     for t in range(h.shape[0]):
-        picked = choose(s[t] + w[p + "correction"].to(s.dtype), mlp["router"])
-        total = s[t, picked].sum() + 1e-20
-        for e in picked:
-            out[t] += s[t, e] / total * mlp["router"].get("scale", 1.0) * expert(h[t:t + 1], w, f"{p}e{e}.")[0]
+        picked = choose(s[t] + w[p + "correction"].to(s.dtype), r)
+        weight[t, picked] = s[t, picked] / (s[t, picked].sum() + 1e-20) * r.get("scale", 1.0)
+    out = torch.zeros_like(h)
+    for e in range(r["experts"]):
+        rows = weight[:, e].nonzero()[:, 0]
+        out[rows] += weight[rows, e:e + 1] * expert(h[rows], w, f"{p}e{e}.")
     return out
 
 
@@ -200,3 +201,67 @@ def forward(cfg, w, tokens, dtype=torch.float64, layers_out=None):
         if layers_out is not None:
             layers_out.append(x)
     return linear(w["head"], layer_norm(x, w["final.norm"], eps))
+
+
+def random_weights(cfg, seed=0, scale=1.0):
+    """bfloat16 weights of the right names and shapes (norm weights around one)."""
+    g = torch.Generator().manual_seed(seed)
+    E, V = cfg["width"], cfg["vocab"]
+    w = {}
+
+    def mat(name, n, k, s=1.0):
+        w[name] = (torch.randn(n, k, generator=g) * (s * scale / k ** 0.5)).to(torch.bfloat16)
+
+    def vec(name, n, mean=1.0, s=0.2):
+        w[name] = (mean + s * torch.randn(n, generator=g)).to(torch.bfloat16)
+
+    w["embed"] = torch.randn(V, E, generator=g).to(torch.bfloat16)
+    for i, spec in enumerate(cfg["layers"]):
+        p, mx, ff = f"l{i}.", spec["mixer"], spec.get("mlp")
+        vec(p + "norm1", E)
+        mat(p + "rg1", E, E, 1.5)
+        vec(p + "rg1.b", E, 0.5, 0.5)
+        if spec["type"] == "rglru":
+            W, n = mx["width"], mx["width"] // mx["blocks"]
+            for z in "yx":
+                mat(p + "mix." + z, W, E)
+                vec(p + f"mix.{z}.b", W, 0.2, 0.3)
+            mat(p + "mix.conv", W, mx["conv"], 1.2)
+            vec(p + "mix.conv.b", W, 0.0, 0.3)
+            for z in ("ra", "ri"):
+                w[p + "mix." + z] = (torch.randn(mx["blocks"], n, n, generator=g) * 1.5 / n ** 0.5).to(torch.bfloat16)
+                w[p + f"mix.{z}.b"] = (0.5 * torch.randn(mx["blocks"], n, generator=g)).to(torch.bfloat16)
+            w[p + "mix.lam"] = torch.linspace(-7.0, 0.5, W)[torch.randperm(W, generator=g)].to(torch.bfloat16)      # memories of one to thousands of tokens
+            mat(p + "mix.o", E, W, 1.5)
+        elif spec["type"] == "latent_attention":
+            H, D, R, Vd = mx["heads"], mx["dim"], mx["rot_dim"], mx["vdim"]
+            mat(p + "mix.dq", mx["q_rank"], E)
+            vec(p + "mix.dq.norm", mx["q_rank"], 1.3)
+            mat(p + "mix.uq", H * (D + R), mx["q_rank"])
+            mat(p + "mix.dkv", mx["kv_rank"] + R, E, 1.3)
+            vec(p + "mix.dkv.norm", mx["kv_rank"])
+            mat(p + "mix.uk", H * D, mx["kv_rank"])
+            mat(p + "mix.uv", H * Vd, mx["kv_rank"], 1.5)
+            mat(p + "mix.g", H, E, 1.5)
+            mat(p + "mix.o", E, H * Vd, 1.5)
+        else:
+            H, G = mx["heads"], mx["kv_heads"]
+            mat(p + "mix.q", H * mx["dim"], E)
+            mat(p + "mix.k", G * mx["dim"], E)
+            mat(p + "mix.v", G * mx["vdim"], E)
+            vec(p + "mix.pb", H, -3.0, 0.5)
+            mat(p + "mix.o", E, H * mx["vdim"], 0.5)
+        if ff:
+            vec(p + "norm2", E)
+            mat(p + "rg2", E, E, 1.5)
+            vec(p + "rg2.b", E, 0.5, 0.5)
+            n, f = ff["router"]["experts"], ff["expert"]["ff"]
+            mat(p + "mlp.router", n, E, 1.5)
+            vec(p + "mlp.correction", n, -0.4, 0.5)
+            for e in range(n):
+                mat(p + f"mlp.e{e}.gate", f, E, 1.5)
+                mat(p + f"mlp.e{e}.up", f, E)
+                mat(p + f"mlp.e{e}.down", E, f)
+    vec("final.norm", E)
+    mat("head", V, E)
+    return w

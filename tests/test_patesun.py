@@ -14,6 +14,7 @@ from .listed_common import DEVICES, PAGE, assert_close, few_threads, portions, s
 from fastllm_b200.engine import EngineConfig, GenerationConfig, LLMEngine
 from fastllm_b200.engine.replay import Replay, open_engine
 from fastllm_b200.loader.hf import load_model
+from fastllm_b200.models.config import LatentSpec
 from fastllm_b200.models.decoder import ForwardBatch
 from fastllm_b200.ops import latent as LA
 from fastllm_b200.ops import stream32 as S
@@ -206,7 +207,7 @@ def test_norms(width, where):
     pool = torch.full((3, PAGE, 1, ld), 7.0, device=device, dtype=dtype)
     slots = torch.tensor([5, -1, 130, 0, 127, 128, -1], dtype=torch.int32)
     xs = x.to(device, dtype)
-    S.latent_norm(xs, w.to(device, dtype), slots.to(device), pool, width, 1e-3)
+    S.latent_post(xs, 0, w.to(device, dtype), width, slots.to(device), pool, 1e-3)
     flat = pool.view(-1, ld).cpu().double()
     want = O.rms_norm(xs.cpu().double(), w.double(), 1e-3)
     for t, s in enumerate(slots.tolist()):
@@ -228,12 +229,10 @@ def _latent_case(spec, lens, news, device, dtype, seed=0, strong=()):
         k = O.linear(uk, c[b][j:j + 1].double()).reshape(H, D)
         q[b][i] = (k * (score / spec["scale"] / k.pow(2).sum(-1, keepdim=True))).reshape(-1).to(torch.bfloat16)
     want = torch.cat([O.latent_core(q[b].double(), c[b].double(), uk.double(), uv.double(), gate[b].double(), spec) for b in range(len(lens))])
-
-    class Spec:
-        heads, dim, vdim, kv_rank, scale, window = H, D, V, R, spec["scale"], (spec.get("mask") or {}).get("size") or 0
+    sp = LatentSpec(H, D, V, R, spec["scale"], (spec.get("mask") or {}).get("size") or 0)
     zero = torch.zeros(H * D, 16)
     to = lambda t: t.to(device, dtype)
-    lw, _ = LA.build(Spec, to(zero), to(torch.zeros(H * V, 16)), to(torch.zeros(R, 16)), to(torch.ones(R)), to(uk), to(uv))
+    lw, _, _ = LA.build(sp, to(zero), to(torch.zeros(H * V, 16)), to(torch.zeros(R, 16)), to(torch.ones(R)), to(uk), to(uv))
     # pages are handed out in a shuffled order; a page of every request starts dirty
     npg = [(n + PAGE - 1) // PAGE for n in lens]
     order = torch.randperm(sum(npg), generator=g).tolist()
