@@ -195,7 +195,16 @@ struct LatentPostParams {
   float eps;
 };
 
-template <int DT>
+template <int DT, int VEC>
+__device__ __forceinline__ void ldv(const typename Act<DT>::T* p, float* v) {
+  if (VEC == 4) ld4<DT>(p, v); else v[0] = Act<DT>::ld(p[0]);
+}
+template <int DT, int VEC>
+__device__ __forceinline__ void stv(typename Act<DT>::T* p, const float* v) {
+  if (VEC == 4) st4<DT>(p, v); else p[0] = Act<DT>::st(v[0]);
+}
+
+template <int DT, int VEC>
 __global__ void latent_post_kernel(const LatentPostParams p) {
   typedef typename Act<DT>::T T;
   extern __shared__ float row[];
@@ -206,10 +215,18 @@ __global__ void latent_post_kernel(const LatentPostParams p) {
   const T* xp = reinterpret_cast<const T*>(p.x) + (size_t)t * p.ldx;
   const int slot = p.slots[t];
   T* yp = reinterpret_cast<T*>(p.pool) + (size_t)(slot < 0 ? p.spare : (long long)slot) * p.ld;
-  float qs = 0.f, ks = 0.f;
+  float sum[2] = {0.f, 0.f};
   float* krow = row + p.q_rank;
-  for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) { const float v = Act<DT>::ld(xp[p.q_col + i]); row[i] = v; qs += v * v; }
-  for (int i = threadIdx.x; i < p.rank; i += blockDim.x) { const float v = Act<DT>::ld(xp[p.kv_col + i]); krow[i] = v; ks += v * v; }
+  auto take = [&](const T* src, float* dst, int n, float& s) {
+    for (int i = threadIdx.x * VEC; i < n; i += blockDim.x * VEC) {
+      float v[VEC];
+      ldv<DT, VEC>(src + i, v);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) { dst[i + j] = v[j]; s += v[j] * v[j]; }
+    }
+  };
+  take(xp + p.q_col, row, p.q_rank, sum[0]);
+  take(xp + p.kv_col, krow, p.rank, sum[1]);
   for (int i = threadIdx.x; i < p.n_gates; i += blockDim.x) p.gates[(size_t)t * p.n_gates + i] = Act<DT>::ld(xp[p.gate_col + i]);
   if (p.rot > 0) {
     int pos = p.positions[t];
@@ -227,17 +244,33 @@ __global__ void latent_post_kernel(const LatentPostParams p) {
       }
     }
   }
-  if (p.q_rank > 0) {
-    qs = block_sum32(qs, sh[0]);
-    const float inv = 1.0f / sqrtf(qs / (float)p.q_rank + p.eps);
-    const T* w = reinterpret_cast<const T*>(p.q_norm);
-    T* cp = reinterpret_cast<T*>(p.cq) + (size_t)t * p.q_pad;
-    for (int i = threadIdx.x; i < p.q_pad; i += blockDim.x) cp[i] = Act<DT>::st(i < p.q_rank ? row[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+  // both sums in one exchange
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum[k] += __shfl_xor_sync(0xffffffffu, sum[k], o);
+    if ((threadIdx.x & 31) == 0) sh[k][threadIdx.x >> 5] = sum[k];
   }
-  ks = block_sum32(ks, sh[1]);
-  const float inv = 1.0f / sqrtf(ks / (float)p.rank + p.eps);
-  const T* w = reinterpret_cast<const T*>(p.kv_norm);
-  for (int i = threadIdx.x; i < p.lv; i += blockDim.x) yp[i] = Act<DT>::st(i < p.rank ? krow[i] * inv * Act<DT>::ld(w[i]) : 0.f);
+  __syncthreads();
+  float qs = 0.f, ks = 0.f;
+  for (int w = 0; w < (int)(blockDim.x >> 5); ++w) { qs += sh[0][w]; ks += sh[1][w]; }
+  auto put = [&](const float* src, const T* w, T* dst, int n, int width, float inv) {
+    for (int i = threadIdx.x * VEC; i < width; i += blockDim.x * VEC) {
+      float v[VEC];
+      if (i < n) {                                         // (n is a multiple of VEC)
+        ldv<DT, VEC>(w + i, v);
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[j] *= src[i + j] * inv;
+      } else {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) v[j] = 0.f;
+      }
+      stv<DT, VEC>(dst + i, v);
+    }
+  };
+  if (p.q_rank > 0)
+    put(row, reinterpret_cast<const T*>(p.q_norm), reinterpret_cast<T*>(p.cq) + (size_t)t * p.q_pad, p.q_rank, p.q_pad, 1.0f / sqrtf(qs / (float)p.q_rank + p.eps));
+  put(krow, reinterpret_cast<const T*>(p.kv_norm), yp, p.rank, p.lv, 1.0f / sqrtf(ks / (float)p.rank + p.eps));
 }
 
 // dst[t, h, :width] = src[t, h, :width] with the first `rot` dimensions turned, pairs (2j, 2j + 1) or (neox) (j, j + rot / 2); dst may be src
@@ -291,11 +324,6 @@ struct JoinParams {
 };
 
 __device__ __forceinline__ float sigmoid32(float z) { return 1.0f / (1.0f + expf(-z)); }
-
-template <int DT, int VEC>
-__device__ __forceinline__ void ldv(const typename Act<DT>::T* p, float* v) {
-  if (VEC == 4) ld4<DT>(p, v); else v[0] = Act<DT>::ld(p[0]);
-}
 
 template <int DT, int VEC>
 __global__ void gated_join_kernel(const JoinParams p) {
@@ -654,9 +682,12 @@ extern "C" int fb_latent_post(const void* x, long long ldx, int q_col, int q_ran
       (q_rank > 0 && (cq == nullptr || q_norm == nullptr)) || (n_gates > 0 && gates == nullptr))
     return -1;
   LatentPostParams p{x, ldx, q_col, q_rank, q_pad, kv_col, rank, lv, rot_col, rot, ld, neox, gate_col, n_gates, q_norm, kv_norm, cos_tab, sin_tab, tab_rows, positions, slots, cq, pool, gates, spare, eps};
-  const int th = row_threads(ld > q_pad ? ld : q_pad, 2);
-#define GO(DT) S32_LAUNCH((latent_post_kernel<DT>), T, th, q_rank + rank, stream, p)
-  if (dt == 0) GO(0) else if (dt == 1) GO(1) else GO(2)
+  const bool vec = !((q_col | q_rank | q_pad | kv_col | rank | lv | ld | ldx) & 3) && !((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(pool) | reinterpret_cast<uintptr_t>(cq) |
+                                                                                         reinterpret_cast<uintptr_t>(q_norm) | reinterpret_cast<uintptr_t>(kv_norm)) & 15);
+  const int th = row_threads(ld > q_pad ? ld : q_pad, vec ? 4 : 2);
+#define GO(DT, V) S32_LAUNCH((latent_post_kernel<DT, V>), T, th, q_rank + rank, stream, p)
+  if (vec) { if (dt == 0) GO(0, 4) else if (dt == 1) GO(1, 4) else GO(2, 4) }
+  else { if (dt == 0) GO(0, 1) else if (dt == 1) GO(1, 1) else GO(2, 1) }
 #undef GO
   return (int)cudaGetLastError();
 }

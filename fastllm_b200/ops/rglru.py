@@ -7,8 +7,8 @@
 request's state.  Both live in the engine's state slots: ``[width, taps - 1]`` inputs in the activation type and ``[width]`` in fp32.
 
 Three steps on CUDA (``csrc/rglru.cu``): the convolution, the gates' logits as one block-diagonal tensor-core product with fp32 results
-(``basic.linear_blocks``), and the recurrence with the output gate -- for prompts cut into chunks of 128 tokens that run in parallel
-behind a launch that sums every chunk up.  CPU tensors evaluate the PyTorch definition.
+(``basic.linear_blocks``), and the recurrence with the output gate: token by token for short portions, in chunks of 128 tokens that run
+in parallel behind a launch that sums every chunk up for longer ones.  CPU tensors evaluate the PyTorch definition.
 """
 from __future__ import annotations
 
@@ -29,6 +29,7 @@ _lib.register_sigs({
 }, ["rglru"])
 
 CHUNK = 128
+ROW_TOKENS = 16                  # requests that bring at most this many tokens walk them one by one
 DECAY = 8.0                      # log a = -DECAY * r * softplus(lam)
 
 
@@ -81,17 +82,23 @@ def out_proj(o, spec):
 
 
 class _Plan:
-    """The batch's requests in chunks: (first row, rows, slot, the request's rows before it, its first chunk, last)."""
+    """The batch's requests: ``conv`` all of them in chunks, ``short`` those that are walked token by token, ``long`` the others in chunks.  Items are
+    (first row, rows, slot, the request's rows before it, its first item in the list, last)."""
 
     def __init__(self, fb):
-        cu, chunks = fb.cu_q_host, []
+        cu, lists = fb.cu_q_host, ([], [], [])
         for b, s in enumerate(fb.state_slots_host):
-            n, first = cu[b + 1] - cu[b], len(chunks)
-            chunks += [(cu[b] + c, min(CHUNK, n - c), s, c, first, int(c + CHUNK >= n)) for c in range(0, n, CHUNK)]
-        self.n = len(chunks)
-        self.max_rows = max((c[1] for c in chunks), default=1)
-        self.multi = any(not c[5] for c in chunks)
-        self.chunks = torch.tensor(chunks, dtype=torch.int32).reshape(-1).to(fb.page_table.device, non_blocking=True)
+            n = cu[b + 1] - cu[b]
+            for l in (lists[0], lists[2])[:1 if n <= ROW_TOKENS else 2]:
+                first = len(l)
+                l.extend((cu[b] + c, min(CHUNK, n - c), s, c, first, int(c + CHUNK >= n)) for c in range(0, n, CHUNK))
+            if 0 < n <= ROW_TOKENS:
+                lists[1].append((cu[b], n, s, 0, 0, 1))
+        self.max_rows = max((c[1] for c in lists[0]), default=1)
+        self.multi = any(not c[5] for c in lists[2])
+        self.sizes = [len(l) for l in lists]
+        meta = torch.tensor([x for l in lists for t in l for x in t], dtype=torch.int32).to(fb.page_table.device, non_blocking=True)
+        self.conv, self.short, self.long = meta.split([6 * n for n in self.sizes])
 
 
 def mix(w: RGLRUWeights, proj, fb, state):
@@ -100,26 +107,27 @@ def mix(w: RGLRUWeights, proj, fb, state):
     if not proj.is_cuda:
         return mix_ref(w, proj, fb, state)
     T, W = proj.shape[0], w.width
-    conv, rec = state
     u = torch.empty((T, W), device=proj.device, dtype=proj.dtype)
     out = torch.empty_like(u)
-    if fb.is_decode:
-        slots, chunks, n, rows, multi = fb.state_slots, None, T, 1, 0
-    else:
-        pl = fb.__dict__.get("_rglru_plan")
-        if pl is None:
-            pl = fb._rglru_plan = _Plan(fb)
-        slots, chunks, n, rows, multi = None, pl.chunks, pl.n, pl.max_rows, int(pl.multi)
-    sums = torch.empty((3, n, W), device=proj.device, dtype=torch.float32) if multi else (None,) * 3
 
-    def step(which, z):
+    def step(which, z, slots, items, n, rows=1, sums=None):
         rc = _lib.kernels().fb_rglru(which, _ptr(proj[:, W:]), _ptr(proj), proj.stride(0), _ptr(w.conv_w), _ptr(w.conv_b), _ptr(w.gate_b), _ptr(w.decay), _ptr(z), _ptr(u),
-                                     _ptr(out), out.stride(0), _ptr(conv), _ptr(rec), _ptr(slots), _ptr(chunks), n, rows, multi, *(_ptr(t) for t in sums),
-                                     W, w.part, w.taps, S.act_code(proj.dtype), _stream())
+                                     _ptr(out), out.stride(0), _ptr(state[0]), _ptr(state[1]), _ptr(slots), _ptr(items), n, rows, int(sums is not None),
+                                     *(_ptr(t) for t in (sums if sums is not None else (None,) * 3)), W, w.part, w.taps, S.act_code(proj.dtype), _stream())
         _lib.check(rc, "fb_rglru")
 
-    step(0, None)
-    step(1, B.linear_blocks(u, w.gates))
+    if fb.is_decode:
+        step(0, None, fb.state_slots, None, T)
+        step(1, B.linear_blocks(u, w.gates), fb.state_slots, None, T)
+        return out
+    pl = fb.__dict__.get("_rglru_plan")
+    if pl is None:
+        pl = fb._rglru_plan = _Plan(fb)
+    n_conv, n_short, n_long = pl.sizes
+    step(0, None, None, pl.conv, n_conv, pl.max_rows)
+    z = B.linear_blocks(u, w.gates)
+    step(1, z, None, pl.short, n_short)
+    step(2, z, None, pl.long, n_long, pl.max_rows, torch.empty((3, n_long, W), device=proj.device, dtype=torch.float32) if pl.multi else None)
     return out
 
 
