@@ -298,16 +298,38 @@ def mlstm(heads=16, batch=64, tokens=8192, step=False, iters=4):
     torch.cuda.synchronize()
 
 
-def capped_prompt(tokens=8192, heads=16, kv=4, iters=3, window=0, keep=0):
-    """Soft-capped grouped-query prompt attention with sinks and head gates."""
+def rglru_prompt(tokens=8192, width=2048, part=256, iters=3):
+    """Recurrent unit over one prompt."""
+    from ..models.config import RGLRUSpec
+    from ..models.decoder import ForwardBatch
+    from ..ops import rglru as RG
+
+    dev, blocks = "cuda", width // part
+    rnd = lambda *s: (torch.randn(*s, device=dev) * 0.05).bfloat16()
+    i32 = lambda v: torch.tensor(v, device=dev, dtype=torch.int32)
+    w, _ = RG.build(RGLRUSpec(width, blocks, 4), rnd(width, 16), rnd(width, 16), rnd(width, 4), rnd(width), rnd(blocks, part, part), rnd(blocks, part), rnd(blocks, part, part),
+                    rnd(blocks, part), torch.linspace(-6, -2, width, device=dev).bfloat16())
+    state = (torch.zeros((1, width, 3), device=dev, dtype=torch.bfloat16), torch.zeros((1, width), device=dev))
+    fb = ForwardBatch(ids=None, positions=None, slots=None, page_table=i32([[0]]), kv_lens=None, cu_q=i32([0, tokens]), cu_q_host=[0, tokens], state_slots=i32([0]), state_slots_host=[0])
+    proj = rnd(tokens, 2 * width)
+    for _ in range(iters):
+        RG.mix(w, proj, fb, state)
+    torch.cuda.synchronize()
+
+
+def capped_prompt(tokens=8192, heads=16, kv=4, iters=3, window=0, keep=0, sigmoid=False):
+    """Soft-capped grouped-query prompt attention with sinks and head gates, or with sigmoid weights and rotated values."""
+    from ..ops import attention as A
     from ..models.config import AttnSpec
     from ..models.decoder import ForwardBatch
     from ..ops import grouped as GR
 
     dev, D, pages = "cuda", 128, tokens // 128
     rnd = lambda *s: (torch.randn(*s, device=dev) * 0.1).bfloat16()
-    spec = AttnSpec(heads, kv, D, D, D ** -0.5, softcap=50.0, sinks=True, qk_norm=False, gate="head", window=window, keep=keep)
-    w, _ = GR.build(spec, rnd(heads * D, 16), rnd(kv * D, 16), rnd(kv * D, 16), None, None, None, None, rnd(heads))
+    part = dict(gate="", weights="sigmoid", rope_values={"theta": 5e5, "rot_dim": D, "scaling": None, "mode": "neox"}) if sigmoid else dict(gate="head", sinks=True)
+    spec = AttnSpec(heads, kv, D, D, D ** -0.5, softcap=50.0, qk_norm=False, window=window, keep=keep, **part)
+    w, _ = GR.build(spec, rnd(heads * D, 16), rnd(kv * D, 16), rnd(kv * D, 16), None, None, None, None, None if sigmoid else rnd(heads), rnd(heads) - 4.0)
+    w.turn = A.build_rope_tables(D, tokens, 5e5, None, dev)
     pool = (rnd(pages, 128, kv, D), rnd(pages, 128, kv, D))
     pos = torch.arange(tokens, device=dev, dtype=torch.int32)
     fb = ForwardBatch(ids=pos, positions=pos, slots=pos, page_table=torch.arange(pages, device=dev, dtype=torch.int32).view(1, pages),
@@ -315,7 +337,7 @@ def capped_prompt(tokens=8192, heads=16, kv=4, iters=3, window=0, keep=0):
                       cu_q_host=[0, tokens], kv_lens_host=[tokens])
     proj, gates = rnd(tokens, w.v_col + kv * D), torch.randn(tokens, heads, device=dev)
     for _ in range(iters):
-        GR.attention(w, proj, pool, fb, head_gate=gates)
+        GR.attention(w, proj, pool, fb, head_gate=None if sigmoid else gates)
     torch.cuda.synchronize()
 
 
@@ -343,6 +365,8 @@ CASES = {
     "mlstm_prompt": mlstm,
     "mlstm_step": lambda: mlstm(step=True),
     "capped_prompt": capped_prompt,
+    "sigmoid_prompt": lambda: capped_prompt(sigmoid=True),
+    "rglru_prompt": rglru_prompt,
     "gla_step": lambda: gla(heads=32, step=True),
     "model_kernel_table_qwen3_moe_fp8": model_kernel_table,
     "gemm_qkv_post": gemm_qkv_post,
